@@ -136,8 +136,12 @@ class ModelPlan:
     final_norm: PartSpec
     head: PartSpec
     stop_token_ids: Tuple[int, ...] = ()
+    streams: int = 1          # copies of the width that the residual stream holds side by side (the embedding makes them, the
+                              # layers' arrangement works on them, the model's end is their sum)
 
     def validate(self) -> None:
+        if self.streams < 1:
+            raise SpecError(f"arch spec error: a model with {self.streams} residual streams")
         if not self.layers:
             raise SpecError("arch spec error: a model needs at least one layer")
         for i, call in enumerate(self.schedule):

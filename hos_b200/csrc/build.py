@@ -25,7 +25,7 @@ Libraries and what needs them:
               over keys and values of unequal sizes
   mixers      a norm after the residual sum, the norm-and-gate of a mixer's heads, and the
               matrix-state recurrences with a decay per head (constant, or per token with the
-              delta rule and short convolutions)
+              delta rule and short convolutions) or per key channel, hyper-connections
 A model builds only the libraries whose parts it has.
 """
 from __future__ import annotations
@@ -57,7 +57,7 @@ _STATIC_LIBS: Dict[str, Tuple[List[str], List[str]]] = {
     "experts": (["moe.cu"], []),
     "blocks": (["latent_attention.cu", "wkv.cu"], []),
     "gated_attn": (["gated_attention.cu", "gated_attention_mma.cu"], []),
-    "mixers": (["postnorm.cu", "state_scan.cu"], []),
+    "mixers": (["postnorm.cu", "state_scan.cu", "hyper.cu"], []),
 }
 
 _loaded: Dict[str, ctypes.CDLL] = {}

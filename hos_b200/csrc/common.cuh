@@ -210,4 +210,17 @@ __device__ __forceinline__ float clamped_swish_fast(float g, float u, float limi
     return g * rcp_approx(1.f + ex2_approx(-1.44269504f * kSwishAlpha * g)) * (u + 1.f);
 }
 
+// erf-form GELU: 0.5 x (1 + erf(x / sqrt 2)) = 0.5 x erfc(-x / sqrt 2), which does not cancel for negative x.
+__device__ __forceinline__ float gelu_erf(float x) { return 0.5f * x * erfcf(-0.70710678f * x); }
+// The same for the bfloat16 products' epilogues: erf by the rational approximation 7.1.26 of Abramowitz and Stegun
+// (Handbook of Mathematical Functions), erfc(a) = t (a1 + t (a2 + ...)) exp(-a^2), t = 1 / (1 + p a), a >= 0, absolute error
+// 1.5e-7; a dozen instructions per element.
+__device__ __forceinline__ float gelu_erf_fast(float x) {
+    const float a = 0.70710678f * fabsf(x);
+    const float t = rcp_approx(fmaf(0.3275911f, a, 1.f));
+    const float poly = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+    const float half_erfc = 0.5f * poly * ex2_approx(-1.44269504f * a * a);
+    return x * (x >= 0.f ? 1.f - half_erfc : half_erfc);
+}
+
 }  // namespace hos

@@ -12,17 +12,20 @@ namespace hos {
 // which marks padding, gives a zero row).
 template <typename TW>
 __global__ void embed_kernel(const int* __restrict__ tokens, const TW* __restrict__ table,
-                             float scale, float* __restrict__ out, int D) {
+                             float scale, float* __restrict__ out, int D, int copies) {
     pdl_enter();      // the kernels before this one are complete from here on
     const int n = blockIdx.x;
     const int tok = tokens[n];
-    float* o = out + (size_t)n * D;
+    float* o = out + (size_t)n * copies * D;         // a row is `copies` copies of the embedding, side by side
     if (tok < 0) {
-        for (int d = threadIdx.x; d < D; d += blockDim.x) o[d] = 0.f;
+        for (int d = threadIdx.x; d < copies * D; d += blockDim.x) o[d] = 0.f;
         return;
     }
     const TW* row = table + (size_t)tok * D;
-    for (int d = threadIdx.x; d < D; d += blockDim.x) o[d] = to_float(row[d]) * scale;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+        const float v = to_float(row[d]) * scale;
+        for (int c = 0; c < copies; ++c) o[(size_t)c * D + d] = v;
+    }
 }
 
 // ---- RMSNorm -----------------------------------------------------------------------
@@ -606,12 +609,13 @@ using namespace hos;
 extern "C" const char* hos_last_error() { return error_buffer(); }
 
 extern "C" int hos_embed(const int* tokens, const void* table, int table_dtype, float scale,
-                         float* out, int N, int D, cudaStream_t stream) {
+                         float* out, int N, int D, int copies, cudaStream_t stream) {
     if (N <= 0) return 0;
+    if (copies < 1) HOS_REFUSE("embed: %d copies", copies);
     if (table_dtype == kBF16)
-        launch_pdl(embed_kernel<bf16>, dim3(N), dim3(256), 0, stream, tokens, (const bf16*)table, scale, out, D);
+        launch_pdl(embed_kernel<bf16>, dim3(N), dim3(256), 0, stream, tokens, (const bf16*)table, scale, out, D, copies);
     else if (table_dtype == kF32)
-        launch_pdl(embed_kernel<float>, dim3(N), dim3(256), 0, stream, tokens, (const float*)table, scale, out, D);
+        launch_pdl(embed_kernel<float>, dim3(N), dim3(256), 0, stream, tokens, (const float*)table, scale, out, D, copies);
     else
         HOS_REFUSE("embed: unknown table dtype %d", table_dtype);
     return check_launch("embed");

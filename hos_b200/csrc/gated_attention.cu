@@ -10,7 +10,9 @@
 //   (2i, 2i+1) by the angle position * freq[i], cosine and sine times `magnitude`; queries are written as 32-bit
 //   rows, keys and values (in the cache's type) to their places in the paged cache.  With v_first the values
 //   are first blended with another layer's values of the same token, v <- (1 - v_mix) v + v_mix v_first, and the
-//   blend is what the cache holds.
+//   blend is what the cache holds.  With a short convolution (conv.w) every channel of q, k and v passes one over
+//   time right after the projection and its bias; its last inputs are the slot's state.  With q_every > 0 a query at
+//   position p is multiplied by 1 + q_coef ln(floor((p + 1) / q_every) + 1) at the end.
 // gated_attn: one warp per (token, up to 8 query heads that share a kv head, share of the keys).  A lane takes a
 //   key: 32 scores per head at a time, then the lanes turn to the value columns; a key or value row is read once
 //   for all of the warp's heads.  Keys j of position i: j <= i and, with chunks of size C,
@@ -19,6 +21,7 @@
 //   partial (maximum, sum, weighted values) go to a workspace and attn_merge adds them.
 #include "common.cuh"
 #include "kv_layout.cuh"
+#include "short_conv.cuh"
 
 namespace hos {
 
@@ -36,13 +39,23 @@ __device__ __forceinline__ int table_entry(const PagedKV2& c, int lp) { return c
 
 constexpr int kPrepMaxPL = 16;    // a head of up to 32 * 16 numbers in a warp's registers
 
-template <typename TC, int kPrepPL, int kThreads>
+// The short convolution of the q, k and v channels: w [taps][C] over the row's first C = H kd + G (kd + vd) columns.
+struct QkvConv {
+    const float* w;           // null: no convolution
+    const float* keep;        // [slots][taps - 1][C]
+    float* keep_w;            // the same memory where the kept inputs move on in this launch, else null
+    const int* cu_seqlens;
+    int taps;
+};
+
+template <typename TC, int kPrepPL, int kThreads, bool CONV>
 __global__ void __launch_bounds__(kThreads)
 qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ bias, const float* __restrict__ q_norm,
                const float* __restrict__ k_norm, float eps, const float* __restrict__ freq, int rot_dims, float magnitude,
                const int* __restrict__ token_pos, const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
                float* __restrict__ q_out, PagedKV2 cache, int H, int G, int kd, int vd, int norm_whole,
-               const float* __restrict__ v_first, long long v_first_ld, float v_mix, int q_maps) {
+               const float* __restrict__ v_first, long long v_first_ld, float v_mix, int q_maps, QkvConv conv, float q_coef,
+               int q_every) {
     pdl_enter();
     __shared__ float scratch[32];
     const int n = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -57,6 +70,19 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
     const int slot = seq_slot[seq];
     const int page = G > 0 ? cache.page_table[(size_t)slot * cache.table_stride + table_entry(cache, pos / kPageTokens)] : 0;
     const int r = pos % kPageTokens;
+    // The row that tap j of the convolution reads, from column 0 on: a row of this step (as projected, the bias is still to
+    // be added), one of the slot's kept inputs, or null before the sequence's start.
+    const int conv_C = H * kd + G * (kd + vd);
+    const int conv_r0 = CONV ? conv.cu_seqlens[seq] : 0;
+    const bool conv_fresh = CONV ? token_pos[conv_r0] == 0 : false;
+    const size_t keep_at = CONV ? (size_t)slot * (conv.taps - 1) * conv_C : 0;
+    auto tap_row = [&](int j, bool& raw) -> const float* {
+        const int src = n - (conv.taps - 1) + j;
+        raw = src >= conv_r0;
+        if (raw) return proj + (size_t)src * ld;
+        return conv_fresh ? nullptr : conv.keep + keep_at + (size_t)((conv.taps - 1) + (src - conv_r0)) * conv_C;
+    };
+    const float q_mult = q_every > 0 ? 1.f + q_coef * logf((float)((pos + 1) / q_every + 1)) : 1.f;
     float inv_all[2] = {0.f, 0.f};                       // norm_whole: one root mean square for all q heads, one for all k heads
     if (norm_whole) {
         for (int part = 0; part < (G > 0 ? 2 : 1); ++part) {
@@ -78,12 +104,34 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
         if (nw != nullptr && norm_whole) nw += (is_q ? item : item - H) * kd;
         float v[kPrepPL];
         float ss = 0.f;
+        if (CONV) {
 #pragma unroll
-        for (int i = 0; i < kPrepPL; ++i) {
-            const int d = lane + 32 * i;
-            v[i] = d < kd ? row[col0 + d] + (bias ? bias[col0 + d] : 0.f) : 0.f;
-            ss = fmaf(v[i], v[i], ss);
+            for (int i = 0; i < kPrepPL; ++i) v[i] = 0.f;
+#pragma unroll 1
+            for (int j = 0; j < conv.taps; ++j) {
+                bool raw;
+                const float* src = tap_row(j, raw);
+                // the kept inputs move on: row j - 1 was read in the turn before, by this thread
+                float* kw = conv.keep_w != nullptr && j >= 1 ? conv.keep_w + keep_at + (size_t)(j - 1) * conv_C + col0 : nullptr;
+#pragma unroll
+                for (int i = 0; i < kPrepPL; ++i) {
+                    const int d = lane + 32 * i;
+                    if (d < kd) {
+                        const float x = src == nullptr ? 0.f : src[col0 + d] + (raw && bias ? bias[col0 + d] : 0.f);
+                        v[i] = fmaf(conv.w[(size_t)j * conv_C + col0 + d], x, v[i]);
+                        if (kw != nullptr) kw[d] = x;
+                    }
+                }
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < kPrepPL; ++i) {
+                const int d = lane + 32 * i;
+                v[i] = d < kd ? row[col0 + d] + (bias ? bias[col0 + d] : 0.f) : 0.f;
+            }
         }
+#pragma unroll
+        for (int i = 0; i < kPrepPL; ++i) ss = fmaf(v[i], v[i], ss);
         if (nw != nullptr) {
             ss = warp_sum(ss);
             const float inv = norm_whole ? inv_all[is_q ? 0 : 1] : 1.f / sqrtf(ss / (float)kd + eps);
@@ -105,6 +153,9 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
                 v[i] = (d & 1) ? fmaf(v[i], cs, other * sn) : fmaf(v[i], cs, -other * sn);
             }
         }
+        if (is_q && q_every > 0)
+#pragma unroll
+            for (int i = 0; i < kPrepPL; ++i) v[i] *= q_mult;
         if (is_q && q_maps > 1) {
             // a head's kd numbers are q_maps queries of kd / q_maps numbers each, one per attention map over the same
             // key row: query m is written as a head of its own, zero outside its own part of the key row
@@ -138,7 +189,19 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
         for (int i = threadIdx.x; i < G * vd; i += blockDim.x) {
             const int g = i / vd, d = i % vd;
             TC* vp = (TC*)cache.v_pages + ((size_t)page * G + g) * (size_t)kPageTokens * vd;
-            float x = row[col0 + i] + (bias ? bias[col0 + i] : 0.f);
+            float x = 0.f;
+            if (CONV) {
+#pragma unroll 1
+                for (int j = 0; j < conv.taps; ++j) {
+                    bool raw;
+                    const float* src = tap_row(j, raw);
+                    const float u = src == nullptr ? 0.f : src[col0 + i] + (raw && bias ? bias[col0 + i] : 0.f);
+                    x = fmaf(conv.w[(size_t)j * conv_C + col0 + i], u, x);
+                    if (conv.keep_w != nullptr && j >= 1) conv.keep_w[keep_at + (size_t)(j - 1) * conv_C + col0 + i] = u;
+                }
+            } else {
+                x = row[col0 + i] + (bias ? bias[col0 + i] : 0.f);
+            }
             if (v_first != nullptr) x = fmaf(v_mix, v_first[(size_t)n * v_first_ld + i], (1.f - v_mix) * x);
             vp[kv_elem_offset(r, d, vd)] = from_float<TC>(x);
         }
@@ -167,9 +230,9 @@ template <typename TC, int VPL, int QH>
 __global__ void __launch_bounds__(kAttnWarps * 32)
 gated_attn_kernel(const float* __restrict__ q, PagedKV2 cache, const float* __restrict__ sink, const float* __restrict__ gate,
                   long long gate_stride, const int* __restrict__ token_pos, const int* __restrict__ token_seq,
-                  const int* __restrict__ seq_slot, void* __restrict__ out, int out_bf16, float* __restrict__ part_acc,
-                  float* __restrict__ part_ml, int n_splits, int n_tokens, int H, int G, int kd, int vd, float scale,
-                  int chunk, int window, int keep_first) {
+                  const int* __restrict__ seq_slot, void* __restrict__ out, int out_bf16, long long ldo, float out_scale,
+                  float* __restrict__ part_acc, float* __restrict__ part_ml, int n_splits, int n_tokens, int H, int G, int kd,
+                  int vd, float scale, int chunk, int window, int keep_first) {
     pdl_enter();
     extern __shared__ float qs_all[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -182,7 +245,7 @@ gated_attn_kernel(const float* __restrict__ q, PagedKV2 cache, const float* __re
     if (seq < 0) {
 #pragma unroll
         for (int hh = 0; hh < QH; ++hh) {
-            const size_t orow = ((size_t)n * H + h0 + hh) * vd;
+            const size_t orow = (size_t)n * ldo + (size_t)(h0 + hh) * vd;
             if (n_splits == 1)
                 for (int d = lane; d < vd; d += 32) {
                     if (out_bf16) ((bf16*)out)[orow + d] = from_float<bf16>(0.f);
@@ -292,7 +355,7 @@ gated_attn_kernel(const float* __restrict__ q, PagedKV2 cache, const float* __re
 #pragma unroll
     for (int hh = 0; hh < QH; ++hh) {
         const int h = h0 + hh;
-        const size_t orow = ((size_t)n * H + h) * vd;
+        const size_t orow = (size_t)n * ldo + (size_t)h * vd;
         if (n_splits > 1) {
             const size_t pi = ((size_t)n * H + h) * n_splits + split;
             if (lane == 0) {
@@ -306,7 +369,7 @@ gated_attn_kernel(const float* __restrict__ q, PagedKV2 cache, const float* __re
             }
             continue;
         }
-        float f = l[hh] > 0.f ? 1.f / l[hh] : 0.f;
+        float f = l[hh] > 0.f ? out_scale / l[hh] : 0.f;
         if (gate != nullptr) f *= 1.f / (1.f + expf(-gate[(size_t)n * gate_stride + h]));
 #pragma unroll
         for (int i = 0; i < VPL; ++i) {
@@ -324,7 +387,7 @@ gated_attn_kernel(const float* __restrict__ q, PagedKV2 cache, const float* __re
 __global__ void __launch_bounds__(128)
 attn_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, int n_splits,
                   const float* __restrict__ gate, long long gate_stride, const int* __restrict__ token_seq,
-                  void* __restrict__ out, int out_bf16, int n_tokens, int H, int vd) {
+                  void* __restrict__ out, int out_bf16, long long ldo, float out_scale, int n_tokens, int H, int vd) {
     pdl_enter();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * 4 + warp;
@@ -340,9 +403,10 @@ attn_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ 
     if (live)
         for (int s = lane; s < n_splits; s += 32) l += ml[2 * s + 1] > 0.f ? ml[2 * s + 1] * expf(ml[2 * s] - m) : 0.f;
     l = warp_sum(l);
-    float f = l > 0.f ? 1.f / l : 0.f;
+    float f = l > 0.f ? out_scale / l : 0.f;
     if (live && gate != nullptr) f *= 1.f / (1.f + expf(-gate[(size_t)n * gate_stride + h]));
     const float* acc_rows = part_acc + (size_t)item * n_splits * vd;
+    const size_t orow = (size_t)n * ldo + (size_t)h * vd;
     for (int d0 = 0; d0 < vd; d0 += 128) {
         float a[4] = {0.f, 0.f, 0.f, 0.f};
         if (live) {
@@ -363,8 +427,8 @@ attn_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ 
         for (int i = 0; i < 4; ++i) {
             const int d = d0 + lane + 32 * i;
             if (d >= vd) continue;
-            if (out_bf16) ((bf16*)out)[(size_t)item * vd + d] = from_float<bf16>(a[i] * f);
-            else ((float*)out)[(size_t)item * vd + d] = a[i] * f;
+            if (out_bf16) ((bf16*)out)[orow + d] = from_float<bf16>(a[i] * f);
+            else ((float*)out)[orow + d] = a[i] * f;
         }
     }
 }
@@ -414,13 +478,20 @@ extern "C" const char* hos_last_error() { return error_buffer(); }
 // columns' biases or null.  q_norm / k_norm: [kd] or null (norm_whole: [H * kd] and [G * kd]).  freq: [rot_dims / 2] or
 // null.  v_first: row n's values of another layer at v_first[n * v_first_ld + ...] (G * vd numbers), or null.
 // q_maps > 1: q_out is [N][H * q_maps][kd]: each head's kd numbers are q_maps queries, written as heads of their own.
+// conv_w ([taps][C], C = H kd + G (kd + vd), or null): the short convolution of q, k and v with its kept inputs conv_state [slots]
+// [taps - 1][C]; keep_here: 1 only where every sequence of the step brings exactly one token (the kept inputs move on
+// inside this launch; otherwise hos_qkv_conv_keep does it afterwards).  q_every > 0: the queries' factor by position.
 extern "C" int hos_qk_prep(const float* proj, int ld, const float* bias, const float* q_norm, const float* k_norm, float eps,
                            const float* freq, int rot_dims, float magnitude, const int* token_pos, const int* token_seq,
                            const int* seq_slot, float* q_out, void* k_pages, void* v_pages, int cache_dtype,
                            const int* page_table, int table_stride, int ring_pages, int N, int H, int G, int kd, int vd,
                            int norm_whole, const float* v_first, long long v_first_ld, float v_mix, int q_maps,
-                           cudaStream_t stream) {
+                           const float* conv_w, int taps, float* conv_state, const int* cu_seqlens, int keep_here, float q_coef,
+                           int q_every, cudaStream_t stream) {
     if (N <= 0) return 0;
+    if (conv_w != nullptr && (taps < 1 || taps > kMaxTaps || norm_whole || cu_seqlens == nullptr || (taps > 1 && conv_state == nullptr)))
+        HOS_REFUSE("qk_prep: a convolution of %d taps (1..%d; not with a norm over the whole projection)", taps, kMaxTaps);
+    const QkvConv conv{conv_w, conv_state, keep_here && taps > 1 ? conv_state : nullptr, cu_seqlens, taps};
     if (q_maps < 1 || kd % q_maps != 0) HOS_REFUSE("qk_prep: heads of %d numbers do not hold %d queries", kd, q_maps);
     if (kd <= 0 || kd > 32 * kPrepMaxPL) HOS_REFUSE("qk_prep: heads of %d numbers are outside 1..%d", kd, 32 * kPrepMaxPL);
     if (freq == nullptr) rot_dims = 0;
@@ -428,10 +499,15 @@ extern "C" int hos_qk_prep(const float* proj, int ld, const float* bias, const f
     PagedKV2 c{k_pages, v_pages, page_table, table_stride, ring_pages, G, kd, vd};
     // few rows (single-token steps): a block of 16 warps shortens the row's chain of loads; many rows: 4 warps
     const bool wide = N <= 592 && H + G > 4;
-#define HOS_QKP_N(TC, PL, NT)                                                                                        \
-    launch_pdl(qk_prep_kernel<TC, PL, NT>, dim3(N), dim3(NT), 0, stream, proj, ld, bias, q_norm, k_norm, eps, freq,   \
+#define HOS_QKP_C(TC, PL, NT, CV)                                                                                    \
+    launch_pdl(qk_prep_kernel<TC, PL, NT, CV>, dim3(N), dim3(NT), 0, stream, proj, ld, bias, q_norm, k_norm, eps, freq, \
                rot_dims, magnitude, token_pos, token_seq, seq_slot, q_out, c, H, G, kd, vd, norm_whole, v_first,     \
-               v_first_ld, v_mix, q_maps)
+               v_first_ld, v_mix, q_maps, conv, q_coef, q_every)
+#define HOS_QKP_N(TC, PL, NT)                                                                                        \
+    do {                                                                                                             \
+        if (conv_w != nullptr) HOS_QKP_C(TC, PL, NT, true);                                                          \
+        else HOS_QKP_C(TC, PL, NT, false);                                                                           \
+    } while (0)
 #define HOS_QKP(TC, PL)                                                                                              \
     do {                                                                                                             \
         if (wide) HOS_QKP_N(TC, PL, 512);                                                                            \
@@ -450,18 +526,31 @@ extern "C" int hos_qk_prep(const float* proj, int ld, const float* bias, const f
 #undef HOS_QKP_T
 #undef HOS_QKP
 #undef HOS_QKP_N
+#undef HOS_QKP_C
     return check_launch("qk_prep");
 }
 
-// q: float32 [N][H][kd].  out: [N][H][vd] of out_dtype.  gate: row n's logit of head h at gate[n * gate_stride + h], or
+// The last taps - 1 inputs (with their bias) of every sequence's q, k, v channels go to the slot's state.
+extern "C" int hos_qkv_conv_keep(const float* proj, long long ld, const float* bias, int taps, float* conv_state,
+                                 const int* token_pos, const int* token_seq, const int* cu_seqlens, const int* seq_slot,
+                                 int n_seqs, int C, cudaStream_t stream) {
+    if (n_seqs <= 0 || taps <= 1) return 0;
+    if (taps > kMaxTaps) HOS_REFUSE("qkv_conv_keep: %d taps are outside 1..%d", taps, kMaxTaps);
+    launch_pdl(short_conv_keep_kernel, dim3((C + 127) / 128, n_seqs), dim3(128), 0, stream, proj, ld, bias, taps, conv_state,
+               token_pos, token_seq, cu_seqlens, seq_slot, C);
+    return check_launch("qkv_conv_keep");
+}
+
+// q: float32 [N][H][kd].  out: H * vd numbers of out_dtype from the start of rows that lie ldo apart, the heads' outputs times
+// out_scale.  gate: row n's logit of head h at gate[n * gate_stride + h], or
 // null.  sink: [H] or null.  chunk, window: 0 for none; keep_first: with a window, that many of a sequence's first keys
 // stay in sight.  n_splits > 1: part_acc [N][H][n_splits][vd] and part_ml
 // [N][H][n_splits][2] float32 must be given.
 extern "C" int hos_gated_attn(const float* q, void* k_pages, void* v_pages, int cache_dtype, const int* page_table,
                               int table_stride, int ring_pages, const float* sink, const float* gate, long long gate_stride,
                               const int* token_pos, const int* token_seq, const int* seq_slot, void* out, int out_dtype,
-                              float* part_acc, float* part_ml, int n_splits, int N, int H, int G, int kd, int vd, float scale,
-                              int chunk, int window, int keep_first, cudaStream_t stream) {
+                              long long ldo, float out_scale, float* part_acc, float* part_ml, int n_splits, int N, int H, int G,
+                              int kd, int vd, float scale, int chunk, int window, int keep_first, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (G <= 0 || H % G != 0) HOS_REFUSE("gated_attn: %d heads are not a multiple of %d kv heads", H, G);
     if (vd <= 0 || vd > 32 * kMaxVPL) HOS_REFUSE("gated_attn: value heads of %d numbers are outside 1..%d", vd, 32 * kMaxVPL);
@@ -483,8 +572,8 @@ extern "C" int hos_gated_attn(const float* q, void* k_pages, void* v_pages, int 
     const int out_bf16 = out_dtype == kBF16;
 #define HOS_GA(TC, VPL, QH)                                                                                          \
     launch_pdl(gated_attn_kernel<TC, VPL, QH>, dim3(blocks), dim3(kAttnWarps * 32), smem, stream, q, c, sink, gate,  \
-               gate_stride, token_pos, token_seq, seq_slot, out, out_bf16, part_acc, part_ml, n_splits, N, H, G, kd, vd, \
-               scale, chunk, window, keep_first)
+               gate_stride, token_pos, token_seq, seq_slot, out, out_bf16, ldo, out_scale, part_acc, part_ml, n_splits, N, H, \
+               G, kd, vd, scale, chunk, window, keep_first)
 #define HOS_GA_Q(TC, VPL)                                                                                            \
     do {                                                                                                             \
         if (qh == 8) { if constexpr (VPL <= 4) HOS_GA(TC, VPL, 8); }                                                 \
@@ -508,17 +597,17 @@ extern "C" int hos_gated_attn(const float* q, void* k_pages, void* v_pages, int 
     int rc = check_launch("gated_attn");
     if (rc != 0 || n_splits == 1) return rc;
     launch_pdl(attn_merge_kernel, dim3((unsigned)(((long long)N * H + 3) / 4)), dim3(128), 0, stream, (const float*)part_acc,
-               (const float*)part_ml, n_splits, gate, gate_stride, token_seq, out, out_bf16, N, H, vd);
+               (const float*)part_ml, n_splits, gate, gate_stride, token_seq, out, out_bf16, ldo, out_scale, N, H, vd);
     return check_launch("attn_merge");
 }
 
 // The shares' partial results under one maximum: out [N][H][vd] from part_acc [N][H][n_splits][vd], part_ml [..][2].
 extern "C" int hos_attn_merge(const float* part_acc, const float* part_ml, int n_splits, const float* gate,
-                              long long gate_stride, const int* token_seq, void* out, int out_dtype, int N, int H, int vd,
-                              cudaStream_t stream) {
+                              long long gate_stride, const int* token_seq, void* out, int out_dtype, long long ldo,
+                              float out_scale, int N, int H, int vd, cudaStream_t stream) {
     if (N <= 0) return 0;
     launch_pdl(attn_merge_kernel, dim3((unsigned)(((long long)N * H + 3) / 4)), dim3(128), 0, stream, part_acc, part_ml,
-               n_splits, gate, gate_stride, token_seq, out, out_dtype == kBF16 ? 1 : 0, N, H, vd);
+               n_splits, gate, gate_stride, token_seq, out, out_dtype == kBF16 ? 1 : 0, ldo, out_scale, N, H, vd);
     return check_launch("attn_merge");
 }
 

@@ -5,19 +5,21 @@
 // tensor-core kernel refuses.  Any M, N, K.
 //
 // Epilogues: none; soft-cap (logits); gated (W holds gate rows then up rows,
-// out = act(gate) * up), so that the 2F-wide intermediate is never written.
+// out = act(gate) * up), so that the 2F-wide intermediate is never written; bias (out = act(x + bias[n]), act
+// none or the erf-form GELU).
 #include "common.cuh"
 
 namespace hos {
 
 constexpr int BM = 64, BN = 64, BK = 16;
 
-enum Epilogue : int { kEpiNone = 0, kEpiSoftcap = 1, kEpiGated = 2 };
+enum Epilogue : int { kEpiNone = 0, kEpiSoftcap = 1, kEpiGated = 2, kEpiBias = 3 };
 
 template <typename TA, typename TW, typename TO, int EPI>
 __global__ void __launch_bounds__(256)
 gemm_plain_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TO* __restrict__ out,
-                  int M, int N, int K, int lda, int ldw, int ldo, float cap, int act, int gate_rows) {
+                  int M, int N, int K, int lda, int ldw, int ldo, float cap, int act, int gate_rows,
+                  const float* __restrict__ bias) {
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[BK][BN + 4];
     __shared__ float Us[EPI == kEpiGated ? BK : 1][BN + 4];
@@ -70,6 +72,10 @@ gemm_plain_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TO* __rest
             if (n >= N) continue;
             float v = acc[i][j];
             if (EPI == kEpiSoftcap) v = softcap_precise(v, cap);
+            if (EPI == kEpiBias) {
+                v += bias[n];
+                if (act == 1) v = gelu_erf(v);
+            }
             if (EPI == kEpiGated) {
                 if (act == 2) {
                     v = clamped_swish(v, acc_u[i][j], cap);          // the clamp's limit rides in `cap`
@@ -85,21 +91,26 @@ gemm_plain_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TO* __rest
 
 template <typename TA, typename TW, typename TO>
 static int launch_plain(const void* A, const void* W, void* out, int M, int N, int K, int lda,
-                        int ldw, int ldo, int epi, float cap, int act, cudaStream_t stream) {
+                        int ldw, int ldo, int epi, float cap, int act, const float* bias, cudaStream_t stream) {
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
     if (grid.y > 65535) HOS_REFUSE("gemm_plain: %d rows are more than one launch takes", M);
     switch (epi) {
     case kEpiNone:
         gemm_plain_kernel<TA, TW, TO, kEpiNone><<<grid, 256, 0, stream>>>(
-            (const TA*)A, (const TW*)W, (TO*)out, M, N, K, lda, ldw, ldo, cap, act, 0);
+            (const TA*)A, (const TW*)W, (TO*)out, M, N, K, lda, ldw, ldo, cap, act, 0, bias);
         break;
     case kEpiSoftcap:
         gemm_plain_kernel<TA, TW, TO, kEpiSoftcap><<<grid, 256, 0, stream>>>(
-            (const TA*)A, (const TW*)W, (TO*)out, M, N, K, lda, ldw, ldo, cap, act, 0);
+            (const TA*)A, (const TW*)W, (TO*)out, M, N, K, lda, ldw, ldo, cap, act, 0, bias);
         break;
     case kEpiGated:
         gemm_plain_kernel<TA, TW, TO, kEpiGated><<<grid, 256, 0, stream>>>(
-            (const TA*)A, (const TW*)W, (TO*)out, M, N, K, lda, ldw, ldo, cap, act, N);
+            (const TA*)A, (const TW*)W, (TO*)out, M, N, K, lda, ldw, ldo, cap, act, N, bias);
+        break;
+    case kEpiBias:
+        if (bias == nullptr) HOS_REFUSE("gemm_plain: the bias epilogue needs a bias");
+        gemm_plain_kernel<TA, TW, TO, kEpiBias><<<grid, 256, 0, stream>>>(
+            (const TA*)A, (const TW*)W, (TO*)out, M, N, K, lda, ldw, ldo, cap, act, 0, bias);
         break;
     default:
         HOS_REFUSE("gemm_plain: unknown epilogue %d", epi);
@@ -111,16 +122,17 @@ static int launch_plain(const void* A, const void* W, void* out, int M, int N, i
 
 using namespace hos;
 
-// out[M, N] = A[M, K] . W[N, K]^T.  For the gated epilogue W has 2N rows (gate, then up).
+// out[M, N] = A[M, K] . W[N, K]^T.  For the gated epilogue W has 2N rows (gate, then up); for the bias epilogue `bias` has N
+// numbers and act 1 is the erf-form GELU (0: none).
 // Leading dimensions are in elements.
 extern "C" int hos_gemm_plain(const void* A, int a_dtype, const void* W, int w_dtype, void* out,
                               int out_dtype, int M, int N, int K, int lda, int ldw, int ldo,
-                              int epilogue, float cap, int act, cudaStream_t stream) {
+                              int epilogue, float cap, int act, const float* bias, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0) HOS_REFUSE("gemm_plain: K must be positive");
 #define HOS_CASE(da, dw, dout, TA, TW, TO)                                         \
     if (a_dtype == da && w_dtype == dw && out_dtype == dout)                       \
-        return launch_plain<TA, TW, TO>(A, W, out, M, N, K, lda, ldw, ldo, epilogue, cap, act, stream);
+        return launch_plain<TA, TW, TO>(A, W, out, M, N, K, lda, ldw, ldo, epilogue, cap, act, bias, stream);
     HOS_CASE(kF32, kF32, kF32, float, float, float)
     HOS_CASE(kBF16, kBF16, kBF16, bf16, bf16, bf16)
     HOS_CASE(kBF16, kBF16, kF32, bf16, bf16, float)

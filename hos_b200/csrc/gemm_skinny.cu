@@ -14,7 +14,8 @@
 //    memory and the result does not depend on timing.
 //
 // Epilogues: none (bf16 or f32 output); gated, where the CTA owns 16 gate rows and the 16
-// matching up rows (4 warps each) and writes act(gate) * up.
+// matching up rows (4 warps each) and writes act(gate) * up; bias (out = act(x + bias[n]), act none or the erf-form
+// GELU, bf16 output).
 #include "common.cuh"
 #include "kv_layout.cuh"
 #include "mma_utils.cuh"
@@ -56,7 +57,7 @@ template <int MT, int kUnroll, bool GATED, typename OutT, int WARPS = kSkinnyWar
 __global__ void __launch_bounds__(WARPS * 32, 16 / WARPS)
 gemm_skinny_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, OutT* __restrict__ out,
                    int M, int N, int K, int lda, int ldw, int ldo, int gate_rows, int act, int late,
-                   float act_limit) {
+                   float act_limit, const float* __restrict__ bias) {
     // The kernel may be launched ahead of the end of the kernel before it: its CTAs are placed and a warp's first
     // round of weights, which no kernel writes, is on its way before the activations exist.
     // (`late`: the kernel after this one is let go only when the kernel before this one has ended: this kernel was
@@ -172,6 +173,10 @@ gemm_skinny_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, OutT*
             v = 0.f;
 #pragma unroll
             for (int w = 0; w < WARPS; ++w) v += part[w][m][r][t];
+            if (bias != nullptr) {
+                v += bias[n];
+                if (act == 1) v = gelu_erf_fast(v);
+            }
         }
         out[(size_t)tok * ldo + n] = from_float<OutT>(v);
     }
@@ -359,19 +364,22 @@ static bool skinny_ahead(int kind) { return (skinny_ahead_mode() & kind) != 0 ||
 // everywhere else (2, 4 or 8 sequences; one sequence at 32,768 keys): it stays behind its attention kernel.
 
 // out[M, N] = A[M, K] . W[N, K]^T for M <= 32.  epilogue 0: none (out bf16 or f32); 2: gated (W has
-// 2N rows: gate rows, then up rows at row N; out bf16; act 0, 1, or 2, the clamped form with its limit in act_limit).
+// 2N rows: gate rows, then up rows at row N; out bf16; act 0, 1, or 2, the clamped form with its limit in act_limit);
+// 3: bias (bias[N] added, act 1: erf-form GELU; out bf16).
 // K and the leading dimensions must be
 // multiples of 8 elements, A and W 16-byte aligned.
 // k_splits > 1: `out` is [k_splits][M][ldo] 32-bit partial sums for a consumer that adds them (no epilogue).
 extern "C" int hos_gemm_skinny(const void* A, const void* W, void* out, int out_dtype, int M, int N, int K,
-                               int lda, int ldw, int ldo, int epilogue, int act, float act_limit, int k_splits,
-                               int room_before, cudaStream_t stream) {
+                               int lda, int ldw, int ldo, int epilogue, int act, float act_limit, const float* bias,
+                               int k_splits, int room_before, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M > 8 * kMaxTokenTiles) HOS_REFUSE("gemm_skinny: %d rows are more than %d", M, 8 * kMaxTokenTiles);
     if (K <= 0 || (K % 8) || (lda % 8) || (ldw % 8) || ((uintptr_t)A % 16) || ((uintptr_t)W % 16))
         HOS_REFUSE("gemm_skinny: K and the leading dimensions must be multiples of 8 elements and the operands "
                    "16-byte aligned (K %d lda %d ldw %d)", K, lda, ldw);
-    if (epilogue != 0 && epilogue != 2) HOS_REFUSE("gemm_skinny: epilogue %d is not offered", epilogue);
+    if (epilogue != 0 && epilogue != 2 && epilogue != 3) HOS_REFUSE("gemm_skinny: epilogue %d is not offered", epilogue);
+    if (epilogue == 3 && (out_dtype != kBF16 || bias == nullptr)) HOS_REFUSE("gemm_skinny: the bias epilogue writes bfloat16 and needs a bias");
+    if (epilogue != 3) bias = nullptr;
     if (epilogue == 2 && out_dtype != kBF16) HOS_REFUSE("gemm_skinny: the gated epilogue writes bfloat16");
     if (k_splits < 1 || k_splits > 64) HOS_REFUSE("gemm_skinny: %d splits of K (1..64)", k_splits);
     if (k_splits > 1 && (epilogue != 0 || out_dtype != kF32))
@@ -384,14 +392,15 @@ extern "C" int hos_gemm_skinny(const void* A, const void* W, void* out, int out_
     const int k_ways = epilogue == 2 ? kGatedWarps / 2 : kSkinnyWarps;
     const int k_blocks = (K + 31) / 32, per_cta = (k_blocks + k_splits - 1) / k_splits;
     const int unroll = unroll_for((per_cta + k_ways - 1) / k_ways, (M + 7) / 8);
-    const int kind = (M > 8) ? (epilogue == 2 ? 16 : 0) : (epilogue == 2 ? 1 : (out_dtype == kBF16 ? 2 : 4));
+    const bool behind_norm = epilogue == 2 || epilogue == 3;       // gate/up, or the up product with its bias
+    const int kind = (M > 8) ? (behind_norm ? 16 : 0) : (behind_norm ? 1 : (out_dtype == kBF16 ? 2 : 4));
     // `room_before` (the caller's word that the kernel before this one leaves at least half of the SMs free, as the
     // attention of one sequence does): the o product is then launched ahead as well
     const bool ahead = skinny_ahead(kind) || (kind == 2 && room_before != 0);
     const int late = (kind == 2 || kind == 4) && ahead ? 1 : 0;     // o and down, when launched ahead
 #define HOS_SK_W(MT, U, G, T, WP)                                                                                \
     launch_ahead(ahead, gemm_skinny_kernel<MT, U, G, T, WP>, dim3(grid, k_splits), dim3(WP * 32), 0, stream, (const bf16*)A, (const bf16*)W, (T*)out, \
-                                                                       M, N, K, lda, ldw, ldo, N, act, late, act_limit)
+                                                                       M, N, K, lda, ldw, ldo, N, act, late, act_limit, bias)
 #define HOS_SK(MT, U, G, T) HOS_SK_W(MT, U, G, T, (G ? kGatedWarps : kSkinnyWarps))
 #define HOS_SK_U(MT, G, T)                              \
     do {                                                \

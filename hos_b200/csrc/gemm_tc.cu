@@ -19,7 +19,8 @@
 // that a small kernel adds in a fixed order.
 //
 // Epilogues: none; soft-cap c*tanh(x/c) with 32-bit output (logits); gated act(gate)*up,
-// where W holds the gate rows followed by the up rows and a tile loads matching rows of both.
+// where W holds the gate rows followed by the up rows and a tile loads matching rows of both; act(x + bias[n]), act
+// none or the erf-form GELU.
 //
 // Every wait on an mbarrier is bounded in time: a wait that runs out sets an error flag,
 // the roles leave their loops, tensor memory is freed and the kernel returns.
@@ -37,7 +38,7 @@ constexpr int kGemmThreads = 192;
 constexpr int kPairThreads = 320;         // the kernel on pairs of SMs: TMA warp, MMA warp, 8 epilogue warps
 constexpr long long kWaitCycles = 1ll << 31;     // about a second
 
-enum { kGEpiNone = 0, kGEpiSoftcap = 1, kGEpiGated = 2, kGEpiRope = 3 };
+enum { kGEpiNone = 0, kGEpiSoftcap = 1, kGEpiGated = 2, kGEpiBias = 3, kGEpiRope = 4 };
 
 __device__ int g_gemm_error = 0;
 __device__ int* g_gemm_error_host = nullptr;     // a word in pinned host memory, if the host gave one
@@ -156,9 +157,31 @@ struct GemmParams {
     int k_splits;
     int gate_rows;        // gated: row of W where the up rows begin
     float cap;            // the soft-cap; with the gated epilogue's activation 2, the clamp's limit
-    int act;              // gated: 0 tanh-form GELU, 1 x logistic(x), 2 the clamped form (common.cuh)
+    int act;              // gated: 0 tanh-form GELU, 1 x logistic(x), 2 the clamped form (common.cuh); bias: 0 none, 1 erf-form GELU
+    const float* bias;    // kGEpiBias: [N]
     RopeEpi rope;         // kGEpiRope only
 };
+
+// Thirty-two columns n0.. of one row, with their bias and activation (all lanes of a warp read the same bias: one line).
+__device__ __forceinline__ void bias_act_32(const uint32_t (&v)[32], float (&f)[32], const float* __restrict__ bias, int n0, int N, int act) {
+    if (n0 + 32 <= N && ((uintptr_t)(bias + n0) & 15) == 0) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const float4 b = __ldg(reinterpret_cast<const float4*>(bias + n0) + j);
+            f[4 * j] = __uint_as_float(v[4 * j]) + b.x;
+            f[4 * j + 1] = __uint_as_float(v[4 * j + 1]) + b.y;
+            f[4 * j + 2] = __uint_as_float(v[4 * j + 2]) + b.z;
+            f[4 * j + 3] = __uint_as_float(v[4 * j + 3]) + b.w;
+        }
+    } else {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) f[j] = __uint_as_float(v[j]) + (n0 + j < N ? __ldg(bias + n0 + j) : 0.f);
+    }
+    if (act == 1) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) f[j] = gelu_erf_fast(f[j]);
+    }
+}
 
 template <int BN, bool SWAP>
 struct GemmCfg {
@@ -326,6 +349,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_m,     // the 128-row ope
 #pragma unroll
                                 for (int j = 0; j < 32; ++j) f[j] = silu_fast(__uint_as_float(v[j])) * __uint_as_float(u[j]);
                             }
+                        } else if (EPI == kGEpiBias) {
+                            bias_act_32(v, f, p.bias, n0, p.N, p.act);
                         } else {
 #pragma unroll
                             for (int j = 0; j < 32; ++j) {
@@ -358,6 +383,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_m,     // the 128-row ope
                 const bool gated = EPI == kGEpiGated;
                 const int feat = gated ? mt * 64 + (r & 63) : mt * GM + r;
                 const int feat_count = p.N;
+                const float feat_bias = EPI == kGEpiBias && feat < feat_count ? __ldg(p.bias + feat) : 0.f;
                 OutT* obase = reinterpret_cast<OutT*>(p.out) + (p.k_splits > 1 ? (size_t)ks * p.M * p.ldo : 0);
                 constexpr int CH = BN < 32 ? BN : 32;
 #pragma unroll 1
@@ -405,6 +431,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_m,     // the 128-row ope
                             if (tok < p.M) {
                                 float x = f[j];
                                 if (EPI == kGEpiSoftcap) x = softcap_precise(x, p.cap);
+                                if (EPI == kGEpiBias) {
+                                    x += feat_bias;
+                                    if (p.act == 1) x = gelu_erf_fast(x);
+                                }
                                 obase[(size_t)tok * p.ldo + feat] = from_float<OutT>(x);
                             }
                         }
@@ -740,6 +770,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a,     // A: boxes o
 #pragma unroll
                             for (int j = 0; j < 32; ++j) f[j] = silu_fast(__uint_as_float(v[j])) * __uint_as_float(u[j]);
                         }
+                    } else if (EPI == kGEpiBias) {
+                        bias_act_32(v, f, p.bias, nt * COLS + c0 + 32 * h, p.N, p.act);
                     } else {
 #pragma unroll
                         for (int j = 0; j < 32; ++j) {
@@ -868,7 +900,7 @@ static int launch(const CUtensorMap& mm, const CUtensorMap& mn, const GemmParams
     // dependents go only after its wait, so nothing piles up behind them (64 sequences 8.04 -> 7.97 ms a step, 40
     // sequences 5.80 -> 5.75, 128 sequences 14.50 -> 14.44; the head launched ahead changes nothing).
     static const bool swapped_ahead = !(getenv("HOS_GEMM_TC_AHEAD") && getenv("HOS_GEMM_TC_AHEAD")[0] == '0');
-    const bool ahead = swapped_ahead && SWAP && (EPI == kGEpiGated || (EPI == kGEpiNone && sizeof(OutT) == 4));
+    const bool ahead = swapped_ahead && SWAP && (EPI == kGEpiGated || EPI == kGEpiBias || (EPI == kGEpiNone && sizeof(OutT) == 4));
     launch_ahead(pdl_enabled() || ahead, kernel, dim3(grid), dim3(kGemmThreads),
                  Cfg::kSmem, stream, mm, mn, p);
     return check_launch("gemm_tc");
@@ -964,13 +996,14 @@ extern "C" long long hos_gemm_tc_workspace(int M, int N, int k_splits) {
 }
 
 // out[M, N] = A[M, K] . W[N, K]^T, bf16 operands.  out_dtype: 1 bf16, 0 f32.  epilogue: 0 none,
-// 1 soft-cap (f32 output), 2 gated (W has 2N rows: gate rows, then up rows at row N).
+// 1 soft-cap (f32 output), 2 gated (W has 2N rows: gate rows, then up rows at row N), 3 bias (bias[N] added, act 1: the
+// erf-form GELU; bf16 output).
 // M <= 128 runs swapped; k_splits > 1 is allowed only then and only without an epilogue, and
 // needs `workspace` (see hos_gemm_tc_workspace).  With reduce_now == 0 the partial sums are left
 // in the workspace as [k_splits_used][M][N] floats for the consumer to add, `out` is not written,
 // and the number of parts is returned through *parts_used.  lda, ldw, ldo in elements.
 extern "C" int hos_gemm_tc(const void* A, const void* W, void* out, int out_dtype, int M, int N, int K, int lda,
-                           int ldw, int ldo, int epilogue, float cap, int act, int k_splits, float* workspace,
+                           int ldw, int ldo, int epilogue, float cap, int act, const float* bias, int k_splits, float* workspace,
                            int reduce_now, int* parts_used, cudaStream_t stream) {
     if (parts_used) *parts_used = 1;
     if (M <= 0 || N <= 0) return 0;
@@ -980,6 +1013,9 @@ extern "C" int hos_gemm_tc(const void* A, const void* W, void* out, int out_dtyp
                    "16-byte aligned (K %d lda %d ldw %d)", K, lda, ldw);
     if (epilogue == kGEpiSoftcap && out_dtype != kF32) HOS_REFUSE("gemm_tc: the soft-cap epilogue writes 32-bit");
     if (epilogue == kGEpiGated && out_dtype != kBF16) HOS_REFUSE("gemm_tc: the gated epilogue writes bfloat16");
+    if (epilogue == kGEpiBias && (out_dtype != kBF16 || bias == nullptr))
+        HOS_REFUSE("gemm_tc: the bias epilogue writes bfloat16 and needs a bias");
+    if (epilogue < kGEpiNone || epilogue > kGEpiBias) HOS_REFUSE("gemm_tc: unknown epilogue %d", epilogue);
     if (k_splits < 1) k_splits = 1;
     const bool swap = M <= kSwapMaxRows;
     const bool pairs = !swap && M >= pair_min_rows() && pair_enabled();
@@ -987,7 +1023,7 @@ extern "C" int hos_gemm_tc(const void* A, const void* W, void* out, int out_dtyp
         HOS_REFUSE("gemm_tc: K splits need up to %d rows or the kernel on pairs of SMs, no epilogue and a workspace", kSwapMaxRows);
     const int w_rows = epilogue == kGEpiGated ? 2 * N : N;
     GemmParams p;
-    p.out = out; p.M = M; p.N = N; p.K = K; p.ldo = ldo; p.k_splits = k_splits; p.gate_rows = N; p.cap = cap; p.act = act;
+    p.out = out; p.M = M; p.N = N; p.K = K; p.ldo = ldo; p.k_splits = k_splits; p.gate_rows = N; p.cap = cap; p.act = act; p.bias = bias;
     CUtensorMap mm, mn;
     const int k_blocks = (K + GK - 1) / GK;
     if (k_splits > k_blocks) k_splits = p.k_splits = k_blocks;
@@ -1017,6 +1053,7 @@ extern "C" int hos_gemm_tc(const void* A, const void* W, void* out, int out_dtyp
         if (epilogue == kGEpiGated) return launch_pair<kGEpiGated, bf16>(mm, mn, p, m_tiles * ((N + 127) / 128), stream);
         const int tiles = m_tiles * ((N + 255) / 256);
         if (epilogue == kGEpiSoftcap) return launch_pair<kGEpiSoftcap, float>(mm, mn, p, tiles, stream);
+        if (epilogue == kGEpiBias) return launch_pair<kGEpiBias, bf16>(mm, mn, p, tiles, stream);
         if (out_dtype == kBF16) return launch_pair<kGEpiNone, bf16>(mm, mn, p, tiles, stream);
         return launch_pair<kGEpiNone, float>(mm, mn, p, tiles, stream);
     }
@@ -1031,6 +1068,7 @@ extern "C" int hos_gemm_tc(const void* A, const void* W, void* out, int out_dtyp
         if ((rc = make_map(&mn, W, w_rows, K, ldw, BN))) return rc;
         const int tiles = m_tiles * ((N + BN - 1) / BN);
         if (epilogue == kGEpiSoftcap) HOS_GO(256, kGEpiSoftcap, false, float, tiles);
+        if (epilogue == kGEpiBias) HOS_GO(256, kGEpiBias, false, bf16, tiles);
         if (out_dtype == kBF16) HOS_GO(256, kGEpiNone, false, bf16, tiles);
         HOS_GO(256, kGEpiNone, false, float, tiles);
     }
@@ -1068,6 +1106,12 @@ extern "C" int hos_gemm_tc(const void* A, const void* W, void* out, int out_dtyp
         if (bn == 32) HOS_GO(32, kGEpiSoftcap, true, float, tiles);
         if (bn == 64) HOS_GO(64, kGEpiSoftcap, true, float, tiles);
         HOS_GO(128, kGEpiSoftcap, true, float, tiles);
+    }
+    if (epilogue == kGEpiBias) {
+        if (bn == 16) HOS_GO(16, kGEpiBias, true, bf16, tiles);
+        if (bn == 32) HOS_GO(32, kGEpiBias, true, bf16, tiles);
+        if (bn == 64) HOS_GO(64, kGEpiBias, true, bf16, tiles);
+        HOS_GO(128, kGEpiBias, true, bf16, tiles);
     }
     if (out_dtype == kBF16) {
         if (bn == 16) HOS_GO(16, kGEpiNone, true, bf16, tiles);
@@ -1109,7 +1153,7 @@ extern "C" int hos_gemm_tc_qkv_rope(const void* A, const void* W, void* out, int
                         seq_slot == nullptr || seq_len_after == nullptr))
         HOS_REFUSE("gemm_tc_qkv_rope: the cache write needs kv heads, pages, a page table, slots and lengths");
     GemmParams p;
-    p.out = out; p.M = M; p.N = N; p.K = K; p.ldo = ldo; p.k_splits = 1; p.gate_rows = N; p.cap = 0.f; p.act = 0;
+    p.out = out; p.M = M; p.N = N; p.K = K; p.ldo = ldo; p.k_splits = 1; p.gate_rows = N; p.cap = 0.f; p.act = 0; p.bias = nullptr;
     p.rope.token_pos = token_pos; p.rope.token_seq = token_seq; p.rope.seq_slot = seq_slot;
     p.rope.seq_len_after = seq_len_after; p.rope.angles = reinterpret_cast<const float2*>(angles);
     p.rope.cache = PagedKV{k_pages, v_pages, page_table, table_stride, ring_pages, n_kv_heads, head_dim};

@@ -9,6 +9,8 @@
 // group_norm_gate: out[n][g][:] = o[n][g][:] / sqrt(mean_g(o^2) + eps) * w * act(gate[n][g][:]), the
 //   groups being heads (a weight shared by all heads) or the whole row (one group, a weight per column);
 //   act is the logistic function or x times it.  Statistics, weight and gate are 32-bit.
+// skip_gate_norm: y = (o + D[head] x) * z logistic(z), then in equal parts y / sqrt(mean_part(y^2) + eps) * w: a state
+//   mixer's heads with a skip from the input, the gate BEFORE the norm.
 #include "common.cuh"
 
 namespace hos {
@@ -135,13 +137,13 @@ template <typename TH>
 __global__ void __launch_bounds__(128)
 group_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_per_group,
                        const float* __restrict__ gate, long long gate_stride, int act, const int* __restrict__ token_seq,
-                       TH* __restrict__ out, float eps, int G, int gs) {
+                       TH* __restrict__ out, long long ldo, float eps, int G, int gs) {
     pdl_enter();
     __shared__ float scratch[32];
     const int n = blockIdx.x, g = blockIdx.y;
-    const size_t base = ((size_t)n * G + g) * gs;
+    const size_t base = ((size_t)n * G + g) * gs, obase = (size_t)n * ldo + (size_t)g * gs;
     if (token_seq != nullptr && token_seq[n] < 0) {        // padding: a defined row, nothing read
-        for (int d = threadIdx.x; d < gs; d += blockDim.x) out[base + d] = from_float<TH>(0.f);
+        for (int d = threadIdx.x; d < gs; d += blockDim.x) out[obase + d] = from_float<TH>(0.f);
         return;
     }
     float ss = 0.f;
@@ -156,7 +158,7 @@ group_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w,
     for (int d = threadIdx.x; d < gs; d += blockDim.x) {
         const float z = gt[d];
         const float s = 1.f / (1.f + expf(-z));
-        out[base + d] = from_float<TH>(o[base + d] * inv * wg[d] * (act == 1 ? z * s : s));
+        out[obase + d] = from_float<TH>(o[base + d] * inv * wg[d] * (act == 1 ? z * s : s));
     }
 }
 
@@ -166,14 +168,14 @@ template <typename TH>
 __global__ void __launch_bounds__(256)
 group_norm_gate_warp_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_per_group,
                             const float* __restrict__ gate, long long gate_stride, int act, const int* __restrict__ token_seq,
-                            TH* __restrict__ out, float eps, int G, int gs) {
+                            TH* __restrict__ out, long long ldo, float eps, int G, int gs) {
     pdl_enter();
     const int n = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bool pad = token_seq != nullptr && token_seq[n] < 0;
     for (int g = warp; g < G; g += 8) {
-        const size_t base = ((size_t)n * G + g) * gs;
+        const size_t base = ((size_t)n * G + g) * gs, obase = (size_t)n * ldo + (size_t)g * gs;
         if (pad) {
-            for (int d = lane * 4; d < gs; d += 128) store4(out + base + d, make_float4(0.f, 0.f, 0.f, 0.f));
+            for (int d = lane * 4; d < gs; d += 128) store4(out + obase + d, make_float4(0.f, 0.f, 0.f, 0.f));
             continue;
         }
         float ss = 0.f;
@@ -194,8 +196,71 @@ group_norm_gate_warp_kernel(const float* __restrict__ o, const float* __restrict
             r.y = v.y * inv * wv.y * (act == 1 ? z.y * s1 : s1);
             r.z = v.z * inv * wv.z * (act == 1 ? z.z * s2 : s2);
             r.w = v.w * inv * wv.w * (act == 1 ? z.w * s3 : s3);
-            store4(out + base + d, r);
+            store4(out + obase + d, r);
         }
+    }
+}
+
+// The state mixer's read-out o [N][I] (I = heads x vd), its input x (rows ldx apart), the gate z (rows ldz apart); the row
+// is normed in `parts` equal parts.  TPG threads take a part, NV times four numbers each in registers; NV = 0: any size,
+// the numbers formed again in the second pass.
+template <typename TH, int TPG, int NV>
+__global__ void __launch_bounds__(256)
+skip_gate_norm_kernel(const float* __restrict__ o, const float* __restrict__ x, long long ldx, const float* __restrict__ skip, int vd,
+                      const float* __restrict__ z, long long ldz, const float* __restrict__ w, float eps,
+                      const int* __restrict__ token_seq, TH* __restrict__ out, int N, int parts, int ps) {
+    pdl_enter();
+    __shared__ float scratch[32];
+    constexpr int PER_BLOCK = 256 / TPG;
+    const long long item = (long long)blockIdx.x * PER_BLOCK + threadIdx.x / TPG;
+    const int t = threadIdx.x % TPG;
+    if (TPG == 32 && item >= (long long)N * parts) return;               // a whole warp: no barrier is shared with others
+    const int n = (int)(item / parts), part = (int)(item % parts);
+    const size_t base = (size_t)n * parts * ps + (size_t)part * ps;
+    const float* xr = x + (size_t)n * ldx + (size_t)part * ps;
+    const float* zr = z + (size_t)n * ldz + (size_t)part * ps;
+    const float* wr = w + (size_t)part * ps;
+    const bool pad = token_seq[n] < 0;                                   // padding: a defined row
+    auto one = [&](int d) {
+        const float g = zr[d];
+        return fmaf(skip[(part * ps + d) / vd], xr[d], o[base + d]) * (g / (1.f + expf(-g)));
+    };
+    float ss = 0.f;
+    float4 v[NV > 0 ? NV : 1];
+    if (NV > 0) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int d = (t + i * TPG) * 4;
+            v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (d < ps && !pad) {
+                const float4 a = load4(o + base + d), b = load4(xr + d), g = load4(zr + d);
+                const float s = skip[(part * ps + d) / vd];              // vd is a multiple of four here
+                v[i].x = fmaf(s, b.x, a.x) * (g.x / (1.f + expf(-g.x)));
+                v[i].y = fmaf(s, b.y, a.y) * (g.y / (1.f + expf(-g.y)));
+                v[i].z = fmaf(s, b.z, a.z) * (g.z / (1.f + expf(-g.z)));
+                v[i].w = fmaf(s, b.w, a.w) * (g.w / (1.f + expf(-g.w)));
+                ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+            }
+        }
+    } else if (!pad) {
+        for (int d = t; d < ps; d += TPG) {
+            const float y = one(d);
+            ss = fmaf(y, y, ss);
+        }
+    }
+    ss = TPG == 32 ? warp_sum(ss) : block_sum(ss, scratch);
+    const float inv = 1.f / sqrtf(ss / (float)ps + eps);
+    if (NV > 0) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int d = (t + i * TPG) * 4;
+            if (d < ps) {
+                const float4 wv = load4(wr + d);
+                store4(out + base + d, make_float4(v[i].x * inv * wv.x, v[i].y * inv * wv.y, v[i].z * inv * wv.z, v[i].w * inv * wv.w));
+            }
+        }
+    } else {
+        for (int d = t; d < ps; d += TPG) out[base + d] = from_float<TH>(pad ? 0.f : one(d) * inv * wr[d]);
     }
 }
 
@@ -254,26 +319,57 @@ extern "C" int hos_cast_rows(const float* x, void* h, int h_dtype, long long n, 
 
 // o: [N][G][gs] float32.  w: [gs] if w_per_group (one weight for every group) else [G][gs].  gate: row n's gate of
 // group g, column d at gate[n * gate_stride + g * gs + d].  act: 0 logistic, 1 x times logistic.
+// out: G * gs numbers from the start of rows ldo apart.
 extern "C" int hos_group_norm_gate(const float* o, const float* w, int w_per_group, const float* gate, long long gate_stride,
-                                   int act, const int* token_seq, void* out, int out_dtype, float eps, int N, int G, int gs,
-                                   cudaStream_t stream) {
+                                   int act, const int* token_seq, void* out, int out_dtype, long long ldo, float eps, int N, int G,
+                                   int gs, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (G <= 0 || gs <= 0 || G > 65535) HOS_REFUSE("group_norm_gate: %d groups of %d", G, gs);
-    if (G >= 2 && gs <= 2048 && gs % 4 == 0 && gate_stride % 4 == 0 && (uintptr_t)o % 16 == 0 && (uintptr_t)gate % 16 == 0 &&
+    if (G >= 2 && gs <= 2048 && gs % 4 == 0 && gate_stride % 4 == 0 && ldo % 4 == 0 && (uintptr_t)o % 16 == 0 && (uintptr_t)gate % 16 == 0 &&
         (uintptr_t)w % 16 == 0 && (uintptr_t)out % 16 == 0) {
         if (out_dtype == kBF16)
             launch_pdl(group_norm_gate_warp_kernel<bf16>, dim3(N), dim3(256), 0, stream, o, w, w_per_group, gate, gate_stride,
-                       act, token_seq, (bf16*)out, eps, G, gs);
+                       act, token_seq, (bf16*)out, ldo, eps, G, gs);
         else
             launch_pdl(group_norm_gate_warp_kernel<float>, dim3(N), dim3(256), 0, stream, o, w, w_per_group, gate, gate_stride,
-                       act, token_seq, (float*)out, eps, G, gs);
+                       act, token_seq, (float*)out, ldo, eps, G, gs);
         return check_launch("group_norm_gate");
     }
     if (out_dtype == kBF16)
         launch_pdl(group_norm_gate_kernel<bf16>, dim3(N, G), dim3(128), 0, stream, o, w, w_per_group, gate, gate_stride, act,
-                   token_seq, (bf16*)out, eps, G, gs);
+                   token_seq, (bf16*)out, ldo, eps, G, gs);
     else
         launch_pdl(group_norm_gate_kernel<float>, dim3(N, G), dim3(128), 0, stream, o, w, w_per_group, gate, gate_stride, act,
-                   token_seq, (float*)out, eps, G, gs);
+                   token_seq, (float*)out, ldo, eps, G, gs);
     return check_launch("group_norm_gate");
+}
+
+// o: float32 [N][H * vd]; x: the rows' H * vd inputs from `x` on, ldx apart; skip: [H]; z: the rows' gates, ldz apart; w: [H * vd];
+// the row is normed in `parts` equal parts; out: [N][H * vd] of out_dtype.
+extern "C" int hos_skip_gate_norm(const float* o, const float* x, long long ldx, const float* skip, const float* z, long long ldz,
+                                  const float* w, float eps, const int* token_seq, void* out, int out_dtype, int N, int H, int vd,
+                                  int parts, cudaStream_t stream) {
+    if (N <= 0) return 0;
+    if (H <= 0 || vd <= 0 || parts <= 0 || (H * vd) % parts != 0) HOS_REFUSE("skip_gate_norm: %d heads of %d in %d parts", H, vd, parts);
+    const int ps = H * vd / parts;
+    const bool vec = ps % 4 == 0 && vd % 4 == 0 && ldx % 4 == 0 && ldz % 4 == 0 && (uintptr_t)o % 16 == 0 && (uintptr_t)x % 16 == 0 &&
+                     (uintptr_t)z % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)out % 16 == 0 && ps <= 256 * 4 * 16;
+    const long long items = (long long)N * parts;
+#define HOS_SGN(TH, TPG, NV)                                                                                         \
+    launch_pdl(skip_gate_norm_kernel<TH, TPG, NV>, dim3((unsigned)((items + 256 / TPG - 1) / (256 / TPG))), dim3(256), 0, stream, \
+               o, x, ldx, skip, vd, z, ldz, w, eps, token_seq, (TH*)out, N, parts, ps)
+#define HOS_SGN_T(TH)                                                                                                \
+    do {                                                                                                             \
+        if (!vec) HOS_SGN(TH, 256, 0);                                                                               \
+        else if (ps <= 128) HOS_SGN(TH, 32, 1);                                                                      \
+        else if (ps <= 512) HOS_SGN(TH, 32, 4);                                                                      \
+        else if (ps <= 2048) HOS_SGN(TH, 256, 2);                                                                    \
+        else if (ps <= 4096) HOS_SGN(TH, 256, 4);                                                                    \
+        else HOS_SGN(TH, 256, 16);                                                                                   \
+    } while (0)
+    if (out_dtype == kBF16) HOS_SGN_T(bf16);
+    else HOS_SGN_T(float);
+#undef HOS_SGN_T
+#undef HOS_SGN
+    return check_launch("skip_gate_norm");
 }

@@ -1,9 +1,10 @@
-// Linear recurrences with a matrix state per head, S [dim keys][vdim values] in 32-bit, one kernel for two rules:
+// Linear recurrences with a matrix state per head, S [dim keys][vdim values] in 32-bit, one kernel for three rules:
 //
-//   decay rule   S <- g S + k v^T                                o = S^T q     (g a constant per head)
-//   delta rule   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q  (g, beta per token and head)
+//   decay rule    S <- g S + beta k v^T                           o = S^T q     (g, beta per head, or per token and head)
+//   delta rule    S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q  (g, beta per token and head)
+//   channel rule  S <- diag(g) S + k v^T                          o = S^T q     (g per token, head and key channel)
 //
-// The read-out sees the current token's write.  A sequence's state lives per slot as S^T ([head][vdim][dim]: a
+// (The decay rule's beta may be left out; o may be multiplied by a constant.)  The read-out sees the current token's write.  A sequence's state lives per slot as S^T ([head][vdim][dim]: a
 // thread's run of rows of one column is contiguous), starts at zero (a sequence whose first row is position 0
 // ignores what the slot holds), and is carried from step to step.
 //
@@ -19,7 +20,11 @@
 //   row from the slot's state), x sigmoid(x) of it, q and k divided by their length per head
 //   (sqrt(sum + 1e-6)), q times dim^-1/2; beta = logistic(b); g = exp(-exp(A_log) softplus(a + dt_bias)).
 // conv_keep: the last taps - 1 inputs of every sequence go to the slot's state.
+// conv_act_rows: the short convolution with a bias and an activation on a run of columns, many tokens to a thread; with
+//   per-head step sizes: dt = softplus(raw + dt_bias) and the decay exp(-exp(A_log) dt) in the same launch.
+// channel_decay: logistic(W z + b)^(1 / tau) per key channel from a low-rank row z.
 #include "common.cuh"
+#include "short_conv.cuh"
 
 namespace hos {
 
@@ -84,14 +89,17 @@ rotate_rows_kernel(float* __restrict__ x, long long ld, int Hq, int Hk, int dim,
     }
 }
 
-template <int DR, int R, bool DELTA>
+enum ScanRule : int { kDecayRule = 0, kDeltaRule = 1, kChannelRule = 2 };
+
+template <int DR, int R, int RULE>
 __global__ void __launch_bounds__(256)
 state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, long long ld,
                   int aligned, int act_in_walk, const float* __restrict__ g, long long g_ld, const float* __restrict__ beta,
                   long long beta_ld, float* __restrict__ state, const int* __restrict__ token_pos,
                   const int* __restrict__ token_seq, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
                   float* __restrict__ out, int H, int Gk, int dim, int vdim, int CC, const float* __restrict__ rot_freq,
-                  int rot_dims, int rot_style, float k_mult) {
+                  int rot_dims, int rot_style, float k_mult, float o_mult) {
+    constexpr bool DELTA = RULE == kDeltaRule, CHANNEL = RULE == kChannelRule;
     pdl_enter();
     extern __shared__ __align__(16) float sm[];
     const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * CC;
@@ -105,9 +113,8 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
     const bool live = c < CC && col < vdim;
     const int dpad = R * (DR + kPad);
     // two buffers of staged tokens: while one chunk is walked the next one's rows are on their way (cp.async)
-    const int per_buf = kScanChunk * (2 * dpad + 2 * CC) + 2 * kScanChunk;      // q, k, v, o, g, beta
-    const int CC4 = (CC + 3) & ~3;
-    (void)CC4;
+    const int per_buf = kScanChunk * ((CHANNEL ? 3 : 2) * dpad + 2 * CC) + 2 * kScanChunk;      // q, k, (g,) v, o, g, beta
+    const bool v_scaled = RULE == kDecayRule && beta != nullptr;
 
     float S[DR];
     float* st = state + (((size_t)slot * H + head) * vdim + (live ? col : 0)) * dim + r * DR;
@@ -133,7 +140,8 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
     auto stage = [&](int t0, int nt, float* buf) {
         float* qs = buf;
         float* ks = qs + kScanChunk * dpad;
-        float* vs = ks + kScanChunk * dpad;
+        float* gk = ks + kScanChunk * dpad;          // the channel rule's decays, laid out as the keys
+        float* vs = ks + (CHANNEL ? 2 : 1) * kScanChunk * dpad;
         float* gs = vs + 2 * kScanChunk * CC;        // after v and o
         float* bs = gs + kScanChunk;
         if (aligned) {
@@ -143,6 +151,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                 const int at = t * dpad + d + (d / DR) * kPad;
                 cp_async16(qs + at, q + (size_t)(t0 + t) * ld + kh * dim + d);
                 cp_async16(ks + at, k + (size_t)(t0 + t) * ld + kh * dim + d);
+                if (CHANNEL) cp_async16(gk + at, g + (size_t)(t0 + t) * g_ld + head * dim + d);
             }
         } else {
             for (int idx = threadIdx.x; idx < nt * dim; idx += blockDim.x) {
@@ -150,6 +159,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                 const int at = t * dpad + d + (d / DR) * kPad;
                 cp_async4(qs + at, q + (size_t)(t0 + t) * ld + kh * dim + d);
                 cp_async4(ks + at, k + (size_t)(t0 + t) * ld + kh * dim + d);
+                if (CHANNEL) cp_async4(gk + at, g + (size_t)(t0 + t) * g_ld + head * dim + d);
             }
         }
         const int ncol = min(CC, vdim - col0);
@@ -158,8 +168,8 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
             cp_async4(vs + t * CC + cc, v + (size_t)(t0 + t) * ld + head * vdim + col0 + cc);
         }
         if (threadIdx.x < nt) {
-            cp_async4(gs + threadIdx.x, g + (size_t)(t0 + threadIdx.x) * g_ld + head);
-            if (DELTA) cp_async4(bs + threadIdx.x, beta + (size_t)(t0 + threadIdx.x) * beta_ld + head);
+            if (!CHANNEL) cp_async4(gs + threadIdx.x, g + (size_t)(t0 + threadIdx.x) * g_ld + head);
+            if (DELTA || v_scaled) cp_async4(bs + threadIdx.x, beta + (size_t)(t0 + threadIdx.x) * beta_ld + head);
         }
         cp_async_commit_all();
     };
@@ -198,7 +208,8 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
             }
             __syncthreads();
         }
-        float* vs = ks + kScanChunk * dpad;
+        float* gk = ks + kScanChunk * dpad;
+        float* vs = ks + (CHANNEL ? 2 : 1) * kScanChunk * dpad;
         float* os = vs + kScanChunk * CC;
         float* gs = os + kScanChunk * CC;
         float* bs = gs + kScanChunk;
@@ -210,9 +221,11 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                 if (t >= nt) continue;
                 const float4* k4 = (const float4*)(ks + t * dpad + r * (DR + kPad));
                 const float4* q4 = (const float4*)(qs + t * dpad + r * (DR + kPad));
-                const float gt = gs[t];
+                const float4* g4 = (const float4*)(gk + t * dpad + r * (DR + kPad));
+                const float gt = CHANNEL ? 0.f : gs[t];
                 float u = c < CC ? vs[t * CC + c] : 0.f;
-                if (!DELTA && act_in_walk) u = silu_precise(u);      // single tokens: the activation rides here
+                if (RULE == kDecayRule && act_in_walk) u = silu_precise(u);      // single tokens: the activation rides here
+                if (v_scaled) u *= bs[t];
                 if (DELTA) {
                     float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;       // four chains, not one of DR links
 #pragma unroll
@@ -233,7 +246,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
 #pragma unroll
                 for (int i = 0; i < DR / 4; ++i) {
                     float4 kk = k4[i], qq = q4[i];
-                    if (!DELTA && act_in_walk) {
+                    if (RULE == kDecayRule && act_in_walk) {
                         kk = make_float4(silu_precise(kk.x), silu_precise(kk.y), silu_precise(kk.z), silu_precise(kk.w));
                         qq = make_float4(silu_precise(qq.x), silu_precise(qq.y), silu_precise(qq.z), silu_precise(qq.w));
                     }
@@ -242,6 +255,12 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                         S[4 * i + 1] = fmaf(kk.y, u, S[4 * i + 1]);
                         S[4 * i + 2] = fmaf(kk.z, u, S[4 * i + 2]);
                         S[4 * i + 3] = fmaf(kk.w, u, S[4 * i + 3]);
+                    } else if (CHANNEL) {
+                        const float4 gg = g4[i];
+                        S[4 * i] = fmaf(gg.x, S[4 * i], kk.x * u);
+                        S[4 * i + 1] = fmaf(gg.y, S[4 * i + 1], kk.y * u);
+                        S[4 * i + 2] = fmaf(gg.z, S[4 * i + 2], kk.z * u);
+                        S[4 * i + 3] = fmaf(gg.w, S[4 * i + 3], kk.w * u);
                     } else {
                         S[4 * i] = fmaf(gt, S[4 * i], kk.x * u);
                         S[4 * i + 1] = fmaf(gt, S[4 * i + 1], kk.y * u);
@@ -261,7 +280,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                 float acc = part[t];
 #pragma unroll
                 for (int o = 1; o < R; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-                if (r == 0 && c < CC) os[t * CC + c] = acc;
+                if (r == 0 && c < CC) os[t * CC + c] = acc * o_mult;
             }
         }
         __syncthreads();
@@ -279,8 +298,6 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
             if (r * DR + i < dim) st[i] = S[i];
     }
 }
-
-constexpr int kMaxTaps = 16;
 
 // raw: float32 [N][ld]: q (Gk * dim) | k (Gk * dim) | v (H * vdim) | b (H) | a (H) | ... ; conv_w: [C][taps] over
 // the first C = 2 Gk dim + H vdim columns; conv_state: [slots][taps - 1][C], row j the input taps - 1 - j tokens back.
@@ -313,15 +330,7 @@ conv_prep_kernel(const float* __restrict__ raw, long long ld, const float* __res
     // inputs (a thread the channels it convolves): they move on by one here instead of in a launch of their own
     float* keep_w = keep_here != nullptr ? keep_here + (size_t)seq_slot[seq] * (taps - 1) * C : nullptr;
     for (int ch = threadIdx.x; ch < C; ch += blockDim.x) {
-        float acc = 0.f;
-        for (int j = 0; j < taps; ++j) {
-            const int src = n - (taps - 1) + j;          // the row of this step that holds the input, if it is one
-            float x = 0.f;
-            if (src >= r0) x = raw[(size_t)src * ld + ch];
-            else if (!fresh) x = keep[(size_t)((taps - 1) + (src - r0)) * C + ch];
-            acc = fmaf(conv_w[(size_t)ch * taps + j], x, acc);
-            if (keep_w != nullptr && j >= 1) keep_w[(size_t)(j - 1) * C + ch] = x;      // row j - 1 is read before this
-        }
+        const float acc = short_conv(raw + ch, ld, 0.f, conv_w, taps, keep, keep_w, C, ch, n, r0, fresh);
         const float y = silu_precise(acc);
         if (ch < QK) qk[ch] = y;
         else arow[ch] = y;
@@ -348,27 +357,151 @@ conv_prep_kernel(const float* __restrict__ raw, long long ld, const float* __res
     }
 }
 
-__global__ void conv_keep_kernel(const float* __restrict__ raw, long long ld, int taps, float* __restrict__ conv_state,
-                                 const int* __restrict__ token_pos, const int* __restrict__ token_seq,
-                                 const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot, int C) {
+// act(x): 0 none, 1 x logistic(x)
+__device__ __forceinline__ float conv_act(float x, int act) { return act == 1 ? silu_precise(x) : x; }
+
+constexpr int kConvTokens = 16;      // consecutive rows that a thread of conv_act_rows walks
+
+// out[n][c] = act(sum_j w[c][j] u_(n - taps + 1 + j)[c] + bias[c]) for C columns of 32-bit rows.  A thread takes VEC channels
+// of up to kConvTokens consecutive rows (one where the sequences bring single tokens) and keeps the inputs in sight in
+// registers, so that a column is read once; rows of a sequence's start, or of this run's, fetch them from the rows
+// before or from the slot's kept inputs.  The last block of a row run takes the per-head step sizes: dt = softplus(raw
+// + dt_bias), decay = exp(-exp(A_log) dt).
+template <int TAPS, int VEC>
+__global__ void __launch_bounds__(128)
+conv_act_rows_kernel(const float* raw, long long ld, const float* __restrict__ w, const float* __restrict__ bias, int taps_rt,
+                     const float* keep_all, float* keep_w_all, int act, const int* __restrict__ token_pos,
+                     const int* __restrict__ token_seq, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
+                     float* __restrict__ out, int N, int C, int run, int conv_blocks, const float* __restrict__ dt_raw,
+                     const float* __restrict__ dt_bias, const float* __restrict__ a_log, float* __restrict__ dt_out,
+                     float* __restrict__ g_out, int H) {
     pdl_enter();
-    const int seq = blockIdx.y;
-    const int ch = blockIdx.x * blockDim.x + threadIdx.x;
-    const int r0 = cu_seqlens[seq], r1 = cu_seqlens[seq + 1];
-    if (ch >= C || r1 <= r0 || token_seq[r0] < 0) return;
-    const bool fresh = token_pos[r0] == 0;
-    float* keep = conv_state + (size_t)seq_slot[seq] * (taps - 1) * C;
-    float nv[kMaxTaps];
+    const int n0 = blockIdx.y * run, n1 = min(N, n0 + run);
+    if ((int)blockIdx.x >= conv_blocks) {
+        for (int i = threadIdx.x; i < (n1 - n0) * H; i += blockDim.x) {
+            const int n = n0 + i / H, h = i % H;
+            float dt = 0.f, g = 1.f;
+            if (token_seq[n] >= 0) {
+                const float a = dt_raw[(size_t)n * ld + h] + dt_bias[h];
+                dt = a > 20.f ? a : log1pf(expf(a));
+                g = expf(-expf(a_log[h]) * dt);
+            }
+            dt_out[(size_t)n * H + h] = dt;
+            g_out[(size_t)n * H + h] = g;
+        }
+        return;
+    }
+    const int ch = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (ch >= C) return;
+    const int taps = TAPS > 0 ? TAPS : taps_rt;
+    constexpr int MAXT = TAPS > 0 ? TAPS : kMaxTaps;
+    float wr[VEC][MAXT], win[VEC][MAXT], b[VEC];
 #pragma unroll
-    for (int j = 0; j < kMaxTaps; ++j) {
-        if (j < taps - 1) {
-            const int src = r1 - (taps - 1) + j;
-            nv[j] = src >= r0 ? raw[(size_t)src * ld + ch] : (fresh ? 0.f : keep[(size_t)((taps - 1) + (src - r0)) * C + ch]);
+    for (int v = 0; v < VEC; ++v) {
+        b[v] = bias != nullptr ? bias[ch + v] : 0.f;
+#pragma unroll
+        for (int j = 0; j < MAXT; ++j) wr[v][j] = j < taps ? w[(size_t)(ch + v) * taps + j] : 0.f;
+    }
+    auto load = [&](const float* p, float (&x)[VEC]) {
+        if (VEC == 4) {
+            const float4 t = *(const float4*)p;
+            x[0] = t.x; x[VEC > 1 ? 1 : 0] = t.y; x[VEC > 2 ? 2 : 0] = t.z; x[VEC > 3 ? 3 : 0] = t.w;
+        } else {
+            x[0] = *p;
+        }
+    };
+    auto store = [&](float* p, const float (&x)[VEC]) {
+        if (VEC == 4) *(float4*)p = make_float4(x[0], x[VEC > 1 ? 1 : 0], x[VEC > 2 ? 2 : 0], x[VEC > 3 ? 3 : 0]);
+        else *p = x[0];
+    };
+    int last_seq = -2;
+    for (int n = n0; n < n1; ++n) {
+        const int seq = token_seq[n];
+        float y[VEC];
+        if (seq < 0) {
+#pragma unroll
+            for (int v = 0; v < VEC; ++v) y[v] = 0.f;
+            store(out + (size_t)n * C + ch, y);
+            last_seq = -2;
+            continue;
+        }
+        if (seq != last_seq) {                   // the inputs before this row: win[.][j] of place j - 1 after the shift below
+            const int r0 = cu_seqlens[seq];
+            const bool fresh = token_pos[r0] == 0;
+            const float* keep = keep_all + (size_t)seq_slot[seq] * (taps - 1) * C + ch;
+#pragma unroll
+            for (int j = 1; j < MAXT; ++j) {
+                if (j >= taps) continue;
+                const int src = n - taps + j;
+                float x[VEC];
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) x[v] = 0.f;
+                if (src >= r0) load(raw + (size_t)src * ld + ch, x);
+                else if (!fresh) load(keep + (size_t)((taps - 1) + (src - r0)) * C, x);
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) win[v][j] = x[v];
+            }
+            last_seq = seq;
+        }
+        float x[VEC];
+        load(raw + (size_t)n * ld + ch, x);
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) {
+            float acc = 0.f;
+#pragma unroll
+            for (int j = 0; j < MAXT; ++j) {
+                if (j + 1 < taps) win[v][j] = win[v][j + 1 < MAXT ? j + 1 : j];
+                else if (j + 1 == taps) win[v][j] = x[v];
+                if (j < taps) acc = fmaf(wr[v][j], win[v][j], acc);
+            }
+            y[v] = conv_act(acc + b[v], act);
+        }
+        store(out + (size_t)n * C + ch, y);
+        if (keep_w_all != nullptr) {             // single tokens: the kept inputs (the last taps - 1 in sight) move on here
+            float* keep = keep_w_all + (size_t)seq_slot[seq] * (taps - 1) * C + ch;
+#pragma unroll
+            for (int j = 1; j < MAXT; ++j) {
+                if (j >= taps) continue;
+                float k[VEC];
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) k[v] = win[v][j];
+                store(keep + (size_t)(j - 1) * C, k);
+            }
         }
     }
+}
+
+// out[n][c] = logistic(z)^(1 / tau), z = sum_r w[c][r] low[n][r] + b[c]: exp(-softplus(-z) / tau), 32-bit.  A block takes
+// kDecayRows rows and 128 channels; the low-rank rows are staged in shared memory.
+constexpr int kDecayRows = 8;
+__global__ void __launch_bounds__(128)
+channel_decay_kernel(const float* __restrict__ low, long long ld, const float* __restrict__ w, const float* __restrict__ b,
+                     int rank, float inv_tau, float* __restrict__ out, int N, int C) {
+    pdl_enter();
+    extern __shared__ float low_s[];             // [kDecayRows][rank]
+    const int n0 = blockIdx.y * kDecayRows, rows = min(kDecayRows, N - n0);
+    for (int i = threadIdx.x; i < kDecayRows * rank; i += blockDim.x) {
+        const int r = i / rank;
+        low_s[i] = r < rows ? low[(size_t)(n0 + r) * ld + i % rank] : 0.f;
+    }
+    __syncthreads();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= C) return;
+    float acc[kDecayRows];
 #pragma unroll
-    for (int j = 0; j < kMaxTaps; ++j)
-        if (j < taps - 1) keep[(size_t)j * C + ch] = nv[j];
+    for (int r = 0; r < kDecayRows; ++r) acc[r] = b[c];
+    for (int k = 0; k < rank; ++k) {
+        const float wv = w[(size_t)k * C + c];   // [rank][C]: neighbouring channels side by side
+#pragma unroll
+        for (int r = 0; r < kDecayRows; ++r) acc[r] = fmaf(wv, low_s[r * rank + k], acc[r]);
+    }
+#pragma unroll
+    for (int r = 0; r < kDecayRows; ++r) {
+        if (r >= rows) break;
+        const float z = acc[r];
+        const float sp = fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)));      // softplus(-z) without overflow
+        out[(size_t)(n0 + r) * C + c] = expf(-sp * inv_tau);
+    }
 }
 
 }  // namespace hos
@@ -376,13 +509,14 @@ __global__ void conv_keep_kernel(const float* __restrict__ raw, long long ld, in
 using namespace hos;
 
 // q, k: rows of Gk heads of `dim` numbers; v: rows of H heads of `vdim`; all float32 with `ld` numbers between rows.
-// g: [.][H] with g_ld between rows (0: one row of constants).  beta: null for the decay rule.  state: [slots][H][vdim][dim].
+// rule: 0 decay, 1 delta, 2 channel.  g: [.][H] (channel rule: [.][H * dim]) with g_ld between rows (0: one row of constants).
+// beta: the delta rule's; with the decay rule, if given, the factor on v; o_mult: a constant on the read-outs.  state: [slots][H][vdim][dim].
 // out: float32 [N][H][vdim].  act_in_walk (decay rule only, meant for single-token steps): q, k, v are taken through
 // x logistic(x) as they are read, instead of by hos_act_rows before.  rot_freq ([rot_dims / 2], or null), rot_style, k_mult:
 // the staged q and k are turned by their tokens' positions and the keys multiplied, as hos_rotate_rows would have done
 // before (meant for single-token steps; it follows the rows as they are, so it does not go with act_in_walk).
-extern "C" int hos_state_scan(const float* q, const float* k, const float* v, long long ld, int act_in_walk, const float* g,
-                              long long g_ld, const float* beta, long long beta_ld, float* state, const int* token_pos,
+extern "C" int hos_state_scan(const float* q, const float* k, const float* v, long long ld, int act_in_walk, int rule,
+                              float o_mult, const float* g, long long g_ld, const float* beta, long long beta_ld, float* state, const int* token_pos,
                               const int* token_seq, const int* cu_seqlens, const int* seq_slot, float* out, int n_rows,
                               int n_seqs, int H, int Gk, int dim, int vdim, const float* rot_freq, int rot_dims, int rot_style,
                               float k_mult, cudaStream_t stream) {
@@ -410,11 +544,15 @@ extern "C" int hos_state_scan(const float* q, const float* k, const float* v, lo
         while (CC * R > 64 && (long long)n_seqs * H * ((vdim + CC - 1) / CC) < 2 * sm_count_cached()) CC = (CC + 1) / 2;
     const int threads = (CC * R + 31) / 32 * 32;
     const int dpad = R * (DR + kPad);
-    const size_t smem = (size_t)2 * (2 * kScanChunk * dpad + 2 * kScanChunk * CC + 2 * kScanChunk) * sizeof(float);
-    const int aligned = (dim % 4 == 0 && ld % 4 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)k % 16 == 0) ? 1 : 0;
+    if (rule < kDecayRule || rule > kChannelRule || (rule == kDeltaRule && beta == nullptr) || (rule == kChannelRule && beta != nullptr))
+        HOS_REFUSE("state_scan: rule %d and its inputs do not fit", rule);
+    if (rule == kChannelRule && Gk != H) HOS_REFUSE("state_scan: the channel rule has a key head per head");
+    const int wide_rows = rule == kChannelRule ? 3 : 2;
+    const size_t smem = (size_t)2 * (wide_rows * kScanChunk * dpad + 2 * kScanChunk * CC + 2 * kScanChunk) * sizeof(float);
+    const int aligned = (dim % 4 == 0 && ld % 4 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)k % 16 == 0 &&
+                         (rule != kChannelRule || (g_ld % 4 == 0 && (uintptr_t)g % 16 == 0))) ? 1 : 0;
     const dim3 grid(n_seqs, H, (vdim + CC - 1) / CC);
-    const bool delta = beta != nullptr;
-    if (delta && act_in_walk) HOS_REFUSE("state_scan: the activation in the walk is the decay rule's");
+    if (rule != kDecayRule && act_in_walk) HOS_REFUSE("state_scan: the activation in the walk is the decay rule's");
     if (smem > 200 * 1024) HOS_REFUSE("state_scan: heads of %d x %d do not fit a block's shared memory", dim, vdim);
 #define HOS_SCAN(DRv, Rv, DL)                                                                                        \
     do {                                                                                                             \
@@ -422,12 +560,13 @@ extern "C" int hos_state_scan(const float* q, const float* k, const float* v, lo
             cudaFuncSetAttribute(state_scan_kernel<DRv, Rv, DL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         launch_pdl(state_scan_kernel<DRv, Rv, DL>, grid, dim3(threads), smem, stream, q, k, v, ld, aligned, act_in_walk, g, g_ld, beta, \
                    beta_ld, state, token_pos, token_seq, cu_seqlens, seq_slot, out, H, Gk, dim, vdim, CC, rot_freq,  \
-                   rot_dims, rot_style, k_mult);                                                                     \
+                   rot_dims, rot_style, k_mult, o_mult);                                                             \
     } while (0)
 #define HOS_SCAN_D(DRv, Rv)                                                                                          \
     do {                                                                                                             \
-        if (delta) HOS_SCAN(DRv, Rv, true);                                                                          \
-        else HOS_SCAN(DRv, Rv, false);                                                                               \
+        if (rule == kDeltaRule) HOS_SCAN(DRv, Rv, kDeltaRule);                                                       \
+        else if (rule == kChannelRule) HOS_SCAN(DRv, Rv, kChannelRule);                                              \
+        else HOS_SCAN(DRv, Rv, kDecayRule);                                                                          \
     } while (0)
     // the shapes that the choice of DR above can give: (4; 1, 2, 4), (8; 4 to 32), (16; 32), (32; 32)
     if (DR == 4 && R == 1) HOS_SCAN_D(4, 1);
@@ -490,7 +629,60 @@ extern "C" int hos_conv_keep(const float* raw, long long ld, int taps, float* co
                              cudaStream_t stream) {
     if (n_seqs <= 0 || taps <= 1) return 0;
     if (taps > kMaxTaps) HOS_REFUSE("conv_keep: %d taps are outside 1..%d", taps, kMaxTaps);
-    launch_pdl(conv_keep_kernel, dim3((C + 127) / 128, n_seqs), dim3(128), 0, stream, raw, ld, taps, conv_state, token_pos,
-               token_seq, cu_seqlens, seq_slot, C);
+    launch_pdl(short_conv_keep_kernel, dim3((C + 127) / 128, n_seqs), dim3(128), 0, stream, raw, ld, (const float*)nullptr, taps,
+               conv_state, token_pos, token_seq, cu_seqlens, seq_slot, C);
     return check_launch("conv_keep");
+}
+
+// raw: the rows from the first convolved column on, ld apart; w: [C][taps]; bias: [C] or null; act: 0 none, 1 x logistic(x);
+// conv_state: [slots][taps - 1][C]; out: float32 [N][C].  single: 1 where every sequence of the step brings exactly one token:
+// the kept inputs then move on inside this launch and hos_conv_keep is not needed.  dt_raw (or null): the rows from the
+// first step-size column on, H of them, ld apart: dt_out [N][H] = softplus(dt_raw + dt_bias), g_out [N][H] = exp(-exp(a_log) dt).
+extern "C" int hos_conv_act_rows(const float* raw, long long ld, const float* w, const float* bias, int taps, float* conv_state,
+                                 int act, const int* token_pos, const int* token_seq, const int* cu_seqlens, const int* seq_slot,
+                                 float* out, int N, int C, int single, const float* dt_raw, const float* dt_bias, const float* a_log,
+                                 float* dt_out, float* g_out, int H, cudaStream_t stream) {
+    if (N <= 0 || C <= 0) return 0;
+    if (taps < 1 || taps > kMaxTaps) HOS_REFUSE("conv_act_rows: %d taps are outside 1..%d", taps, kMaxTaps);
+    if (act != 0 && act != 1) HOS_REFUSE("conv_act_rows: unknown activation %d", act);
+    if (dt_raw != nullptr && (dt_bias == nullptr || a_log == nullptr || dt_out == nullptr || g_out == nullptr || H <= 0))
+        HOS_REFUSE("conv_act_rows: step sizes need their bias, their rates and two outputs");
+    const bool vec = taps >= 2 && taps <= 4 && C % 4 == 0 && ld % 4 == 0 && (uintptr_t)raw % 16 == 0 && (uintptr_t)out % 16 == 0 &&
+                     (uintptr_t)conv_state % 16 == 0;
+    const int per_block = 128 * (vec ? 4 : 1);
+    const int conv_blocks = (C + per_block - 1) / per_block;
+    // runs as long as leave every SM several blocks; a single-token step's rows are sequences of their own
+    int run = 1;
+    while (!single && run < kConvTokens && (long long)((N + 2 * run - 1) / (2 * run)) * conv_blocks >= 4 * sm_count_cached()) run *= 2;
+    const dim3 grid(conv_blocks + (dt_raw != nullptr ? 1 : 0), (N + run - 1) / run);
+    if (grid.y > 65535) HOS_REFUSE("conv_act_rows: %d rows are more than one launch takes", N);
+    float* keep_w = single && taps > 1 ? conv_state : nullptr;
+#define HOS_CAR(T, V)                                                                                                \
+    launch_pdl(conv_act_rows_kernel<T, V>, grid, dim3(128), 0, stream, raw, ld, w, bias, taps, (const float*)conv_state, keep_w, \
+               act, token_pos, token_seq, cu_seqlens, seq_slot, out, N, C, run, conv_blocks, dt_raw, dt_bias, a_log, dt_out, \
+               g_out, H)
+#define HOS_CAR_V(T)                                                                                                 \
+    do {                                                                                                             \
+        if (vec) HOS_CAR(T, 4);                                                                                      \
+        else HOS_CAR(T, 1);                                                                                          \
+    } while (0)
+    if (taps == 2) HOS_CAR_V(2);
+    else if (taps == 3) HOS_CAR_V(3);
+    else if (taps == 4) HOS_CAR_V(4);
+    else HOS_CAR(0, 1);
+#undef HOS_CAR_V
+#undef HOS_CAR
+    return check_launch("conv_act_rows");
+}
+
+// low: the rows' low-rank numbers from column 0 of `low` on, ld apart; w: [rank][C] (transposed), b: [C]; out: float32 [N][C].
+extern "C" int hos_channel_decay(const float* low, long long ld, const float* w, const float* b, int rank, float tau, float* out,
+                                 int N, int C, cudaStream_t stream) {
+    if (N <= 0 || C <= 0) return 0;
+    if (rank <= 0 || rank > 1024 || !(tau > 0.f)) HOS_REFUSE("channel_decay: a rank of %d and tau %g", rank, tau);
+    const dim3 grid((C + 127) / 128, (N + kDecayRows - 1) / kDecayRows);
+    if (grid.y > 65535) HOS_REFUSE("channel_decay: %d rows are more than one launch takes", N);
+    launch_pdl(channel_decay_kernel, grid, dim3(128), (size_t)kDecayRows * rank * sizeof(float), stream, low, ld, w, b, rank,
+               1.f / tau, out, N, C);
+    return check_launch("channel_decay");
 }

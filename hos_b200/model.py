@@ -27,6 +27,7 @@ class Model:
         self.final_norm = part_impl("norm", plan.final_norm.kind)(plan.final_norm, rt)
         self.head = part_impl("head", plan.head.kind)(plan.head, rt)
         self.schedule = list(plan.schedule)
+        self.streams = plan.streams
         self.graph_safe = all(p.graph_safe for p in self.all_parts())
 
     def all_parts(self):
@@ -63,8 +64,8 @@ class Model:
                             max_slots, chunk_tokens, self.embedding.state_needs())
 
     def hidden(self, step: StepInfo, cache: CacheManager, tap: Optional[list] = None) -> torch.Tensor:
-        """The residual stream after the last entry of the run order, float32 [N, width].  With `tap`
-        (a list) a copy of the residual stream is appended after the embedding and after every entry
+        """The residual stream after the last entry of the run order, float32 [N, streams * width].  With `tap`
+        (a list) a copy of the residual stream (the sum of its streams) is appended after the embedding and after every entry
         of the run order: what tells where two paths begin to differ (the reference keeps such a tap
         per layer, src/forward.rs:45-103)."""
         return self._run_layers(step, cache, tap, None)[0]
@@ -77,7 +78,7 @@ class Model:
         else:
             x = self.embedding.forward(step.tokens, step)
         if tap is not None:
-            tap.append(x.clone())
+            tap.append(self._sum(x))
         h = None
         for i, call in enumerate(self.schedule):
             layer = self.layers[call.layer]
@@ -92,10 +93,16 @@ class Model:
                     next_norm = nxt.entry_norm() if nxt.chains else None
                 h = layer.forward(x, step, cache.stores[i], h_in=h, next_norm=next_norm)
             if tap is not None:
-                tap.append(x.clone())
+                tap.append(self._sum(x))
         if last_norm is None:
             return x, None
-        return x, (h if h is not None else last_norm.forward(x))
+        if h is None:
+            h = last_norm.forward(self._sum(x) if self.streams > 1 else x)
+        return x, h
+
+    def _sum(self, x: torch.Tensor) -> torch.Tensor:
+        """A copy of the residual stream's rows, or, where it is several streams, their sum: float32 [N, width]."""
+        return x.clone() if self.streams == 1 else ops.stream_sums(x, self.streams)
 
     def step_logits(self, step: StepInfo, cache: CacheManager) -> torch.Tensor:
         """float32 [N, vocab]: the logits of every row of the step (what a decoding step wants): no rows are
@@ -107,8 +114,11 @@ class Model:
         """float32 [len(rows), vocab] for the given rows of the residual stream."""
         if rows.shape[0] == 0:
             return torch.empty((0, self.plan.vocab_size), dtype=torch.float32, device=x.device)
-        picked = torch.empty((rows.shape[0], x.shape[1]), dtype=torch.float32, device=x.device)
-        ops.gather_rows(x, rows, picked)
+        if self.streams > 1:
+            picked = ops.stream_sums(x, self.streams, rows)
+        else:
+            picked = torch.empty((rows.shape[0], x.shape[1]), dtype=torch.float32, device=x.device)
+            ops.gather_rows(x, rows, picked)
         return self.head.forward(self.final_norm.forward(picked))
 
 

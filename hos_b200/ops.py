@@ -21,9 +21,10 @@ from .errors import KernelError
 
 F32, BF16 = 0, 1
 PAGE_TOKENS = 64
-EPI_NONE, EPI_SOFTCAP, EPI_GATED = 0, 1, 2
+EPI_NONE, EPI_SOFTCAP, EPI_GATED, EPI_BIAS = 0, 1, 2, 3
 ACT_GELU_TANH, ACT_SILU, ACT_CLAMPED_SWISH = 0, 1, 2
 ACTIVATIONS = {"gelu_tanh": ACT_GELU_TANH, "silu": ACT_SILU}
+BIAS_ACTIVATIONS = {"none": 0, "gelu_erf": 1}          # what EPI_BIAS applies after the bias
 # the clamped form as the products' gated epilogues know it: g logistic(SWISH_ALPHA g) (u + SWISH_SHIFT), the limit a parameter
 SWISH_ALPHA, SWISH_SHIFT = 1.702, 1.0
 ROPE_STYLES = {"rotate_half": 0, "interleaved": 1}
@@ -289,15 +290,16 @@ class PagedKVArgs:
 
 # ---- element-wise and norms ------------------------------------------------------------
 
-def embed(tokens: torch.Tensor, table: torch.Tensor, scale: float, out: torch.Tensor) -> None:
+def embed(tokens: torch.Tensor, table: torch.Tensor, scale: float, out: torch.Tensor, copies: int = 1) -> None:
+    """out[n] = `copies` copies of table[token] * scale, side by side."""
     _check(tokens, "tokens", torch.int32, 1)
     _check(table, "embedding table", None, 2)
     _check(out, "embedding output", torch.float32, 2)
-    n, d = out.shape
-    if tokens.shape[0] != n or table.shape[1] != d:
+    n, d = out.shape[0], table.shape[1]
+    if tokens.shape[0] != n or out.shape[1] != copies * d:
         raise KernelError("embed: sizes of tokens, table and output disagree")
     core().call("hos_embed", _ptr(tokens), _ptr(table), dtype_code(table.dtype), float(scale),
-                _ptr(out), n, d, _stream())
+                _ptr(out), n, d, int(copies), _stream())
 
 
 def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, add_one: bool, out: torch.Tensor) -> None:
@@ -419,9 +421,9 @@ def gather_rows(x: torch.Tensor, idx: torch.Tensor, out: torch.Tensor) -> None:
 # ---- matrix product (plain) --------------------------------------------------------------
 
 def gemm_plain(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = EPI_NONE,
-               cap: float = 0.0, act: int = 0) -> None:
+               cap: float = 0.0, act: int = 0, bias: Optional[torch.Tensor] = None) -> None:
     """out[M, N] = a[M, K] . w[N, K]^T with 32-bit accumulation on the CUDA cores.
-    Gated epilogue: w has 2N rows (gate rows, then up rows), out = act(gate) * up."""
+    Gated epilogue: w has 2N rows (gate rows, then up rows), out = act(gate) * up.  Bias epilogue: act(product + bias)."""
     _check(a, "left operand", None, 2)
     _check(w, "weight", None, 2)
     _check(out, "product", None, 2)
@@ -431,7 +433,7 @@ def gemm_plain(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: in
     if out.shape[0] != m or w.shape != (want_rows, k):
         raise KernelError(f"gemm: sizes disagree: a {tuple(a.shape)} w {tuple(w.shape)} out {tuple(out.shape)}")
     core().call("hos_gemm_plain", _ptr(a), dtype_code(a.dtype), _ptr(w), dtype_code(w.dtype),
-                _ptr(out), dtype_code(out.dtype), m, n, k, k, k, n, epilogue, float(cap), act,
+                _ptr(out), dtype_code(out.dtype), m, n, k, k, k, n, epilogue, float(cap), act, _ptr(bias),
                 _stream())
 
 
@@ -877,38 +879,116 @@ def cast_rows(x: torch.Tensor, h: torch.Tensor) -> None:
     mixers().call("hos_cast_rows", _ptr(x), _ptr(h), dtype_code(h.dtype), x.numel(), _stream())
 
 
+def _at(t: torch.Tensor, col: int):
+    """The address of a row-major matrix's column `col`."""
+    return ctypes.c_void_p(t.data_ptr() + col * t.element_size())
+
+
 def group_norm_gate(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, gate_col: int, act: int, token_seq,
-                    out: torch.Tensor, eps: float, groups: int, group_size: int) -> None:
-    """out[n, g, :] = o[n, g, :] / rms * w * act(gate[n, gate_col + g * group_size + :]); w: [group_size] (shared by
-    the groups) or [groups * group_size]."""
+                    out: torch.Tensor, eps: float, groups: int, group_size: int, out_col: int = 0) -> None:
+    """out[n, out_col + (g, :)] = o[n, g, :] / rms * w * act(gate[n, gate_col + g * group_size + :]); w: [group_size]
+    (shared by the groups) or [groups * group_size]."""
     _check(o, "mixer output", torch.float32, 2)
     _check(gate, "gate rows", torch.float32, 2)
     _check(w, "norm weight", torch.float32, 1)
     n = o.shape[0]
-    if o.shape[1] != groups * group_size or out.shape != o.shape or w.shape[0] not in (group_size, groups * group_size) \
+    _check(out, "gated heads", None, 2)
+    if o.shape[1] != groups * group_size or out.shape[0] != n or out_col + o.shape[1] > out.shape[1] or w.shape[0] not in (group_size, groups * group_size) \
             or gate.shape[0] != n or gate_col + groups * group_size > gate.shape[1]:
         raise KernelError("group_norm_gate: sizes disagree")
     shared = 1 if (w.shape[0] == group_size and groups > 1) else 0
     mixers().call("hos_group_norm_gate", _ptr(o), _ptr(w), shared,
-                  ctypes.c_void_p(gate.data_ptr() + gate_col * 4), gate.shape[1], int(act), _ptr(token_seq), _ptr(out),
-                  dtype_code(out.dtype), float(eps), n, int(groups), int(group_size), _stream())
+                  _at(gate, gate_col), gate.shape[1], int(act), _ptr(token_seq), _at(out, out_col),
+                  dtype_code(out.dtype), out.shape[1], float(eps), n, int(groups), int(group_size), _stream())
+
+
+def skip_gate_norm(o: torch.Tensor, x: torch.Tensor, x_col: int, skip: torch.Tensor, z: torch.Tensor, z_col: int,
+                   w: torch.Tensor, eps: float, token_seq, out: torch.Tensor, heads: int, vdim: int, parts: int) -> None:
+    """y = (o + skip[head] * x[:, x_col:]) * z logistic(z) with z = z[:, z_col:]; out = y in `parts` equal parts, each divided by
+    its own root mean square, times w ([heads * vdim])."""
+    for t, what in ((o, "read-outs"), (x, "inputs"), (z, "gates")):
+        _check(t, what, torch.float32, 2)
+    _check(w, "norm weight", torch.float32, 1)
+    _check(skip, "skip factors", torch.float32, 1)
+    _check(out, "gated heads", None, 2)
+    n, inner = o.shape
+    if inner != heads * vdim or out.shape != o.shape or w.shape[0] != inner or skip.shape[0] != heads or inner % parts != 0 \
+            or x.shape[0] != n or z.shape[0] != n or x_col + inner > x.shape[1] or z_col + inner > z.shape[1]:
+        raise KernelError("skip_gate_norm: sizes disagree")
+    mixers().call("hos_skip_gate_norm", _ptr(o), _at(x, x_col), x.shape[1], _ptr(skip), _at(z, z_col), z.shape[1], _ptr(w),
+                  float(eps), _ptr(token_seq), _ptr(out), dtype_code(out.dtype), n, int(heads), int(vdim), int(parts), _stream())
+
+
+# ---- hyper-connections (csrc/hyper.cu) -----------------------------------------------------------------------------
+
+def hyper_norm(x: torch.Tensor, streams: int, y: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+               mix: Optional[torch.Tensor] = None, out_w: Optional[torch.Tensor] = None, in_next: Optional[torch.Tensor] = None,
+               w: Optional[torch.Tensor] = None, eps: float = 0.0, h: Optional[torch.Tensor] = None) -> None:
+    """x: float32 [N, streams * D].  With y ([N, D] of any type, or [parts, N, D] float32 partial sums): x_t <- sum_s
+    mix[s, t] x_s + out_w[t] (y + bias).  With h: h = RMSNorm(sum_s in_next[s] x_s; w, eps) (in_next None: ones)."""
+    _check(x, "residual streams", torch.float32, 2)
+    n, d = x.shape[0], x.shape[1] // streams
+    parts = 1
+    if x.shape[1] != streams * d:
+        raise KernelError("hyper_norm: the row is no whole number of streams")
+    if y is not None:
+        _check(y, "branch output")
+        parts = y.shape[0] if y.dim() == 3 else 1
+        if y.dim() not in (2, 3) or tuple(y.shape[-2:]) != (n, d) or mix.shape != (streams, streams) or out_w.shape != (streams,):
+            raise KernelError("hyper_norm: sizes of the branch output or its weights disagree")
+    for t, shape, what in ((bias, (d,), "bias"), (mix, (streams, streams), "mixing weights"), (out_w, (streams,), "output weights"),
+                           (in_next, (streams,), "input weights"), (w, (d,), "norm weight")):
+        if t is not None:
+            _check(t, what, torch.float32)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"hyper_norm: {what} of shape {tuple(t.shape)}, {shape} is needed")
+    if h is not None:
+        _check(h, "norm output", None, 2)
+        if tuple(h.shape) != (n, d) or w is None:
+            raise KernelError("hyper_norm: sizes of the norm disagree")
+    mixers().call("hos_hyper_norm", _ptr(y), dtype_code(y.dtype) if y is not None else 0, parts, _ptr(bias), _ptr(x), int(streams),
+                  _ptr(mix), _ptr(out_w), _ptr(in_next), _ptr(w), float(eps), _ptr(h),
+                  dtype_code(h.dtype) if h is not None else 0, n, d, _stream())
+
+
+def stream_sums(x: torch.Tensor, streams: int, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """float32 [n, D]: the sum of the streams of the given rows (all rows where none are given)."""
+    _check(x, "residual streams", torch.float32, 2)
+    n, d = (x.shape[0] if rows is None else rows.shape[0]), x.shape[1] // streams
+    if rows is not None:
+        _check(rows, "row indices", torch.int32, 1)
+    out = torch.empty((n, d), dtype=torch.float32, device=x.device)
+    mixers().call("hos_stream_sums", _ptr(x), _ptr(rows), _ptr(out), n, int(streams), d, _stream())
+    return out
 
 
 def qk_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor],
             eps: float, freq: Optional[torch.Tensor], rot_dims: int, magnitude: float, step, q_out: torch.Tensor,
             cache: PagedKVArgs, n_heads: int, n_kv: int, kd: int, vd: int, norm_whole: bool = False,
-            v_first: Optional[torch.Tensor] = None, v_first_col: int = 0, v_mix: float = 0.0, q_maps: int = 1) -> None:
-    """proj: float32 [N, >= H kd + G (kd + vd)] = [q | k | v | ...] (G = n_kv; 0: a call that stores nothing).  Adds the
+            v_first: Optional[torch.Tensor] = None, v_first_col: int = 0, v_mix: float = 0.0, q_maps: int = 1,
+            proj_col: int = 0, conv_w: Optional[torch.Tensor] = None, conv_state: Optional[torch.Tensor] = None,
+            keep_here: bool = False, q_temp=None) -> None:
+    """proj: float32 rows whose columns from proj_col on are [q | k | v | ...] (G = n_kv; 0: a call that stores nothing).  Adds the
     biases, norms and rotates the q and k heads, writes q_out float32 [N, H, kd] and stores k, v in the cache.
     norm_whole: one root mean square over all q heads and one over all k heads (weights [H kd], [G kd]).  v_first
     (float32 [N, ld], the values from column v_first_col on): v <- (1 - v_mix) v + v_mix v_first before the store.
     q_maps > 1: a head's kd numbers are q_maps queries, one per attention map over the same key row; q_out is then
-    [N, H * q_maps, kd], every query a head of its own that is zero outside its part of the key row."""
+    [N, H * q_maps, kd], every query a head of its own that is zero outside its part of the key row.  conv_w ([taps, C],
+    C = H kd + G (kd + vd)): a short convolution over time on every channel, right after the bias, with its kept inputs
+    conv_state [slots, taps - 1, C] (keep_here, only where every sequence brings one token: they move on in this launch;
+    else call qkv_conv_keep).  q_temp = (coef, every): q times 1 + coef ln(floor((p + 1) / every) + 1)."""
     _check(proj, "projection rows", torch.float32, 2)
     _check(q_out, "queries", torch.float32, 3)
     n = proj.shape[0]
-    if q_out.shape != (n, n_heads * q_maps, kd) or proj.shape[1] < n_heads * kd + n_kv * (kd + vd):
+    c = n_heads * kd + n_kv * (kd + vd)
+    if q_out.shape != (n, n_heads * q_maps, kd) or proj.shape[1] < proj_col + c:
         raise KernelError("qk_prep: sizes disagree")
+    taps = 0
+    if conv_w is not None:
+        _check(conv_w, "convolution weights", torch.float32, 2)
+        taps = conv_w.shape[0]
+        if conv_w.shape[1] != c or (taps > 1 and tuple(conv_state.shape[1:]) != (taps - 1, c)):
+            raise KernelError("qk_prep: the convolution does not fit the projection")
     if n_kv and (cache.head_dim != kd or cache.v_dim != vd or cache.n_kv_heads != n_kv):
         raise KernelError("qk_prep: the cache does not fit the keys and values")
     for wn, cols in ((q_norm, n_heads * kd), (k_norm, n_kv * kd)):
@@ -920,12 +1000,22 @@ def qk_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional[t
         if v_first.shape[0] != n or v_first_col + n_kv * vd > v_first.shape[1]:
             raise KernelError("qk_prep: the other layer's values do not fit this layer's")
         vf_ptr, vf_ld = ctypes.c_void_p(v_first.data_ptr() + 4 * v_first_col), v_first.shape[1]
-    gated_attn_lib().call("hos_qk_prep", _ptr(proj), proj.shape[1], _ptr(bias), _ptr(q_norm), _ptr(k_norm), float(eps), _ptr(freq),
+    coef, every = q_temp if q_temp else (0.0, 0)
+    gated_attn_lib().call("hos_qk_prep", _at(proj, proj_col), proj.shape[1], _ptr(bias), _ptr(q_norm), _ptr(k_norm), float(eps), _ptr(freq),
                   int(rot_dims), float(magnitude), _ptr(step.token_pos), _ptr(step.token_seq), _ptr(step.seq_slot),
                   _ptr(q_out), _ptr(cache.k_pages) if n_kv else None, _ptr(cache.v_pages) if n_kv else None,
                   dtype_code(cache.k_pages.dtype), _ptr(cache.page_table), cache.table_stride, cache.ring_pages, n,
                   int(n_heads), int(n_kv), int(kd), int(vd), 1 if norm_whole else 0, vf_ptr, vf_ld, float(v_mix),
-                  int(q_maps), _stream())
+                  int(q_maps), _ptr(conv_w), taps, _ptr(conv_state) if taps > 1 else None, _ptr(step.cu_seqlens),
+                  1 if keep_here else 0, float(coef), int(every), _stream())
+
+
+def qkv_conv_keep(proj: torch.Tensor, proj_col: int, bias: Optional[torch.Tensor], taps: int, conv_state: torch.Tensor, step,
+                  channels: int) -> None:
+    """The last taps - 1 projected inputs of every sequence's q, k and v channels go to the slot's state."""
+    gated_attn_lib().call("hos_qkv_conv_keep", _at(proj, proj_col), proj.shape[1], _ptr(bias), int(taps), _ptr(conv_state),
+                          _ptr(step.token_pos), _ptr(step.token_seq), _ptr(step.cu_seqlens), _ptr(step.seq_slot),
+                          int(step.n_seqs), int(channels), _stream())
 
 
 def diff_combine(a: torch.Tensor, lam: float, mult: float, eps: float, gate: Optional[torch.Tensor], gate_col: int, step,
@@ -945,13 +1035,14 @@ def diff_combine(a: torch.Tensor, lam: float, mult: float, eps: float, gate: Opt
 
 def gated_attn(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor],
                gate_col: int, step, out: torch.Tensor, scale: float, chunk: int, window: int, n_splits: int = 1,
-               keep_first: int = 0) -> None:
-    """q: float32 [N, H, kd]; keys and values from the paged cache; out: [N, H * vd].  gate: float32 rows whose column
-    gate_col + h is head h's gate logit."""
+               keep_first: int = 0, out_col: int = 0, out_scale: float = 1.0) -> None:
+    """q: float32 [N, H, kd]; keys and values from the paged cache; out: [N, >= out_col + H * vd], the heads' outputs times
+    out_scale from column out_col on.  gate: float32 rows whose column gate_col + h is head h's gate logit."""
     _check(q, "queries", torch.float32, 3)
+    _check(out, "attention output", None, 2)
     n, heads, kd = q.shape
     vd = cache.v_dim
-    if out.shape != (n, heads * vd) or kd != cache.head_dim:
+    if out.shape[0] != n or out_col + heads * vd > out.shape[1] or kd != cache.head_dim:
         raise KernelError("gated_attn: sizes disagree")
     part_acc = part_ml = None
     if n_splits > 1:
@@ -961,41 +1052,42 @@ def gated_attn(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[torch.Tensor]
                   _ptr(cache.page_table), cache.table_stride, cache.ring_pages, _ptr(sink),
                   ctypes.c_void_p(gate.data_ptr() + gate_col * 4) if gate is not None else None,
                   gate.shape[1] if gate is not None else 0, _ptr(step.token_pos), _ptr(step.token_seq), _ptr(step.seq_slot),
-                  _ptr(out), dtype_code(out.dtype), _ptr(part_acc), _ptr(part_ml), int(n_splits), n, heads,
+                  _at(out, out_col), dtype_code(out.dtype), out.shape[1], float(out_scale), _ptr(part_acc), _ptr(part_ml),
+                  int(n_splits), n, heads,
                   cache.n_kv_heads, kd, vd, float(scale), int(chunk or 0), int(window or 0), int(keep_first or 0), _stream())
 
 
 def gated_attn_mma(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor],
                    gate_col: int, step, out: torch.Tensor, scale: float, chunk: int, window: int, n_q_tiles: int,
-                   keep_first: int = 0) -> bool:
+                   keep_first: int = 0, out_col: int = 0, out_scale: float = 1.0) -> bool:
     """The same attention on the tensor cores, for bfloat16 caches and rows that come many to a sequence.  False: the
     sizes are not that kernel's and nothing ran."""
     n, heads, kd = q.shape
     vd = cache.v_dim
     if out.dtype not in (torch.bfloat16, torch.float32) or cache.k_pages.dtype != torch.bfloat16 \
-            or out.shape != (n, heads * vd):
+            or out.shape[0] != n or out_col + heads * vd > out.shape[1]:
         return False
-    if kd not in (64, 128) or vd not in (64, 128) or q.data_ptr() % 16 or out.data_ptr() % 8:
+    if kd not in (64, 128) or vd not in (64, 128) or q.data_ptr() % 16 or out.data_ptr() % 8 or out.shape[1] % 2 or out_col % 4:
         return False
     gated_attn_lib().call("hos_gated_attn_mma", _ptr(q), _ptr(cache.k_pages), _ptr(cache.v_pages), _ptr(cache.page_table),
                   cache.table_stride, cache.ring_pages, _ptr(sink),
                   ctypes.c_void_p(gate.data_ptr() + gate_col * 4) if gate is not None else None,
                   gate.shape[1] if gate is not None else 0, _ptr(step.cu_seqlens), _ptr(step.token_pos),
-                  _ptr(step.token_seq), _ptr(step.seq_slot), _ptr(out), 1 if out.dtype == torch.float32 else 0,
-                  int(step.n_seqs), int(n_q_tiles), heads,
+                  _ptr(step.token_seq), _ptr(step.seq_slot), _at(out, out_col), 1 if out.dtype == torch.float32 else 0,
+                  out.shape[1], float(out_scale), int(step.n_seqs), int(n_q_tiles), heads,
                   cache.n_kv_heads, kd, vd, float(scale), int(chunk or 0), int(window or 0), int(keep_first or 0), _stream())
     return True
 
 
 def gated_attn_mma_decode(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor],
                           gate_col: int, step, out: torch.Tensor, scale: float, chunk: int, window: int,
-                          n_splits: int = 1, keep_first: int = 0) -> bool:
+                          n_splits: int = 1, keep_first: int = 0, out_col: int = 0, out_scale: float = 1.0) -> bool:
     """Single tokens on the tensor cores: the query heads that share a kv head are the rows of one tile.  False: the
     sizes are not that kernel's and nothing ran."""
     n, heads, kd = q.shape
     vd = cache.v_dim
     if out.dtype not in (torch.bfloat16, torch.float32) or cache.k_pages.dtype != torch.bfloat16 \
-            or out.shape != (n, heads * vd):
+            or out.shape[0] != n or out_col + heads * vd > out.shape[1]:
         return False
     if kd not in (64, 128) or vd not in (64, 128) or heads // cache.n_kv_heads > 16 or q.data_ptr() % 16:
         return False
@@ -1007,20 +1099,23 @@ def gated_attn_mma_decode(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[to
     gate_ld = gate.shape[1] if gate is not None else 0
     gated_attn_lib().call("hos_gated_attn_mma_decode", _ptr(q), _ptr(cache.k_pages), _ptr(cache.v_pages), _ptr(cache.page_table),
                   cache.table_stride, cache.ring_pages, _ptr(sink), gate_ptr, gate_ld, _ptr(step.token_pos),
-                  _ptr(step.token_seq), _ptr(step.seq_slot), _ptr(out), 1 if out.dtype == torch.float32 else 0,
-                  _ptr(part_acc), _ptr(part_ml), int(n_splits), n,
+                  _ptr(step.token_seq), _ptr(step.seq_slot), _at(out, out_col), 1 if out.dtype == torch.float32 else 0,
+                  out.shape[1], float(out_scale), _ptr(part_acc), _ptr(part_ml), int(n_splits), n,
                   heads, cache.n_kv_heads, kd, vd, float(scale), int(chunk or 0), int(window or 0), int(keep_first or 0),
                   _stream())
     if n_splits > 1:
         gated_attn_lib().call("hos_attn_merge", _ptr(part_acc), _ptr(part_ml), int(n_splits), gate_ptr, gate_ld,
-                      _ptr(step.token_seq), _ptr(out), dtype_code(out.dtype), n, heads, vd, _stream())
+                      _ptr(step.token_seq), _at(out, out_col), dtype_code(out.dtype), out.shape[1], float(out_scale), n, heads,
+                      vd, _stream())
     return True
 
 
 def state_scan(rows: torch.Tensor, q_col: int, k_col: int, v_col: int, silu_on_load: bool, g: torch.Tensor,
                per_token_g: bool, beta: Optional[torch.Tensor], state: torch.Tensor, step, out: torch.Tensor,
-               heads: int, key_heads: int, dim: int, vdim: int, rot=None) -> None:
-    """The matrix-state recurrence over the step's sequences.  rot = (freq, rot_dims, style, k_mult): q and k turn with
+               heads: int, key_heads: int, dim: int, vdim: int, rot=None, v_factor: Optional[torch.Tensor] = None,
+               channel_g: bool = False, o_mult: float = 1.0) -> None:
+    """The matrix-state recurrence over the step's sequences.  v_factor ([N, heads]): with the decay rule, the factor on v.
+    channel_g: g is [N, heads * dim], a decay per key channel.  o_mult: a constant on the read-outs.  rot = (freq, rot_dims, style, k_mult): q and k turn with
     their positions and the keys take a factor inside the walk (single-token steps), instead of by rotate_rows before.  rows: float32 [N, ld] holding q, k (key_heads x dim) and
     v (heads x vdim) from the given columns on.  g: [heads] constants, or [N, heads] per token; beta ([N, heads]): the
     delta rule, None: the plain decay rule.  state: [slots, heads, vdim, dim] float32.  out: float32 [N, heads * vdim]."""
@@ -1031,17 +1126,26 @@ def state_scan(rows: torch.Tensor, q_col: int, k_col: int, v_col: int, silu_on_l
     n, ld = rows.shape
     if out.shape != (n, heads * vdim) or tuple(state.shape[1:]) != (heads, vdim, dim):
         raise KernelError("state_scan: sizes disagree")
+    if channel_g and (tuple(g.shape) != (n, heads * dim) or beta is not None or v_factor is not None or key_heads != heads):
+        raise KernelError("state_scan: the decays per key channel do not fit")
+    if v_factor is not None:
+        _check(v_factor, "factors on v", torch.float32, 2)
+        if beta is not None or silu_on_load or tuple(v_factor.shape) != (n, heads):
+            raise KernelError("state_scan: factors on v go with the plain decay rule")
     base = rows.data_ptr()
     if rot is not None and (silu_on_load or beta is not None or key_heads != heads):
         raise KernelError("state_scan: the rotation in the walk goes with the plain decay rule on rows as they are")
+    rule = 1 if beta is not None else (2 if channel_g else 0)
+    second = beta if beta is not None else v_factor
+    g_ld = heads * dim if channel_g else (heads if per_token_g else 0)
     in_walk = bool(silu_on_load) and beta is None and step.max_new == 1      # single tokens: no launch of its own for it
     if silu_on_load and not in_walk:        # q, k, v lie side by side from q_col on: x logistic(x) in place, once, before the walk
         if not (q_col < k_col < v_col) or v_col + heads * vdim - q_col != 2 * key_heads * dim + heads * vdim:
             raise KernelError("state_scan: q, k, v must lie side by side for the activation")
         mixers().call("hos_act_rows", ctypes.c_void_p(base + 4 * q_col), ld, 2 * key_heads * dim + heads * vdim, n, _stream())
     mixers().call("hos_state_scan", ctypes.c_void_p(base + 4 * q_col), ctypes.c_void_p(base + 4 * k_col),
-                  ctypes.c_void_p(base + 4 * v_col), ld, 1 if in_walk else 0, _ptr(g), heads if per_token_g else 0,
-                  _ptr(beta), heads if beta is not None else 0, _ptr(state), _ptr(step.token_pos), _ptr(step.token_seq),
+                  ctypes.c_void_p(base + 4 * v_col), ld, 1 if in_walk else 0, rule, float(o_mult), _ptr(g), g_ld,
+                  _ptr(second), heads if second is not None else 0, _ptr(state), _ptr(step.token_pos), _ptr(step.token_seq),
                   _ptr(step.cu_seqlens), _ptr(step.seq_slot), _ptr(out), n, int(step.n_seqs), int(heads), int(key_heads),
                   int(dim), int(vdim), _ptr(rot[0]) if rot else None, int(rot[1]) if rot else 0, int(rot[2]) if rot else 0,
                   float(rot[3]) if rot else 1.0, _stream())
@@ -1081,7 +1185,48 @@ def conv_prep(raw: torch.Tensor, conv_w: torch.Tensor, conv_state: torch.Tensor,
                   _ptr(beta), _ptr(g), n, int(heads), int(key_heads), int(dim), int(vdim), 1 if keep_here else 0, _stream())
 
 
-def conv_keep(raw: torch.Tensor, taps: int, conv_state: torch.Tensor, step, channels: int) -> None:
-    mixers().call("hos_conv_keep", _ptr(raw), raw.shape[1], int(taps), _ptr(conv_state), _ptr(step.token_pos),
+def conv_keep(raw: torch.Tensor, taps: int, conv_state: torch.Tensor, step, channels: int, col: int = 0) -> None:
+    mixers().call("hos_conv_keep", _at(raw, col), raw.shape[1], int(taps), _ptr(conv_state), _ptr(step.token_pos),
                   _ptr(step.token_seq), _ptr(step.cu_seqlens), _ptr(step.seq_slot), int(step.n_seqs), int(channels),
+                  _stream())
+
+
+def conv_act_rows(raw: torch.Tensor, col: int, conv_w: torch.Tensor, bias: Optional[torch.Tensor], conv_state: torch.Tensor,
+                  act: str, step, out: torch.Tensor, single: bool, dt=None) -> None:
+    """out ([N, C] float32) = act(short convolution of raw[:, col:col + C] + bias), act "none" or "x_logistic"; conv_w: [C, taps];
+    conv_state: [slots, taps - 1, C] (single, only where every sequence brings one token: the kept inputs move on in this
+    launch; else call conv_keep).  dt = (column, dt_bias, a_log, dt_out, g_out): per head, dt_out = softplus(raw + dt_bias) and
+    g_out = exp(-exp(a_log) dt) in the same launch."""
+    _check(raw, "projection rows", torch.float32, 2)
+    _check(conv_w, "convolution weights", torch.float32, 2)
+    _check(out, "convolved rows", torch.float32, 2)
+    n, (c, taps) = raw.shape[0], conv_w.shape
+    if tuple(out.shape) != (n, c) or col + c > raw.shape[1] or tuple(conv_state.shape[1:]) != (taps - 1, c):
+        raise KernelError("conv_act_rows: sizes disagree")
+    dt_args = (None, None, None, None, None, 0)
+    if dt is not None:
+        dt_col, dt_bias, a_log, dt_out, g_out = dt
+        heads = dt_bias.shape[0]
+        for t in (dt_out, g_out):
+            _check(t, "step sizes", torch.float32, 2)
+            if tuple(t.shape) != (n, heads):
+                raise KernelError("conv_act_rows: sizes of the step sizes disagree")
+        if dt_col + heads > raw.shape[1] or a_log.shape[0] != heads:
+            raise KernelError("conv_act_rows: sizes of the step sizes disagree")
+        dt_args = (_at(raw, dt_col), _ptr(dt_bias), _ptr(a_log), _ptr(dt_out), _ptr(g_out), heads)
+    mixers().call("hos_conv_act_rows", _at(raw, col), raw.shape[1], _ptr(conv_w), _ptr(bias), int(taps),
+                  _ptr(conv_state) if taps > 1 else None, {"none": 0, "x_logistic": 1}[act], _ptr(step.token_pos), _ptr(step.token_seq),
+                  _ptr(step.cu_seqlens), _ptr(step.seq_slot), _ptr(out), n, int(c), 1 if single else 0, *dt_args, _stream())
+
+
+def channel_decay(rows: torch.Tensor, col: int, rank: int, w: torch.Tensor, b: torch.Tensor, tau: float, out: torch.Tensor) -> None:
+    """out ([N, C] float32) = logistic(rows[:, col:col + rank] . w + b)^(1 / tau); w: [rank, C]."""
+    _check(rows, "projection rows", torch.float32, 2)
+    _check(w, "decay projection", torch.float32, 2)
+    _check(b, "decay bias", torch.float32, 1)
+    _check(out, "decays", torch.float32, 2)
+    n, c = out.shape
+    if rows.shape[0] != n or col + rank > rows.shape[1] or tuple(w.shape) != (rank, c) or b.shape[0] != c:
+        raise KernelError("channel_decay: sizes disagree")
+    mixers().call("hos_channel_decay", _at(rows, col), rows.shape[1], _ptr(w), _ptr(b), int(rank), float(tau), _ptr(out), n, int(c),
                   _stream())

@@ -10,6 +10,7 @@ from typing import List, Mapping, Optional
 import torch
 
 from .. import ops
+from ..errors import SpecError
 from ..registry import part_impl, register_part
 from . import linear
 from .base import CallStore, Part, StateNeed, StepInfo, WeightSpec
@@ -24,7 +25,10 @@ class ScaledEmbedding(Part):
         self.width = int(spec.params["width"])
         self.scale = float(spec.params.get("scale", 1.0))
         self.table: Optional[torch.Tensor] = None
+        self.copies = int(spec.params.get("copies", 1))      # a row is that many copies side by side (residual streams)
         norm = spec.params.get("norm")       # the spec of a norm part: the rows are normed, in place, on their way out
+        if self.copies < 1 or (norm is not None and self.copies > 1):
+            raise SpecError("arch spec error: an embedding with a norm has one copy of its rows")
         self.norm = part_impl("norm", norm.kind)(norm, rt) if norm is not None else None
         if self.norm is not None and not self.norm.graph_safe:
             self.graph_safe = False
@@ -39,8 +43,8 @@ class ScaledEmbedding(Part):
             self.norm.bind(tensors)
 
     def forward(self, tokens: torch.Tensor, step: StepInfo = None) -> torch.Tensor:
-        x = torch.empty((tokens.shape[0], self.width), dtype=torch.float32, device=tokens.device)
-        ops.embed(tokens, self.table, self.scale, x)
+        x = torch.empty((tokens.shape[0], self.copies * self.width), dtype=torch.float32, device=tokens.device)
+        ops.embed(tokens, self.table, self.scale, x, self.copies)
         if self.norm is not None:
             self.norm.forward(x, out=x)
         return x

@@ -7,7 +7,12 @@ floor(j / C) = floor(i / C), counted from the sequence's position 0) or of a win
 `keep_first` also the sequence's first keep_first keys), or plain causal; a sink (`sink` true: a learned number per
 head whose exponential joins the softmax's denominator, without a key or a value; "zero": the constant 0, which
 adds one to the denominator); a gate per head (the head's output times the logistic function of a projection of
-the mixer's input); the output projection.
+the mixer's input); the output projection (`o_bias`: with a bias; `out_scale`: times a constant).
+
+`conv`: every channel of the q, k and v projections passes a short causal convolution over time (that many taps, the
+last one the current token's, no bias, zeros before a sequence's start) right after the projection and its bias; its last
+conv - 1 projected inputs are per-sequence state.  `q_temp` {"coef": c, "every": n}: the query at position p is
+multiplied by 1 + c ln(floor((p + 1) / n) + 1).
 
 Values mixed across layers (`value_mix`): {"key": name, "role": "source"} leaves the layer's values, as projected,
 in the step's shared store under that name; {"key": name, "role": "mixed"} blends its own values with them,
@@ -36,7 +41,7 @@ from .. import ops
 from ..errors import KernelError, SpecError
 from ..registry import part_impl, register_part
 from . import linear
-from .base import FEW_TOKENS, CallStore, KVNeed, Mixer, StepInfo, WeightSpec
+from .base import FEW_TOKENS, CallStore, KVNeed, Mixer, StateNeed, StepInfo, WeightSpec
 
 SPLIT_MIN_KEYS = 256        # rows that see fewer keys are never cut into shares
 
@@ -67,6 +72,16 @@ class GatedSoftmaxAttention(Mixer):
         if self.keep_first < 0 or (self.keep_first and not p.get("window")):
             raise SpecError("arch spec error: kept first keys go with a window")
         self.shares_kv = bool(p.get("shares_kv", False))
+        self.taps = int(p.get("conv") or 0)
+        if self.taps < 0 or (self.taps and (self.shares_kv or self.norm_whole)):
+            raise SpecError("arch spec error: a short convolution goes with keys and values of the layer's own and no norm over "
+                            "the whole projection")
+        temp = p.get("q_temp")
+        self.q_temp = (float(temp["coef"]), int(temp["every"])) if temp else None
+        if self.q_temp and self.q_temp[1] <= 0:
+            raise SpecError("arch spec error: the query factor's step must be positive")
+        self.has_o_bias, self.out_scale = bool(p.get("o_bias", False)), float(p.get("out_scale", 1.0))
+        self.out_bias: Optional[torch.Tensor] = None
         if min(self.n_heads, self.n_kv_heads, self.dim, self.vdim) <= 0 or self.n_heads % self.n_kv_heads != 0:
             raise SpecError(f"arch spec error: {self.n_heads} heads of {self.dim}/{self.vdim} numbers over "
                             f"{self.n_kv_heads} kv heads")
@@ -90,6 +105,10 @@ class GatedSoftmaxAttention(Mixer):
             roles += [("k", self.n_kv_heads * self.dim), ("v", self.n_kv_heads * self.vdim)]
         if self.has_bias:
             out += [WeightSpec(w[r + "_bias"], (n,), "vector", 0.1) for r, n in roles]
+        if self.taps:
+            out += [WeightSpec(w[r + "_conv"], (n, self.taps), "matrix", 0.4) for r, n in roles]
+        if self.has_o_bias:
+            out.append(WeightSpec(w["o_bias"], (self.width,), "vector", 0.1))
         if self.qk_norm:
             out += [WeightSpec(w[r + "_norm"], (n if self.norm_whole else self.dim,), "vector", 0.1)
                     for r, n in roles if r != "v"]
@@ -126,6 +145,13 @@ class GatedSoftmaxAttention(Mixer):
                          else self._vector32(tensors[w["sink"]]))
         self.v_mix = float(tensors[w["value_mix"]].float().reshape(-1)[0].item()) if self.mix_role == "mixed" else 0.0
         self.w_o = self._matrix(tensors[w["o"]])
+        self.conv_w = None
+        if self.taps:
+            self.conv_w = torch.cat([tensors[w[r + "_conv"]].to(torch.float32) for r in roles], dim=0).t().contiguous()  # [taps, C]
+        self.out_bias = (self._vector32(tensors[w["o_bias"]]) * self.out_scale).contiguous() if self.has_o_bias else None
+
+    def state_needs(self) -> List[StateNeed]:
+        return [StateNeed("conv", (self.taps - 1, self.q_cols + self.kv_cols), torch.float32)] if self.taps > 1 else []
 
     def kv_need(self) -> KVNeed:
         # every position is kept: rows attend over the cache in the step that stores them too, and a prompt may
@@ -152,23 +178,49 @@ class GatedSoftmaxAttention(Mixer):
         return max(1, min(room // warps, keys // 64, 64))
 
     def forward(self, h, step: StepInfo, store: CallStore):
-        return self._run(h, step, store, False)
+        att = self._heads(h, step, store)
+        if self.out_bias is not None:
+            return linear.matmul(att, self.w_o, epilogue=ops.EPI_BIAS, bias=self.out_bias)
+        return linear.matmul(att, self.w_o)
 
     def forward_partial(self, h, step: StepInfo, store: CallStore):
-        return self._run(h, step, store, True)
+        if self.out_bias is not None:
+            return self.forward(h, step, store)
+        return self.forward_unbiased(h, step, store)
 
-    def _run(self, h: torch.Tensor, step: StepInfo, store: CallStore, partial_ok: bool) -> torch.Tensor:
+    def forward_unbiased(self, h, step: StepInfo, store: CallStore):
+        """As forward, without `out_bias`, for a consumer that adds it; may hand back 32-bit partial sums."""
+        return linear.matmul_or_partials(self._heads(h, step, store), self.w_o)
+
+    def _heads(self, h, step: StepInfo, store: CallStore) -> torch.Tensor:
+        proj = linear.matmul(h, self.w_in, out_dtype=torch.float32)
+        att = torch.empty((h.shape[0], self.n_heads * self.vdim), dtype=h.dtype, device=h.device)
+        self.run_heads(proj, 0, step, store, att, 0)
+        return att
+
+    # the mixer between its projections (see parts/parallel_mixers.py): input columns in, output columns out
+    @property
+    def in_cols(self) -> int:
+        return self.q_cols + self.kv_cols + (self.n_heads if self.head_gate else 0)
+
+    @property
+    def out_cols(self) -> int:
+        return self.n_heads * self.vdim
+
+    def run_heads(self, proj: torch.Tensor, col: int, step: StepInfo, store: CallStore, att: torch.Tensor, out_col: int) -> None:
+        """From the projections, 32-bit rows `proj` whose columns from `col` on are [q | k | v | gate logits], to the heads'
+        outputs times out_scale in att's columns from out_col on."""
         cache = store.kv
         if cache is None:
             raise KernelError("attention needs a cache view")
         if store.owns_kv == self.shares_kv:
             raise KernelError("attention: the call's cache and the mixer's tensors do not fit (a mixer without key and "
                               "value tensors reads another call's cache, and only such a mixer does)")
-        n = h.shape[0]
-        proj = linear.matmul(h, self.w_in, out_dtype=torch.float32)
-        q = torch.empty((n, self.n_heads, self.dim), dtype=torch.float32, device=h.device)
+        n = proj.shape[0]
+        q = torch.empty((n, self.n_heads, self.dim), dtype=torch.float32, device=proj.device)
         freq, rot_dims, _ = self.position.kernel_args() if self.position else (None, 0, 0)
-        v_col = self.q_cols + self.n_kv_heads * self.dim
+        v_col = col + self.q_cols + self.n_kv_heads * self.dim
+        gate_col = col + self.gate_col
         v_first = None
         if self.mix_role == "source":
             step.shared[self.mix_key] = (proj, v_col)          # the values as projected, for the layers that mix them in
@@ -176,31 +228,35 @@ class GatedSoftmaxAttention(Mixer):
             if self.mix_key not in step.shared:
                 raise KernelError(f"attention: no layer of this step has left values under {self.mix_key!r}")
             v_first = step.shared[self.mix_key]
+        kept = store.state["conv"] if self.taps > 1 else None
+        single = step.max_new == 1           # every sequence brings one token: the kept inputs move on in qk_prep itself
         ops.qk_prep(proj, self.bias, self.q_norm, self.k_norm, self.eps, freq, rot_dims,
                     getattr(self.position, "magnitude", 1.0), step, q, cache, self.n_heads,
                     0 if self.shares_kv else self.n_kv_heads, self.dim, self.vdim, self.norm_whole,
-                    v_first[0] if v_first else None, v_first[1] if v_first else 0, self.v_mix)
-        att = torch.empty((n, self.n_heads * self.vdim), dtype=h.dtype, device=h.device)
+                    v_first[0] if v_first else None, v_first[1] if v_first else 0, self.v_mix,
+                    proj_col=col, conv_w=self.conv_w, conv_state=kept, keep_here=single, q_temp=self.q_temp)
+        if self.taps > 1 and not single:
+            ops.qkv_conv_keep(proj, col, self.bias, self.taps, kept, step, self.q_cols + self.kv_cols)
         gate = proj if self.head_gate else None
-        if self.use_tensor_cores and h.dtype == torch.bfloat16 and step.max_new > FEW_TOKENS:
+        where = dict(keep_first=self.keep_first, out_col=out_col, out_scale=self.out_scale)
+        if self.use_tensor_cores and att.dtype == torch.bfloat16 and step.max_new > FEW_TOKENS:
             # rows that come many to a sequence: 64 queries to a key tile on the tensor cores
             if step.cu_host:
                 tiles = sum((step.cu_host[i + 1] - step.cu_host[i] + 63) // 64 for i in range(len(step.cu_host) - 1))
             else:
                 tiles = (n + 63) // 64 + step.n_seqs
-            if ops.gated_attn_mma(q, cache, self.sink, gate, self.gate_col, step, att, self.scale, self.chunk or 0,
-                                  self.window or 0, tiles, self.keep_first):
-                return linear.matmul_or_partials(att, self.w_o) if partial_ok else linear.matmul(att, self.w_o)
-        if self.use_tensor_cores and h.dtype == torch.bfloat16 and step.max_new == 1:
+            if ops.gated_attn_mma(q, cache, self.sink, gate, gate_col, step, att, self.scale, self.chunk or 0,
+                                  self.window or 0, tiles, **where):
+                return
+        if self.use_tensor_cores and att.dtype == torch.bfloat16 and step.max_new == 1:
             # single tokens: the query heads of a kv head are the rows of one tile; few rows: the key tiles in shares
             tiles = (self.keys_seen(step.max_len_after) + 63) // 64 + 1
             shares = max(1, min(tiles, 2 * ops.sm_count() // max(1, n * self.n_kv_heads), 32))
-            if ops.gated_attn_mma_decode(q, cache, self.sink, gate, self.gate_col, step, att, self.scale, self.chunk or 0,
-                                         self.window or 0, shares, self.keep_first):
-                return linear.matmul_or_partials(att, self.w_o) if partial_ok else linear.matmul(att, self.w_o)
-        ops.gated_attn(q, cache, self.sink, proj if self.head_gate else None, self.gate_col, step, att, self.scale,
-                       self.chunk or 0, self.window or 0, self.n_splits(n, step.max_len_after), self.keep_first)
-        return linear.matmul_or_partials(att, self.w_o) if partial_ok else linear.matmul(att, self.w_o)
+            if ops.gated_attn_mma_decode(q, cache, self.sink, gate, gate_col, step, att, self.scale, self.chunk or 0,
+                                         self.window or 0, shares, **where):
+                return
+        ops.gated_attn(q, cache, self.sink, gate, gate_col, step, att, self.scale, self.chunk or 0, self.window or 0,
+                       self.n_splits(n, step.max_len_after), **where)
 
 
 register_part("mixer", "gated_softmax_attention", GatedSoftmaxAttention)

@@ -1,5 +1,5 @@
 """Python face of the matrix product for up to 32 rows (csrc/gemm_skinny.cu): what decoding at
-small batch runs.  bfloat16 operands, K a multiple of 8; epilogues none and gated."""
+small batch runs.  bfloat16 operands, K a multiple of 8; epilogues none, gated and bias."""
 from __future__ import annotations
 
 from typing import Optional
@@ -29,18 +29,19 @@ def operands_ok(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def can_take(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int) -> bool:
-    if not operands_ok(x, w) or epilogue not in (ops.EPI_NONE, ops.EPI_GATED) or not out.is_contiguous():
+    if not operands_ok(x, w) or epilogue not in (ops.EPI_NONE, ops.EPI_GATED, ops.EPI_BIAS) or not out.is_contiguous():
         return False
-    if epilogue == ops.EPI_GATED:
+    if epilogue in (ops.EPI_GATED, ops.EPI_BIAS):
         return out.dtype == torch.bfloat16
     return out.dtype in (torch.bfloat16, torch.float32)
 
 
-def matmul(x, w, out, epilogue: int = ops.EPI_NONE, act: int = 0, act_limit: float = 0.0) -> None:
+def matmul(x, w, out, epilogue: int = ops.EPI_NONE, act: int = 0, act_limit: float = 0.0,
+           bias: Optional[torch.Tensor] = None) -> None:
     m, k = x.shape
     n = out.shape[1]
     lib().call("hos_gemm_skinny", ops._ptr(x), ops._ptr(w), ops._ptr(out), ops.dtype_code(out.dtype), m, n, k,
-               x.stride(0), w.stride(0), out.stride(0), epilogue, act, float(act_limit), 1,
+               x.stride(0), w.stride(0), out.stride(0), epilogue, act, float(act_limit), ops._ptr(bias), 1,
                1 if ops.take_room_left() else 0, ops._stream())
 
 
@@ -65,7 +66,7 @@ def matmul_partials(x, w, k_splits: Optional[int] = None) -> Optional[torch.Tens
         return None
     parts = torch.empty((k_splits, m, n), dtype=torch.float32, device=x.device)
     lib().call("hos_gemm_skinny", ops._ptr(x), ops._ptr(w), ops._ptr(parts), ops.F32, m, n, k,
-               x.stride(0), w.stride(0), n, ops.EPI_NONE, 0, 0.0, k_splits, 1 if ops.take_room_left() else 0, ops._stream())
+               x.stride(0), w.stride(0), n, ops.EPI_NONE, 0, 0.0, None, k_splits, 1 if ops.take_room_left() else 0, ops._stream())
     return parts
 
 

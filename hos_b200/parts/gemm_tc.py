@@ -44,7 +44,7 @@ def can_take(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int)
         return False
     if x.data_ptr() % 16 or w.data_ptr() % 16 or out.data_ptr() % 16 or not out.is_contiguous():
         return False
-    if epilogue == ops.EPI_GATED and out.dtype != torch.bfloat16:
+    if epilogue in (ops.EPI_GATED, ops.EPI_BIAS) and out.dtype != torch.bfloat16:
         return False
     if epilogue == ops.EPI_SOFTCAP and out.dtype != torch.float32:
         return False
@@ -71,7 +71,7 @@ def k_splits_for(m: int, n: int, k: int, epilogue: int) -> int:
 
 
 def matmul(x, w, out, epilogue: int = ops.EPI_NONE, cap: float = 0.0, act: int = 0,
-           k_splits: Optional[int] = None) -> None:
+           k_splits: Optional[int] = None, bias: Optional[torch.Tensor] = None) -> None:
     m, k = x.shape
     n = out.shape[1]
     if k_splits is None:
@@ -80,7 +80,7 @@ def matmul(x, w, out, epilogue: int = ops.EPI_NONE, cap: float = 0.0, act: int =
     if k_splits > 1:
         ws = torch.empty(k_splits * m * n, dtype=torch.float32, device=x.device)
     lib().call("hos_gemm_tc", ops._ptr(x), ops._ptr(w), ops._ptr(out), ops.dtype_code(out.dtype), m, n, k,
-               x.stride(0), w.stride(0), out.stride(0), epilogue, float(cap), act, k_splits, ops._ptr(ws),
+               x.stride(0), w.stride(0), out.stride(0), epilogue, float(cap), act, ops._ptr(bias), k_splits, ops._ptr(ws),
                1, None, ops._stream())
 
 
@@ -96,7 +96,7 @@ def matmul_partials(x, w, k_splits: Optional[int] = None) -> Optional[torch.Tens
     ws = torch.empty((k_splits, m, n), dtype=torch.float32, device=x.device)
     used = ctypes.c_int(0)
     lib().call("hos_gemm_tc", ops._ptr(x), ops._ptr(w), None, ops.F32, m, n, k, x.stride(0), w.stride(0), n,
-               ops.EPI_NONE, 0.0, 0, k_splits, ops._ptr(ws), 0, ctypes.byref(used), ops._stream())
+               ops.EPI_NONE, 0.0, 0, None, k_splits, ops._ptr(ws), 0, ctypes.byref(used), ops._stream())
     return ws[: used.value]
 
 

@@ -24,11 +24,18 @@ def plain_forced() -> bool:
     return _force_plain
 
 
+def pad_rows(w: torch.Tensor, multiple: int = 8) -> torch.Tensor:
+    """The matrix with zero rows appended up to a multiple: the product's rows are then whole 16-byte pieces apart, which
+    its stores and its readers' loads want (the extra columns are zeros that nobody reads)."""
+    more = -w.shape[0] % multiple
+    return torch.cat([w, w.new_zeros((more, w.shape[1]))], dim=0).contiguous() if more else w
+
+
 def matmul(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
            epilogue: int = ops.EPI_NONE, cap: float = 0.0, act: int = 0,
-           out: Optional[torch.Tensor] = None) -> torch.Tensor:
+           out: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[M, N] = x[M, K] . w[N or 2N, K]^T (2N rows with the gated epilogue; with its clamped activation the limit
-    rides in `cap`)."""
+    rides in `cap`; the bias epilogue adds `bias` ([N] float32) and applies `act`, one of ops.BIAS_ACTIVATIONS)."""
     m = x.shape[0]
     n = w.shape[0] // 2 if epilogue == ops.EPI_GATED else w.shape[0]
     if out is None:
@@ -38,12 +45,12 @@ def matmul(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
     if (not _force_plain and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16):
         from . import gemm_skinny, gemm_tc
         if gemm_skinny.can_take(x, w, out, epilogue):
-            gemm_skinny.matmul(x, w, out, epilogue, act, cap)
+            gemm_skinny.matmul(x, w, out, epilogue, act, cap, bias=bias)
             return out
         if gemm_tc.can_take(x, w, out, epilogue):
-            gemm_tc.matmul(x, w, out, epilogue, cap, act)
+            gemm_tc.matmul(x, w, out, epilogue, cap, act, bias=bias)
             return out
-    ops.gemm_plain(x, w, out, epilogue, cap, act)
+    ops.gemm_plain(x, w, out, epilogue, cap, act, bias)
     return out
 
 

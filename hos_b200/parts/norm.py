@@ -2,7 +2,8 @@
 `add_one` is Gemma's (1 + w) convention, src/hf.rs:101-107).  Statistics in 32-bit.
 A norm may name a second tensor, `scale`: a multiplier per column on the norm's output (the layer scale of a
 branch whose last act is this norm).  It is folded into the weight when the tensors are bound, (w + add_one) * scale
-in 32-bit, which is exact for weights stored in bfloat16 (16 bits of product) and one rounding otherwise."""
+in 32-bit, which is exact for weights stored in bfloat16 (16 bits of product) and one rounding otherwise.  `mult`: a constant
+on the norm's output (a factor on the logits of the head that reads it, for instance), folded into the weight the same way."""
 from __future__ import annotations
 
 from typing import List, Mapping, Optional
@@ -22,6 +23,7 @@ class RMSNorm(Norm):
         self.width = int(spec.params["width"])
         self.eps = float(spec.params["eps"])
         self.add_one = bool(spec.params.get("add_one", False))
+        self.mult = float(spec.params.get("mult", 1.0))
         self.weight: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> List[WeightSpec]:
@@ -36,6 +38,8 @@ class RMSNorm(Norm):
             # y * w * scale == y * (w * scale); with Gemma's convention the kernel adds one, so that is taken here
             scale = self._vector32(tensors[self.spec.weights["scale"]])
             self.weight = ((self.weight + 1.0) * scale - 1.0 if self.add_one else self.weight * scale).contiguous()
+        if self.mult != 1.0:
+            self.weight = ((self.weight + 1.0) * self.mult - 1.0 if self.add_one else self.weight * self.mult).contiguous()
 
     def forward(self, x: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         if out is None:

@@ -1,4 +1,4 @@
-"""Two mixers that keep a matrix state S [dim keys x vdim values] per head and sequence instead of keys and values.
+"""Mixers that keep a matrix state S [dim keys x vdim values] per head and sequence instead of keys and values.
 
 decay_linear_attention: q, k = act(W_q h), act(W_k h) (heads x dim), v = act(W_v h) (heads x vdim), act(x) = x
     logistic(x); per head S <- decay_h S + k v^T, o = S^T q with a constant decay per head and no other scale; the
@@ -14,6 +14,16 @@ gated_delta_rule: q, k (kv_heads x dim) and v (heads x vdim) each pass a short c
     key head h // (heads / kv_heads)):  S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.  Each head's o
     is divided by its root mean square, multiplied by a weight shared by the heads and by W_g h times its logistic
     function, and projected by W_o.
+
+channel_decay_attention: q = W_q h, k = W_k h (heads x dim), v = W_v h (heads x vdim) as projected; a decay per key channel
+    alpha = logistic(W_a2 (W_a1 h) + b)^(1 / tau).  Per head S <- diag(alpha) S + k v^T, o = dim^-1/2 S^T q; each head's o is
+    divided by its root mean square, multiplied by a weight shared by the heads and by W_g h times its logistic
+    function (`out_scale`: and by a constant), and projected by W_o.
+state_space: one projection gives [z | x | B | C | dt] (x, z: heads x vdim; B, C: groups x state; dt: heads).  x, B and C
+    pass a short causal convolution over time per channel with a bias, and x logistic(x); dt = softplus(dt + dt_bias).
+    Per head (head h reads group h // (heads / groups)):  S <- exp(-exp(A_log) dt) S + dt B x^T,  y = S^T C + D x.  The
+    heads' y, side by side, are multiplied by z logistic(z), then divided by their root mean square in `norm_groups`
+    equal parts and multiplied by a weight per column, and projected by W_o.
 
 The state (and the convolution's last taps - 1 inputs) is per-sequence state of fixed size: zero at a sequence's
 start, carried from step to step.  Everything between the projections and the output projection is 32-bit: the
@@ -187,5 +197,155 @@ class GatedDeltaRule(Mixer):
         return linear.matmul_or_partials(y, self.w_o) if partial_ok else linear.matmul(y, self.w_o)
 
 
+class ChannelDecayAttention(Mixer):
+    graph_safe = True
+    out_bias = None
+
+    def __init__(self, spec, rt):
+        super().__init__(spec, rt)
+        p = spec.params
+        self.width, self.n_heads = int(p["width"]), int(p["n_heads"])
+        self.dim, self.vdim, self.eps, self.tau = int(p["dim"]), int(p["vdim"]), float(p["eps"]), float(p["tau"])
+        self.rank = int(p["decay_rank"]) if p.get("decay_rank") else -1          # -1: the a1 tensor's shape gives it
+        self.out_scale = float(p.get("out_scale", 1.0))
+        if min(self.width, self.n_heads, self.dim, self.vdim) <= 0 or not self.tau > 0.0:
+            raise SpecError("arch spec error: the mixer with a decay per key channel needs positive sizes and a positive tau")
+        self.qk_cols, self.v_cols = self.n_heads * self.dim, self.n_heads * self.vdim
+
+    def weight_specs(self) -> List[WeightSpec]:
+        w = self.spec.weights
+        return [WeightSpec(w["q"], (self.qk_cols, self.width), "matrix", 0.05),
+                WeightSpec(w["k"], (self.qk_cols, self.width), "matrix", 0.05),
+                WeightSpec(w["v"], (self.v_cols, self.width), "matrix", 0.05),
+                WeightSpec(w["gate"], (self.v_cols, self.width), "matrix", 0.05),
+                WeightSpec(w["a1"], (self.rank, self.width), "matrix", 0.05),
+                WeightSpec(w["a2"], (self.qk_cols, self.rank), "matrix", 0.1),
+                WeightSpec(w["a2_bias"], (self.qk_cols,), "vector", 0.5),
+                WeightSpec(w["norm"], (self.vdim,), "vector", 0.1),
+                WeightSpec(w["o"], (self.width, self.v_cols), "matrix", 0.02)]
+
+    def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        w = self.spec.weights
+        mats = [self._matrix(tensors[w[r]]) for r in ("q", "k", "v", "gate", "a1")]
+        if len({m.dtype for m in mats}) > 1:
+            mats = [m.float() for m in mats]
+        self.bound_rank = mats[-1].shape[0]
+        if tensors[w["a2"]].shape[1] != self.bound_rank:
+            raise SpecError(f"arch spec error: the decay's two projections do not fit ({tuple(mats[-1].shape)}, "
+                            f"{tuple(tensors[w['a2']].shape)})")
+        self.w_in = torch.cat(mats, dim=0).contiguous()                          # q | k | v | gate | low-rank decay
+        self.a2_t = tensors[w["a2"]].to(torch.float32).t().contiguous()          # [rank, heads * dim]
+        self.a2_bias = self._vector32(tensors[w["a2_bias"]])
+        self.norm_w = (self._vector32(tensors[w["norm"]]) * self.out_scale).contiguous()
+        self.w_o = self._matrix(tensors[w["o"]])
+
+    def state_needs(self) -> List[StateNeed]:
+        return [StateNeed("S", (self.n_heads, self.vdim, self.dim), torch.float32)]      # kept as S^T per head
+
+    def forward(self, h, step: StepInfo, store: CallStore):
+        return linear.matmul(self._heads(h, step, store), self.w_o)
+
+    def forward_partial(self, h, step: StepInfo, store: CallStore):
+        return linear.matmul_or_partials(self._heads(h, step, store), self.w_o)
+
+    def _heads(self, h, step, store):
+        proj = linear.matmul(h, self.w_in, out_dtype=torch.float32)
+        y = torch.empty((h.shape[0], self.v_cols), dtype=h.dtype, device=h.device)
+        self.run_heads(proj, 0, step, store, y, 0)
+        return y
+
+    # the mixer between its projections (see parts/parallel_mixers.py)
+    @property
+    def in_cols(self) -> int:
+        return 2 * self.qk_cols + 2 * self.v_cols + self.bound_rank
+
+    @property
+    def out_cols(self) -> int:
+        return self.v_cols
+
+    def run_heads(self, proj, col: int, step: StepInfo, store: CallStore, y, out_col: int) -> None:
+        """From the projections (32-bit rows, columns from `col` on) to the gated heads in y's columns from out_col on."""
+        n, dev = proj.shape[0], proj.device
+        gate_col = col + 2 * self.qk_cols + self.v_cols
+        alpha = torch.empty((n, self.qk_cols), dtype=torch.float32, device=dev)
+        ops.channel_decay(proj, gate_col + self.v_cols, self.bound_rank, self.a2_t, self.a2_bias, self.tau, alpha)
+        o = torch.empty((n, self.v_cols), dtype=torch.float32, device=dev)
+        ops.state_scan(proj, col, col + self.qk_cols, col + 2 * self.qk_cols, False, alpha, True, None, store.state["S"], step, o,
+                       self.n_heads, self.n_heads, self.dim, self.vdim, channel_g=True, o_mult=float(self.dim) ** -0.5)
+        ops.group_norm_gate(o, self.norm_w, proj, gate_col, ops.ACT_X_LOGISTIC, step.token_seq, y, self.eps, self.n_heads, self.vdim,
+                            out_col)
+
+
+class StateSpace(Mixer):
+    graph_safe = True
+
+    def __init__(self, spec, rt):
+        super().__init__(spec, rt)
+        p = spec.params
+        self.width, self.n_heads, self.vdim = int(p["width"]), int(p["n_heads"]), int(p["vdim"])
+        self.state, self.groups, self.taps = int(p["state"]), int(p["groups"]), int(p["taps"])
+        self.norm_groups, self.eps = int(p["norm_groups"]), float(p["eps"])
+        if min(self.width, self.n_heads, self.vdim, self.state, self.groups, self.taps, self.norm_groups) <= 0 \
+                or self.n_heads % self.groups != 0 or (self.n_heads * self.vdim) % self.norm_groups != 0:
+            raise SpecError("arch spec error: the state-space mixer needs positive sizes, heads that are a multiple of its groups "
+                            "and an inner size that is a multiple of its norm groups")
+        self.inner, self.bc_cols = self.n_heads * self.vdim, self.groups * self.state
+        self.conv_cols = self.inner + 2 * self.bc_cols
+        self.rows = self.inner + self.conv_cols + self.n_heads
+
+    def weight_specs(self) -> List[WeightSpec]:
+        w = self.spec.weights
+        return [WeightSpec(w["in"], (self.rows, self.width), "matrix", 0.05),
+                WeightSpec(w["conv"], (self.conv_cols, self.taps), "matrix", 0.4),
+                WeightSpec(w["conv_bias"], (self.conv_cols,), "vector", 0.1),
+                WeightSpec(w["dt_bias"], (self.n_heads,), "vector", 0.5),
+                WeightSpec(w["A_log"], (self.n_heads,), "vector", 0.5),
+                WeightSpec(w["D"], (self.n_heads,), "vector", 0.5),
+                WeightSpec(w["norm"], (self.inner,), "vector", 0.1),
+                WeightSpec(w["o"], (self.width, self.inner), "matrix", 0.02)]
+
+    def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        w = self.spec.weights
+        self.w_in = linear.pad_rows(self._matrix(tensors[w["in"]]))              # z | x | B | C | dt
+        self.conv_w, self.conv_bias = tensors[w["conv"]].to(torch.float32).contiguous(), self._vector32(tensors[w["conv_bias"]])
+        self.dt_bias, self.a_log, self.skip = (self._vector32(tensors[w[r]]) for r in ("dt_bias", "A_log", "D"))
+        self.norm_w = self._vector32(tensors[w["norm"]])
+        self.w_o = self._matrix(tensors[w["o"]])
+
+    def state_needs(self) -> List[StateNeed]:
+        out = [StateNeed("S", (self.n_heads, self.vdim, self.state), torch.float32)]     # kept as S^T per head
+        if self.taps > 1:
+            out.append(StateNeed("conv", (self.taps - 1, self.conv_cols), torch.float32))
+        return out
+
+    def forward(self, h, step: StepInfo, store: CallStore):
+        return linear.matmul(self._heads(h, step, store), self.w_o)
+
+    def forward_partial(self, h, step: StepInfo, store: CallStore):
+        return linear.matmul_or_partials(self._heads(h, step, store), self.w_o)
+
+    def _heads(self, h, step, store):
+        n, dev = h.shape[0], h.device
+        raw = linear.matmul(h, self.w_in, out_dtype=torch.float32)
+        act = torch.empty((n, self.conv_cols), dtype=torch.float32, device=dev)
+        dt = torch.empty((n, self.n_heads), dtype=torch.float32, device=dev)
+        g = torch.empty_like(dt)
+        kept = store.state["conv"] if self.taps > 1 else raw.new_empty((0, 0, self.conv_cols))
+        single = step.max_new == 1           # every sequence brings one token: the kept inputs move on in the same launch
+        ops.conv_act_rows(raw, self.inner, self.conv_w, self.conv_bias, kept, "x_logistic", step, act, single,
+                          (self.inner + self.conv_cols, self.dt_bias, self.a_log, dt, g))
+        if self.taps > 1 and not single:
+            ops.conv_keep(raw, self.taps, kept, step, self.conv_cols, self.inner)
+        o = torch.empty((n, self.inner), dtype=torch.float32, device=dev)
+        ops.state_scan(act, self.inner + self.bc_cols, self.inner, 0, False, g, True, None, store.state["S"], step, o,
+                       self.n_heads, self.groups, self.state, self.vdim, v_factor=dt)
+        y = torch.empty((n, self.inner), dtype=h.dtype, device=dev)
+        ops.skip_gate_norm(o, act, 0, self.skip, raw, 0, self.norm_w, self.eps, step.token_seq, y, self.n_heads, self.vdim,
+                           self.norm_groups)
+        return y
+
+
+register_part("mixer", "channel_decay_attention", ChannelDecayAttention)
+register_part("mixer", "state_space", StateSpace)
 register_part("mixer", "decay_linear_attention", DecayLinearAttention)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)
