@@ -59,9 +59,10 @@ def query_factor(q_temp: Optional[dict], pos: int) -> float:
 
 def softmax_branch(m, w, p, h):
     T, H, G, d, vd = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    q = short_conv(h @ w[p + "q"].T + w[p + "q.b"], w[p + "q.conv"]).view(T, H, d)
-    k = short_conv(h @ w[p + "k"].T + w[p + "k.b"], w[p + "k.conv"]).view(T, G, d)
-    v = short_conv(h @ w[p + "v"].T + w[p + "v.b"], w[p + "v.conv"]).view(T, G, vd)
+    def channels(name):             # a layer whose constants name no taps has no convolution
+        u = h @ w[p + name].T + w[p + name + ".b"]
+        return short_conv(u, w[p + name + ".conv"]) if m.get("conv") else u
+    q, k, v = channels("q").view(T, H, d), channels("k").view(T, G, d), channels("v").view(T, G, vd)
     out = torch.zeros(T, H, vd, dtype=h.dtype)
     for i in range(T):
         lo = max(0, i + 1 - m["only_last"]) if m.get("only_last") else 0      # a test may take far keys away
