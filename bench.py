@@ -12,7 +12,7 @@ back to the host, where the loop reads them one step late.  `prefill` is one pro
 step must read (every weight once, and the cache of the live sequences) to its time.
 `points` holds decoding at batch 1 and 64.  One JSON line is printed.
 
-`--design satapel` (or `vagonex`, `fobilorn`, `tofodra`) is another measurement (not the line above): prompt and decode throughput of that design at
+`--design satapel` (or `vagonex`, `fobilorn`, `tofodra`, `ravutar`) is another measurement (not the line above): prompt and decode throughput of that design at
 a few sizes beside Gemma-2 at equal size, and each of the design's kernels against its roofline; one JSON line per size.
 With `--profile prefill|decode` it measures nothing and runs two such steps of one block of layers kernel by kernel, for a profiler.
 
@@ -577,13 +577,112 @@ def tofodra_kernel_work(z, tokens, batch, ctx):
     }
 
 
+# ---- --design ravutar: the Ravutar design beside Vagonex at equal size -----------------------------------
+# Layers (state space, side by side, state space, side by side) x blocks on four residual streams, dense feed-forwards with
+# biases.  The closest existing model is Vagonex (layers listed one by one, a matrix state behind short convolutions, the
+# same scan kernel, attention through the same grouped-query kernels, dense feed-forwards): "Vagonex at equal size" has the
+# same width, layer count and vocabulary, a delta-rule layer (short convolutions, as many cells of state) where Ravutar has
+# the first state-space layer of a block and a decay-rule layer where it has the second, attention of the same heads where
+# Ravutar has attention and linear attention side by side (in chunks longer than any measured sequence), and a gated
+# feed-forward of as many weights (two thirds as wide).
+RAVUTAR_SIZES = {
+    "s": dict(width=1024, vocab=32000, blocks=2, streams=4, ss_heads=32, ss_vdim=64, state=128, groups=1, conv=4, heads=8,
+              kv_heads=2, dim=128, vdim=128, lin_heads=8, lin_dim=64, lin_vdim=128, rank=16, ff=4096),
+    "m": dict(width=2048, vocab=32000, blocks=2, streams=4, ss_heads=64, ss_vdim=64, state=128, groups=1, conv=4, heads=16,
+              kv_heads=4, dim=128, vdim=128, lin_heads=16, lin_dim=64, lin_vdim=128, rank=16, ff=8192),
+    "l": dict(width=4096, vocab=64000, blocks=1, streams=4, ss_heads=128, ss_vdim=64, state=128, groups=8, conv=4, heads=32,
+              kv_heads=8, dim=128, vdim=128, lin_heads=32, lin_dim=64, lin_vdim=128, rank=16, ff=14336),
+}
+
+
+def ravutar_raw(z):
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    ss = {"heads": z["ss_heads"], "vdim": z["ss_vdim"], "state": z["state"], "groups": z["groups"], "conv": z["conv"], "norm_groups": 1}
+    both = {"left": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5,
+                     "conv": z["conv"], "q_temp": {"coef": 0.1, "every": 4096}},
+            "right": {"heads": z["lin_heads"], "dim": z["lin_dim"], "vdim": z["lin_vdim"], "tau": 16.0, "decay_rank": z["rank"]},
+            "left_scale": 1.0, "right_scale": 1.0}
+    layers = [{"type": "mamba2", "mixer": ss, "mlp": mlp}, {"type": "parallel", "mixer": both, "mlp": mlp}] * (2 * z["blocks"])
+    return {"architecture": "Ravutar", "vocab": z["vocab"], "width": z["width"], "streams": z["streams"], "norm": {"eps": 1e-6},
+            "logit_scale": 1.0, "layers": layers}
+
+
+def vagonex_raw_like_ravutar(z):
+    mlp = {"kind": "dense", "ff": z["ff"] * 2 // 3 // 64 * 64}
+    heads = z["ss_heads"] * z["ss_vdim"] // 128          # heads of 128 x 128: the same cells of state per layer
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5,
+                     "mask": {"size": 1 << 16}}}
+    dec = {"type": "lightning", "mlp": mlp, "mixer": {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -7] * heads}}
+    dlt = {"type": "delta", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": z["conv"]}}
+    return {"architecture": "Vagonex", "vocab": z["vocab"], "width": z["width"], "postln_alpha": 2.0, "norm": {"eps": 1e-6},
+            "embedding": {"scale": float(z["width"]) ** 0.5}, "layers": [dlt, att, dec, att] * z["blocks"]}
+
+
+def _both(fn, tokens, batch):
+    return {"prefill": fn(tokens, 1), "decode": fn(batch, batch)}
+
+
+def ravutar_kernel_work(z, tokens, batch, ctx):
+    """Per launch of each of the design's own kernels: (bytes that must move, FLOPs of the mathematics) for a prompt of
+    `tokens` tokens and for a decode step of `batch` sequences at length `ctx` (bfloat16 cache and products, 32-bit rows,
+    states and streams)."""
+    H, G, kd, vd, width, S = z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["width"], z["streams"]
+    pairs = tokens * (tokens + 1) // 2
+    attn = {"prefill": (tokens * G * (kd + vd) * 2 + tokens * H * (kd * 4 + vd * 2), 2.0 * pairs * H * (kd + vd)),
+            "decode": (batch * ctx * G * (kd + vd) * 2, 2.0 * batch * ctx * H * (kd + vd))}
+    sh, sv, N, g, t = z["ss_heads"], z["ss_vdim"], z["state"], z["groups"], z["conv"] - 1
+    inner, C = sh * sv, sh * sv + 2 * g * N
+    lh, ld, lv = z["lin_heads"], z["lin_dim"], z["lin_vdim"]
+    kept = lambda n, seqs, cols: seqs * 2 * t * cols * 4          # the convolution's kept inputs, in and out
+    return {
+        "hos_gated_attn": attn, "hos_gated_attn_mma": attn, "hos_gated_attn_mma_decode": attn,
+        # x, B, C rows and the step sizes in, read-outs out, the state in and out; update and read-out: 4 per cell
+        "hos_state_scan/v_factor": _both(lambda n, q: (n * (C + inner + 2 * sh) * 4 + q * sh * N * sv * 8, 4.0 * n * sh * N * sv), tokens, batch),
+        # q, k, v and the decays in
+        "hos_state_scan/channel": _both(lambda n, q: (n * (3 * lh * ld + 2 * lh * lv) * 4 + q * lh * ld * lv * 8, 4.0 * n * lh * ld * lv),
+                                        tokens, batch),
+        "hos_conv_act_rows": _both(lambda n, q: (n * C * 8 + (kept(n, q, C) if q == n else 0), 0.0), tokens, batch),
+        "hos_skip_gate_norm": _both(lambda n, q: (n * inner * 14, 0.0), tokens, batch),
+        "hos_group_norm_gate": _both(lambda n, q: (n * lh * lv * 10, 0.0), tokens, batch),
+        "hos_channel_decay": _both(lambda n, q: (n * (lh * ld + z["rank"]) * 4 + lh * ld * z["rank"] * 4, 2.0 * n * lh * ld * z["rank"]),
+                                   tokens, batch),
+        "hos_qk_prep": _both(lambda n, q: (n * (H * kd * 8 + G * (kd + vd) * 6) + (kept(n, q, H * kd + G * (kd + vd)) if q == n else 0), 0.0),
+                             tokens, batch),
+        # the streams in and out (32-bit), the branch's output in, the normed rows out
+        "hos_hyper_norm": _both(lambda n, q: (n * width * (8 * S + 4), 0.0), tokens, batch),
+    }
+
+
+def _vagonex_work_like_ravutar(z, tokens, batch, ctx):
+    """The compared model's kernels at the equal-size configuration; the scan's row is the mean of a delta-rule and a
+    decay-rule launch (as many of each)."""
+    H, G, kd, vd, width = z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["width"]
+    pairs = tokens * (tokens + 1) // 2
+    sh = z["ss_heads"] * z["ss_vdim"] // 128
+    cells, cols = sh * 128 * 128, 2 * (sh // 2) * 128 + sh * 128
+    attn = {"prefill": (tokens * G * (kd + vd) * 2 + tokens * H * (kd * 4 + vd * 2), 2.0 * pairs * H * (kd + vd)),
+            "decode": (batch * ctx * G * (kd + vd) * 2, 2.0 * batch * ctx * H * (kd + vd))}
+    return {
+        "hos_gated_attn": attn, "hos_gated_attn_mma": attn, "hos_gated_attn_mma_decode": attn,
+        "hos_state_scan": _both(lambda n, q: (n * (cols + 5 * sh * 128) * 2 + q * cells * 8, 5.5 * n * cells), tokens, batch),
+        "hos_conv_prep": _both(lambda n, q: (n * cols * 8 + (q * 2 * (z["conv"] - 1) * cols * 4 if q == n else 0), 0.0), tokens, batch),
+        "hos_group_norm_gate": _both(lambda n, q: (n * sh * 128 * 10, 0.0), tokens, batch),
+        "hos_qk_prep": _both(lambda n, q: (n * (H * kd * 8 + G * (kd + vd) * 6), 0.0), tokens, batch),
+        "hos_scale_add_norm": _both(lambda n, q: (n * width * 12, 0.0), tokens, batch),
+    }
+
+
 DESIGNS = {"fobilorn": lambda: (FOBILORN_SIZES, fobilorn_raw, gemma_raw_like_fobilorn, fobilorn_kernel_work,
                                 ("hos_gated_attn",)),
            "satapel": lambda: (SATAPEL_SIZES, satapel_raw, gemma_raw_like, satapel_kernel_work, ("hos_wkv_scan",)),
            "vagonex": lambda: (VAGONEX_SIZES, vagonex_raw, gemma_raw_like_vagonex, vagonex_kernel_work,
                                ("hos_state_scan", "hos_gated_attn")),
            "tofodra": lambda: (TOFODRA_SIZES, tofodra_raw, vagonex_raw_like_tofodra, tofodra_kernel_work,
-                               ("hos_state_scan", "hos_gated_attn"))}
+                               ("hos_state_scan", "hos_gated_attn")),
+           "ravutar": lambda: (RAVUTAR_SIZES, ravutar_raw, vagonex_raw_like_ravutar, ravutar_kernel_work,
+                               ("hos_state_scan", "hos_state_scan/channel", "hos_state_scan/v_factor", "hos_gated_attn",
+                                "hos_channel_decay"))}
 
 
 def _vagonex_work_like_tofodra(z, tokens, batch, ctx):
@@ -605,8 +704,8 @@ def _vagonex_work_like_tofodra(z, tokens, batch, ctx):
             "hos_scale_add_norm": {"prefill": (tokens * z["width"] * 12, 0.0), "decode": (batch * z["width"] * 12, 0.0)}}
 
 
-OTHER_WORK = {"tofodra": _vagonex_work_like_tofodra}
-OTHER_ARM = {"tofodra": "vagonex_equal_size"}      # the closest existing model per design (Gemma-2 where none is named)
+OTHER_WORK = {"tofodra": _vagonex_work_like_tofodra, "ravutar": _vagonex_work_like_ravutar}
+OTHER_ARM = {"tofodra": "vagonex_equal_size", "ravutar": "vagonex_equal_size"}      # the closest existing model per design (Gemma-2 where none is named)
 
 
 def run_design_profile_step(args) -> int:

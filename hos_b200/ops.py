@@ -125,7 +125,8 @@ class Library:
             self._fns[name] = f
         return f
 
-    def call(self, name: str, *args, signature: Optional[str] = None) -> None:
+    def call(self, name: str, *args, signature: Optional[str] = None, label: Optional[str] = None) -> None:
+        """`label`: what the measurement aid below calls it (a function that runs several kinds of work)."""
         global launch_count
         launch_count += 1
         if _call_times is not None:
@@ -133,7 +134,7 @@ class Library:
             e0.record()
             rc = self.fn(name, signature)(*args)
             e1.record()
-            _call_times.append((name, e0, e1))
+            _call_times.append((label or name, e0, e1))
         else:
             rc = self.fn(name, signature)(*args)
         if rc != 0:
@@ -1148,7 +1149,8 @@ def state_scan(rows: torch.Tensor, q_col: int, k_col: int, v_col: int, silu_on_l
                   _ptr(second), heads if second is not None else 0, _ptr(state), _ptr(step.token_pos), _ptr(step.token_seq),
                   _ptr(step.cu_seqlens), _ptr(step.seq_slot), _ptr(out), n, int(step.n_seqs), int(heads), int(key_heads),
                   int(dim), int(vdim), _ptr(rot[0]) if rot else None, int(rot[1]) if rot else 0, int(rot[2]) if rot else 0,
-                  float(rot[3]) if rot else 1.0, _stream())
+                  float(rot[3]) if rot else 1.0, _stream(),
+                  label="hos_state_scan/channel" if channel_g else ("hos_state_scan/v_factor" if v_factor is not None else None))
 
 
 def act_rows(rows: torch.Tensor, cols: int) -> None:
