@@ -647,7 +647,7 @@ def ravutar_kernel_work(z, tokens, batch, ctx):
         "hos_group_norm_gate": _both(lambda n, q: (n * lh * lv * 10, 0.0), tokens, batch),
         "hos_channel_decay": _both(lambda n, q: (n * (lh * ld + z["rank"]) * 4 + lh * ld * z["rank"] * 4, 2.0 * n * lh * ld * z["rank"]),
                                    tokens, batch),
-        "hos_qk_prep": _both(lambda n, q: (n * (H * kd * 8 + G * (kd + vd) * 6) + (kept(n, q, H * kd + G * (kd + vd)) if q == n else 0), 0.0),
+        "hos_qkv_conv_store": _both(lambda n, q: (n * (H * kd * 8 + G * (kd + vd) * 6) + (kept(n, q, H * kd + G * (kd + vd)) if q == n else 0), 0.0),
                              tokens, batch),
         # the streams in and out (32-bit), the branch's output in, the normed rows out
         "hos_hyper_norm": _both(lambda n, q: (n * width * (8 * S + 4), 0.0), tokens, batch),

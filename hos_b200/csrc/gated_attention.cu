@@ -10,9 +10,11 @@
 //   (2i, 2i+1) by the angle position * freq[i], cosine and sine times `magnitude`; queries are written as 32-bit
 //   rows, keys and values (in the cache's type) to their places in the paged cache.  With v_first the values
 //   are first blended with another layer's values of the same token, v <- (1 - v_mix) v + v_mix v_first, and the
-//   blend is what the cache holds.  With a short convolution (conv.w) every channel of q, k and v passes one over
-//   time right after the projection and its bias; its last inputs are the slot's state.  With q_every > 0 a query at
-//   position p is multiplied by 1 + q_coef ln(floor((p + 1) / q_every) + 1) at the end.
+//   blend is what the cache holds.  With q_every > 0 a query at position p is multiplied by 1 + q_coef ln(floor((p + 1) /
+//   q_every) + 1) at the end.
+// qkv_conv_store: the same without norms, rotation and blending for projections whose channels each pass a short causal
+//   convolution over time right after their bias (conv_walk in short_conv.cuh): a thread takes four channels of a run of
+//   rows and writes the queries (with their factor) or the cache.
 // gated_attn: one warp per (token, up to 8 query heads that share a kv head, share of the keys).  A lane takes a
 //   key: 32 scores per head at a time, then the lanes turn to the value columns; a key or value row is read once
 //   for all of the warp's heads.  Keys j of position i: j <= i and, with chunks of size C,
@@ -37,25 +39,20 @@ struct PagedKV2 {            // keys [n_pages][n_kv][64][kd], values [n_pages][n
 
 __device__ __forceinline__ int table_entry(const PagedKV2& c, int lp) { return c.ring_pages > 0 ? lp % c.ring_pages : lp; }
 
+// 1 + coef ln(floor((pos + 1) / every) + 1), or 1 without a step
+__device__ __forceinline__ float query_factor(int pos, float coef, int every) {
+    return every > 0 ? 1.f + coef * logf((float)((pos + 1) / every + 1)) : 1.f;
+}
+
 constexpr int kPrepMaxPL = 16;    // a head of up to 32 * 16 numbers in a warp's registers
 
-// The short convolution of the q, k and v channels: w [taps][C] over the row's first C = H kd + G (kd + vd) columns.
-struct QkvConv {
-    const float* w;           // null: no convolution
-    const float* keep;        // [slots][taps - 1][C]
-    float* keep_w;            // the same memory where the kept inputs move on in this launch, else null
-    const int* cu_seqlens;
-    int taps;
-};
-
-template <typename TC, int kPrepPL, int kThreads, bool CONV>
+template <typename TC, int kPrepPL, int kThreads>
 __global__ void __launch_bounds__(kThreads)
 qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ bias, const float* __restrict__ q_norm,
                const float* __restrict__ k_norm, float eps, const float* __restrict__ freq, int rot_dims, float magnitude,
                const int* __restrict__ token_pos, const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
                float* __restrict__ q_out, PagedKV2 cache, int H, int G, int kd, int vd, int norm_whole,
-               const float* __restrict__ v_first, long long v_first_ld, float v_mix, int q_maps, QkvConv conv, float q_coef,
-               int q_every) {
+               const float* __restrict__ v_first, long long v_first_ld, float v_mix, int q_maps, float q_coef, int q_every) {
     pdl_enter();
     __shared__ float scratch[32];
     const int n = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -70,19 +67,7 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
     const int slot = seq_slot[seq];
     const int page = G > 0 ? cache.page_table[(size_t)slot * cache.table_stride + table_entry(cache, pos / kPageTokens)] : 0;
     const int r = pos % kPageTokens;
-    // The row that tap j of the convolution reads, from column 0 on: a row of this step (as projected, the bias is still to
-    // be added), one of the slot's kept inputs, or null before the sequence's start.
-    const int conv_C = H * kd + G * (kd + vd);
-    const int conv_r0 = CONV ? conv.cu_seqlens[seq] : 0;
-    const bool conv_fresh = CONV ? token_pos[conv_r0] == 0 : false;
-    const size_t keep_at = CONV ? (size_t)slot * (conv.taps - 1) * conv_C : 0;
-    auto tap_row = [&](int j, bool& raw) -> const float* {
-        const int src = n - (conv.taps - 1) + j;
-        raw = src >= conv_r0;
-        if (raw) return proj + (size_t)src * ld;
-        return conv_fresh ? nullptr : conv.keep + keep_at + (size_t)((conv.taps - 1) + (src - conv_r0)) * conv_C;
-    };
-    const float q_mult = q_every > 0 ? 1.f + q_coef * logf((float)((pos + 1) / q_every + 1)) : 1.f;
+    const float q_mult = query_factor(pos, q_coef, q_every);
     float inv_all[2] = {0.f, 0.f};                       // norm_whole: one root mean square for all q heads, one for all k heads
     if (norm_whole) {
         for (int part = 0; part < (G > 0 ? 2 : 1); ++part) {
@@ -104,34 +89,12 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
         if (nw != nullptr && norm_whole) nw += (is_q ? item : item - H) * kd;
         float v[kPrepPL];
         float ss = 0.f;
-        if (CONV) {
 #pragma unroll
-            for (int i = 0; i < kPrepPL; ++i) v[i] = 0.f;
-#pragma unroll 1
-            for (int j = 0; j < conv.taps; ++j) {
-                bool raw;
-                const float* src = tap_row(j, raw);
-                // the kept inputs move on: row j - 1 was read in the turn before, by this thread
-                float* kw = conv.keep_w != nullptr && j >= 1 ? conv.keep_w + keep_at + (size_t)(j - 1) * conv_C + col0 : nullptr;
-#pragma unroll
-                for (int i = 0; i < kPrepPL; ++i) {
-                    const int d = lane + 32 * i;
-                    if (d < kd) {
-                        const float x = src == nullptr ? 0.f : src[col0 + d] + (raw && bias ? bias[col0 + d] : 0.f);
-                        v[i] = fmaf(conv.w[(size_t)j * conv_C + col0 + d], x, v[i]);
-                        if (kw != nullptr) kw[d] = x;
-                    }
-                }
-            }
-        } else {
-#pragma unroll
-            for (int i = 0; i < kPrepPL; ++i) {
-                const int d = lane + 32 * i;
-                v[i] = d < kd ? row[col0 + d] + (bias ? bias[col0 + d] : 0.f) : 0.f;
-            }
+        for (int i = 0; i < kPrepPL; ++i) {
+            const int d = lane + 32 * i;
+            v[i] = d < kd ? row[col0 + d] + (bias ? bias[col0 + d] : 0.f) : 0.f;
+            ss = fmaf(v[i], v[i], ss);
         }
-#pragma unroll
-        for (int i = 0; i < kPrepPL; ++i) ss = fmaf(v[i], v[i], ss);
         if (nw != nullptr) {
             ss = warp_sum(ss);
             const float inv = norm_whole ? inv_all[is_q ? 0 : 1] : 1.f / sqrtf(ss / (float)kd + eps);
@@ -189,23 +152,64 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
         for (int i = threadIdx.x; i < G * vd; i += blockDim.x) {
             const int g = i / vd, d = i % vd;
             TC* vp = (TC*)cache.v_pages + ((size_t)page * G + g) * (size_t)kPageTokens * vd;
-            float x = 0.f;
-            if (CONV) {
-#pragma unroll 1
-                for (int j = 0; j < conv.taps; ++j) {
-                    bool raw;
-                    const float* src = tap_row(j, raw);
-                    const float u = src == nullptr ? 0.f : src[col0 + i] + (raw && bias ? bias[col0 + i] : 0.f);
-                    x = fmaf(conv.w[(size_t)j * conv_C + col0 + i], u, x);
-                    if (conv.keep_w != nullptr && j >= 1) conv.keep_w[keep_at + (size_t)(j - 1) * conv_C + col0 + i] = u;
-                }
-            } else {
-                x = row[col0 + i] + (bias ? bias[col0 + i] : 0.f);
-            }
+            float x = row[col0 + i] + (bias ? bias[col0 + i] : 0.f);
             if (v_first != nullptr) x = fmaf(v_mix, v_first[(size_t)n * v_first_ld + i], (1.f - v_mix) * x);
             vp[kv_elem_offset(r, d, vd)] = from_float<TC>(x);
         }
     }
+}
+
+// Four consecutive numbers of a cache row (d a multiple of four: never across a permuted group), or one.
+template <int VEC>
+__device__ __forceinline__ void cache_store(float* base, int r, int d, int width, const float (&y)[VEC]) {
+    conv_store<VEC>(base + kv_elem_offset(r, d, width), y);
+}
+template <int VEC>
+__device__ __forceinline__ void cache_store(bf16* base, int r, int d, int width, const float (&y)[VEC]) {
+    bf16* p = base + kv_elem_offset(r, d, width);
+    if constexpr (VEC == 4) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(y[0], y[1]), b = __floats2bfloat162_rn(y[2], y[3]);
+        *(uint2*)p = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    } else {
+        *p = from_float<bf16>(y[0]);
+    }
+}
+
+template <typename TC, int TAPS, int VEC>
+__global__ void __launch_bounds__(128)
+qkv_conv_store_kernel(ConvWalk c, float* __restrict__ q_out, PagedKV2 cache, int N, int run, int H, int G, int kd, int vd,
+                      float q_coef, int q_every) {
+    pdl_enter();
+    const int n0 = blockIdx.y * run, n1 = min(N, n0 + run);
+    const int ch = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (ch >= c.C) return;
+    const int k0 = H * kd, v0 = k0 + G * kd;
+    const bool is_q = ch < k0, is_k = !is_q && ch < v0;
+    const int at = is_k ? ch - k0 : ch - v0, width = is_k ? kd : vd;
+    const int g = is_q ? 0 : at / width, d = is_q ? 0 : at % width;
+    TC* pages = (TC*)(is_k ? cache.k_pages : cache.v_pages);
+    conv_walk<TAPS, VEC>(
+        c, ch, n0, n1,
+        [&](int n, float (&y)[VEC]) {
+            const int pos = c.token_pos[n];
+            if (is_q) {
+                const float m = query_factor(pos, q_coef, q_every);
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) y[v] *= m;
+                conv_store<VEC>(q_out + (size_t)n * k0 + ch, y);
+                return;
+            }
+            const int slot = c.seq_slot[c.token_seq[n]];
+            const int page = cache.page_table[(size_t)slot * cache.table_stride + table_entry(cache, pos / kPageTokens)];
+            cache_store<VEC>(pages + ((size_t)page * G + g) * (size_t)kPageTokens * width, pos % kPageTokens, d, width, y);
+        },
+        [&](int n) {
+            if (!is_q) return;
+            float y[VEC];
+#pragma unroll
+            for (int v = 0; v < VEC; ++v) y[v] = 0.f;
+            conv_store<VEC>(q_out + (size_t)n * k0 + ch, y);
+        });
 }
 
 constexpr int kAttnWarps = 4;
@@ -478,20 +482,14 @@ extern "C" const char* hos_last_error() { return error_buffer(); }
 // columns' biases or null.  q_norm / k_norm: [kd] or null (norm_whole: [H * kd] and [G * kd]).  freq: [rot_dims / 2] or
 // null.  v_first: row n's values of another layer at v_first[n * v_first_ld + ...] (G * vd numbers), or null.
 // q_maps > 1: q_out is [N][H * q_maps][kd]: each head's kd numbers are q_maps queries, written as heads of their own.
-// conv_w ([taps][C], C = H kd + G (kd + vd), or null): the short convolution of q, k and v with its kept inputs conv_state [slots]
-// [taps - 1][C]; keep_here: 1 only where every sequence of the step brings exactly one token (the kept inputs move on
-// inside this launch; otherwise hos_qkv_conv_keep does it afterwards).  q_every > 0: the queries' factor by position.
+// q_every > 0: the queries' factor by position.
 extern "C" int hos_qk_prep(const float* proj, int ld, const float* bias, const float* q_norm, const float* k_norm, float eps,
                            const float* freq, int rot_dims, float magnitude, const int* token_pos, const int* token_seq,
                            const int* seq_slot, float* q_out, void* k_pages, void* v_pages, int cache_dtype,
                            const int* page_table, int table_stride, int ring_pages, int N, int H, int G, int kd, int vd,
                            int norm_whole, const float* v_first, long long v_first_ld, float v_mix, int q_maps,
-                           const float* conv_w, int taps, float* conv_state, const int* cu_seqlens, int keep_here, float q_coef,
-                           int q_every, cudaStream_t stream) {
+                           float q_coef, int q_every, cudaStream_t stream) {
     if (N <= 0) return 0;
-    if (conv_w != nullptr && (taps < 1 || taps > kMaxTaps || norm_whole || cu_seqlens == nullptr || (taps > 1 && conv_state == nullptr)))
-        HOS_REFUSE("qk_prep: a convolution of %d taps (1..%d; not with a norm over the whole projection)", taps, kMaxTaps);
-    const QkvConv conv{conv_w, conv_state, keep_here && taps > 1 ? conv_state : nullptr, cu_seqlens, taps};
     if (q_maps < 1 || kd % q_maps != 0) HOS_REFUSE("qk_prep: heads of %d numbers do not hold %d queries", kd, q_maps);
     if (kd <= 0 || kd > 32 * kPrepMaxPL) HOS_REFUSE("qk_prep: heads of %d numbers are outside 1..%d", kd, 32 * kPrepMaxPL);
     if (freq == nullptr) rot_dims = 0;
@@ -499,15 +497,10 @@ extern "C" int hos_qk_prep(const float* proj, int ld, const float* bias, const f
     PagedKV2 c{k_pages, v_pages, page_table, table_stride, ring_pages, G, kd, vd};
     // few rows (single-token steps): a block of 16 warps shortens the row's chain of loads; many rows: 4 warps
     const bool wide = N <= 592 && H + G > 4;
-#define HOS_QKP_C(TC, PL, NT, CV)                                                                                    \
-    launch_pdl(qk_prep_kernel<TC, PL, NT, CV>, dim3(N), dim3(NT), 0, stream, proj, ld, bias, q_norm, k_norm, eps, freq, \
-               rot_dims, magnitude, token_pos, token_seq, seq_slot, q_out, c, H, G, kd, vd, norm_whole, v_first,     \
-               v_first_ld, v_mix, q_maps, conv, q_coef, q_every)
 #define HOS_QKP_N(TC, PL, NT)                                                                                        \
-    do {                                                                                                             \
-        if (conv_w != nullptr) HOS_QKP_C(TC, PL, NT, true);                                                          \
-        else HOS_QKP_C(TC, PL, NT, false);                                                                           \
-    } while (0)
+    launch_pdl(qk_prep_kernel<TC, PL, NT>, dim3(N), dim3(NT), 0, stream, proj, ld, bias, q_norm, k_norm, eps, freq,   \
+               rot_dims, magnitude, token_pos, token_seq, seq_slot, q_out, c, H, G, kd, vd, norm_whole, v_first,     \
+               v_first_ld, v_mix, q_maps, q_coef, q_every)
 #define HOS_QKP(TC, PL)                                                                                              \
     do {                                                                                                             \
         if (wide) HOS_QKP_N(TC, PL, 512);                                                                            \
@@ -526,19 +519,45 @@ extern "C" int hos_qk_prep(const float* proj, int ld, const float* bias, const f
 #undef HOS_QKP_T
 #undef HOS_QKP
 #undef HOS_QKP_N
-#undef HOS_QKP_C
     return check_launch("qk_prep");
 }
 
-// The last taps - 1 inputs (with their bias) of every sequence's q, k, v channels go to the slot's state.
-extern "C" int hos_qkv_conv_keep(const float* proj, long long ld, const float* bias, int taps, float* conv_state,
-                                 const int* token_pos, const int* token_seq, const int* cu_seqlens, const int* seq_slot,
-                                 int n_seqs, int C, cudaStream_t stream) {
-    if (n_seqs <= 0 || taps <= 1) return 0;
-    if (taps > kMaxTaps) HOS_REFUSE("qkv_conv_keep: %d taps are outside 1..%d", taps, kMaxTaps);
-    launch_pdl(short_conv_keep_kernel, dim3((C + 127) / 128, n_seqs), dim3(128), 0, stream, proj, ld, bias, taps, conv_state,
-               token_pos, token_seq, cu_seqlens, seq_slot, C);
-    return check_launch("qkv_conv_keep");
+// proj: float32 [N][ld] from the first q column on: q (H * kd) | k (G * kd) | v (G * vd), C = H kd + G (kd + vd) channels; w:
+// [taps][C], bias: [C] (before the convolution) or null; conv_state: [slots][taps - 1][C]; single: 1 where every sequence of
+// the step brings exactly one token (the kept inputs then move on inside this launch).  q_out: float32 [N][H][kd].
+extern "C" int hos_qkv_conv_store(const float* proj, long long ld, const float* bias, const float* w, int taps, float* conv_state,
+                                  int single, const int* token_pos, const int* token_seq, const int* cu_seqlens, const int* seq_slot,
+                                  float* q_out, void* k_pages, void* v_pages, int cache_dtype, const int* page_table, int table_stride,
+                                  int ring_pages, int N, int H, int G, int kd, int vd, float q_coef, int q_every, cudaStream_t stream) {
+    if (N <= 0) return 0;
+    if (taps < 1 || taps > kMaxTaps) HOS_REFUSE("qkv_conv_store: %d taps are outside 1..%d", taps, kMaxTaps);
+    if (H <= 0 || G <= 0 || kd <= 0 || vd <= 0) HOS_REFUSE("qkv_conv_store: %d heads over %d of %d and %d numbers", H, G, kd, vd);
+    const int C = H * kd + G * (kd + vd);
+    const bool vec = taps >= 2 && taps <= 4 && kd % 4 == 0 && vd % 4 == 0 && ld % 4 == 0 &&
+                     (((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)w | (uintptr_t)conv_state | (uintptr_t)q_out | (uintptr_t)k_pages |
+                       (uintptr_t)v_pages) % 16) == 0;
+    const int per_block = 128 * (vec ? 4 : 1);
+    const int blocks = (C + per_block - 1) / per_block;
+    const int run = conv_run(N, blocks, single != 0);
+    const dim3 grid(blocks, (N + run - 1) / run);
+    if (grid.y > 65535) HOS_REFUSE("qkv_conv_store: %d rows are more than one launch takes", N);
+    const ConvWalk c{proj, ld, w, bias, conv_state, single && taps > 1 ? conv_state : nullptr, token_pos, token_seq, cu_seqlens,
+                     seq_slot, taps, C};
+    PagedKV2 kv{k_pages, v_pages, page_table, table_stride, ring_pages, G, kd, vd};
+#define HOS_QCS(TC, T, V)                                                                                            \
+    launch_pdl(qkv_conv_store_kernel<TC, T, V>, grid, dim3(128), 0, stream, c, q_out, kv, N, run, H, G, kd, vd, q_coef, q_every)
+#define HOS_QCS_T(TC)                                                                                                \
+    do {                                                                                                             \
+        if (vec && taps == 2) HOS_QCS(TC, 2, 4);                                                                     \
+        else if (vec && taps == 3) HOS_QCS(TC, 3, 4);                                                                \
+        else if (vec) HOS_QCS(TC, 4, 4);                                                                             \
+        else HOS_QCS(TC, 0, 1);                                                                                      \
+    } while (0)
+    if (cache_dtype == kBF16) HOS_QCS_T(bf16);
+    else HOS_QCS_T(float);
+#undef HOS_QCS_T
+#undef HOS_QCS
+    return check_launch("qkv_conv_store");
 }
 
 // q: float32 [N][H][kd].  out: H * vd numbers of out_dtype from the start of rows that lie ldo apart, the heads' outputs times

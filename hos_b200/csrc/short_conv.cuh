@@ -26,6 +26,117 @@ __device__ __forceinline__ float short_conv(const float* raw, long long ld, floa
     return acc;
 }
 
+template <int VEC>
+__device__ __forceinline__ void conv_load(const float* p, float (&x)[VEC]) {
+    if constexpr (VEC == 4) {
+        const float4 t = *(const float4*)p;
+        x[0] = t.x; x[1] = t.y; x[2] = t.z; x[3] = t.w;
+    } else {
+        x[0] = *p;
+    }
+}
+template <int VEC>
+__device__ __forceinline__ void conv_store(float* p, const float (&x)[VEC]) {
+    if constexpr (VEC == 4) *(float4*)p = make_float4(x[0], x[1], x[2], x[3]);
+    else *p = x[0];
+}
+
+constexpr int kConvTokens = 16;      // consecutive rows that a thread walks at most
+
+// What a walk needs to know.  w: [taps][C]; in_bias (or null): [C], added to the rows' columns before the convolution;
+// keep / keep_w: as in short_conv above, from slot 0 on.
+struct ConvWalk {
+    const float* raw;
+    long long ld;
+    const float* w;
+    const float* in_bias;
+    const float* keep;
+    float* keep_w;
+    const int* token_pos;
+    const int* token_seq;
+    const int* cu_seqlens;
+    const int* seq_slot;
+    int taps, C;
+};
+
+// The convolution of VEC channels from ch on, over rows n0 .. n1 - 1, with the inputs in sight in registers, so that a
+// column is read once; a sequence's first row, or the walk's, fetches the ones before it from the rows or the slot's kept
+// inputs.  emit(n, y) takes every live row's result, pad(n) the padding rows.
+template <int TAPS, int VEC, typename Emit, typename Pad>
+__device__ __forceinline__ void conv_walk(const ConvWalk& c, int ch, int n0, int n1, Emit emit, Pad pad) {
+    const int taps = TAPS > 0 ? TAPS : c.taps;
+    constexpr int MAXT = TAPS > 0 ? TAPS : kMaxTaps;
+    float wr[MAXT][VEC], win[MAXT][VEC], b[VEC];
+#pragma unroll
+    for (int v = 0; v < VEC; ++v) b[v] = 0.f;
+    if (c.in_bias != nullptr) conv_load<VEC>(c.in_bias + ch, b);
+#pragma unroll
+    for (int j = 0; j < MAXT; ++j) {
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) wr[j][v] = win[j][v] = 0.f;
+        if (j < taps) conv_load<VEC>(c.w + (size_t)j * c.C + ch, wr[j]);
+    }
+    int last_seq = -2;
+    for (int n = n0; n < n1; ++n) {
+        const int seq = c.token_seq[n];
+        if (seq < 0) {
+            pad(n);
+            last_seq = -2;
+            continue;
+        }
+        float x[VEC];
+        conv_load<VEC>(c.raw + (size_t)n * c.ld + ch, x);
+        if (seq != last_seq) {                   // win[j] (j >= 1) holds the input taps - j back; it moves down by one below
+            const int r0 = c.cu_seqlens[seq];
+            const bool fresh = c.token_pos[r0] == 0;
+            const float* keep = c.keep + (size_t)c.seq_slot[seq] * (taps - 1) * c.C + ch;
+#pragma unroll
+            for (int j = 1; j < MAXT; ++j) {
+                if (j >= taps) continue;
+                const int src = n - taps + j;
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) win[j][v] = 0.f;
+                if (src >= r0) {
+                    conv_load<VEC>(c.raw + (size_t)src * c.ld + ch, win[j]);
+#pragma unroll
+                    for (int v = 0; v < VEC; ++v) win[j][v] += b[v];
+                } else if (!fresh) {
+                    conv_load<VEC>(keep + (size_t)((taps - 1) + (src - r0)) * c.C, win[j]);
+                }
+            }
+            last_seq = seq;
+        }
+        float y[VEC];
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) {
+            float acc = 0.f;
+            x[v] += b[v];
+#pragma unroll
+            for (int j = 0; j < MAXT; ++j) {
+                if (j + 1 < taps) win[j][v] = win[j + 1 < MAXT ? j + 1 : j][v];
+                else if (j + 1 == taps) win[j][v] = x[v];
+                if (j < taps) acc = fmaf(wr[j][v], win[j][v], acc);
+            }
+            y[v] = acc;
+        }
+        emit(n, y);
+        if (c.keep_w != nullptr) {               // single tokens: the kept inputs (the last taps - 1 in sight) move on here
+            float* keep = c.keep_w + (size_t)c.seq_slot[seq] * (taps - 1) * c.C + ch;
+#pragma unroll
+            for (int j = 1; j < MAXT; ++j)
+                if (j < taps) conv_store<VEC>(keep + (size_t)(j - 1) * c.C, win[j]);
+        }
+    }
+}
+
+// How many rows a thread walks: runs as long as leave every SM several blocks; a single-token step's rows are sequences of
+// their own.
+inline int conv_run(int N, int blocks, bool single) {
+    int run = 1;
+    while (!single && run < kConvTokens && (long long)((N + 2 * run - 1) / (2 * run)) * blocks >= 4 * sm_count_cached()) run *= 2;
+    return run;
+}
+
 // The last taps - 1 inputs of every sequence of the step go to the slot's kept inputs: a thread per (sequence, channel).
 // raw: the rows from the first channel's column on; bias: [C] or null.
 static __global__ void short_conv_keep_kernel(const float* __restrict__ raw, long long ld, const float* __restrict__ bias, int taps,

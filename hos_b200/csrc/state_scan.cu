@@ -11,7 +11,11 @@
 // state_scan: one block per (sequence, head, run of value columns); a column of S is cut into R runs of DR rows,
 //   one thread each (R lanes side by side, so that sums over a column are shuffles); tokens in order, a chunk of
 //   them staged in shared memory while the chunk before it is walked (cp.async, two buffers).  Columns are
-//   independent of one another in both rules.
+//   independent of one another in all rules.
+//   A long sequence of the decay or the channel rule (whose state at a segment's end is linear in the state at its start,
+//   cell by cell) is cut into segments that are walked side by side: first every segment from a zero state (its first
+//   one from the sequence's), without read-outs, leaving its state and the product of its decays; then segment_starts
+//   turns those into the states at the segments' starts, and a second walk from these makes the read-outs.
 // act_rows: x logistic(x) in place on the leading columns of 32-bit rows (the decay rule's q, k, v).
 // rotate_rows: rotary positions in place on the q and k heads of 32-bit rows (either pairing, the first rot_dims
 //   numbers of a head; angle = position * freq in 32-bit, sincosf), the keys then multiplied by a constant.
@@ -89,22 +93,43 @@ rotate_rows_kernel(float* __restrict__ x, long long ld, int Hq, int Hk, int dim,
     }
 }
 
+constexpr int kDecayPerThread = 4;
+
 enum ScanRule : int { kDecayRule = 0, kDeltaRule = 1, kChannelRule = 2 };
 
-template <int DR, int R, int RULE>
+// What a walk by segments needs: seg_len rows to a segment, `count` segments to a sequence at most (blockIdx.x is sequence x
+// count + segment; count 1: the whole sequence); states: [sequences][count][H][vdim][dim]; decays: [sequences][count][H]
+// (channel rule: [H][dim]).
+struct Segments {
+    float* states;
+    float* decays;
+    int len, count;
+};
+
+template <int DR, int R, int RULE, bool LOCAL>
 __global__ void __launch_bounds__(256)
 state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, long long ld,
                   int aligned, int act_in_walk, const float* __restrict__ g, long long g_ld, const float* __restrict__ beta,
                   long long beta_ld, float* __restrict__ state, const int* __restrict__ token_pos,
                   const int* __restrict__ token_seq, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
                   float* __restrict__ out, int H, int Gk, int dim, int vdim, int CC, const float* __restrict__ rot_freq,
-                  int rot_dims, int rot_style, float k_mult, float o_mult) {
+                  int rot_dims, int rot_style, float k_mult, float o_mult, Segments sg) {
     constexpr bool DELTA = RULE == kDeltaRule, CHANNEL = RULE == kChannelRule;
     pdl_enter();
     extern __shared__ __align__(16) float sm[];
-    const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * CC;
-    const int lo = cu_seqlens[seq], hi = cu_seqlens[seq + 1];
+    const int seq = blockIdx.x / sg.count, seg = blockIdx.x % sg.count, head = blockIdx.y, col0 = blockIdx.z * CC;
+    int lo = cu_seqlens[seq], hi = cu_seqlens[seq + 1];
     if (hi <= lo || token_seq[lo] < 0) return;
+    const bool fresh = token_pos[lo] == 0;
+    bool last = true;
+    if (sg.count > 1) {
+        const int end = hi;
+        lo += seg * sg.len;
+        if (lo >= end) return;
+        hi = min(end, lo + sg.len);
+        last = hi == end;
+        if (LOCAL && last) return;               // nothing starts from the last segment's state but the slot's, which the second walk makes
+    }
     const int slot = seq_slot[seq];
     const int kh = head / (H / Gk);
     const int r = threadIdx.x % R, c = threadIdx.x / R;
@@ -117,19 +142,25 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
     const bool v_scaled = RULE == kDecayRule && beta != nullptr;
 
     float S[DR];
-    float* st = state + (((size_t)slot * H + head) * vdim + (live ? col : 0)) * dim + r * DR;
-    const bool fresh = token_pos[lo] == 0;
+    const size_t cell = ((size_t)head * vdim + (live ? col : 0)) * dim + r * DR, cells = (size_t)H * vdim * dim;
+    float* st = state + (size_t)slot * cells + cell;                                  // the slot's
+    float* seg_st = sg.states + ((size_t)seq * sg.count + seg) * cells + cell;        // the segment's, where there are several
+    // where this walk starts: the slot's state (whole sequences, and the first segment of a first walk), zero, or the
+    // segment's start
+    const bool from_seg = sg.count > 1 && !LOCAL;
+    const float* src = from_seg ? seg_st : st;
+    const bool zero = from_seg ? false : (fresh || seg > 0);
     // a thread's run of rows is contiguous in the kept S^T: 16 bytes at a time where the run is whole and aligned
     const bool whole = live && r * DR + DR <= dim && (dim & 3) == 0;
-    if (!fresh && whole) {
+    if (!zero && whole) {
 #pragma unroll
         for (int i = 0; i < DR / 4; ++i) {
-            const float4 t = ((const float4*)st)[i];
+            const float4 t = ((const float4*)src)[i];
             S[4 * i] = t.x; S[4 * i + 1] = t.y; S[4 * i + 2] = t.z; S[4 * i + 3] = t.w;
         }
     } else {
 #pragma unroll
-        for (int i = 0; i < DR; ++i) S[i] = (!fresh && live && r * DR + i < dim) ? st[i] : 0.f;
+        for (int i = 0; i < DR; ++i) S[i] = (!zero && live && r * DR + i < dim) ? src[i] : 0.f;
     }
     // rows beyond dim and columns beyond vdim are read by the walk and never staged: they stay zero for good
     if (R * DR != dim || col0 + CC > vdim) {
@@ -149,7 +180,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
             for (int idx = threadIdx.x; idx < nt * d4; idx += blockDim.x) {
                 const int t = idx / d4, d = (idx % d4) << 2;
                 const int at = t * dpad + d + (d / DR) * kPad;
-                cp_async16(qs + at, q + (size_t)(t0 + t) * ld + kh * dim + d);
+                if (!LOCAL) cp_async16(qs + at, q + (size_t)(t0 + t) * ld + kh * dim + d);
                 cp_async16(ks + at, k + (size_t)(t0 + t) * ld + kh * dim + d);
                 if (CHANNEL) cp_async16(gk + at, g + (size_t)(t0 + t) * g_ld + head * dim + d);
             }
@@ -157,7 +188,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
             for (int idx = threadIdx.x; idx < nt * dim; idx += blockDim.x) {
                 const int t = idx / dim, d = idx % dim;
                 const int at = t * dpad + d + (d / DR) * kPad;
-                cp_async4(qs + at, q + (size_t)(t0 + t) * ld + kh * dim + d);
+                if (!LOCAL) cp_async4(qs + at, q + (size_t)(t0 + t) * ld + kh * dim + d);
                 cp_async4(ks + at, k + (size_t)(t0 + t) * ld + kh * dim + d);
                 if (CHANNEL) cp_async4(gk + at, g + (size_t)(t0 + t) * g_ld + head * dim + d);
             }
@@ -176,6 +207,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
 
     stage(lo, min(kScanChunk, hi - lo), sm);
     int which = 0;
+    float dec[kDecayPerThread] = {1.f, 1.f, 1.f, 1.f};       // first walks: the product of the segment's decays
     for (int t0 = lo; t0 < hi; t0 += kScanChunk, which ^= 1) {
         const int nt = min(kScanChunk, hi - t0);
         cp_async_wait_all();
@@ -183,7 +215,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
         if (t0 + kScanChunk < hi) stage(t0 + kScanChunk, min(kScanChunk, hi - t0 - kScanChunk), sm + (which ^ 1) * per_buf);
         float* qs = sm + which * per_buf;
         float* ks = qs + kScanChunk * dpad;
-        if (rot_in_walk) {
+        if (!LOCAL && rot_in_walk) {
             // the staged q and k turn with their tokens' positions, and the keys take their factor, as rotate_rows would
             // have done in a launch of its own (meant for single-token steps: every block of a head repeats it)
             const int half = rot_dims >> 1, per = half + (dim - rot_dims);
@@ -245,7 +277,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                 float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
 #pragma unroll
                 for (int i = 0; i < DR / 4; ++i) {
-                    float4 kk = k4[i], qq = q4[i];
+                    float4 kk = k4[i], qq = LOCAL ? make_float4(0.f, 0.f, 0.f, 0.f) : q4[i];
                     if (RULE == kDecayRule && act_in_walk) {
                         kk = make_float4(silu_precise(kk.x), silu_precise(kk.y), silu_precise(kk.z), silu_precise(kk.w));
                         qq = make_float4(silu_precise(qq.x), silu_precise(qq.y), silu_precise(qq.z), silu_precise(qq.w));
@@ -267,6 +299,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                         S[4 * i + 2] = fmaf(gt, S[4 * i + 2], kk.z * u);
                         S[4 * i + 3] = fmaf(gt, S[4 * i + 3], kk.w * u);
                     }
+                    if (LOCAL) continue;
                     a0 = fmaf(S[4 * i], qq.x, a0);
                     a1 = fmaf(S[4 * i + 1], qq.y, a1);
                     a2 = fmaf(S[4 * i + 2], qq.z, a2);
@@ -276,18 +309,42 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
             }
 #pragma unroll
             for (int t = 0; t < kScanChunk; ++t) {
-                if (t >= nt) break;
+                if (LOCAL || t >= nt) break;
                 float acc = part[t];
 #pragma unroll
                 for (int o = 1; o < R; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
                 if (r == 0 && c < CC) os[t * CC + c] = acc * o_mult;
             }
         }
+        if (LOCAL) {
+            if (blockIdx.z == 0) {
+#pragma unroll
+                for (int i = 0; i < kDecayPerThread; ++i) {
+                    const int d = threadIdx.x + i * blockDim.x;
+                    if (d >= (CHANNEL ? dim : 1)) break;
+                    for (int t = 0; t < nt; ++t) dec[i] *= CHANNEL ? gk[t * dpad + d + (d / DR) * kPad] : gs[t];
+                }
+            }
+            continue;
+        }
         __syncthreads();
         for (int idx = threadIdx.x; idx < nt * CC; idx += blockDim.x) {
             const int t = idx / CC, cc = idx % CC;
             if (col0 + cc < vdim) out[((size_t)(t0 + t) * H + head) * vdim + col0 + cc] = os[idx];
         }
+    }
+    if (LOCAL) {
+        if (blockIdx.z == 0) {
+            float* dp = sg.decays + (((size_t)seq * sg.count + seg) * H + head) * (CHANNEL ? dim : 1);
+#pragma unroll
+            for (int i = 0; i < kDecayPerThread; ++i) {
+                const int d = threadIdx.x + i * blockDim.x;
+                if (d < (CHANNEL ? dim : 1)) dp[d] = dec[i];
+            }
+        }
+        st = seg_st;
+    } else if (!last) {
+        return;                                  // only the last segment's state is the sequence's
     }
     if (whole) {
 #pragma unroll
@@ -296,6 +353,44 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
 #pragma unroll
         for (int i = 0; i < DR; ++i)
             if (r * DR + i < dim) st[i] = S[i];
+    }
+}
+
+// states: what the first walk left, [count][cells] per sequence; becomes the states at the segments' starts (the first one's:
+// the slot's, or zero).  A thread per cell; decays: a number per head, or (channel) per head and key number.
+__global__ void __launch_bounds__(256)
+segment_starts_kernel(const float* __restrict__ state, Segments sg, const int* __restrict__ token_pos, const int* __restrict__ token_seq,
+                      const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot, int H, int dim, int vdim, int channel) {
+    pdl_enter();
+    const int seq = blockIdx.y;
+    const int lo = cu_seqlens[seq], len = cu_seqlens[seq + 1] - lo;
+    if (len <= 0 || token_seq[lo] < 0) return;
+    const long long cells = (long long)H * vdim * dim;
+    const long long cell = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (cell >= cells) return;
+    const int n = (len + sg.len - 1) / sg.len;
+    const int head = (int)(cell / ((long long)vdim * dim));
+    const int per = channel ? H * dim : H, at = channel ? head * dim + (int)(cell % dim) : head;
+    float* st = sg.states + (size_t)seq * sg.count * cells + cell;
+    const float* dp = sg.decays + (size_t)seq * sg.count * per + at;
+    float cur = token_pos[lo] == 0 ? 0.f : state[(size_t)seq_slot[seq] * cells + cell];
+    constexpr int B = 8;                          // loads under way together
+    for (int s0 = 0; s0 < n; s0 += B) {
+        float local[B], d[B];
+#pragma unroll
+        for (int i = 0; i < B; ++i) {
+            const int s = s0 + i;
+            const bool in = s < n - 1;            // the last segment has left nothing
+            local[i] = in ? st[(size_t)s * cells] : 0.f;
+            d[i] = in ? dp[(size_t)s * per] : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < B; ++i) {
+            const int s = s0 + i;
+            if (s >= n) break;
+            st[(size_t)s * cells] = cur;
+            cur = s == 0 ? local[i] : fmaf(d[i], cur, local[i]);      // the first segment's walk began with the sequence's state
+        }
     }
 }
 
@@ -360,29 +455,21 @@ conv_prep_kernel(const float* __restrict__ raw, long long ld, const float* __res
 // act(x): 0 none, 1 x logistic(x)
 __device__ __forceinline__ float conv_act(float x, int act) { return act == 1 ? silu_precise(x) : x; }
 
-constexpr int kConvTokens = 16;      // consecutive rows that a thread of conv_act_rows walks
-
-// out[n][c] = act(sum_j w[c][j] u_(n - taps + 1 + j)[c] + bias[c]) for C columns of 32-bit rows.  A thread takes VEC channels
-// of up to kConvTokens consecutive rows (one where the sequences bring single tokens) and keeps the inputs in sight in
-// registers, so that a column is read once; rows of a sequence's start, or of this run's, fetch them from the rows
-// before or from the slot's kept inputs.  The last block of a row run takes the per-head step sizes: dt = softplus(raw
-// + dt_bias), decay = exp(-exp(A_log) dt).
+// out[n][c] = act(convolution + bias[c]) for C columns of 32-bit rows (conv_walk in short_conv.cuh).  The last block of a row
+// run takes the per-head step sizes: dt = softplus(raw + dt_bias), decay = exp(-exp(A_log) dt).
 template <int TAPS, int VEC>
 __global__ void __launch_bounds__(128)
-conv_act_rows_kernel(const float* raw, long long ld, const float* __restrict__ w, const float* __restrict__ bias, int taps_rt,
-                     const float* keep_all, float* keep_w_all, int act, const int* __restrict__ token_pos,
-                     const int* __restrict__ token_seq, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
-                     float* __restrict__ out, int N, int C, int run, int conv_blocks, const float* __restrict__ dt_raw,
-                     const float* __restrict__ dt_bias, const float* __restrict__ a_log, float* __restrict__ dt_out,
-                     float* __restrict__ g_out, int H) {
+conv_act_rows_kernel(ConvWalk c, const float* __restrict__ bias, int act, float* __restrict__ out, int N, int run, int conv_blocks,
+                     const float* __restrict__ dt_raw, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
+                     float* __restrict__ dt_out, float* __restrict__ g_out, int H) {
     pdl_enter();
     const int n0 = blockIdx.y * run, n1 = min(N, n0 + run);
     if ((int)blockIdx.x >= conv_blocks) {
         for (int i = threadIdx.x; i < (n1 - n0) * H; i += blockDim.x) {
             const int n = n0 + i / H, h = i % H;
             float dt = 0.f, g = 1.f;
-            if (token_seq[n] >= 0) {
-                const float a = dt_raw[(size_t)n * ld + h] + dt_bias[h];
+            if (c.token_seq[n] >= 0) {
+                const float a = dt_raw[(size_t)n * c.ld + h] + dt_bias[h];
                 dt = a > 20.f ? a : log1pf(expf(a));
                 g = expf(-expf(a_log[h]) * dt);
             }
@@ -392,83 +479,23 @@ conv_act_rows_kernel(const float* raw, long long ld, const float* __restrict__ w
         return;
     }
     const int ch = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
-    if (ch >= C) return;
-    const int taps = TAPS > 0 ? TAPS : taps_rt;
-    constexpr int MAXT = TAPS > 0 ? TAPS : kMaxTaps;
-    float wr[VEC][MAXT], win[VEC][MAXT], b[VEC];
+    if (ch >= c.C) return;
+    float b[VEC];
 #pragma unroll
-    for (int v = 0; v < VEC; ++v) {
-        b[v] = bias != nullptr ? bias[ch + v] : 0.f;
+    for (int v = 0; v < VEC; ++v) b[v] = bias != nullptr ? bias[ch + v] : 0.f;
+    conv_walk<TAPS, VEC>(
+        c, ch, n0, n1,
+        [&](int n, float (&y)[VEC]) {
 #pragma unroll
-        for (int j = 0; j < MAXT; ++j) wr[v][j] = j < taps ? w[(size_t)(ch + v) * taps + j] : 0.f;
-    }
-    auto load = [&](const float* p, float (&x)[VEC]) {
-        if (VEC == 4) {
-            const float4 t = *(const float4*)p;
-            x[0] = t.x; x[VEC > 1 ? 1 : 0] = t.y; x[VEC > 2 ? 2 : 0] = t.z; x[VEC > 3 ? 3 : 0] = t.w;
-        } else {
-            x[0] = *p;
-        }
-    };
-    auto store = [&](float* p, const float (&x)[VEC]) {
-        if (VEC == 4) *(float4*)p = make_float4(x[0], x[VEC > 1 ? 1 : 0], x[VEC > 2 ? 2 : 0], x[VEC > 3 ? 3 : 0]);
-        else *p = x[0];
-    };
-    int last_seq = -2;
-    for (int n = n0; n < n1; ++n) {
-        const int seq = token_seq[n];
-        float y[VEC];
-        if (seq < 0) {
+            for (int v = 0; v < VEC; ++v) y[v] = conv_act(y[v] + b[v], act);
+            conv_store<VEC>(out + (size_t)n * c.C + ch, y);
+        },
+        [&](int n) {
+            float y[VEC];
 #pragma unroll
             for (int v = 0; v < VEC; ++v) y[v] = 0.f;
-            store(out + (size_t)n * C + ch, y);
-            last_seq = -2;
-            continue;
-        }
-        if (seq != last_seq) {                   // the inputs before this row: win[.][j] of place j - 1 after the shift below
-            const int r0 = cu_seqlens[seq];
-            const bool fresh = token_pos[r0] == 0;
-            const float* keep = keep_all + (size_t)seq_slot[seq] * (taps - 1) * C + ch;
-#pragma unroll
-            for (int j = 1; j < MAXT; ++j) {
-                if (j >= taps) continue;
-                const int src = n - taps + j;
-                float x[VEC];
-#pragma unroll
-                for (int v = 0; v < VEC; ++v) x[v] = 0.f;
-                if (src >= r0) load(raw + (size_t)src * ld + ch, x);
-                else if (!fresh) load(keep + (size_t)((taps - 1) + (src - r0)) * C, x);
-#pragma unroll
-                for (int v = 0; v < VEC; ++v) win[v][j] = x[v];
-            }
-            last_seq = seq;
-        }
-        float x[VEC];
-        load(raw + (size_t)n * ld + ch, x);
-#pragma unroll
-        for (int v = 0; v < VEC; ++v) {
-            float acc = 0.f;
-#pragma unroll
-            for (int j = 0; j < MAXT; ++j) {
-                if (j + 1 < taps) win[v][j] = win[v][j + 1 < MAXT ? j + 1 : j];
-                else if (j + 1 == taps) win[v][j] = x[v];
-                if (j < taps) acc = fmaf(wr[v][j], win[v][j], acc);
-            }
-            y[v] = conv_act(acc + b[v], act);
-        }
-        store(out + (size_t)n * C + ch, y);
-        if (keep_w_all != nullptr) {             // single tokens: the kept inputs (the last taps - 1 in sight) move on here
-            float* keep = keep_w_all + (size_t)seq_slot[seq] * (taps - 1) * C + ch;
-#pragma unroll
-            for (int j = 1; j < MAXT; ++j) {
-                if (j >= taps) continue;
-                float k[VEC];
-#pragma unroll
-                for (int v = 0; v < VEC; ++v) k[v] = win[v][j];
-                store(keep + (size_t)(j - 1) * C, k);
-            }
-        }
-    }
+            conv_store<VEC>(out + (size_t)n * c.C + ch, y);
+        });
 }
 
 // out[n][c] = logistic(z)^(1 / tau), z = sum_r w[c][r] low[n][r] + b[c]: exp(-softplus(-z) / tau), 32-bit.  A block takes
@@ -508,42 +535,78 @@ channel_decay_kernel(const float* __restrict__ low, long long ld, const float* _
 
 using namespace hos;
 
+namespace hos {
+// How a walk is cut: DR rows of a column to a thread, R threads to a column, CC columns to a block.
+struct ScanShape {
+    int DR, R, CC;
+    ScanShape(int dim, int vdim) {
+        // short runs of rows per thread: a token's walk is a chain of dependent instructions (scale, dot, sum over the
+        // runs, update, read-out, sum), and with few (sequence, head) pairs nothing else hides its latency; the sums over
+        // 16 or 32 runs are shuffles
+        // (heads of 128 x 128, 2,048 tokens, decay / delta rule: 4 rows to a thread 477 / 628 us, 8 rows 459 / 598, 16 rows
+        // 584 / 679, 32 rows 900 / 961)
+        DR = dim <= 16 ? 4 : (dim <= 256 ? 8 : (dim <= 512 ? 16 : 32));
+        R = 1;
+        while (R * DR < dim) R <<= 1;
+        if (DR == 8 && R < 4) R = 4;          // the compiled shapes (rows beyond dim are zeros)
+        if (DR >= 16) R = 32;
+        CC = 256 / R;
+        if (CC > vdim) CC = vdim;
+    }
+    int threads() const { return (CC * R + 31) / 32 * 32; }
+};
+constexpr int kMinSegment = 64;       // tokens
+}  // namespace hos
+
+// How many tokens a segment has where sequences that bring up to max_new tokens are worth walking in segments (see the file's
+// head); 0 where they are not.  The caller then gives hos_state_scan the workspace: with n = ceil(max_new / that),
+// n_seqs * n * H * vdim * dim and n_seqs * n * H (channel rule: H * dim) floats.
+extern "C" int hos_state_scan_segment(int n_seqs, int H, int dim, int vdim, int max_new, int rule) {
+    if (rule == kDeltaRule || n_seqs <= 0 || max_new < 3 * kMinSegment || dim <= 0 || dim > 1024 || vdim <= 0) return 0;
+    const ScanShape shape(dim, vdim);
+    if (rule == kChannelRule && dim > kDecayPerThread * shape.threads()) return 0;
+    const long long blocks = (long long)n_seqs * H * ((vdim + shape.CC - 1) / shape.CC);
+    // a walk is bound by its chain until several blocks share an SM; two walks instead of one must be paid for
+    const long long want = 8ll * sm_count_cached() / blocks;
+    if (want < 3) return 0;
+    const int count = (int)(want < max_new / kMinSegment ? want : max_new / kMinSegment);
+    const int len = (max_new + count - 1) / count;
+    return (len + kScanChunk - 1) / kScanChunk * kScanChunk;
+}
+
 // q, k: rows of Gk heads of `dim` numbers; v: rows of H heads of `vdim`; all float32 with `ld` numbers between rows.
 // rule: 0 decay, 1 delta, 2 channel.  g: [.][H] (channel rule: [.][H * dim]) with g_ld between rows (0: one row of constants).
 // beta: the delta rule's; with the decay rule, if given, the factor on v; o_mult: a constant on the read-outs.  state: [slots][H][vdim][dim].
 // out: float32 [N][H][vdim].  act_in_walk (decay rule only, meant for single-token steps): q, k, v are taken through
 // x logistic(x) as they are read, instead of by hos_act_rows before.  rot_freq ([rot_dims / 2], or null), rot_style, k_mult:
 // the staged q and k are turned by their tokens' positions and the keys multiplied, as hos_rotate_rows would have done
-// before (meant for single-token steps; it follows the rows as they are, so it does not go with act_in_walk).
+// before (meant for single-token steps; it follows the rows as they are, so it does not go with act_in_walk).  seg_len, seg_count > 1: the
+// walk in segments (hos_state_scan_segment), seg_count of them to a sequence at most, with its workspace.
 extern "C" int hos_state_scan(const float* q, const float* k, const float* v, long long ld, int act_in_walk, int rule,
                               float o_mult, const float* g, long long g_ld, const float* beta, long long beta_ld, float* state, const int* token_pos,
                               const int* token_seq, const int* cu_seqlens, const int* seq_slot, float* out, int n_rows,
                               int n_seqs, int H, int Gk, int dim, int vdim, const float* rot_freq, int rot_dims, int rot_style,
-                              float k_mult, cudaStream_t stream) {
+                              float k_mult, int seg_len, int seg_count, float* seg_states, float* seg_decays, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (rot_freq == nullptr) rot_dims = 0;
     if (rot_dims < 0 || rot_dims % 2 != 0 || rot_dims > dim || (rot_style != 0 && rot_style != 1))
         HOS_REFUSE("state_scan: %d rotated numbers in heads of %d", rot_dims, dim);
     if (Gk <= 0 || H % Gk != 0) HOS_REFUSE("state_scan: %d heads are not a multiple of %d key heads", H, Gk);
     if (dim <= 0 || dim > 1024 || vdim <= 0) HOS_REFUSE("state_scan: heads of %d x %d", dim, vdim);
-    // short runs of rows per thread: a token's walk is a chain of dependent instructions (scale, dot, sum over the
-    // runs, update, read-out, sum), and with few (sequence, head) pairs nothing else hides its latency; the sums over
-    // 16 or 32 runs are shuffles
-    // (heads of 128 x 128, 2,048 tokens, decay / delta rule: 4 rows to a thread 477 / 628 us, 8 rows 459 / 598, 16 rows
-    // 584 / 679, 32 rows 900 / 961)
-    const int DR = dim <= 16 ? 4 : (dim <= 256 ? 8 : (dim <= 512 ? 16 : 32));
-    int R = 1;
-    while (R * DR < dim) R <<= 1;
-    if (DR == 8 && R < 4) R = 4;          // the compiled shapes (rows beyond dim are zeros)
-    if (DR >= 16) R = 32;
-    int CC = 256 / R;
-    if (CC > vdim) CC = vdim;
+    const ScanShape shape(dim, vdim);
+    const int DR = shape.DR, R = shape.R;
+    int CC = shape.CC;
     // single tokens and few (sequence, head) pairs: fewer columns to a block, so that the blocks fill the GPU (columns
     // are independent; every block stages the whole q and k rows, which a long walk would pay for token by token)
     if (n_rows <= 2 * n_seqs)
         while (CC * R > 64 && (long long)n_seqs * H * ((vdim + CC - 1) / CC) < 2 * sm_count_cached()) CC = (CC + 1) / 2;
     const int threads = (CC * R + 31) / 32 * 32;
     const int dpad = R * (DR + kPad);
+    const bool segments = seg_count > 1;
+    if (segments && (rule == kDeltaRule || act_in_walk || rot_dims > 0 || k_mult != 1.f || seg_len <= 0 || seg_states == nullptr ||
+                     seg_decays == nullptr || (rule == kChannelRule && dim > kDecayPerThread * threads)))
+        HOS_REFUSE("state_scan: %d segments of %d tokens do not fit this walk", seg_count, seg_len);
+    const Segments sg{seg_states, seg_decays, segments ? seg_len : 1, segments ? seg_count : 1};
     if (rule < kDecayRule || rule > kChannelRule || (rule == kDeltaRule && beta == nullptr) || (rule == kChannelRule && beta != nullptr))
         HOS_REFUSE("state_scan: rule %d and its inputs do not fit", rule);
     if (rule == kChannelRule && Gk != H) HOS_REFUSE("state_scan: the channel rule has a key head per head");
@@ -551,22 +614,31 @@ extern "C" int hos_state_scan(const float* q, const float* k, const float* v, lo
     const size_t smem = (size_t)2 * (wide_rows * kScanChunk * dpad + 2 * kScanChunk * CC + 2 * kScanChunk) * sizeof(float);
     const int aligned = (dim % 4 == 0 && ld % 4 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)k % 16 == 0 &&
                          (rule != kChannelRule || (g_ld % 4 == 0 && (uintptr_t)g % 16 == 0))) ? 1 : 0;
-    const dim3 grid(n_seqs, H, (vdim + CC - 1) / CC);
+    const dim3 grid(n_seqs * sg.count, H, (vdim + CC - 1) / CC);
     if (rule != kDecayRule && act_in_walk) HOS_REFUSE("state_scan: the activation in the walk is the decay rule's");
     if (smem > 200 * 1024) HOS_REFUSE("state_scan: heads of %d x %d do not fit a block's shared memory", dim, vdim);
-#define HOS_SCAN(DRv, Rv, DL)                                                                                        \
+#define HOS_SCAN(DRv, Rv, DL, LOC)                                                                                   \
     do {                                                                                                             \
         if (smem > 48 * 1024)                                                                                        \
-            cudaFuncSetAttribute(state_scan_kernel<DRv, Rv, DL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        launch_pdl(state_scan_kernel<DRv, Rv, DL>, grid, dim3(threads), smem, stream, q, k, v, ld, aligned, act_in_walk, g, g_ld, beta, \
+            cudaFuncSetAttribute(state_scan_kernel<DRv, Rv, DL, LOC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        launch_pdl(state_scan_kernel<DRv, Rv, DL, LOC>, grid, dim3(threads), smem, stream, q, k, v, ld, aligned, act_in_walk, g, g_ld, beta, \
                    beta_ld, state, token_pos, token_seq, cu_seqlens, seq_slot, out, H, Gk, dim, vdim, CC, rot_freq,  \
-                   rot_dims, rot_style, k_mult, o_mult);                                                             \
+                   rot_dims, rot_style, k_mult, o_mult, sg);                                                         \
+    } while (0)
+#define HOS_SCAN_S(DRv, Rv, DL)                                                                                      \
+    do {                                                                                                             \
+        if (segments) {                                                                                              \
+            HOS_SCAN(DRv, Rv, DL, true);                                                                             \
+            launch_pdl(segment_starts_kernel, dim3((unsigned)(((long long)H * vdim * dim + 255) / 256), n_seqs), dim3(256), 0, stream, \
+                       (const float*)state, sg, token_pos, token_seq, cu_seqlens, seq_slot, H, dim, vdim, DL == kChannelRule ? 1 : 0); \
+        }                                                                                                            \
+        HOS_SCAN(DRv, Rv, DL, false);                                                                                \
     } while (0)
 #define HOS_SCAN_D(DRv, Rv)                                                                                          \
     do {                                                                                                             \
-        if (rule == kDeltaRule) HOS_SCAN(DRv, Rv, kDeltaRule);                                                       \
-        else if (rule == kChannelRule) HOS_SCAN(DRv, Rv, kChannelRule);                                              \
-        else HOS_SCAN(DRv, Rv, kDecayRule);                                                                          \
+        if (rule == kDeltaRule) HOS_SCAN(DRv, Rv, kDeltaRule, false);                                                \
+        else if (rule == kChannelRule) HOS_SCAN_S(DRv, Rv, kChannelRule);                                            \
+        else HOS_SCAN_S(DRv, Rv, kDecayRule);                                                                        \
     } while (0)
     // the shapes that the choice of DR above can give: (4; 1, 2, 4), (8; 4 to 32), (16; 32), (32; 32)
     if (DR == 4 && R == 1) HOS_SCAN_D(4, 1);
@@ -579,6 +651,7 @@ extern "C" int hos_state_scan(const float* q, const float* k, const float* v, lo
     else if (DR == 16) HOS_SCAN_D(16, 32);
     else HOS_SCAN_D(32, 32);
 #undef HOS_SCAN_D
+#undef HOS_SCAN_S
 #undef HOS_SCAN
     return check_launch("state_scan");
 }
@@ -624,43 +697,42 @@ extern "C" int hos_conv_prep(const float* raw, long long ld, const float* conv_w
     return check_launch("conv_prep");
 }
 
-extern "C" int hos_conv_keep(const float* raw, long long ld, int taps, float* conv_state, const int* token_pos,
+extern "C" int hos_conv_keep(const float* raw, long long ld, const float* in_bias, int taps, float* conv_state, const int* token_pos,
                              const int* token_seq, const int* cu_seqlens, const int* seq_slot, int n_seqs, int C,
                              cudaStream_t stream) {
     if (n_seqs <= 0 || taps <= 1) return 0;
     if (taps > kMaxTaps) HOS_REFUSE("conv_keep: %d taps are outside 1..%d", taps, kMaxTaps);
-    launch_pdl(short_conv_keep_kernel, dim3((C + 127) / 128, n_seqs), dim3(128), 0, stream, raw, ld, (const float*)nullptr, taps,
-               conv_state, token_pos, token_seq, cu_seqlens, seq_slot, C);
+    launch_pdl(short_conv_keep_kernel, dim3((C + 127) / 128, n_seqs), dim3(128), 0, stream, raw, ld, in_bias, taps, conv_state,
+               token_pos, token_seq, cu_seqlens, seq_slot, C);
     return check_launch("conv_keep");
 }
 
-// raw: the rows from the first convolved column on, ld apart; w: [C][taps]; bias: [C] or null; act: 0 none, 1 x logistic(x);
-// conv_state: [slots][taps - 1][C]; out: float32 [N][C].  single: 1 where every sequence of the step brings exactly one token:
-// the kept inputs then move on inside this launch and hos_conv_keep is not needed.  dt_raw (or null): the rows from the
-// first step-size column on, H of them, ld apart: dt_out [N][H] = softplus(dt_raw + dt_bias), g_out [N][H] = exp(-exp(a_log) dt).
-extern "C" int hos_conv_act_rows(const float* raw, long long ld, const float* w, const float* bias, int taps, float* conv_state,
-                                 int act, const int* token_pos, const int* token_seq, const int* cu_seqlens, const int* seq_slot,
-                                 float* out, int N, int C, int single, const float* dt_raw, const float* dt_bias, const float* a_log,
-                                 float* dt_out, float* g_out, int H, cudaStream_t stream) {
+// raw: the rows from the first convolved column on, ld apart; w: [taps][C]; in_bias ([C] or null): added before the
+// convolution; bias ([C] or null): after it; act: 0 none, 1 x logistic(x); conv_state: [slots][taps - 1][C]; out: float32
+// [N][C].  single: 1 where every sequence of the step brings exactly one token: the kept inputs then move on inside this
+// launch (otherwise hos_conv_keep does it afterwards).  dt_raw (or null): the rows from the first step-size column on, H of
+// them, ld apart: dt_out [N][H] = softplus(dt_raw + dt_bias), g_out [N][H] = exp(-exp(a_log) dt).
+extern "C" int hos_conv_act_rows(const float* raw, long long ld, const float* w, const float* in_bias, const float* bias, int taps,
+                                 float* conv_state, int act, const int* token_pos, const int* token_seq, const int* cu_seqlens,
+                                 const int* seq_slot, float* out, int N, int C, int single, const float* dt_raw, const float* dt_bias,
+                                 const float* a_log, float* dt_out, float* g_out, int H, cudaStream_t stream) {
     if (N <= 0 || C <= 0) return 0;
     if (taps < 1 || taps > kMaxTaps) HOS_REFUSE("conv_act_rows: %d taps are outside 1..%d", taps, kMaxTaps);
     if (act != 0 && act != 1) HOS_REFUSE("conv_act_rows: unknown activation %d", act);
     if (dt_raw != nullptr && (dt_bias == nullptr || a_log == nullptr || dt_out == nullptr || g_out == nullptr || H <= 0))
         HOS_REFUSE("conv_act_rows: step sizes need their bias, their rates and two outputs");
-    const bool vec = taps >= 2 && taps <= 4 && C % 4 == 0 && ld % 4 == 0 && (uintptr_t)raw % 16 == 0 && (uintptr_t)out % 16 == 0 &&
-                     (uintptr_t)conv_state % 16 == 0;
+    const bool vec = taps >= 2 && taps <= 4 && C % 4 == 0 && ld % 4 == 0 &&
+                     (((uintptr_t)raw | (uintptr_t)out | (uintptr_t)conv_state | (uintptr_t)w | (uintptr_t)in_bias) % 16) == 0;
     const int per_block = 128 * (vec ? 4 : 1);
     const int conv_blocks = (C + per_block - 1) / per_block;
-    // runs as long as leave every SM several blocks; a single-token step's rows are sequences of their own
-    int run = 1;
-    while (!single && run < kConvTokens && (long long)((N + 2 * run - 1) / (2 * run)) * conv_blocks >= 4 * sm_count_cached()) run *= 2;
+    const int run = conv_run(N, conv_blocks, single != 0);
     const dim3 grid(conv_blocks + (dt_raw != nullptr ? 1 : 0), (N + run - 1) / run);
     if (grid.y > 65535) HOS_REFUSE("conv_act_rows: %d rows are more than one launch takes", N);
-    float* keep_w = single && taps > 1 ? conv_state : nullptr;
+    const ConvWalk c{raw, ld, w, in_bias, conv_state, single && taps > 1 ? conv_state : nullptr, token_pos, token_seq, cu_seqlens,
+                     seq_slot, taps, C};
 #define HOS_CAR(T, V)                                                                                                \
-    launch_pdl(conv_act_rows_kernel<T, V>, grid, dim3(128), 0, stream, raw, ld, w, bias, taps, (const float*)conv_state, keep_w, \
-               act, token_pos, token_seq, cu_seqlens, seq_slot, out, N, C, run, conv_blocks, dt_raw, dt_bias, a_log, dt_out, \
-               g_out, H)
+    launch_pdl(conv_act_rows_kernel<T, V>, grid, dim3(128), 0, stream, c, bias, act, out, N, run, conv_blocks, dt_raw, dt_bias, \
+               a_log, dt_out, g_out, H)
 #define HOS_CAR_V(T)                                                                                                 \
     do {                                                                                                             \
         if (vec) HOS_CAR(T, 4);                                                                                      \

@@ -967,29 +967,20 @@ def qk_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional[t
             eps: float, freq: Optional[torch.Tensor], rot_dims: int, magnitude: float, step, q_out: torch.Tensor,
             cache: PagedKVArgs, n_heads: int, n_kv: int, kd: int, vd: int, norm_whole: bool = False,
             v_first: Optional[torch.Tensor] = None, v_first_col: int = 0, v_mix: float = 0.0, q_maps: int = 1,
-            proj_col: int = 0, conv_w: Optional[torch.Tensor] = None, conv_state: Optional[torch.Tensor] = None,
-            keep_here: bool = False, q_temp=None) -> None:
+            proj_col: int = 0, q_temp=None) -> None:
     """proj: float32 rows whose columns from proj_col on are [q | k | v | ...] (G = n_kv; 0: a call that stores nothing).  Adds the
     biases, norms and rotates the q and k heads, writes q_out float32 [N, H, kd] and stores k, v in the cache.
     norm_whole: one root mean square over all q heads and one over all k heads (weights [H kd], [G kd]).  v_first
     (float32 [N, ld], the values from column v_first_col on): v <- (1 - v_mix) v + v_mix v_first before the store.
     q_maps > 1: a head's kd numbers are q_maps queries, one per attention map over the same key row; q_out is then
-    [N, H * q_maps, kd], every query a head of its own that is zero outside its part of the key row.  conv_w ([taps, C],
-    C = H kd + G (kd + vd)): a short convolution over time on every channel, right after the bias, with its kept inputs
-    conv_state [slots, taps - 1, C] (keep_here, only where every sequence brings one token: they move on in this launch;
-    else call qkv_conv_keep).  q_temp = (coef, every): q times 1 + coef ln(floor((p + 1) / every) + 1)."""
+    [N, H * q_maps, kd], every query a head of its own that is zero outside its part of the key row.  q_temp = (coef, every): q times
+    1 + coef ln(floor((p + 1) / every) + 1) at position p."""
     _check(proj, "projection rows", torch.float32, 2)
     _check(q_out, "queries", torch.float32, 3)
     n = proj.shape[0]
     c = n_heads * kd + n_kv * (kd + vd)
     if q_out.shape != (n, n_heads * q_maps, kd) or proj.shape[1] < proj_col + c:
         raise KernelError("qk_prep: sizes disagree")
-    taps = 0
-    if conv_w is not None:
-        _check(conv_w, "convolution weights", torch.float32, 2)
-        taps = conv_w.shape[0]
-        if conv_w.shape[1] != c or (taps > 1 and tuple(conv_state.shape[1:]) != (taps - 1, c)):
-            raise KernelError("qk_prep: the convolution does not fit the projection")
     if n_kv and (cache.head_dim != kd or cache.v_dim != vd or cache.n_kv_heads != n_kv):
         raise KernelError("qk_prep: the cache does not fit the keys and values")
     for wn, cols in ((q_norm, n_heads * kd), (k_norm, n_kv * kd)):
@@ -1007,16 +998,30 @@ def qk_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional[t
                   _ptr(q_out), _ptr(cache.k_pages) if n_kv else None, _ptr(cache.v_pages) if n_kv else None,
                   dtype_code(cache.k_pages.dtype), _ptr(cache.page_table), cache.table_stride, cache.ring_pages, n,
                   int(n_heads), int(n_kv), int(kd), int(vd), 1 if norm_whole else 0, vf_ptr, vf_ld, float(v_mix),
-                  int(q_maps), _ptr(conv_w), taps, _ptr(conv_state) if taps > 1 else None, _ptr(step.cu_seqlens),
-                  1 if keep_here else 0, float(coef), int(every), _stream())
+                  int(q_maps), float(coef), int(every), _stream())
 
 
-def qkv_conv_keep(proj: torch.Tensor, proj_col: int, bias: Optional[torch.Tensor], taps: int, conv_state: torch.Tensor, step,
-                  channels: int) -> None:
-    """The last taps - 1 projected inputs of every sequence's q, k and v channels go to the slot's state."""
-    gated_attn_lib().call("hos_qkv_conv_keep", _at(proj, proj_col), proj.shape[1], _ptr(bias), int(taps), _ptr(conv_state),
-                          _ptr(step.token_pos), _ptr(step.token_seq), _ptr(step.cu_seqlens), _ptr(step.seq_slot),
-                          int(step.n_seqs), int(channels), _stream())
+def qkv_conv_store(proj: torch.Tensor, col: int, bias: Optional[torch.Tensor], conv_w: torch.Tensor, conv_state, step, q_out: torch.Tensor,
+                   cache: PagedKVArgs, n_heads: int, n_kv: int, kd: int, vd: int, single: bool, q_temp=None) -> None:
+    """proj: float32 rows whose C = H kd + G (kd + vd) columns from `col` on are [q | k | v]: every channel passes a short
+    convolution over time (conv_w [taps, C]) right after its bias, with its kept inputs conv_state [slots, taps - 1, C]
+    (single, only where every sequence brings one token: they move on in this launch; else call conv_keep); queries (times
+    their factor, as qk_prep) go to q_out float32 [N, H, kd], keys and values to the cache."""
+    _check(proj, "projection rows", torch.float32, 2)
+    _check(conv_w, "convolution weights", torch.float32, 2)
+    _check(q_out, "queries", torch.float32, 3)
+    n, (taps, c) = proj.shape[0], conv_w.shape
+    if c != n_heads * kd + n_kv * (kd + vd) or col + c > proj.shape[1] or q_out.shape != (n, n_heads, kd) \
+            or (taps > 1 and tuple(conv_state.shape[1:]) != (taps - 1, c)) or (bias is not None and bias.shape[0] < c):
+        raise KernelError("qkv_conv_store: sizes disagree")
+    if cache.head_dim != kd or cache.v_dim != vd or cache.n_kv_heads != n_kv:
+        raise KernelError("qkv_conv_store: the cache does not fit the keys and values")
+    coef, every = q_temp if q_temp else (0.0, 0)
+    gated_attn_lib().call("hos_qkv_conv_store", _at(proj, col), proj.shape[1], _ptr(bias), _ptr(conv_w), int(taps),
+                          _ptr(conv_state) if taps > 1 else None, 1 if single else 0, _ptr(step.token_pos), _ptr(step.token_seq),
+                          _ptr(step.cu_seqlens), _ptr(step.seq_slot), _ptr(q_out), _ptr(cache.k_pages), _ptr(cache.v_pages),
+                          dtype_code(cache.k_pages.dtype), _ptr(cache.page_table), cache.table_stride, cache.ring_pages, n,
+                          int(n_heads), int(n_kv), int(kd), int(vd), float(coef), int(every), _stream())
 
 
 def diff_combine(a: torch.Tensor, lam: float, mult: float, eps: float, gate: Optional[torch.Tensor], gate_col: int, step,
@@ -1111,6 +1116,9 @@ def gated_attn_mma_decode(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[to
     return True
 
 
+segmented_scans = True        # tests switch it off to compare the walk by segments with the whole one
+
+
 def state_scan(rows: torch.Tensor, q_col: int, k_col: int, v_col: int, silu_on_load: bool, g: torch.Tensor,
                per_token_g: bool, beta: Optional[torch.Tensor], state: torch.Tensor, step, out: torch.Tensor,
                heads: int, key_heads: int, dim: int, vdim: int, rot=None, v_factor: Optional[torch.Tensor] = None,
@@ -1139,6 +1147,14 @@ def state_scan(rows: torch.Tensor, q_col: int, k_col: int, v_col: int, silu_on_l
     rule = 1 if beta is not None else (2 if channel_g else 0)
     second = beta if beta is not None else v_factor
     g_ld = heads * dim if channel_g else (heads if per_token_g else 0)
+    seg_len, seg_count, seg_states, seg_decays = 0, 1, None, None
+    if rot is None and rule != 1 and segmented_scans:
+        seg_len = int(mixers().fn("hos_state_scan_segment")(int(step.n_seqs), int(heads), int(dim), int(vdim), int(step.max_new), rule))
+        if seg_len > 0:
+            seg_count = -(-int(step.max_new) // seg_len)
+            places = int(step.n_seqs) * seg_count * heads
+            seg_states = torch.empty(places * vdim * dim, dtype=torch.float32, device=rows.device)
+            seg_decays = torch.empty(places * (dim if channel_g else 1), dtype=torch.float32, device=rows.device)
     in_walk = bool(silu_on_load) and beta is None and step.max_new == 1      # single tokens: no launch of its own for it
     if silu_on_load and not in_walk:        # q, k, v lie side by side from q_col on: x logistic(x) in place, once, before the walk
         if not (q_col < k_col < v_col) or v_col + heads * vdim - q_col != 2 * key_heads * dim + heads * vdim:
@@ -1149,7 +1165,7 @@ def state_scan(rows: torch.Tensor, q_col: int, k_col: int, v_col: int, silu_on_l
                   _ptr(second), heads if second is not None else 0, _ptr(state), _ptr(step.token_pos), _ptr(step.token_seq),
                   _ptr(step.cu_seqlens), _ptr(step.seq_slot), _ptr(out), n, int(step.n_seqs), int(heads), int(key_heads),
                   int(dim), int(vdim), _ptr(rot[0]) if rot else None, int(rot[1]) if rot else 0, int(rot[2]) if rot else 0,
-                  float(rot[3]) if rot else 1.0, _stream(),
+                  float(rot[3]) if rot else 1.0, seg_len, seg_count, _ptr(seg_states), _ptr(seg_decays), _stream(),
                   label="hos_state_scan/channel" if channel_g else ("hos_state_scan/v_factor" if v_factor is not None else None))
 
 
@@ -1187,22 +1203,24 @@ def conv_prep(raw: torch.Tensor, conv_w: torch.Tensor, conv_state: torch.Tensor,
                   _ptr(beta), _ptr(g), n, int(heads), int(key_heads), int(dim), int(vdim), 1 if keep_here else 0, _stream())
 
 
-def conv_keep(raw: torch.Tensor, taps: int, conv_state: torch.Tensor, step, channels: int, col: int = 0) -> None:
-    mixers().call("hos_conv_keep", _at(raw, col), raw.shape[1], int(taps), _ptr(conv_state), _ptr(step.token_pos),
+def conv_keep(raw: torch.Tensor, taps: int, conv_state: torch.Tensor, step, channels: int, col: int = 0,
+              in_bias: Optional[torch.Tensor] = None) -> None:
+    """The last taps - 1 inputs (raw[:, col:col + channels] + in_bias) of every sequence go to the slot's kept inputs."""
+    mixers().call("hos_conv_keep", _at(raw, col), raw.shape[1], _ptr(in_bias), int(taps), _ptr(conv_state), _ptr(step.token_pos),
                   _ptr(step.token_seq), _ptr(step.cu_seqlens), _ptr(step.seq_slot), int(step.n_seqs), int(channels),
                   _stream())
 
 
 def conv_act_rows(raw: torch.Tensor, col: int, conv_w: torch.Tensor, bias: Optional[torch.Tensor], conv_state: torch.Tensor,
-                  act: str, step, out: torch.Tensor, single: bool, dt=None) -> None:
-    """out ([N, C] float32) = act(short convolution of raw[:, col:col + C] + bias), act "none" or "x_logistic"; conv_w: [C, taps];
-    conv_state: [slots, taps - 1, C] (single, only where every sequence brings one token: the kept inputs move on in this
+                  act: str, step, out: torch.Tensor, single: bool, dt=None, in_bias: Optional[torch.Tensor] = None) -> None:
+    """out ([N, C] float32) = act(short convolution of (raw[:, col:col + C] + in_bias) + bias), act "none" or "x_logistic"; conv_w:
+    [taps, C]; conv_state: [slots, taps - 1, C] (single, only where every sequence brings one token: the kept inputs move on in this
     launch; else call conv_keep).  dt = (column, dt_bias, a_log, dt_out, g_out): per head, dt_out = softplus(raw + dt_bias) and
     g_out = exp(-exp(a_log) dt) in the same launch."""
     _check(raw, "projection rows", torch.float32, 2)
     _check(conv_w, "convolution weights", torch.float32, 2)
     _check(out, "convolved rows", torch.float32, 2)
-    n, (c, taps) = raw.shape[0], conv_w.shape
+    n, (taps, c) = raw.shape[0], conv_w.shape
     if tuple(out.shape) != (n, c) or col + c > raw.shape[1] or tuple(conv_state.shape[1:]) != (taps - 1, c):
         raise KernelError("conv_act_rows: sizes disagree")
     dt_args = (None, None, None, None, None, 0)
@@ -1216,7 +1234,7 @@ def conv_act_rows(raw: torch.Tensor, col: int, conv_w: torch.Tensor, bias: Optio
         if dt_col + heads > raw.shape[1] or a_log.shape[0] != heads:
             raise KernelError("conv_act_rows: sizes of the step sizes disagree")
         dt_args = (_at(raw, dt_col), _ptr(dt_bias), _ptr(a_log), _ptr(dt_out), _ptr(g_out), heads)
-    mixers().call("hos_conv_act_rows", _at(raw, col), raw.shape[1], _ptr(conv_w), _ptr(bias), int(taps),
+    mixers().call("hos_conv_act_rows", _at(raw, col), raw.shape[1], _ptr(conv_w), _ptr(in_bias), _ptr(bias), int(taps),
                   _ptr(conv_state) if taps > 1 else None, {"none": 0, "x_logistic": 1}[act], _ptr(step.token_pos), _ptr(step.token_seq),
                   _ptr(step.cu_seqlens), _ptr(step.seq_slot), _ptr(out), n, int(c), 1 if single else 0, *dt_args, _stream())
 

@@ -73,9 +73,9 @@ class GatedSoftmaxAttention(Mixer):
             raise SpecError("arch spec error: kept first keys go with a window")
         self.shares_kv = bool(p.get("shares_kv", False))
         self.taps = int(p.get("conv") or 0)
-        if self.taps < 0 or (self.taps and (self.shares_kv or self.norm_whole)):
-            raise SpecError("arch spec error: a short convolution goes with keys and values of the layer's own and no norm over "
-                            "the whole projection")
+        if self.taps < 0 or (self.taps and (self.shares_kv or self.mix_role)):
+            raise SpecError("arch spec error: a short convolution goes with keys and values of the layer's own, not blended with "
+                            "another's")
         temp = p.get("q_temp")
         self.q_temp = (float(temp["coef"]), int(temp["every"])) if temp else None
         if self.q_temp and self.q_temp[1] <= 0:
@@ -228,15 +228,27 @@ class GatedSoftmaxAttention(Mixer):
             if self.mix_key not in step.shared:
                 raise KernelError(f"attention: no layer of this step has left values under {self.mix_key!r}")
             v_first = step.shared[self.mix_key]
-        kept = store.state["conv"] if self.taps > 1 else None
-        single = step.max_new == 1           # every sequence brings one token: the kept inputs move on in qk_prep itself
-        ops.qk_prep(proj, self.bias, self.q_norm, self.k_norm, self.eps, freq, rot_dims,
-                    getattr(self.position, "magnitude", 1.0), step, q, cache, self.n_heads,
-                    0 if self.shares_kv else self.n_kv_heads, self.dim, self.vdim, self.norm_whole,
-                    v_first[0] if v_first else None, v_first[1] if v_first else 0, self.v_mix,
-                    proj_col=col, conv_w=self.conv_w, conv_state=kept, keep_here=single, q_temp=self.q_temp)
-        if self.taps > 1 and not single:
-            ops.qkv_conv_keep(proj, col, self.bias, self.taps, kept, step, self.q_cols + self.kv_cols)
+        rows, bias = proj, self.bias
+        if self.taps:
+            c = self.q_cols + self.kv_cols
+            kept = store.state["conv"] if self.taps > 1 else proj.new_empty((0, 0, c))
+            single = step.max_new == 1           # every sequence brings one token: the kept inputs move on in the same launch
+            stored = not self.qk_norm and self.position is None
+            if stored:
+                ops.qkv_conv_store(proj, col, self.bias, self.conv_w, kept, step, q, cache, self.n_heads, self.n_kv_heads, self.dim,
+                                   self.vdim, single, self.q_temp)
+            else:                                # norms or a rotation follow: the convolved rows first
+                rows, bias = torch.empty((n, c), dtype=torch.float32, device=proj.device), None
+                ops.conv_act_rows(proj, col, self.conv_w, None, kept, "none", step, rows, single,
+                                  in_bias=self.bias[:c] if self.bias is not None else None)
+            if self.taps > 1 and not single:
+                ops.conv_keep(proj, self.taps, kept, step, c, col, self.bias)
+        if not self.taps or not stored:
+            ops.qk_prep(rows, bias, self.q_norm, self.k_norm, self.eps, freq, rot_dims,
+                        getattr(self.position, "magnitude", 1.0), step, q, cache, self.n_heads,
+                        0 if self.shares_kv else self.n_kv_heads, self.dim, self.vdim, self.norm_whole,
+                        v_first[0] if v_first else None, v_first[1] if v_first else 0, self.v_mix,
+                        proj_col=col if rows is proj else 0, q_temp=self.q_temp)
         gate = proj if self.head_gate else None
         where = dict(keep_first=self.keep_first, out_col=out_col, out_scale=self.out_scale)
         if self.use_tensor_cores and att.dtype == torch.bfloat16 and step.max_new > FEW_TOKENS:

@@ -307,7 +307,8 @@ class StateSpace(Mixer):
     def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
         w = self.spec.weights
         self.w_in = linear.pad_rows(self._matrix(tensors[w["in"]]))              # z | x | B | C | dt
-        self.conv_w, self.conv_bias = tensors[w["conv"]].to(torch.float32).contiguous(), self._vector32(tensors[w["conv_bias"]])
+        self.conv_w = tensors[w["conv"]].to(torch.float32).t().contiguous()      # [taps, channels]
+        self.conv_bias = self._vector32(tensors[w["conv_bias"]])
         self.dt_bias, self.a_log, self.skip = (self._vector32(tensors[w[r]]) for r in ("dt_bias", "A_log", "D"))
         self.norm_w = self._vector32(tensors[w["norm"]])
         self.w_o = self._matrix(tensors[w["o"]])

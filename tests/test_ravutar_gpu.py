@@ -530,16 +530,16 @@ def test_the_convolution_kernel_alone(taps, c, act):
         step, cu = _ragged(dev, lens, starts, [6, 0, 3, 5, 2][:len(lens)])
         n, ld = sum(lens) + 1, -(-(col + c + H) // 4) * 4
         raw = torch.randn(n, ld, device=dev)
-        w, b = torch.randn(c, taps, device=dev), torch.randn(c, device=dev)
+        w, b, ib = torch.randn(taps, c, device=dev), torch.randn(c, device=dev), torch.randn(c, device=dev)
         keep = torch.randn(7, taps - 1, c, device=dev)
         dt_bias, a_log = torch.randn(H, device=dev), torch.randn(H, device=dev)
         out, dt, g = torch.empty(n, c, device=dev), torch.empty(n, H, device=dev), torch.empty(n, H, device=dev)
         single = max(lens) == 1
         kept = keep.clone()
-        ops.conv_act_rows(raw, col, w, b, kept, act, step, out, single, (col + c, dt_bias, a_log, dt, g))
+        ops.conv_act_rows(raw, col, w, b, kept, act, step, out, single, (col + c, dt_bias, a_log, dt, g), in_bias=ib)
         if not single:
-            ops.conv_keep(raw, taps, kept, step, c, col)
-        U, W = raw.double().cpu()[:, col:col + c], w.double().cpu()
+            ops.conv_keep(raw, taps, kept, step, c, col, ib)
+        U, W = (raw[:, col:col + c] + ib).double().cpu(), w.double().cpu().T
         for i, k in enumerate(lens):
             slot = int(step.seq_slot[i])
             before = keep[slot].double().cpu() if starts[i] else torch.zeros(taps - 1, c, dtype=torch.float64)
@@ -734,9 +734,8 @@ def test_attention_into_columns_of_a_wider_row():
         step = StepInfo(T, 1, None, i32(list(range(T))), i32([0] * T), i32([0, T]), i32([1]), i32([T]), True, False, T, T)
         q = torch.empty(T, H, kd, device=dev)
         kept = torch.randn(2, taps - 1, c, device=dev)
-        ops.qk_prep(proj, bias, None, None, 1e-6, None, 0, 1.0, step, q, cache, H, G, kd, vd, proj_col=4, conv_w=w, conv_state=kept,
-                    q_temp=(0.4, 50))
-        ops.qkv_conv_keep(proj, 4, bias, taps, kept, step, c)
+        ops.qkv_conv_store(proj, 4, bias, w, kept, step, q, cache, H, G, kd, vd, False, (0.4, 50))
+        ops.conv_keep(proj, taps, kept, step, c, 4, bias)
         assert float((q.double().cpu() - Q).abs().max()) < 1e-5
         assert float((kept[1].double().cpu() - U[-(taps - 1):]).abs().max()) < 1e-6
         want = torch.zeros(T, H, vd, dtype=torch.float64)
@@ -758,8 +757,7 @@ def test_attention_into_columns_of_a_wider_row():
         kept[1] = U[-taps:-1].float().to(dev)
         one = StepInfo(1, 1, None, i32([T - 1]), i32([0]), i32([0, 1]), i32([1]), i32([T]), False, True, 1, T)
         q1 = torch.empty(1, H, kd, device=dev)
-        ops.qk_prep(proj[T - 1:].contiguous(), bias, None, None, 1e-6, None, 0, 1.0, one, q1, cache, H, G, kd, vd, proj_col=4, conv_w=w,
-                    conv_state=kept, keep_here=True, q_temp=(0.4, 50))
+        ops.qkv_conv_store(proj[T - 1:].contiguous(), 4, bias, w, kept, one, q1, cache, H, G, kd, vd, True, (0.4, 50))
         assert float((q1.double().cpu() - Q[-1:]).abs().max()) < 1e-5
         assert float((kept[1].double().cpu() - U[-(taps - 1):]).abs().max()) < 1e-6
         for shares in (1, 3):
@@ -770,3 +768,85 @@ def test_attention_into_columns_of_a_wider_row():
                 ops.gated_attn(q1, cache, sink, None, 0, one, out, scale, 0, 0, shares, out_col=16, out_scale=factor)
             assert float((out[:, 16:16 + H * vd].double().cpu() - want[-1:]).abs().max()) < tol * float(want.abs().max())
             assert float((out[:, :16] - 9).abs().max()) == 0.0 and float((out[:, 16 + H * vd:] - 9).abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("H, G, d, vd", [(3, 3, 16, 20), (4, 2, 64, 48), (2, 1, 200, 8), (1, 1, 7, 5), (1, 1, 300, 2)])
+def test_a_scan_in_segments_gives_what_a_whole_walk_gives(H, G, d, vd):
+    """Long sequences of the decay rule (decays and factors per token, or constants) and of the channel rule are walked in
+    segments side by side: the same read-outs and states as the whole walk, for sequences that start and that go on,
+    some of them shorter than a segment, with decays near one and decays that vanish within a segment."""
+    from hos_b200 import ops
+    dev = "cuda"
+    torch.manual_seed(5)
+    lens, starts = [1, 700, 65, 401], [0, 0, 12, 7]
+    step, cu = _ragged(dev, lens, starts, [2, 0, 3, 1])
+    n = sum(lens) + 1
+    assert ops.mixers().fn("hos_state_scan_segment")(len(lens), H, d, vd, max(lens), 0) > 0, "these sizes are not walked in segments"
+    for kind in ("token", "constant", "channel"):
+        channel, g_heads = kind == "channel", H if kind == "channel" else G
+        ld = -(-(2 * g_heads * d + H * vd + 3) // 4) * 4
+        rows = torch.randn(n, ld, device=dev) * 0.3
+        shape = {"token": (n, H), "constant": (H,), "channel": (n, H * d)}[kind]
+        g = 1.0 - torch.rand(shape, device=dev) * 0.02
+        if kind != "constant":
+            g[::97] = 1e-3
+            g[300:340] = 1e-12           # a product of these is below what 32 bits hold
+        f = torch.rand(n, H, device=dev) + 0.3 if kind == "token" else None
+        state = torch.randn(4, H, vd, d, device=dev)
+        outs = []
+        for on in (True, False):
+            ops.segmented_scans = on
+            try:
+                kept, out = state.clone(), torch.zeros(n, H * vd, device=dev)
+                ops.state_scan(rows, 0, g_heads * d, 2 * g_heads * d, False, g, kind != "constant", None, kept, step, out, H, g_heads, d, vd,
+                               v_factor=f, channel_g=channel, o_mult=0.5)
+                outs.append((out, kept))
+            finally:
+                ops.segmented_scans = True
+        for a, b in zip(*outs):
+            assert float((a - b).abs().max()) < 1e-5 * float(b.abs().max()), kind
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_convolution_before_norms_and_a_rotation(dtype):
+    """The attention mixer with a convolution and what may follow it (a norm per head or over the projection, a rotation):
+    the same as the mixer without a convolution on rows that were convolved outside."""
+    from hos_b200.cache.kv import KVGroup
+    from hos_b200.config.base import PartSpec
+    from hos_b200.parts.base import CallStore, Runtime, StepInfo
+    from hos_b200.registry import part_impl
+    dev, dt = "cuda", {"float32": torch.float32, "bfloat16": torch.bfloat16}[dtype]
+    torch.manual_seed(3)
+    H, G, kd, vd, width, T, taps = 4, 2, 16, 12, 24, 90, 3
+    c = H * kd + G * (kd + vd)
+    for norm, rot in (("head", True), ("whole", False), (False, True)):
+        base = {"width": width, "n_heads": H, "n_kv_heads": G, "dim": kd, "vdim": vd, "scale": 0.3, "bias": True, "qk_norm": norm,
+                "position": PartSpec("rotary", {"theta": 100.0, "rotary_dim": 8, "style": "interleaved"}) if rot else None}
+        names = {r: r for r in ("q", "k", "v", "o", "q_bias", "k_bias", "v_bias", "q_norm", "k_norm", "q_conv", "k_conv", "v_conv")}
+        outs = []
+        rt = Runtime(torch.device(dev), dt)
+        with_conv = part_impl("mixer", "gated_softmax_attention")(PartSpec("gated_softmax_attention", dict(base, conv=taps), names), rt)
+        plain = part_impl("mixer", "gated_softmax_attention")(PartSpec("gated_softmax_attention", dict(base, bias=False), names), rt)
+        g = torch.Generator().manual_seed(1)
+        tensors = {s.name: torch.randn(tuple(s.shape), generator=g).to(dev) for s in with_conv.weight_specs()}
+        with_conv.bind(tensors)
+        plain.bind(tensors)
+        proj = torch.randn(T, c, device=dev)
+        u = torch.cat([torch.zeros(taps - 1, c, device=dev), proj + with_conv.bias])
+        convolved = sum(u[j:j + T] * with_conv.conv_w[j] for j in range(taps)).contiguous()
+        i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        cuts = [(0, 50), (50, 89), (89, 90)]
+        for m, rows in ((with_conv, proj), (plain, convolved)):
+            group = KVGroup(m.kv_need(), 1, 4, 2, 128, dt, torch.device(dev))
+            group.open_slot(1)
+            group.grow(1, T)
+            group.flush()
+            store = CallStore(group.view(0), True, {"conv": torch.full((2, taps - 1, c), 5.0, device=dev)})
+            att = torch.empty(T, H * vd, device=dev, dtype=dt)
+            for a, b in cuts:
+                step = StepInfo(b - a, 1, None, i32(list(range(a, b))), i32([0] * (b - a)), i32([0, b - a]), i32([1]), i32([b]), a == 0,
+                                b - a == 1, b - a, b)
+                m.run_heads(rows[a:b].contiguous(), 0, step, store, att[a:b], 0)
+            outs.append(att.float())
+        tol = 2e-5 if dtype == "float32" else 2e-2
+        assert float((outs[0] - outs[1]).abs().max()) < tol * float(outs[1].abs().max()), (norm, rot)
