@@ -106,7 +106,9 @@ struct Segments {
     int len, count;
 };
 
-template <int DR, int R, int RULE, bool LOCAL>
+// A thread's cells: DR rows of DC neighbouring columns (DC > 1, the walks by segments: what is read of k, q and the decays
+// serves DC columns).
+template <int DR, int R, int DC, int RULE, bool LOCAL>
 __global__ void __launch_bounds__(256)
 state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, long long ld,
                   int aligned, int act_in_walk, const float* __restrict__ g, long long g_ld, const float* __restrict__ beta,
@@ -133,16 +135,18 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
     const int slot = seq_slot[seq];
     const int kh = head / (H / Gk);
     const int r = threadIdx.x % R, c = threadIdx.x / R;
-    const int col = col0 + c;
+    const int col = col0 + c * DC;
     const bool rot_in_walk = rot_dims > 0 || k_mult != 1.f;
-    const bool live = c < CC && col < vdim;
+    const int n_cols = CC / DC;                  // threads' columns of this block
+    auto live = [&](int j) { return c < n_cols && col + j < vdim; };
     const int dpad = R * (DR + kPad);
     // two buffers of staged tokens: while one chunk is walked the next one's rows are on their way (cp.async)
     const int per_buf = kScanChunk * ((CHANNEL ? 3 : 2) * dpad + 2 * CC) + 2 * kScanChunk;      // q, k, (g,) v, o, g, beta
+    const bool v_aligned = DC == 4 && (vdim & 3) == 0 && (ld & 3) == 0 && ((uintptr_t)v & 15) == 0;
     const bool v_scaled = RULE == kDecayRule && beta != nullptr;
 
-    float S[DR];
-    const size_t cell = ((size_t)head * vdim + (live ? col : 0)) * dim + r * DR, cells = (size_t)H * vdim * dim;
+    float S[DC][DR];
+    const size_t cell = ((size_t)head * vdim + (live(0) ? col : 0)) * dim + r * DR, cells = (size_t)H * vdim * dim;
     float* st = state + (size_t)slot * cells + cell;                                  // the slot's
     float* seg_st = sg.states + ((size_t)seq * sg.count + seg) * cells + cell;        // the segment's, where there are several
     // where this walk starts: the slot's state (whole sequences, and the first segment of a first walk), zero, or the
@@ -151,16 +155,20 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
     const float* src = from_seg ? seg_st : st;
     const bool zero = from_seg ? false : (fresh || seg > 0);
     // a thread's run of rows is contiguous in the kept S^T: 16 bytes at a time where the run is whole and aligned
-    const bool whole = live && r * DR + DR <= dim && (dim & 3) == 0;
-    if (!zero && whole) {
+    const bool whole = r * DR + DR <= dim && (dim & 3) == 0;
 #pragma unroll
-        for (int i = 0; i < DR / 4; ++i) {
-            const float4 t = ((const float4*)src)[i];
-            S[4 * i] = t.x; S[4 * i + 1] = t.y; S[4 * i + 2] = t.z; S[4 * i + 3] = t.w;
+    for (int j = 0; j < DC; ++j) {
+        const float* from = src + (size_t)j * dim;
+        if (!zero && whole && live(j)) {
+#pragma unroll
+            for (int i = 0; i < DR / 4; ++i) {
+                const float4 t = ((const float4*)from)[i];
+                S[j][4 * i] = t.x; S[j][4 * i + 1] = t.y; S[j][4 * i + 2] = t.z; S[j][4 * i + 3] = t.w;
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < DR; ++i) S[j][i] = (!zero && live(j) && r * DR + i < dim) ? from[i] : 0.f;
         }
-    } else {
-#pragma unroll
-        for (int i = 0; i < DR; ++i) S[i] = (!zero && live && r * DR + i < dim) ? src[i] : 0.f;
     }
     // rows beyond dim and columns beyond vdim are read by the walk and never staged: they stay zero for good
     if (R * DR != dim || col0 + CC > vdim) {
@@ -194,6 +202,13 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
             }
         }
         const int ncol = min(CC, vdim - col0);
+        if (DC == 4 && v_aligned) {
+            const int c4 = ncol >> 2;
+            for (int idx = threadIdx.x; idx < nt * c4; idx += blockDim.x) {
+                const int t = idx / c4, cc = (idx % c4) << 2;
+                cp_async16(vs + t * CC + cc, v + (size_t)(t0 + t) * ld + head * vdim + col0 + cc);
+            }
+        } else
         for (int idx = threadIdx.x; idx < nt * ncol; idx += blockDim.x) {
             const int t = idx / ncol, cc = idx % ncol;
             cp_async4(vs + t * CC + cc, v + (size_t)(t0 + t) * ld + head * vdim + col0 + cc);
@@ -246,7 +261,7 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
         float* gs = os + kScanChunk * CC;
         float* bs = gs + kScanChunk;
         {       // every thread walks (a warp's shuffles want all its lanes); only live columns are written
-            float part[kScanChunk];       // the read-outs' partial sums: added up after the walk, off its chain
+            float part[kScanChunk];       // one column: the read-outs' partial sums, added up after the walk, off its chain
 #pragma unroll
             for (int t = 0; t < kScanChunk; ++t) {
                 part[t] = 0.f;
@@ -255,26 +270,37 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                 const float4* q4 = (const float4*)(qs + t * dpad + r * (DR + kPad));
                 const float4* g4 = (const float4*)(gk + t * dpad + r * (DR + kPad));
                 const float gt = CHANNEL ? 0.f : gs[t];
-                float u = c < CC ? vs[t * CC + c] : 0.f;
-                if (RULE == kDecayRule && act_in_walk) u = silu_precise(u);      // single tokens: the activation rides here
-                if (v_scaled) u *= bs[t];
+                float u[DC];
+                if constexpr (DC == 4) {
+                    const float4 t4 = c < n_cols ? *(const float4*)(vs + t * CC + c * DC) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    u[0] = t4.x; u[1] = t4.y; u[2] = t4.z; u[3] = t4.w;
+                } else {
+                    u[0] = c < n_cols ? vs[t * CC + c] : 0.f;
+                }
+#pragma unroll
+                for (int j = 0; j < DC; ++j) {
+                    if (RULE == kDecayRule && act_in_walk) u[j] = silu_precise(u[j]);      // single tokens: the activation rides here
+                    if (v_scaled) u[j] *= bs[t];
+                }
                 if (DELTA) {
                     float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;       // four chains, not one of DR links
 #pragma unroll
                     for (int i = 0; i < DR / 4; ++i) {
                         const float4 kk = k4[i];
-                        S[4 * i] *= gt; S[4 * i + 1] *= gt; S[4 * i + 2] *= gt; S[4 * i + 3] *= gt;
-                        d0 = fmaf(S[4 * i], kk.x, d0);
-                        d1 = fmaf(S[4 * i + 1], kk.y, d1);
-                        d2 = fmaf(S[4 * i + 2], kk.z, d2);
-                        d3 = fmaf(S[4 * i + 3], kk.w, d3);
+                        S[0][4 * i] *= gt; S[0][4 * i + 1] *= gt; S[0][4 * i + 2] *= gt; S[0][4 * i + 3] *= gt;
+                        d0 = fmaf(S[0][4 * i], kk.x, d0);
+                        d1 = fmaf(S[0][4 * i + 1], kk.y, d1);
+                        d2 = fmaf(S[0][4 * i + 2], kk.z, d2);
+                        d3 = fmaf(S[0][4 * i + 3], kk.w, d3);
                     }
                     float dot = (d0 + d1) + (d2 + d3);
 #pragma unroll
                     for (int o = 1; o < R; o <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
-                    u = bs[t] * (u - dot);
+                    u[0] = bs[t] * (u[0] - dot);
                 }
-                float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+                float a[DC][4];
+#pragma unroll
+                for (int j = 0; j < DC; ++j) a[j][0] = a[j][1] = a[j][2] = a[j][3] = 0.f;
 #pragma unroll
                 for (int i = 0; i < DR / 4; ++i) {
                     float4 kk = k4[i], qq = LOCAL ? make_float4(0.f, 0.f, 0.f, 0.f) : q4[i];
@@ -282,34 +308,50 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                         kk = make_float4(silu_precise(kk.x), silu_precise(kk.y), silu_precise(kk.z), silu_precise(kk.w));
                         qq = make_float4(silu_precise(qq.x), silu_precise(qq.y), silu_precise(qq.z), silu_precise(qq.w));
                     }
-                    if (DELTA) {
-                        S[4 * i] = fmaf(kk.x, u, S[4 * i]);
-                        S[4 * i + 1] = fmaf(kk.y, u, S[4 * i + 1]);
-                        S[4 * i + 2] = fmaf(kk.z, u, S[4 * i + 2]);
-                        S[4 * i + 3] = fmaf(kk.w, u, S[4 * i + 3]);
-                    } else if (CHANNEL) {
-                        const float4 gg = g4[i];
-                        S[4 * i] = fmaf(gg.x, S[4 * i], kk.x * u);
-                        S[4 * i + 1] = fmaf(gg.y, S[4 * i + 1], kk.y * u);
-                        S[4 * i + 2] = fmaf(gg.z, S[4 * i + 2], kk.z * u);
-                        S[4 * i + 3] = fmaf(gg.w, S[4 * i + 3], kk.w * u);
-                    } else {
-                        S[4 * i] = fmaf(gt, S[4 * i], kk.x * u);
-                        S[4 * i + 1] = fmaf(gt, S[4 * i + 1], kk.y * u);
-                        S[4 * i + 2] = fmaf(gt, S[4 * i + 2], kk.z * u);
-                        S[4 * i + 3] = fmaf(gt, S[4 * i + 3], kk.w * u);
+                    const float4 gg = CHANNEL ? g4[i] : make_float4(gt, gt, gt, gt);
+#pragma unroll
+                    for (int j = 0; j < DC; ++j) {
+                        float* s4 = &S[j][4 * i];
+                        if (DELTA) {
+                            s4[0] = fmaf(kk.x, u[j], s4[0]);
+                            s4[1] = fmaf(kk.y, u[j], s4[1]);
+                            s4[2] = fmaf(kk.z, u[j], s4[2]);
+                            s4[3] = fmaf(kk.w, u[j], s4[3]);
+                        } else {
+                            s4[0] = fmaf(gg.x, s4[0], kk.x * u[j]);
+                            s4[1] = fmaf(gg.y, s4[1], kk.y * u[j]);
+                            s4[2] = fmaf(gg.z, s4[2], kk.z * u[j]);
+                            s4[3] = fmaf(gg.w, s4[3], kk.w * u[j]);
+                        }
+                        if (LOCAL) continue;
+                        a[j][0] = fmaf(s4[0], qq.x, a[j][0]);
+                        a[j][1] = fmaf(s4[1], qq.y, a[j][1]);
+                        a[j][2] = fmaf(s4[2], qq.z, a[j][2]);
+                        a[j][3] = fmaf(s4[3], qq.w, a[j][3]);
                     }
-                    if (LOCAL) continue;
-                    a0 = fmaf(S[4 * i], qq.x, a0);
-                    a1 = fmaf(S[4 * i + 1], qq.y, a1);
-                    a2 = fmaf(S[4 * i + 2], qq.z, a2);
-                    a3 = fmaf(S[4 * i + 3], qq.w, a3);
                 }
-                part[t] = (a0 + a1) + (a2 + a3);
+                if constexpr (DC == 1) {
+                    part[t] = (a[0][0] + a[0][1]) + (a[0][2] + a[0][3]);
+                } else if constexpr (!LOCAL) {
+                    // four columns' sums over R threads: a thread hands on the columns it does not end with, two and then
+                    // one, and the rest of the threads add up the one that is left
+                    static_assert(DC == 4 && R >= 4, "the sums of four columns");
+                    float p[4];
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) p[j] = (a[j][0] + a[j][1]) + (a[j][2] + a[j][3]);
+                    const bool up = (r & (R / 2)) != 0, up2 = (r & (R / 4)) != 0;
+                    const float x0 = __shfl_xor_sync(0xffffffffu, up ? p[0] : p[2], R / 2);
+                    const float x1 = __shfl_xor_sync(0xffffffffu, up ? p[1] : p[3], R / 2);
+                    const float y0 = (up ? p[2] : p[0]) + x0, y1 = (up ? p[3] : p[1]) + x1;
+                    float acc = (up2 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, up2 ? y0 : y1, R / 4);
+#pragma unroll
+                    for (int o = R / 8; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+                    if ((r & (R / 4 - 1)) == 0 && c < n_cols) os[t * CC + c * DC + (up ? 2 : 0) + (up2 ? 1 : 0)] = acc * o_mult;
+                }
             }
 #pragma unroll
             for (int t = 0; t < kScanChunk; ++t) {
-                if (LOCAL || t >= nt) break;
+                if (LOCAL || DC > 1 || t >= nt) break;
                 float acc = part[t];
 #pragma unroll
                 for (int o = 1; o < R; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
@@ -346,13 +388,19 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
     } else if (!last) {
         return;                                  // only the last segment's state is the sequence's
     }
-    if (whole) {
 #pragma unroll
-        for (int i = 0; i < DR / 4; ++i) ((float4*)st)[i] = make_float4(S[4 * i], S[4 * i + 1], S[4 * i + 2], S[4 * i + 3]);
-    } else if (live) {
+    for (int j = 0; j < DC; ++j) {
+        if (!live(j)) continue;
+        float* to = st + (size_t)j * dim;
+        if (whole) {
 #pragma unroll
-        for (int i = 0; i < DR; ++i)
-            if (r * DR + i < dim) st[i] = S[i];
+            for (int i = 0; i < DR / 4; ++i)
+                ((float4*)to)[i] = make_float4(S[j][4 * i], S[j][4 * i + 1], S[j][4 * i + 2], S[j][4 * i + 3]);
+        } else {
+#pragma unroll
+            for (int i = 0; i < DR; ++i)
+                if (r * DR + i < dim) to[i] = S[j][i];
+        }
     }
 }
 
@@ -538,8 +586,8 @@ using namespace hos;
 namespace hos {
 // How a walk is cut: DR rows of a column to a thread, R threads to a column, CC columns to a block.
 struct ScanShape {
-    int DR, R, CC;
-    ScanShape(int dim, int vdim) {
+    int DR, R, CC, DC = 1;
+    ScanShape(int dim, int vdim, bool segments = false) {
         // short runs of rows per thread: a token's walk is a chain of dependent instructions (scale, dot, sum over the
         // runs, update, read-out, sum), and with few (sequence, head) pairs nothing else hides its latency; the sums over
         // 16 or 32 runs are shuffles
@@ -550,10 +598,11 @@ struct ScanShape {
         while (R * DR < dim) R <<= 1;
         if (DR == 8 && R < 4) R = 4;          // the compiled shapes (rows beyond dim are zeros)
         if (DR >= 16) R = 32;
-        CC = 256 / R;
-        if (CC > vdim) CC = vdim;
+        if (segments && DR == 8) DC = 4;      // the shapes that are compiled for four columns to a thread
+        CC = 256 / R * DC;
+        if (CC > vdim) CC = (vdim + DC - 1) / DC * DC;
     }
-    int threads() const { return (CC * R + 31) / 32 * 32; }
+    int threads() const { return (CC / DC * R + 31) / 32 * 32; }
 };
 constexpr int kMinSegment = 64;       // tokens
 }  // namespace hos
@@ -563,11 +612,11 @@ constexpr int kMinSegment = 64;       // tokens
 // n_seqs * n * H * vdim * dim and n_seqs * n * H (channel rule: H * dim) floats.
 extern "C" int hos_state_scan_segment(int n_seqs, int H, int dim, int vdim, int max_new, int rule) {
     if (rule == kDeltaRule || n_seqs <= 0 || max_new < 3 * kMinSegment || dim <= 0 || dim > 1024 || vdim <= 0) return 0;
-    const ScanShape shape(dim, vdim);
+    const ScanShape shape(dim, vdim, true);
     if (rule == kChannelRule && dim > kDecayPerThread * shape.threads()) return 0;
     const long long blocks = (long long)n_seqs * H * ((vdim + shape.CC - 1) / shape.CC);
     // a walk is bound by its chain until several blocks share an SM; two walks instead of one must be paid for
-    const long long want = 8ll * sm_count_cached() / blocks;
+    const long long want = (shape.DC > 1 ? 4ll : 8ll) * sm_count_cached() / blocks;
     if (want < 3) return 0;
     const int count = (int)(want < max_new / kMinSegment ? want : max_new / kMinSegment);
     const int len = (max_new + count - 1) / count;
@@ -593,16 +642,16 @@ extern "C" int hos_state_scan(const float* q, const float* k, const float* v, lo
         HOS_REFUSE("state_scan: %d rotated numbers in heads of %d", rot_dims, dim);
     if (Gk <= 0 || H % Gk != 0) HOS_REFUSE("state_scan: %d heads are not a multiple of %d key heads", H, Gk);
     if (dim <= 0 || dim > 1024 || vdim <= 0) HOS_REFUSE("state_scan: heads of %d x %d", dim, vdim);
-    const ScanShape shape(dim, vdim);
-    const int DR = shape.DR, R = shape.R;
+    const bool segments = seg_count > 1;
+    const ScanShape shape(dim, vdim, segments);
+    const int DR = shape.DR, R = shape.R, DC = shape.DC;
     int CC = shape.CC;
     // single tokens and few (sequence, head) pairs: fewer columns to a block, so that the blocks fill the GPU (columns
     // are independent; every block stages the whole q and k rows, which a long walk would pay for token by token)
-    if (n_rows <= 2 * n_seqs)
+    if (n_rows <= 2 * n_seqs && !segments)
         while (CC * R > 64 && (long long)n_seqs * H * ((vdim + CC - 1) / CC) < 2 * sm_count_cached()) CC = (CC + 1) / 2;
-    const int threads = (CC * R + 31) / 32 * 32;
+    const int threads = (CC / DC * R + 31) / 32 * 32;
     const int dpad = R * (DR + kPad);
-    const bool segments = seg_count > 1;
     if (segments && (rule == kDeltaRule || act_in_walk || rot_dims > 0 || k_mult != 1.f || seg_len <= 0 || seg_states == nullptr ||
                      seg_decays == nullptr || (rule == kChannelRule && dim > kDecayPerThread * threads)))
         HOS_REFUSE("state_scan: %d segments of %d tokens do not fit this walk", seg_count, seg_len);
@@ -617,26 +666,29 @@ extern "C" int hos_state_scan(const float* q, const float* k, const float* v, lo
     const dim3 grid(n_seqs * sg.count, H, (vdim + CC - 1) / CC);
     if (rule != kDecayRule && act_in_walk) HOS_REFUSE("state_scan: the activation in the walk is the decay rule's");
     if (smem > 200 * 1024) HOS_REFUSE("state_scan: heads of %d x %d do not fit a block's shared memory", dim, vdim);
-#define HOS_SCAN(DRv, Rv, DL, LOC)                                                                                   \
+#define HOS_SCAN(DRv, Rv, DCv, DL, LOC)                                                                                   \
     do {                                                                                                             \
         if (smem > 48 * 1024)                                                                                        \
-            cudaFuncSetAttribute(state_scan_kernel<DRv, Rv, DL, LOC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        launch_pdl(state_scan_kernel<DRv, Rv, DL, LOC>, grid, dim3(threads), smem, stream, q, k, v, ld, aligned, act_in_walk, g, g_ld, beta, \
+            cudaFuncSetAttribute(state_scan_kernel<DRv, Rv, DCv, DL, LOC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        launch_pdl(state_scan_kernel<DRv, Rv, DCv, DL, LOC>, grid, dim3(threads), smem, stream, q, k, v, ld, aligned, act_in_walk, g, g_ld, beta, \
                    beta_ld, state, token_pos, token_seq, cu_seqlens, seq_slot, out, H, Gk, dim, vdim, CC, rot_freq,  \
                    rot_dims, rot_style, k_mult, o_mult, sg);                                                         \
     } while (0)
 #define HOS_SCAN_S(DRv, Rv, DL)                                                                                      \
     do {                                                                                                             \
+        constexpr int DCs = DRv == 8 ? 4 : 1;                                                                        \
         if (segments) {                                                                                              \
-            HOS_SCAN(DRv, Rv, DL, true);                                                                             \
+            HOS_SCAN(DRv, Rv, DCs, DL, true);                                                                           \
             launch_pdl(segment_starts_kernel, dim3((unsigned)(((long long)H * vdim * dim + 255) / 256), n_seqs), dim3(256), 0, stream, \
                        (const float*)state, sg, token_pos, token_seq, cu_seqlens, seq_slot, H, dim, vdim, DL == kChannelRule ? 1 : 0); \
+            HOS_SCAN(DRv, Rv, DCs, DL, false);                                                                       \
+        } else {                                                                                                     \
+            HOS_SCAN(DRv, Rv, 1, DL, false);                                                                         \
         }                                                                                                            \
-        HOS_SCAN(DRv, Rv, DL, false);                                                                                \
     } while (0)
 #define HOS_SCAN_D(DRv, Rv)                                                                                          \
     do {                                                                                                             \
-        if (rule == kDeltaRule) HOS_SCAN(DRv, Rv, kDeltaRule, false);                                                \
+        if (rule == kDeltaRule) HOS_SCAN(DRv, Rv, 1, kDeltaRule, false);                                              \
         else if (rule == kChannelRule) HOS_SCAN_S(DRv, Rv, kChannelRule);                                            \
         else HOS_SCAN_S(DRv, Rv, kDecayRule);                                                                        \
     } while (0)
