@@ -95,6 +95,24 @@ rotate_rows_kernel(float* __restrict__ x, long long ld, int Hq, int Hk, int dim,
 
 constexpr int kDecayPerThread = 4;
 
+// Two 32-bit multiply-adds (or products) in one instruction: each half is the plain operation with one rounding.
+__device__ __forceinline__ uint64_t pair_of(float x, float y) {
+    uint64_t d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(x), "f"(y));
+    return d;
+}
+__device__ __forceinline__ void halves_of(uint64_t p, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(p)); }
+__device__ __forceinline__ uint64_t fma_pair(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ uint64_t mul_pair(uint64_t a, uint64_t b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+
 enum ScanRule : int { kDecayRule = 0, kDeltaRule = 1, kChannelRule = 2 };
 
 // What a walk by segments needs: seg_len rows to a segment, `count` segments to a sequence at most (blockIdx.x is sequence x
@@ -169,6 +187,13 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
 #pragma unroll
             for (int i = 0; i < DR; ++i) S[j][i] = (!zero && live(j) && r * DR + i < dim) ? from[i] : 0.f;
         }
+    }
+    uint64_t P[DC][DR / 2];                      // four columns: the cells as pairs of rows
+    if (DC == 4) {
+#pragma unroll
+        for (int j = 0; j < DC; ++j)
+#pragma unroll
+            for (int i = 0; i < DR / 2; ++i) P[j][i] = pair_of(S[j][2 * i], S[j][2 * i + 1]);
     }
     // rows beyond dim and columns beyond vdim are read by the walk and never staged: they stay zero for good
     if (R * DR != dim || col0 + CC > vdim) {
@@ -260,8 +285,66 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
         float* os = vs + kScanChunk * CC;
         float* gs = os + kScanChunk * CC;
         float* bs = gs + kScanChunk;
-        {       // every thread walks (a warp's shuffles want all its lanes); only live columns are written
-            float part[kScanChunk];       // one column: the read-outs' partial sums, added up after the walk, off its chain
+        if constexpr (DC == 4) {
+#pragma unroll 2
+            for (int t = 0; t < nt; ++t) {
+                const float4* k4 = (const float4*)(ks + t * dpad + r * (DR + kPad));
+                const float4* q4 = (const float4*)(qs + t * dpad + r * (DR + kPad));
+                const float4* g4 = (const float4*)(gk + t * dpad + r * (DR + kPad));
+                float4 u = c < n_cols ? *(const float4*)(vs + t * CC + c * DC) : make_float4(0.f, 0.f, 0.f, 0.f);
+                if (v_scaled) {
+                    const float f = bs[t];
+                    u = make_float4(u.x * f, u.y * f, u.z * f, u.w * f);
+                }
+                const uint64_t uu[4] = {pair_of(u.x, u.x), pair_of(u.y, u.y), pair_of(u.z, u.z), pair_of(u.w, u.w)};
+                const uint64_t gt = CHANNEL ? 0 : pair_of(gs[t], gs[t]);
+                uint64_t a[4] = {0, 0, 0, 0};
+#pragma unroll
+                for (int i = 0; i < DR / 4; ++i) {
+                    const float4 kk = k4[i];
+                    const uint64_t k2[2] = {pair_of(kk.x, kk.y), pair_of(kk.z, kk.w)};
+                    uint64_t g2[2] = {gt, gt}, q2[2] = {0, 0};
+                    if (CHANNEL) {
+                        const float4 gg = g4[i];
+                        g2[0] = pair_of(gg.x, gg.y);
+                        g2[1] = pair_of(gg.z, gg.w);
+                    }
+                    if (!LOCAL) {
+                        const float4 qq = q4[i];
+                        q2[0] = pair_of(qq.x, qq.y);
+                        q2[1] = pair_of(qq.z, qq.w);
+                    }
+#pragma unroll
+                    for (int e = 0; e < 2; ++e)
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) {
+                            uint64_t& p = P[j][2 * i + e];
+                            p = fma_pair(g2[e], p, mul_pair(k2[e], uu[j]));
+                            if (!LOCAL) a[j] = fma_pair(p, q2[e], a[j]);
+                        }
+                }
+                if (LOCAL) continue;
+                // four columns' sums over R threads: a thread hands on the columns it does not end with, two and then one,
+                // and the rest of the threads add up the one that is left
+                static_assert(R >= 4, "the sums of four columns");
+                float p[4];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    float x, y;
+                    halves_of(a[j], x, y);
+                    p[j] = x + y;
+                }
+                const bool up = (r & (R / 2)) != 0, up2 = (r & (R / 4)) != 0;
+                const float x0 = __shfl_xor_sync(0xffffffffu, up ? p[0] : p[2], R / 2);
+                const float x1 = __shfl_xor_sync(0xffffffffu, up ? p[1] : p[3], R / 2);
+                const float y0 = (up ? p[2] : p[0]) + x0, y1 = (up ? p[3] : p[1]) + x1;
+                float acc = (up2 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, up2 ? y0 : y1, R / 4);
+#pragma unroll
+                for (int o = R / 8; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+                if ((r & (R / 4 - 1)) == 0 && c < n_cols) os[t * CC + c * DC + (up ? 2 : 0) + (up2 ? 1 : 0)] = acc * o_mult;
+            }
+        } else {       // every thread walks (a warp's shuffles want all its lanes); only live columns are written
+            float part[kScanChunk];       // the read-outs' partial sums: added up after the walk, off its chain
 #pragma unroll
             for (int t = 0; t < kScanChunk; ++t) {
                 part[t] = 0.f;
@@ -270,18 +353,9 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                 const float4* q4 = (const float4*)(qs + t * dpad + r * (DR + kPad));
                 const float4* g4 = (const float4*)(gk + t * dpad + r * (DR + kPad));
                 const float gt = CHANNEL ? 0.f : gs[t];
-                float u[DC];
-                if constexpr (DC == 4) {
-                    const float4 t4 = c < n_cols ? *(const float4*)(vs + t * CC + c * DC) : make_float4(0.f, 0.f, 0.f, 0.f);
-                    u[0] = t4.x; u[1] = t4.y; u[2] = t4.z; u[3] = t4.w;
-                } else {
-                    u[0] = c < n_cols ? vs[t * CC + c] : 0.f;
-                }
-#pragma unroll
-                for (int j = 0; j < DC; ++j) {
-                    if (RULE == kDecayRule && act_in_walk) u[j] = silu_precise(u[j]);      // single tokens: the activation rides here
-                    if (v_scaled) u[j] *= bs[t];
-                }
+                float u = c < n_cols ? vs[t * CC + c] : 0.f;
+                if (RULE == kDecayRule && act_in_walk) u = silu_precise(u);      // single tokens: the activation rides here
+                if (v_scaled) u *= bs[t];
                 if (DELTA) {
                     float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;       // four chains, not one of DR links
 #pragma unroll
@@ -296,11 +370,9 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                     float dot = (d0 + d1) + (d2 + d3);
 #pragma unroll
                     for (int o = 1; o < R; o <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
-                    u[0] = bs[t] * (u[0] - dot);
+                    u = bs[t] * (u - dot);
                 }
-                float a[DC][4];
-#pragma unroll
-                for (int j = 0; j < DC; ++j) a[j][0] = a[j][1] = a[j][2] = a[j][3] = 0.f;
+                float a[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int i = 0; i < DR / 4; ++i) {
                     float4 kk = k4[i], qq = LOCAL ? make_float4(0.f, 0.f, 0.f, 0.f) : q4[i];
@@ -309,49 +381,29 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                         qq = make_float4(silu_precise(qq.x), silu_precise(qq.y), silu_precise(qq.z), silu_precise(qq.w));
                     }
                     const float4 gg = CHANNEL ? g4[i] : make_float4(gt, gt, gt, gt);
-#pragma unroll
-                    for (int j = 0; j < DC; ++j) {
-                        float* s4 = &S[j][4 * i];
-                        if (DELTA) {
-                            s4[0] = fmaf(kk.x, u[j], s4[0]);
-                            s4[1] = fmaf(kk.y, u[j], s4[1]);
-                            s4[2] = fmaf(kk.z, u[j], s4[2]);
-                            s4[3] = fmaf(kk.w, u[j], s4[3]);
-                        } else {
-                            s4[0] = fmaf(gg.x, s4[0], kk.x * u[j]);
-                            s4[1] = fmaf(gg.y, s4[1], kk.y * u[j]);
-                            s4[2] = fmaf(gg.z, s4[2], kk.z * u[j]);
-                            s4[3] = fmaf(gg.w, s4[3], kk.w * u[j]);
-                        }
-                        if (LOCAL) continue;
-                        a[j][0] = fmaf(s4[0], qq.x, a[j][0]);
-                        a[j][1] = fmaf(s4[1], qq.y, a[j][1]);
-                        a[j][2] = fmaf(s4[2], qq.z, a[j][2]);
-                        a[j][3] = fmaf(s4[3], qq.w, a[j][3]);
+                    float* s4 = &S[0][4 * i];
+                    if (DELTA) {
+                        s4[0] = fmaf(kk.x, u, s4[0]);
+                        s4[1] = fmaf(kk.y, u, s4[1]);
+                        s4[2] = fmaf(kk.z, u, s4[2]);
+                        s4[3] = fmaf(kk.w, u, s4[3]);
+                    } else {
+                        s4[0] = fmaf(gg.x, s4[0], kk.x * u);
+                        s4[1] = fmaf(gg.y, s4[1], kk.y * u);
+                        s4[2] = fmaf(gg.z, s4[2], kk.z * u);
+                        s4[3] = fmaf(gg.w, s4[3], kk.w * u);
                     }
+                    if (LOCAL) continue;
+                    a[0] = fmaf(s4[0], qq.x, a[0]);
+                    a[1] = fmaf(s4[1], qq.y, a[1]);
+                    a[2] = fmaf(s4[2], qq.z, a[2]);
+                    a[3] = fmaf(s4[3], qq.w, a[3]);
                 }
-                if constexpr (DC == 1) {
-                    part[t] = (a[0][0] + a[0][1]) + (a[0][2] + a[0][3]);
-                } else if constexpr (!LOCAL) {
-                    // four columns' sums over R threads: a thread hands on the columns it does not end with, two and then
-                    // one, and the rest of the threads add up the one that is left
-                    static_assert(DC == 4 && R >= 4, "the sums of four columns");
-                    float p[4];
-#pragma unroll
-                    for (int j = 0; j < 4; ++j) p[j] = (a[j][0] + a[j][1]) + (a[j][2] + a[j][3]);
-                    const bool up = (r & (R / 2)) != 0, up2 = (r & (R / 4)) != 0;
-                    const float x0 = __shfl_xor_sync(0xffffffffu, up ? p[0] : p[2], R / 2);
-                    const float x1 = __shfl_xor_sync(0xffffffffu, up ? p[1] : p[3], R / 2);
-                    const float y0 = (up ? p[2] : p[0]) + x0, y1 = (up ? p[3] : p[1]) + x1;
-                    float acc = (up2 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, up2 ? y0 : y1, R / 4);
-#pragma unroll
-                    for (int o = R / 8; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-                    if ((r & (R / 4 - 1)) == 0 && c < n_cols) os[t * CC + c * DC + (up ? 2 : 0) + (up2 ? 1 : 0)] = acc * o_mult;
-                }
+                part[t] = (a[0] + a[1]) + (a[2] + a[3]);
             }
 #pragma unroll
             for (int t = 0; t < kScanChunk; ++t) {
-                if (LOCAL || DC > 1 || t >= nt) break;
+                if (LOCAL || t >= nt) break;
                 float acc = part[t];
 #pragma unroll
                 for (int o = 1; o < R; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
@@ -387,6 +439,12 @@ state_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
         st = seg_st;
     } else if (!last) {
         return;                                  // only the last segment's state is the sequence's
+    }
+    if (DC == 4) {
+#pragma unroll
+        for (int j = 0; j < DC; ++j)
+#pragma unroll
+            for (int i = 0; i < DR / 2; ++i) halves_of(P[j][i], S[j][2 * i], S[j][2 * i + 1]);
     }
 #pragma unroll
     for (int j = 0; j < DC; ++j) {
