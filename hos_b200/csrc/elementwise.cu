@@ -50,7 +50,8 @@ __global__ void rmsnorm_kernel(const TIn* __restrict__ x, const float* __restric
         out[base + d] = from_float<TOut>(row[d] * r * (w[d] + add_one));
 }
 
-// x += RMSNorm(y; w_post);  optionally h = RMSNorm(x; w_next).
+// x += RMSNorm(y; w_post);  optionally h = RMSNorm(x; w_next), or, without w_next, h = x in h's type (what a branch
+// that reads the residual stream itself takes).
 // The sandwich arrangement's "post norm, residual sum, next pre norm" in one pass
 // over the row: y is read once, x is read and written once, h is written once.
 template <typename TY, typename TH>
@@ -78,6 +79,10 @@ __global__ void norm_add_norm_kernel(const TY* __restrict__ y, const float* __re
         ss2 += v * v;
     }
     if (h == nullptr) return;
+    if (w_next == nullptr) {
+        for (int d = threadIdx.x; d < D; d += blockDim.x) h[base + d] = from_float<TH>(row[d]);
+        return;
+    }
     ss2 = block_sum(ss2, scratch);
     const float r2 = 1.0f / sqrtf(ss2 / (float)D + eps_next);
     for (int d = threadIdx.x; d < D; d += blockDim.x)
@@ -152,7 +157,7 @@ __global__ void norm_add_norm_vec_kernel(const TY* __restrict__ y, int n_parts, 
         const int i = (c * blockDim.x + threadIdx.x) * 4;
         if (i < D) {
             wp[c] = load4(w_post + i);
-            if (h != nullptr) wn[c] = load4(w_next + i);
+            if (w_next != nullptr) wn[c] = load4(w_next + i);
         }
     }
     pdl_wait();       // the kernels before this one are complete from here on
@@ -183,10 +188,11 @@ __global__ void norm_add_norm_vec_kernel(const TY* __restrict__ y, int n_parts, 
             xv[c].z += yv[c].z * r * (wp[c].z + add_one_post);
             xv[c].w += yv[c].w * r * (wp[c].w + add_one_post);
             store4(x + base + i, xv[c]);
+            if (h != nullptr && w_next == nullptr) store4(h + base + i, xv[c]);
             ss2 += xv[c].x * xv[c].x + xv[c].y * xv[c].y + xv[c].z * xv[c].z + xv[c].w * xv[c].w;
         }
     }
-    if (h == nullptr) return;
+    if (h == nullptr || w_next == nullptr) return;
     ss2 = block_sum(ss2, scratch);
     const float r2 = 1.0f / sqrtf(ss2 / (float)D + eps_next);
 #pragma unroll
@@ -245,7 +251,7 @@ __global__ void norm_add_norm_rows_kernel(const TY* __restrict__ y, int n_parts,
     for (int i = 0; i < 8; ++i) wp.v[i] = wn.v[i] = 0.f;
     if (live) {
         wp = load8(w_post + c0);
-        if (h != nullptr) wn = load8(w_next + c0);
+        if (w_next != nullptr) wn = load8(w_next + c0);
     }
     pdl_wait();       // the kernels before this one are complete from here on
     auto fetch_y = [&](int row) {
@@ -278,7 +284,9 @@ __global__ void norm_add_norm_rows_kernel(const TY* __restrict__ y, int n_parts,
             ss2 += xv.v[i] * xv.v[i];
         }
         if (live) store8(x + (size_t)row * D + c0, xv);
-        if (h != nullptr) {
+        if (h != nullptr && w_next == nullptr) {
+            if (live) store8(h + (size_t)row * D + c0, xv);
+        } else if (h != nullptr) {
             ss2 = block_sum(ss2, scratch);
             const float r2 = 1.0f / sqrtf(ss2 / (float)D + eps_next);
             Row8 o;
@@ -651,7 +659,7 @@ extern "C" int hos_rmsnorm(const void* x, int x_dtype, const float* w, float eps
     return check_launch("rmsnorm");
 }
 
-// x += RMSNorm(y; w_post); if h != NULL also h = RMSNorm(x; w_next), written as h_dtype.
+// x += RMSNorm(y; w_post); if h != NULL also h = RMSNorm(x; w_next), or x itself if w_next == NULL, written as h_dtype.
 // n_parts > 1: y is n_parts partial sums of 32-bit floats, [n_parts][N][D], added here.
 extern "C" int hos_norm_add_norm(const void* y, int y_dtype, int n_parts, const float* w_post, float eps_post,
                                  int add_one_post, float* x, const float* w_next, float eps_next,
@@ -686,6 +694,7 @@ extern "C" int hos_norm_add_norm(const void* y, int y_dtype, int n_parts, const 
                 (const TY*)y, w_post, eps_post, a1, x, w_next, eps_next, a2, (TH*)h, D);                    \
         }                                                                                                   \
     } while (0)
+    if (h == nullptr) w_next = nullptr;
     if (h == nullptr) h_dtype = y_dtype == kF32 ? kF32 : kBF16;
     // many rows of a width in steps of 8: CTAs that walk over rows with the next row's loads in flight
     if (N >= kRowsKernelMinRows && chunks != 0 && D % 8 == 0 && D / 8 <= 1024) {

@@ -6,8 +6,10 @@
 // qk_prep: one block per token over the fused projection row [q | k | v | gate logits] (32-bit, biases added
 //   here): each query and key head is divided by its root mean square and multiplied by a weight shared by
 //   the heads (norm_whole: the root mean square is taken over all query heads, and over all key heads, at once,
-//   and the weight has a number per column), its first rot_dims numbers are rotated as neighbouring pairs
-//   (2i, 2i+1) by the angle position * freq[i], cosine and sine times `magnitude`; queries are written as 32-bit
+//   and the weight has a number per column; unit_norm: no weight), its first rot_dims numbers are rotated by the angle
+//   position * freq[i], cosine and sine times `magnitude`, as pairs (2i, 2i+1) (style 1) or (i, i + rot_dims / 2) (style 0;
+//   a rotation keeps a head's root mean square, so a norm without a weight is the same before it and after it, and
+//   a magnitude of 1); queries are written as 32-bit
 //   rows, keys and values (in the cache's type) to their places in the paged cache.  With v_first the values
 //   are first blended with another layer's values of the same token, v <- (1 - v_mix) v + v_mix v_first, and the
 //   blend is what the cache holds.  With q_every > 0 a query at position p is multiplied by 1 + q_coef ln(floor((p + 1) /
@@ -18,7 +20,8 @@
 // gated_attn: one warp per (token, up to 8 query heads that share a kv head, share of the keys).  A lane takes a
 //   key: 32 scores per head at a time, then the lanes turn to the value columns; a key or value row is read once
 //   for all of the warp's heads.  Keys j of position i: j <= i and, with chunks of size C,
-//   floor(j / C) = floor(i / C); with a window W, j > i - W or j < keep_first.  The denominator also holds exp(sink[head]).
+//   floor(j / C) = floor(i / C); with a window W, j > i - W or j < keep_first.  A score is q . k times `scale`, with a
+//   soft-cap c (softcap > 0) then c tanh(score / c).  The denominator also holds exp(sink[head]).
 //   The head's output is multiplied by the logistic function of its gate logit.  With more than one share the
 //   partial (maximum, sum, weighted values) go to a workspace and attn_merge adds them.
 #include "common.cuh"
@@ -52,7 +55,8 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
                const float* __restrict__ k_norm, float eps, const float* __restrict__ freq, int rot_dims, float magnitude,
                const int* __restrict__ token_pos, const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
                float* __restrict__ q_out, PagedKV2 cache, int H, int G, int kd, int vd, int norm_whole,
-               const float* __restrict__ v_first, long long v_first_ld, float v_mix, int q_maps, float q_coef, int q_every) {
+               const float* __restrict__ v_first, long long v_first_ld, float v_mix, int q_maps, float q_coef, int q_every,
+               int style, int unit_norm) {
     pdl_enter();
     __shared__ float scratch[32];
     const int n = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -81,6 +85,20 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
             inv_all[part] = 1.f / sqrtf(ss / (float)cn + eps);
         }
     }
+    // a lane's numbers of a head are the same columns for every head: their sines and cosines are taken once
+    const int half = rot_dims >> 1;
+    float sn[kPrepPL], cs[kPrepPL];
+#pragma unroll
+    for (int i = 0; i < kPrepPL; ++i) {
+        const int d = lane + 32 * i;
+        sn[i] = 0.f;
+        cs[i] = 1.f;
+        if (d < rot_dims) {
+            sincosf(fpos * freq[style == 0 ? (d < half ? d : d - half) : d >> 1], &sn[i], &cs[i]);
+            sn[i] *= magnitude;
+            cs[i] *= magnitude;
+        }
+    }
     // query heads 0..H-1, then key heads H..H+G-1
     for (int item = warp; item < H + G; item += kThreads / 32) {
         const bool is_q = item < H;
@@ -95,25 +113,28 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
             v[i] = d < kd ? row[col0 + d] + (bias ? bias[col0 + d] : 0.f) : 0.f;
             ss = fmaf(v[i], v[i], ss);
         }
-        if (nw != nullptr) {
+        float inv = 1.f;
+        if (nw != nullptr || unit_norm) {
             ss = warp_sum(ss);
-            const float inv = norm_whole ? inv_all[is_q ? 0 : 1] : 1.f / sqrtf(ss / (float)kd + eps);
+            inv = norm_whole ? inv_all[is_q ? 0 : 1] : 1.f / sqrtf(ss / (float)kd + eps);
 #pragma unroll
             for (int i = 0; i < kPrepPL; ++i) {
                 const int d = lane + 32 * i;
-                if (d < kd) v[i] = v[i] * inv * nw[d];
+                if (d < kd) v[i] = v[i] * inv * (nw != nullptr ? nw[d] : 1.f);
             }
         }
 #pragma unroll
         for (int i = 0; i < kPrepPL; ++i) {
             const int d = lane + 32 * i;
-            const float other = __shfl_xor_sync(0xffffffffu, v[i], 1);       // the pair's partner: the lane beside
-            if (d < rot_dims && d < kd) {
-                float sn, cs;
-                sincosf(fpos * freq[d >> 1], &sn, &cs);
-                sn *= magnitude;
-                cs *= magnitude;
-                v[i] = (d & 1) ? fmaf(v[i], cs, other * sn) : fmaf(v[i], cs, -other * sn);
+            float other = __shfl_xor_sync(0xffffffffu, v[i], 1);             // style 1: the pair's partner is the lane beside
+            if (d < rot_dims) {
+                bool upper = d & 1;
+                if (style == 0) {                                            // half a rotation away: formed again from the row
+                    upper = d >= half;
+                    const int o = upper ? d - half : d + half;
+                    other = (row[col0 + o] + (bias ? bias[col0 + o] : 0.f)) * inv * (nw != nullptr ? nw[o] : 1.f);
+                }
+                v[i] = upper ? fmaf(v[i], cs[i], other * sn[i]) : fmaf(v[i], cs[i], -other * sn[i]);
             }
         }
         if (is_q && q_every > 0)
@@ -236,7 +257,7 @@ gated_attn_kernel(const float* __restrict__ q, PagedKV2 cache, const float* __re
                   long long gate_stride, const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                   const int* __restrict__ seq_slot, void* __restrict__ out, int out_bf16, long long ldo, float out_scale,
                   float* __restrict__ part_acc, float* __restrict__ part_ml, int n_splits, int n_tokens, int H, int G, int kd,
-                  int vd, float scale, int chunk, int window, int keep_first) {
+                  int vd, float scale, int chunk, int window, int keep_first, float softcap) {
     pdl_enter();
     extern __shared__ float qs_all[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -324,7 +345,7 @@ gated_attn_kernel(const float* __restrict__ q, PagedKV2 cache, const float* __re
                 }
             }
 #pragma unroll
-            for (int hh = 0; hh < QH; ++hh) s[hh] = dot[hh] * scale;
+            for (int hh = 0; hh < QH; ++hh) s[hh] = softcap_precise(dot[hh] * scale, softcap);
         }
         float p[QH];
 #pragma unroll
@@ -482,25 +503,29 @@ extern "C" const char* hos_last_error() { return error_buffer(); }
 // columns' biases or null.  q_norm / k_norm: [kd] or null (norm_whole: [H * kd] and [G * kd]).  freq: [rot_dims / 2] or
 // null.  v_first: row n's values of another layer at v_first[n * v_first_ld + ...] (G * vd numbers), or null.
 // q_maps > 1: q_out is [N][H * q_maps][kd]: each head's kd numbers are q_maps queries, written as heads of their own.
-// q_every > 0: the queries' factor by position.
+// q_every > 0: the queries' factor by position.  style: the rotation's pairing (0: halves, 1: neighbours).  unit_norm: every
+// q and k head is divided by its root mean square without a weight (then q_norm and k_norm are null).
 extern "C" int hos_qk_prep(const float* proj, int ld, const float* bias, const float* q_norm, const float* k_norm, float eps,
                            const float* freq, int rot_dims, float magnitude, const int* token_pos, const int* token_seq,
                            const int* seq_slot, float* q_out, void* k_pages, void* v_pages, int cache_dtype,
                            const int* page_table, int table_stride, int ring_pages, int N, int H, int G, int kd, int vd,
                            int norm_whole, const float* v_first, long long v_first_ld, float v_mix, int q_maps,
-                           float q_coef, int q_every, cudaStream_t stream) {
+                           float q_coef, int q_every, int style, int unit_norm, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (q_maps < 1 || kd % q_maps != 0) HOS_REFUSE("qk_prep: heads of %d numbers do not hold %d queries", kd, q_maps);
     if (kd <= 0 || kd > 32 * kPrepMaxPL) HOS_REFUSE("qk_prep: heads of %d numbers are outside 1..%d", kd, 32 * kPrepMaxPL);
     if (freq == nullptr) rot_dims = 0;
     if (rot_dims % 2 != 0 || rot_dims > kd) HOS_REFUSE("qk_prep: %d rotated numbers in heads of %d", rot_dims, kd);
+    if (style != 0 && style != 1) HOS_REFUSE("qk_prep: unknown pairing style %d", style);
+    if (unit_norm && (q_norm != nullptr || k_norm != nullptr || norm_whole))
+        HOS_REFUSE("qk_prep: a norm without a weight is one per head and has no weight");
     PagedKV2 c{k_pages, v_pages, page_table, table_stride, ring_pages, G, kd, vd};
     // few rows (single-token steps): a block of 16 warps shortens the row's chain of loads; many rows: 4 warps
     const bool wide = N <= 592 && H + G > 4;
 #define HOS_QKP_N(TC, PL, NT)                                                                                        \
     launch_pdl(qk_prep_kernel<TC, PL, NT>, dim3(N), dim3(NT), 0, stream, proj, ld, bias, q_norm, k_norm, eps, freq,   \
                rot_dims, magnitude, token_pos, token_seq, seq_slot, q_out, c, H, G, kd, vd, norm_whole, v_first,     \
-               v_first_ld, v_mix, q_maps, q_coef, q_every)
+               v_first_ld, v_mix, q_maps, q_coef, q_every, style, unit_norm)
 #define HOS_QKP(TC, PL)                                                                                              \
     do {                                                                                                             \
         if (wide) HOS_QKP_N(TC, PL, 512);                                                                            \
@@ -563,13 +588,13 @@ extern "C" int hos_qkv_conv_store(const float* proj, long long ld, const float* 
 // q: float32 [N][H][kd].  out: H * vd numbers of out_dtype from the start of rows that lie ldo apart, the heads' outputs times
 // out_scale.  gate: row n's logit of head h at gate[n * gate_stride + h], or
 // null.  sink: [H] or null.  chunk, window: 0 for none; keep_first: with a window, that many of a sequence's first keys
-// stay in sight.  n_splits > 1: part_acc [N][H][n_splits][vd] and part_ml
+// stay in sight.  softcap: 0 for none.  n_splits > 1: part_acc [N][H][n_splits][vd] and part_ml
 // [N][H][n_splits][2] float32 must be given.
 extern "C" int hos_gated_attn(const float* q, void* k_pages, void* v_pages, int cache_dtype, const int* page_table,
                               int table_stride, int ring_pages, const float* sink, const float* gate, long long gate_stride,
                               const int* token_pos, const int* token_seq, const int* seq_slot, void* out, int out_dtype,
                               long long ldo, float out_scale, float* part_acc, float* part_ml, int n_splits, int N, int H, int G,
-                              int kd, int vd, float scale, int chunk, int window, int keep_first, cudaStream_t stream) {
+                              int kd, int vd, float scale, int chunk, int window, int keep_first, float softcap, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (G <= 0 || H % G != 0) HOS_REFUSE("gated_attn: %d heads are not a multiple of %d kv heads", H, G);
     if (vd <= 0 || vd > 32 * kMaxVPL) HOS_REFUSE("gated_attn: value heads of %d numbers are outside 1..%d", vd, 32 * kMaxVPL);
@@ -592,7 +617,7 @@ extern "C" int hos_gated_attn(const float* q, void* k_pages, void* v_pages, int 
 #define HOS_GA(TC, VPL, QH)                                                                                          \
     launch_pdl(gated_attn_kernel<TC, VPL, QH>, dim3(blocks), dim3(kAttnWarps * 32), smem, stream, q, c, sink, gate,  \
                gate_stride, token_pos, token_seq, seq_slot, out, out_bf16, ldo, out_scale, part_acc, part_ml, n_splits, N, H, \
-               G, kd, vd, scale, chunk, window, keep_first)
+               G, kd, vd, scale, chunk, window, keep_first, softcap)
 #define HOS_GA_Q(TC, VPL)                                                                                            \
     do {                                                                                                             \
         if (qh == 8) { if constexpr (VPL <= 4) HOS_GA(TC, VPL, 8); }                                                 \

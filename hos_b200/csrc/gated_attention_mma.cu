@@ -5,7 +5,7 @@
 // positions are pages of the cache, copied as they lie (the cache's permutation of 16-byte groups is the one the
 // kernel reads with) through a two-stage cp.async pipeline.  Per tile each warp computes S = Q K^T for its 16
 // queries (m16n8k16, 32-bit accumulators: with bfloat16 operands every product is exact, so the scores are 32-bit
-// sums), scales, masks (causal; the chunk's first key; the window's edge, with or without a sequence's kept first keys), keeps the running maximum and sum in
+// sums), scales, soft-caps (an option), masks (causal; the chunk's first key; the window's edge, with or without a sequence's kept first keys), keeps the running maximum and sum in
 // 32-bit and accumulates O += P V with the 32-bit weights P fed as two bfloat16 terms (P = hi + lo, 16 bits of
 // mantissa) so that the weights are not rounded to 8 bits.  The sink starts the running maximum and the sum
 // (exp(sink - max) counts once); the head's gate multiplies the output.  Keys of KD and values of VD numbers,
@@ -31,7 +31,7 @@ gated_attn_mma_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pa
                       const float* __restrict__ gate, long long gate_stride, const int* __restrict__ cu_seqlens,
                       const int* __restrict__ token_pos, const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
                       void* __restrict__ out_v, int out_f32, long long ldo, float out_scale, int n_seqs, int H, int G,
-                      float scale, int chunk, int window, int keep_first) {
+                      float scale, int chunk, int window, int keep_first, float softcap) {
     pdl_enter();
     extern __shared__ __align__(128) unsigned char smem_raw[];
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);                 // [64][KD]
@@ -109,6 +109,8 @@ gated_attn_mma_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pa
         if (window > 0) qlo_max = max(qlo_max, q_last + 1 - window);
     }
 
+    // with a soft-cap c the score is c tanh(q . k scale / c), taken at once; else q . k scale
+    const float cap_in = softcap > 0.f ? scale / softcap : 0.f, mul = softcap > 0.f ? 1.f : scale;
     for (int it = 0; it < n_kt; ++it) {
         const int stage = it & 1;
         if (it + 1 < n_kt) load_kv(tile_of(it + 1), stage ^ 1);
@@ -138,6 +140,12 @@ gated_attn_mma_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pa
                 mma_bf16(sc[kb * 2 + 1], qa, b[2], b[3]);
             }
         }
+        if (softcap > 0.f) {
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) sc[nt][i] = softcap * tanh_fast(sc[nt][i] * cap_in);
+        }
         float m_new[2] = {m_run[0], m_run[1]};
         // a tile that every query of the warp sees whole (after its first key, up to its own position, or kept) skips the mask
         const bool whole = key0 + MK - 1 <= p0 + warp * 16 && (key0 >= qlo_max || key0 + MK <= keep_first);
@@ -146,7 +154,7 @@ gated_attn_mma_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pa
             for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    sc[nt][i] *= scale;
+                    sc[nt][i] *= mul;
                     m_new[i >> 1] = fmaxf(m_new[i >> 1], sc[nt][i]);
                 }
         } else {
@@ -156,7 +164,7 @@ gated_attn_mma_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pa
                 for (int i = 0; i < 4; ++i) {
                     const int key = key0 + nt * 8 + 2 * t4 + (i & 1);
                     const bool vis = key <= qpos[i >> 1] && (key >= qlo[i >> 1] || key < keep_first);
-                    const float s = vis ? sc[nt][i] * scale : -INFINITY;
+                    const float s = vis ? sc[nt][i] * mul : -INFINITY;
                     sc[nt][i] = s;
                     m_new[i >> 1] = fmaxf(m_new[i >> 1], s);
                 }
@@ -261,7 +269,7 @@ gated_attn_mma_decode_kernel(const float* __restrict__ q, const bf16* __restrict
                              const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                              const int* __restrict__ seq_slot, void* __restrict__ out_v, int out_f32, long long ldo,
                              float out_scale, float* __restrict__ part_acc, float* __restrict__ part_ml, int n_splits, int H, int G,
-                             float scale, int chunk, int window, int keep_first) {
+                             float scale, int chunk, int window, int keep_first, float softcap) {
     pdl_enter();
     extern __shared__ __align__(128) unsigned char smem_raw[];
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);                 // [16][KD]
@@ -345,6 +353,8 @@ gated_attn_mma_decode_kernel(const float* __restrict__ q, const bf16* __restrict
     for (int i = 0; i < VD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     const uint32_t q_base = smem_u32(q_s);
 
+    // with a soft-cap c the score is c tanh(q . k scale / c), taken at once; else q . k scale
+    const float cap_in = softcap > 0.f ? scale / softcap : 0.f, mul = softcap > 0.f ? 1.f : scale;
     for (int it = 0; it < n_kt; ++it) {
         const int stage = it % kDecStages;
         if (it + kDecStages - 1 < n_kt) load_kv(tile_of(kt_lo + it + kDecStages - 1), (it + kDecStages - 1) % kDecStages);
@@ -366,13 +376,19 @@ gated_attn_mma_decode_kernel(const float* __restrict__ q, const bf16* __restrict
             mma_bf16(sc[0], qa, b[0], b[1]);
             mma_bf16(sc[1], qa, b[2], b[3]);
         }
+        if (softcap > 0.f) {
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) sc[nt][i] = softcap * tanh_fast(sc[nt][i] * cap_in);
+        }
         float m_new[2] = {m_run[0], m_run[1]};
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const int key = key0 + nt * 8 + 2 * t4 + (i & 1);
-                const float s = (key <= pos && (key >= lo || key < keep_first)) ? sc[nt][i] * scale : -INFINITY;
+                const float s = (key <= pos && (key >= lo || key < keep_first)) ? sc[nt][i] * mul : -INFINITY;
                 sc[nt][i] = s;
                 m_new[i >> 1] = fmaxf(m_new[i >> 1], s);
             }
@@ -478,7 +494,8 @@ extern "C" int hos_gated_attn_mma(const float* q, const void* k_pages, const voi
                                   int table_stride, int ring_pages, const float* sink, const float* gate,
                                   long long gate_stride, const int* cu_seqlens, const int* token_pos, const int* token_seq,
                                   const int* seq_slot, void* out, int out_f32, long long ldo, float out_scale, int n_seqs,
-                                  int n_q_tiles, int H, int G, int kd, int vd, float scale, int chunk, int window, int keep_first, cudaStream_t stream) {
+                                  int n_q_tiles, int H, int G, int kd, int vd, float scale, int chunk, int window, int keep_first, float softcap,
+                                  cudaStream_t stream) {
     if (n_seqs <= 0 || n_q_tiles <= 0) return 0;
     if (G <= 0 || H % G != 0 || H > 65535) HOS_REFUSE("gated_attn_mma: %d heads over %d kv heads", H, G);
     if ((kd != 64 && kd != 128) || (vd != 64 && vd != 128))
@@ -497,7 +514,7 @@ extern "C" int hos_gated_attn_mma(const float* q, const void* k_pages, const voi
         launch_pdl(gated_attn_mma_kernel<KDv, VDv>, grid, dim3(128), smem, stream, q, (const bf16*)k_pages,          \
                    (const bf16*)v_pages, page_table, table_stride, ring_pages, sink, gate, gate_stride, cu_seqlens,  \
                    token_pos, token_seq, seq_slot, out, out_f32, ldo, out_scale, n_seqs, H, G, scale, chunk, window,  \
-                   keep_first);                                                                                      \
+                   keep_first, softcap);                                                                                      \
     } while (0)
     if (kd == 64 && vd == 64) HOS_GAM(64, 64);
     else if (kd == 64) HOS_GAM(64, 128);
@@ -514,7 +531,7 @@ extern "C" int hos_gated_attn_mma_decode(const float* q, const void* k_pages, co
                                          long long gate_stride, const int* token_pos, const int* token_seq,
                                          const int* seq_slot, void* out, int out_f32, long long ldo, float out_scale,
                                          float* part_acc, float* part_ml, int n_splits, int N, int H, int G, int kd, int vd, float scale, int chunk, int window,
-                                         int keep_first, cudaStream_t stream) {
+                                         int keep_first, float softcap, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (G <= 0 || H % G != 0 || H / G > 16 || G > 65535) HOS_REFUSE("gated_attn_mma_decode: %d heads over %d kv heads", H, G);
     if ((kd != 64 && kd != 128) || (vd != 64 && vd != 128))
@@ -534,7 +551,7 @@ extern "C" int hos_gated_attn_mma_decode(const float* q, const void* k_pages, co
         launch_pdl(gated_attn_mma_decode_kernel<KDv, VDv>, grid, dim3(128), smem, stream, q, (const bf16*)k_pages,   \
                    (const bf16*)v_pages, page_table, table_stride, ring_pages, sink, gate, gate_stride, token_pos,   \
                    token_seq, seq_slot, out, out_f32, ldo, out_scale, part_acc, part_ml, n_splits, H, G, scale, chunk, window, \
-                   keep_first);                                                                                      \
+                   keep_first, softcap);                                                                                      \
     } while (0)
     if (kd == 64 && vd == 64) HOS_GAD(64, 64);
     else if (kd == 64) HOS_GAD(64, 128);

@@ -5,8 +5,8 @@
 // tensor-core kernel refuses.  Any M, N, K.
 //
 // Epilogues: none; soft-cap (logits); gated (W holds gate rows then up rows,
-// out = act(gate) * up), so that the 2F-wide intermediate is never written; bias (out = act(x + bias[n]), act
-// none or the erf-form GELU).
+// out = act(gate) * up), so that the 2F-wide intermediate is never written; bias (out = act(x + bias[n]), or
+// act(x) without a bias, act none, the erf-form or the tanh-form GELU).
 #include "common.cuh"
 
 namespace hos {
@@ -73,8 +73,9 @@ gemm_plain_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TO* __rest
             float v = acc[i][j];
             if (EPI == kEpiSoftcap) v = softcap_precise(v, cap);
             if (EPI == kEpiBias) {
-                v += bias[n];
+                if (bias != nullptr) v += bias[n];
                 if (act == 1) v = gelu_erf(v);
+                else if (act == 2) v = gelu_tanh(v);
             }
             if (EPI == kEpiGated) {
                 if (act == 2) {
@@ -108,7 +109,6 @@ static int launch_plain(const void* A, const void* W, void* out, int M, int N, i
             (const TA*)A, (const TW*)W, (TO*)out, M, N, K, lda, ldw, ldo, cap, act, N, bias);
         break;
     case kEpiBias:
-        if (bias == nullptr) HOS_REFUSE("gemm_plain: the bias epilogue needs a bias");
         gemm_plain_kernel<TA, TW, TO, kEpiBias><<<grid, 256, 0, stream>>>(
             (const TA*)A, (const TW*)W, (TO*)out, M, N, K, lda, ldw, ldo, cap, act, 0, bias);
         break;
@@ -123,7 +123,7 @@ static int launch_plain(const void* A, const void* W, void* out, int M, int N, i
 using namespace hos;
 
 // out[M, N] = A[M, K] . W[N, K]^T.  For the gated epilogue W has 2N rows (gate, then up); for the bias epilogue `bias` has N
-// numbers and act 1 is the erf-form GELU (0: none).
+// numbers or is null, and act 1 is the erf-form GELU, 2 the tanh form (0: none).
 // Leading dimensions are in elements.
 extern "C" int hos_gemm_plain(const void* A, int a_dtype, const void* W, int w_dtype, void* out,
                               int out_dtype, int M, int N, int K, int lda, int ldw, int ldo,

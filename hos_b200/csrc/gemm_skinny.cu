@@ -14,8 +14,8 @@
 //    memory and the result does not depend on timing.
 //
 // Epilogues: none (bf16 or f32 output); gated, where the CTA owns 16 gate rows and the 16
-// matching up rows (4 warps each) and writes act(gate) * up; bias (out = act(x + bias[n]), act none or the erf-form
-// GELU, bf16 output).
+// matching up rows (4 warps each) and writes act(gate) * up; bias (out = act(x + bias[n]), or act(x) without one, act none or the
+// erf-form or tanh-form GELU, bf16 output).
 #include "common.cuh"
 #include "kv_layout.cuh"
 #include "mma_utils.cuh"
@@ -173,10 +173,9 @@ gemm_skinny_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, OutT*
             v = 0.f;
 #pragma unroll
             for (int w = 0; w < WARPS; ++w) v += part[w][m][r][t];
-            if (bias != nullptr) {
-                v += bias[n];
-                if (act == 1) v = gelu_erf_fast(v);
-            }
+            if (bias != nullptr) v += bias[n];
+            if (act == 1) v = gelu_erf_fast(v);
+            else if (act == 2) v = gelu_tanh_fast(v);
         }
         out[(size_t)tok * ldo + n] = from_float<OutT>(v);
     }
@@ -365,7 +364,7 @@ static bool skinny_ahead(int kind) { return (skinny_ahead_mode() & kind) != 0 ||
 
 // out[M, N] = A[M, K] . W[N, K]^T for M <= 32.  epilogue 0: none (out bf16 or f32); 2: gated (W has
 // 2N rows: gate rows, then up rows at row N; out bf16; act 0, 1, or 2, the clamped form with its limit in act_limit);
-// 3: bias (bias[N] added, act 1: erf-form GELU; out bf16).
+// 3: bias (bias[N] added unless null, act 1: erf-form GELU, 2: tanh form; out bf16).
 // K and the leading dimensions must be
 // multiples of 8 elements, A and W 16-byte aligned.
 // k_splits > 1: `out` is [k_splits][M][ldo] 32-bit partial sums for a consumer that adds them (no epilogue).
@@ -378,8 +377,9 @@ extern "C" int hos_gemm_skinny(const void* A, const void* W, void* out, int out_
         HOS_REFUSE("gemm_skinny: K and the leading dimensions must be multiples of 8 elements and the operands "
                    "16-byte aligned (K %d lda %d ldw %d)", K, lda, ldw);
     if (epilogue != 0 && epilogue != 2 && epilogue != 3) HOS_REFUSE("gemm_skinny: epilogue %d is not offered", epilogue);
-    if (epilogue == 3 && (out_dtype != kBF16 || bias == nullptr)) HOS_REFUSE("gemm_skinny: the bias epilogue writes bfloat16 and needs a bias");
+    if (epilogue == 3 && out_dtype != kBF16) HOS_REFUSE("gemm_skinny: the bias epilogue writes bfloat16");
     if (epilogue != 3) bias = nullptr;
+    if (epilogue == 0) act = 0;
     if (epilogue == 2 && out_dtype != kBF16) HOS_REFUSE("gemm_skinny: the gated epilogue writes bfloat16");
     if (k_splits < 1 || k_splits > 64) HOS_REFUSE("gemm_skinny: %d splits of K (1..64)", k_splits);
     if (k_splits > 1 && (epilogue != 0 || out_dtype != kF32))

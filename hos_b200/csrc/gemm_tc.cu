@@ -19,8 +19,8 @@
 // that a small kernel adds in a fixed order.
 //
 // Epilogues: none; soft-cap c*tanh(x/c) with 32-bit output (logits); gated act(gate)*up,
-// where W holds the gate rows followed by the up rows and a tile loads matching rows of both; act(x + bias[n]), act
-// none or the erf-form GELU.
+// where W holds the gate rows followed by the up rows and a tile loads matching rows of both; act(x + bias[n]) or,
+// without a bias, act(x), act none, the erf-form or the tanh-form GELU.
 //
 // Every wait on an mbarrier is bounded in time: a wait that runs out sets an error flag,
 // the roles leave their loops, tensor memory is freed and the kernel returns.
@@ -157,14 +157,17 @@ struct GemmParams {
     int k_splits;
     int gate_rows;        // gated: row of W where the up rows begin
     float cap;            // the soft-cap; with the gated epilogue's activation 2, the clamp's limit
-    int act;              // gated: 0 tanh-form GELU, 1 x logistic(x), 2 the clamped form (common.cuh); bias: 0 none, 1 erf-form GELU
-    const float* bias;    // kGEpiBias: [N]
+    int act;              // gated: 0 tanh-form GELU, 1 x logistic(x), 2 the clamped form (common.cuh); bias: 0 none, 1 erf-form GELU, 2 tanh form
+    const float* bias;    // kGEpiBias: [N], or null
     RopeEpi rope;         // kGEpiRope only
 };
 
 // Thirty-two columns n0.. of one row, with their bias and activation (all lanes of a warp read the same bias: one line).
 __device__ __forceinline__ void bias_act_32(const uint32_t (&v)[32], float (&f)[32], const float* __restrict__ bias, int n0, int N, int act) {
-    if (n0 + 32 <= N && ((uintptr_t)(bias + n0) & 15) == 0) {
+    if (bias == nullptr) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) f[j] = __uint_as_float(v[j]);
+    } else if (n0 + 32 <= N && ((uintptr_t)(bias + n0) & 15) == 0) {
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             const float4 b = __ldg(reinterpret_cast<const float4*>(bias + n0) + j);
@@ -180,6 +183,9 @@ __device__ __forceinline__ void bias_act_32(const uint32_t (&v)[32], float (&f)[
     if (act == 1) {
 #pragma unroll
         for (int j = 0; j < 32; ++j) f[j] = gelu_erf_fast(f[j]);
+    } else if (act == 2) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) f[j] = gelu_tanh_fast(f[j]);
     }
 }
 
@@ -383,7 +389,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_m,     // the 128-row ope
                 const bool gated = EPI == kGEpiGated;
                 const int feat = gated ? mt * 64 + (r & 63) : mt * GM + r;
                 const int feat_count = p.N;
-                const float feat_bias = EPI == kGEpiBias && feat < feat_count ? __ldg(p.bias + feat) : 0.f;
+                const float feat_bias = EPI == kGEpiBias && p.bias != nullptr && feat < feat_count ? __ldg(p.bias + feat) : 0.f;
                 OutT* obase = reinterpret_cast<OutT*>(p.out) + (p.k_splits > 1 ? (size_t)ks * p.M * p.ldo : 0);
                 constexpr int CH = BN < 32 ? BN : 32;
 #pragma unroll 1
@@ -434,6 +440,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_m,     // the 128-row ope
                                 if (EPI == kGEpiBias) {
                                     x += feat_bias;
                                     if (p.act == 1) x = gelu_erf_fast(x);
+                                    else if (p.act == 2) x = gelu_tanh_fast(x);
                                 }
                                 obase[(size_t)tok * p.ldo + feat] = from_float<OutT>(x);
                             }
@@ -996,8 +1003,8 @@ extern "C" long long hos_gemm_tc_workspace(int M, int N, int k_splits) {
 }
 
 // out[M, N] = A[M, K] . W[N, K]^T, bf16 operands.  out_dtype: 1 bf16, 0 f32.  epilogue: 0 none,
-// 1 soft-cap (f32 output), 2 gated (W has 2N rows: gate rows, then up rows at row N), 3 bias (bias[N] added, act 1: the
-// erf-form GELU; bf16 output).
+// 1 soft-cap (f32 output), 2 gated (W has 2N rows: gate rows, then up rows at row N), 3 bias (bias[N] added unless null, act 1:
+// the erf-form GELU, 2: the tanh form; bf16 output).
 // M <= 128 runs swapped; k_splits > 1 is allowed only then and only without an epilogue, and
 // needs `workspace` (see hos_gemm_tc_workspace).  With reduce_now == 0 the partial sums are left
 // in the workspace as [k_splits_used][M][N] floats for the consumer to add, `out` is not written,
@@ -1013,8 +1020,7 @@ extern "C" int hos_gemm_tc(const void* A, const void* W, void* out, int out_dtyp
                    "16-byte aligned (K %d lda %d ldw %d)", K, lda, ldw);
     if (epilogue == kGEpiSoftcap && out_dtype != kF32) HOS_REFUSE("gemm_tc: the soft-cap epilogue writes 32-bit");
     if (epilogue == kGEpiGated && out_dtype != kBF16) HOS_REFUSE("gemm_tc: the gated epilogue writes bfloat16");
-    if (epilogue == kGEpiBias && (out_dtype != kBF16 || bias == nullptr))
-        HOS_REFUSE("gemm_tc: the bias epilogue writes bfloat16 and needs a bias");
+    if (epilogue == kGEpiBias && out_dtype != kBF16) HOS_REFUSE("gemm_tc: the bias epilogue writes bfloat16");
     if (epilogue < kGEpiNone || epilogue > kGEpiBias) HOS_REFUSE("gemm_tc: unknown epilogue %d", epilogue);
     if (k_splits < 1) k_splits = 1;
     const bool swap = M <= kSwapMaxRows;

@@ -14,7 +14,7 @@
 // sink: a learned number per head that joins the softmax's denominator as exp(sink), without a key
 // or a value and unscaled.
 //
-// Kernels: latent_prep (norm of c, rotations, cache write), latent_attn and latent_attn_tc (keys from
+// Kernels: latent_prep (norms of c and of the queries' own latent, rotations, cache write), latent_attn and latent_attn_tc (keys from
 // the step's own rows for sequences that start at position 0, or from the paged cache), latent_merge
 // (the shares of a row's keys put together), heads_product and heads_product_tc (the per-head products
 // W_uk_h^T q_h and W_uv_h o_h as one launch over all heads).
@@ -25,85 +25,119 @@
 namespace hos {
 
 // ---- latent_prep ---------------------------------------------------------------------------
-// proj[n] = [ q: H heads of (dq + P) | c_raw: R | key_rot_raw: P ].  Writes
-//   kc[n]     = [ rms(c_raw) * w_norm | rot(key_rot_raw) ]                (the row the cache keeps)
-//   q_lat[n][h][R : R + P] = rot(q_h[dq : dq + P])                        (32-bit)
-// and stores kc[n] at the token's place in the paged cache (rows of D, not permuted).  With kc null the rows hold
-// the queries only (a call that reads another call's cache): nothing is normed or stored.
-// Rotation: the first rot_dims of the P numbers, pairs (2i, 2i + 1), angle = position * inv_freq[i].
+// What lies between the projections and the attention, for whichever of the three parts are given:
+//   down[n] = [ c_raw: R | key_rot_raw: P ]      -> kc[n] = [ rms(c_raw) * w_norm | rot(key_rot_raw) ], the row the cache
+//                                                   keeps, also stored at the token's place in the paged cache (rows of
+//                                                   R + P, not permuted)
+//   q[n]    = H heads of [ dq | P ]              -> q_lat[n][h][R : R + P] = rot(q_h[dq : dq + P])          (32-bit)
+//   cq[n]   = the queries' own latent, Rq numbers -> cq_out[n] = rms(cq) * cq_norm, what the queries' up projection reads
+// A call without a part passes null for it (a call that reads another call's cache: no `down`; queries that come straight
+// from the layer's input: no `cq`; queries that are not there yet because they wait for cq_out: no `q`).
+// Rotation: the first rot_dims of the P numbers, angle = position * inv_freq[i]; style 0 pairs (i, i + rot_dims / 2),
+// style 1 pairs (2i, 2i + 1).
 template <typename T>
-__global__ void latent_prep_kernel(const T* __restrict__ proj, int proj_stride, int H, int dq, int R, int P,
-                                   const float* __restrict__ w_norm, float eps, const float* __restrict__ inv_freq,
-                                   int rot_dims, const int* __restrict__ token_pos, const int* __restrict__ token_seq,
-                                   const int* __restrict__ seq_slot, const int* __restrict__ seq_len_after,
-                                   T* __restrict__ kc, float* __restrict__ q_lat, T* __restrict__ k_pages,
-                                   const int* __restrict__ page_table, int table_stride, int ring_pages) {
+struct LatentPrep {
+    const T* q;
+    const T* down;
+    const T* cq;
+    int q_stride, down_stride, cq_stride;
+    int H, dq, R, P, Rq;
+    const float* w_norm;
+    const float* cq_norm;
+    float eps;
+    const float* inv_freq;
+    int rot_dims, style;
+    const int* token_pos;
+    const int* token_seq;
+    const int* seq_slot;
+    const int* seq_len_after;
+    T* kc;
+    float* q_lat;
+    T* cq_out;
+    T* k_pages;
+    const int* page_table;
+    int table_stride, ring_pages;
+};
+
+template <typename T>
+__global__ void latent_prep_kernel(LatentPrep<T> a) {
     pdl_enter();
     extern __shared__ float2 sincos_tab[];      // [rot_dims / 2]
     __shared__ float scratch[32];
     const int n = blockIdx.x;
-    const int seq = token_seq[n];
+    const int seq = a.token_seq[n];
     if (seq < 0) return;
-    const int pos = token_pos[n], D = R + P, half = rot_dims >> 1;
+    const int pos = a.token_pos[n], R = a.R, P = a.P, D = R + P, half = a.rot_dims >> 1;
+    const bool keys = a.down != nullptr;
     int page = -1;
-    if (k_pages != nullptr && !(ring_pages > 0 && pos + ring_pages * kPageTokens < seq_len_after[seq])) {
+    if (a.k_pages != nullptr && !(a.ring_pages > 0 && pos + a.ring_pages * kPageTokens < a.seq_len_after[seq])) {
         const int lp = pos / kPageTokens;
-        page = page_table[(size_t)seq_slot[seq] * table_stride + (ring_pages > 0 ? lp % ring_pages : lp)];
+        page = a.page_table[(size_t)a.seq_slot[seq] * a.table_stride + (a.ring_pages > 0 ? lp % a.ring_pages : lp)];
     }
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float s, c;
-        sincosf((float)pos * inv_freq[i], &s, &c);
+        sincosf((float)pos * a.inv_freq[i], &s, &c);
         sincos_tab[i] = make_float2(s, c);
     }
-    const T* row = proj + (size_t)n * proj_stride;
-    const T* craw = row + (size_t)H * (dq + P);
-    const bool keys = kc != nullptr;
+    const T* craw = keys ? a.down + (size_t)n * a.down_stride : nullptr;
     float ss = 0.f;
     if (keys)
         for (int d = threadIdx.x; d < R; d += blockDim.x) {
             const float v = to_float(craw[d]);
             ss = fmaf(v, v, ss);
         }
-    const float rinv = rsqrtf(block_sum(ss, scratch) / (float)R + eps);      // (also orders sincos_tab)
-    T* out = keys ? kc + (size_t)n * D : nullptr;
-    T* cached = page >= 0 ? k_pages + ((size_t)page * kPageTokens + pos % kPageTokens) * D : nullptr;
+    const float rinv = rsqrtf(block_sum(ss, scratch) / (float)R + a.eps);      // (also orders sincos_tab)
+    T* out = keys ? a.kc + (size_t)n * D : nullptr;
+    T* cached = keys && page >= 0 ? a.k_pages + ((size_t)page * kPageTokens + pos % kPageTokens) * D : nullptr;
     if (keys)
         for (int d = threadIdx.x; d < R; d += blockDim.x) {
-            const T v = from_float<T>(to_float(craw[d]) * rinv * w_norm[d]);
+            const T v = from_float<T>(to_float(craw[d]) * rinv * a.w_norm[d]);
             out[d] = v;
             if (cached) cached[d] = v;
         }
-    // the shared rotated key part, then every head's rotated query part: items of one pair (or one
-    // unrotated number beyond rot_dims)
-    const int per = half + (P - rot_dims);
-    for (int it = threadIdx.x; it < (H + (keys ? 1 : 0)) * per; it += blockDim.x) {
-        const int who = it / per, j = it - who * per;       // who == H: the key
-        const T* src = who == H ? craw + R : row + (size_t)who * (dq + P) + dq;
-        float a, b = 0.f;
-        int d0;
+    if (a.cq != nullptr) {
+        const T* src = a.cq + (size_t)n * a.cq_stride;
+        float sq = 0.f;
+        for (int d = threadIdx.x; d < a.Rq; d += blockDim.x) {
+            const float v = to_float(src[d]);
+            sq = fmaf(v, v, sq);
+        }
+        const float qinv = rsqrtf(block_sum(sq, scratch) / (float)a.Rq + a.eps);
+        for (int d = threadIdx.x; d < a.Rq; d += blockDim.x)
+            a.cq_out[(size_t)n * a.Rq + d] = from_float<T>(to_float(src[d]) * qinv * a.cq_norm[d]);
+    }
+    // the shared rotated key part and every head's rotated query part: items of one pair (or one unrotated number
+    // beyond rot_dims); item group 0 is the key if there is one
+    const int per = half + (P - a.rot_dims), first = keys ? 1 : 0;
+    for (int it = threadIdx.x; it < ((a.q != nullptr ? a.H : 0) + first) * per; it += blockDim.x) {
+        const int who = it / per - first, j = it - (it / per) * per;       // who == -1: the key
+        const T* src = who < 0 ? craw + R : a.q + (size_t)n * a.q_stride + (size_t)who * (a.dq + P) + a.dq;
+        float x, y = 0.f;
+        int d0, d1 = 0;
         const bool pair = j < half;
         if (pair) {
-            d0 = 2 * j;
+            d0 = a.style == 0 ? j : 2 * j;
+            d1 = a.style == 0 ? j + half : 2 * j + 1;
             const float2 sc = sincos_tab[j];
-            const float u = to_float(src[d0]), v = to_float(src[d0 + 1]);
-            a = u * sc.y - v * sc.x;
-            b = v * sc.y + u * sc.x;
+            const float u = to_float(src[d0]), v = to_float(src[d1]);
+            x = u * sc.y - v * sc.x;
+            y = v * sc.y + u * sc.x;
         } else {
-            d0 = rot_dims + (j - half);
-            a = to_float(src[d0]);
+            d0 = a.rot_dims + (j - half);
+            x = to_float(src[d0]);
         }
-        if (who == H) {
-            const T ta = from_float<T>(a), tb = from_float<T>(b);
-            out[R + d0] = ta;
-            if (cached) cached[R + d0] = ta;
+        if (who < 0) {
+            const T tx = from_float<T>(x), ty = from_float<T>(y);
+            out[R + d0] = tx;
+            if (cached) cached[R + d0] = tx;
             if (pair) {
-                out[R + d0 + 1] = tb;
-                if (cached) cached[R + d0 + 1] = tb;
+                out[R + d1] = ty;
+                if (cached) cached[R + d1] = ty;
             }
         } else {
-            float* q = q_lat + ((size_t)n * H + who) * D + R;
-            q[d0] = a;
-            if (pair) q[d0 + 1] = b;
+            float* q = a.q_lat + ((size_t)n * a.H + who) * D + R;
+            q[d0] = x;
+            if (pair) q[d1] = y;
         }
     }
 }
@@ -675,17 +709,6 @@ heads_product_tc_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, 
     }
 }
 
-template <typename T>
-static int launch_prep(const void* proj, int proj_stride, int H, int dq, int R, int P, const float* w_norm, float eps,
-                       const float* inv_freq, int rot_dims, const int* token_pos, const int* token_seq,
-                       const int* seq_slot, const int* seq_len_after, void* kc, float* q_lat, void* k_pages,
-                       const int* page_table, int table_stride, int ring_pages, int N, cudaStream_t stream) {
-    launch_pdl(latent_prep_kernel<T>, dim3(N), dim3(128), (size_t)(rot_dims / 2 + 1) * sizeof(float2), stream,
-               (const T*)proj, proj_stride, H, dq, R, P, w_norm, eps, inv_freq, rot_dims, token_pos, token_seq, seq_slot,
-               seq_len_after, (T*)kc, q_lat, (T*)k_pages, page_table, table_stride, ring_pages);
-    return check_launch("latent_prep");
-}
-
 template <typename T, bool PAGED, int NC, int QT>
 static int launch_attn_as(const float* q_lat, const void* kc, const void* k_pages, const int* page_table, int table_stride,
                           int ring_pages, const float* sink, void* o_lat, float* part_acc, float* part_ml, int n_splits,
@@ -780,20 +803,31 @@ using namespace hos;
 
 extern "C" const char* hos_last_error() { return error_buffer(); }
 
-extern "C" int hos_latent_prep(const void* proj, int dtype, int proj_stride, int H, int dq, int R, int P,
-                               const float* w_norm, float eps, const float* inv_freq, int rot_dims,
-                               const int* token_pos, const int* token_seq, const int* seq_slot,
-                               const int* seq_len_after, void* kc, float* q_lat, void* k_pages,
-                               const int* page_table, int table_stride, int ring_pages, int N, cudaStream_t stream) {
+// q, down, cq: rows q_stride, down_stride, cq_stride elements apart, of one dtype; any of them may be null (see the kernel).
+extern "C" int hos_latent_prep(const void* q, int q_stride, const void* down, int down_stride, const void* cq, int cq_stride,
+                               int dtype, int H, int dq, int R, int P, int Rq, const float* w_norm, const float* cq_norm,
+                               float eps, const float* inv_freq, int rot_dims, int style, const int* token_pos,
+                               const int* token_seq, const int* seq_slot, const int* seq_len_after, void* kc, float* q_lat,
+                               void* cq_out, void* k_pages, const int* page_table, int table_stride, int ring_pages, int N,
+                               cudaStream_t stream) {
     if (N <= 0) return 0;
+    if (inv_freq == nullptr) rot_dims = 0;
     if (rot_dims < 0 || rot_dims > P || (rot_dims & 1)) HOS_REFUSE("latent_prep: %d rotated of %d numbers", rot_dims, P);
-    if (dtype == kBF16)
-        return launch_prep<bf16>(proj, proj_stride, H, dq, R, P, w_norm, eps, inv_freq, rot_dims, token_pos, token_seq,
-                                 seq_slot, seq_len_after, kc, q_lat, k_pages, page_table, table_stride, ring_pages, N, stream);
-    if (dtype == kF32)
-        return launch_prep<float>(proj, proj_stride, H, dq, R, P, w_norm, eps, inv_freq, rot_dims, token_pos, token_seq,
-                                  seq_slot, seq_len_after, kc, q_lat, k_pages, page_table, table_stride, ring_pages, N, stream);
-    HOS_REFUSE("latent_prep: unknown dtype %d", dtype);
+    if (style != 0 && style != 1) HOS_REFUSE("latent_prep: unknown pairing style %d", style);
+    if ((q && !q_lat) || (down && (!kc || !w_norm)) || (cq && (!cq_out || !cq_norm || Rq <= 0)))
+        HOS_REFUSE("latent_prep: a part comes without its output or its norm's weight");
+#define HOS_PREP(T)                                                                                                  \
+    do {                                                                                                             \
+        LatentPrep<T> a{(const T*)q, (const T*)down, (const T*)cq, q_stride, down_stride, cq_stride, H, dq, R, P, Rq, w_norm, \
+                        cq_norm, eps, inv_freq, rot_dims, style, token_pos, token_seq, seq_slot, seq_len_after, (T*)kc, \
+                        q_lat, (T*)cq_out, (T*)k_pages, page_table, table_stride, ring_pages};                       \
+        launch_pdl(latent_prep_kernel<T>, dim3(N), dim3(128), (size_t)(rot_dims / 2 + 1) * sizeof(float2), stream, a); \
+    } while (0)
+    if (dtype == kBF16) HOS_PREP(bf16);
+    else if (dtype == kF32) HOS_PREP(float);
+    else HOS_REFUSE("latent_prep: unknown dtype %d", dtype);
+#undef HOS_PREP
+    return check_launch("latent_prep");
 }
 
 // Rows row0 .. row0 + rows - 1 of the step.  paged = 0: keys are the step's own rows `kc` (sequences

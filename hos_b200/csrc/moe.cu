@@ -2,7 +2,8 @@
 //
 //   route     per row: router logits in 32-bit, scores = softmax over all outputs (or, scoring 1, the logistic
 //             function of each logit), the `top` largest of (score + correction) chosen, each weighted by
-//             its plain score (not renormalised).
+//             its plain score (not renormalised).  With groups (equal groups of neighbouring outputs) a group's score is
+//             the sum of its two largest (score + correction), and only the outputs of the `keep` best groups are open.
 //             The last `n_identity` router outputs are experts without tensors: their output is
 //             the row itself.
 //   align     the chosen (row, choice) pairs listed expert by expert, each expert's list padded to
@@ -12,6 +13,7 @@
 //             (limit <= 0: no clamp; the 1 is `up_shift`, 0 for the plain gated form g' sigmoid(alpha g') u').  With
 //             in_weight the pair's weight multiplies the expert's INPUT: gate and up products are linear, so
 //             g and u are multiplied by it before the activation, and down takes no weight.
+//             The kernels' other activation (kReluSquare) has no gate: y = relu(u)^2, W holds the up rows alone.
 //   down      per tile, the expert's down product, times the pair's weight, to the pair's own row
 //             of a 32-bit buffer.
 //   combine   per row, the sum of its pairs' rows in the order of the choices, identity experts added
@@ -31,12 +33,71 @@ __device__ __forceinline__ float4 route_load4(const bf16* p) {
                        __uint_as_float(u.y & 0xffff0000u));
 }
 
+enum ExpertAct : int { kGatedSwish = 0, kReluSquare = 1 };
+
+// y of an expert's inner number from its 32-bit gate and up products (kReluSquare: from the up product, given as g)
+template <int ACT>
+__device__ __forceinline__ float expert_act(float g, float u, float limit, float alpha, float up_shift) {
+    if (ACT == kReluSquare) {
+        const float r = fmaxf(g, 0.f);
+        return r * r;
+    }
+    if (limit > 0.f) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+    }
+    return g / (1.f + expf(-alpha * g)) * (u + up_shift);
+}
+
+// One warp: the outputs outside the `keep` best of `groups` equal groups are marked as taken.  gs: [groups] in shared memory;
+// score(e) is what the groups are judged by.  Equal groups: the first wins.
+template <typename Score>
+__device__ __forceinline__ void route_groups(Score score, float* taken, float* gs, int n_out, int groups, int keep, int lane) {
+    const int size = n_out / groups;
+    for (int g = lane; g < groups; g += 32) {
+        float a = -INFINITY, b = -INFINITY;
+        for (int i = 0; i < size; ++i) {
+            const float c = score(g * size + i);
+            if (c > a) {
+                b = a;
+                a = c;
+            } else if (c > b) {
+                b = c;
+            }
+        }
+        gs[g] = size > 1 ? a + b : a;
+    }
+    for (int e = lane; e < n_out; e += 32) taken[e] = 1.f;
+    __syncwarp();
+    for (int k = 0; k < keep; ++k) {
+        float best = -INFINITY;
+        int arg = 0x7fffffff;
+        for (int g = lane; g < groups; g += 32)
+            if (gs[g] > best || (gs[g] == best && gs[g] != -INFINITY && g < arg)) {
+                best = gs[g];
+                arg = g;
+            }
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+            if (ob > best || (ob == best && oa < arg)) {
+                best = ob;
+                arg = oa;
+            }
+        }
+        if (arg == 0x7fffffff) break;
+        for (int i = lane; i < size; i += 32) taken[arg * size + i] = 0.f;
+        if (lane == 0) gs[arg] = -INFINITY;
+        __syncwarp();
+    }
+}
+
 // One warp: z [n_out] logits of row n (in shared memory) -> scores, the `top` largest of (score + correction)
 // and their plain scores.  A padding row (token_seq < 0) chooses nothing.
 __device__ __forceinline__ void route_choose(float* z, float* taken, const float* __restrict__ correction,
                                              const int* __restrict__ token_seq, int* __restrict__ choice,
                                              float* __restrict__ weight, int n, int n_out, int top, int scoring, int lane,
-                                             float renorm, float wscale) {
+                                             float renorm, float wscale, float* gs, int groups, int keep) {
     if (token_seq[n] < 0) {
         for (int k = lane; k < top; k += 32) {
             choice[(size_t)n * top + k] = -1;
@@ -65,6 +126,11 @@ __device__ __forceinline__ void route_choose(float* z, float* taken, const float
         for (int e = lane; e < n_out; e += 32) z[e] = z[e] / sum;
     }
     __syncwarp();
+    if (groups > 0) {
+        route_groups([&](int e) { return (by_logit ? 1.f / (1.f + expf(-z[e])) : z[e]) + (correction ? correction[e] : 0.f); }, taken,
+                     gs, n_out, groups, keep, lane);
+        __syncwarp();
+    }
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int arg = 0x7fffffff;
@@ -112,12 +178,13 @@ template <typename T, int RT, bool VEC>
 __global__ void __launch_bounds__(256)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
                  const int* __restrict__ token_seq, int* __restrict__ choice, float* __restrict__ weight, int N, int D,
-                 int n_out, int top, int scoring, float* __restrict__ logits, float renorm, float wscale) {
+                 int n_out, int top, int scoring, float* __restrict__ logits, float renorm, float wscale, int groups, int keep) {
     pdl_enter();
     extern __shared__ float route_sm[];
     float* z_all = route_sm;                       // [RT][n_out] scores
     float* taken_all = z_all + RT * n_out;         // [RT][n_out] flags
-    float* part = taken_all + RT * n_out;          // [warps][RT][n_out] partial sums
+    float* gs_all = taken_all + RT * n_out;        // [RT][groups] the groups' scores
+    float* part = gs_all + RT * groups;            // [warps][RT][n_out] partial sums
     const int n0 = blockIdx.x * RT, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
     const T* rows[RT];
 #pragma unroll
@@ -192,27 +259,28 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
     const int n = n0 + warp;
     if (n >= N) return;
     route_choose(z_all + warp * n_out, taken_all + warp * n_out, correction, token_seq, choice, weight, n, n_out, top, scoring,
-                 lane, renorm, wscale);
+                 lane, renorm, wscale, gs_all + warp * groups, groups, keep);
 }
 
 // A warp per row: logits [N][n_out] from moe_route_kernel's blocks -> scores, the `top` largest, their weights.
 __global__ void __launch_bounds__(128)
 moe_choose_kernel(const float* __restrict__ logits, const float* __restrict__ correction, const int* __restrict__ token_seq,
                   int* __restrict__ choice, float* __restrict__ weight, int N, int n_out, int top, int scoring,
-                  float renorm, float wscale) {
+                  float renorm, float wscale, int groups, int keep) {
     pdl_enter();
     extern __shared__ float route_sm[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
     const int n = blockIdx.x * nwarps + warp;
     if (n >= N) return;
-    float* z = route_sm + (size_t)warp * 2 * n_out;
+    float* z = route_sm + (size_t)warp * (2 * n_out + groups);
     float* taken = z + n_out;
     for (int e = lane; e < n_out; e += 32) {
         z[e] = logits[(size_t)n * n_out + e];
         taken[e] = 0.f;
     }
     __syncwarp();
-    route_choose(z, taken, correction, token_seq, choice, weight, n, n_out, top, scoring, lane, renorm, wscale);
+    route_choose(z, taken, correction, token_seq, choice, weight, n, n_out, top, scoring, lane, renorm, wscale, taken + n_out, groups,
+                 keep);
 }
 
 // One block.  listed: [cap] pair ids (row * top + choice) expert by expert, -1 where a tile is padded;
@@ -256,8 +324,9 @@ __global__ void moe_align_kernel(const int* __restrict__ choice, int n_pairs, in
     }
 }
 
-// y[listed position][F] = act(gate, up) of the listed rows; W: [experts][2F][D], gate rows then up rows.
-template <typename T>
+// y[listed position][F] = act(gate, up) of the listed rows; W: [experts][2F][D], gate rows then up rows (kReluSquare:
+// [experts][F][D], the up rows, which stand where the gate rows would).
+template <typename T, int ACT>
 __global__ void __launch_bounds__(256)
 moe_gate_up_kernel(const T* __restrict__ h, const T* __restrict__ W, const int* __restrict__ listed,
                    const int* __restrict__ tile_expert, T* __restrict__ y, int D, int F, int top, float limit,
@@ -266,7 +335,8 @@ moe_gate_up_kernel(const T* __restrict__ h, const T* __restrict__ W, const int* 
     constexpr int BK = 16;
     __shared__ float As[BK][kTile + 4];
     __shared__ float Gs[BK][kTile + 4];
-    __shared__ float Us[BK][kTile + 4];
+    constexpr bool GATED = ACT == kGatedSwish;
+    __shared__ float Us[GATED ? BK : 1][kTile + 4];
     __shared__ int rows[kTile];
     const int tile = blockIdx.y, e = tile_expert[tile];
     if (e < 0) return;
@@ -279,7 +349,7 @@ moe_gate_up_kernel(const T* __restrict__ h, const T* __restrict__ W, const int* 
     const int warp_row0 = (threadIdx.x >> 5) * 8;          // a warp's threads hold rows warp_row0 .. +7
     bool busy = false;
     for (int i = 0; i < 8; ++i) busy = busy || rows[warp_row0 + i] >= 0;
-    const T* Wg = W + (size_t)e * 2 * F * D;
+    const T* Wg = W + (size_t)e * (GATED ? 2 : 1) * F * D;
     const T* Wu = Wg + (size_t)F * D;
     float acc_g[4][4] = {}, acc_u[4][4] = {};
     for (int k0 = 0; k0 < D; k0 += BK) {
@@ -289,7 +359,7 @@ moe_gate_up_kernel(const T* __restrict__ h, const T* __restrict__ W, const int* 
             As[kk][r] = (src >= 0 && k < D) ? to_float(h[(size_t)src * D + k]) : 0.f;
             const bool in = n < F && k < D;
             Gs[kk][r] = in ? to_float(Wg[(size_t)n * D + k]) : 0.f;
-            Us[kk][r] = in ? to_float(Wu[(size_t)n * D + k]) : 0.f;
+            if constexpr (GATED) Us[kk][r] = in ? to_float(Wu[(size_t)n * D + k]) : 0.f;
         }
         __syncthreads();
         if (busy) {
@@ -301,14 +371,14 @@ moe_gate_up_kernel(const T* __restrict__ h, const T* __restrict__ W, const int* 
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     g[j] = Gs[kk][tx * 4 + j];
-                    u[j] = Us[kk][tx * 4 + j];
+                    u[j] = GATED ? Us[GATED ? kk : 0][tx * 4 + j] : 0.f;
                 }
 #pragma unroll
                 for (int i = 0; i < 4; ++i)
 #pragma unroll
                     for (int j = 0; j < 4; ++j) {
                         acc_g[i][j] = fmaf(a[i], g[j], acc_g[i][j]);
-                        acc_u[i][j] = fmaf(a[i], u[j], acc_u[i][j]);
+                        if constexpr (GATED) acc_u[i][j] = fmaf(a[i], u[j], acc_u[i][j]);
                     }
             }
         }
@@ -323,12 +393,7 @@ moe_gate_up_kernel(const T* __restrict__ h, const T* __restrict__ W, const int* 
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
             if (n >= F) continue;
-            float g = acc_g[i][j] * wt, u = acc_u[i][j] * wt;
-            if (limit > 0.f) {
-                g = fminf(g, limit);
-                u = fminf(fmaxf(u, -limit), limit);
-            }
-            const float v = g / (1.f + expf(-alpha * g)) * (u + up_shift);
+            const float v = expert_act<ACT>(acc_g[i][j] * wt, acc_u[i][j] * wt, limit, alpha, up_shift);
             y[(size_t)(tile * kTile + r) * F + n] = from_float<T>(v);
         }
     }
@@ -399,6 +464,7 @@ moe_down_kernel(const T* __restrict__ y, const T* __restrict__ W, const int* __r
 // 32-bit accumulators.  A warp whose 16 rows are all padding issues no MMA (a decode step's tiles hold a
 // few rows each: the launch is then bound by the weights it streams).  K and the row strides must be
 // multiples of 8 (16-byte rows); other sizes take the kernels above.
+template <int ACT>
 __global__ void __launch_bounds__(256)
 moe_gate_up_tc_kernel(const bf16* __restrict__ h, const bf16* __restrict__ W, const int* __restrict__ listed,
                       const int* __restrict__ tile_expert, bf16* __restrict__ y, int D, int F, int top, float limit,
@@ -418,9 +484,10 @@ moe_gate_up_tc_kernel(const bf16* __restrict__ h, const bf16* __restrict__ W, co
     const int warp_m = warp & 3, warp_n = warp >> 2;
     bool busy = false;
     for (int i = 0; i < 16; ++i) busy = busy || rows[warp_m * 16 + i] >= 0;
-    float acc[2][4][4] = {};
-    const bf16* We = W + (size_t)e * 2 * F * D;
-    tc_mainloop<2>(smem, [&](int r) { return rows[r] >= 0 ? h + (size_t)rows[r] * D : (const bf16*)nullptr; }, We, F, n0,
+    constexpr int NB = ACT == kGatedSwish ? 2 : 1;
+    float acc[NB][4][4] = {};
+    const bf16* We = W + (size_t)e * NB * F * D;
+    tc_mainloop<NB>(smem, [&](int r) { return rows[r] >= 0 ? h + (size_t)rows[r] * D : (const bf16*)nullptr; }, We, F, n0,
                    (size_t)F * D, D, busy, acc);
     if (!busy) return;
 #pragma unroll
@@ -434,14 +501,8 @@ moe_gate_up_tc_kernel(const bf16* __restrict__ h, const bf16* __restrict__ W, co
             const float wt = in_weight ? in_weight[listed[tile * kTile + r]] : 1.f;
             float v[2];
 #pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                float g = acc[0][nt][half * 2 + c] * wt, u = acc[1][nt][half * 2 + c] * wt;
-                if (limit > 0.f) {
-                    g = fminf(g, limit);
-                    u = fminf(fmaxf(u, -limit), limit);
-                }
-                v[c] = g / (1.f + expf(-alpha * g)) * (u + up_shift);
-            }
+            for (int c = 0; c < 2; ++c)
+                v[c] = expert_act<ACT>(acc[0][nt][half * 2 + c] * wt, acc[NB - 1][nt][half * 2 + c] * wt, limit, alpha, up_shift);
             *reinterpret_cast<uint32_t*>(y + (size_t)(tile * kTile + r) * F + n) = pack_bf16(v[0], v[1]);
         }
     }
@@ -505,7 +566,7 @@ __device__ __forceinline__ float dot8(const uint4& a, const uint4& b) {
 }
 
 // y[pair][F] = act(gate, up) of row pair / top under expert choice[pair]
-template <int QF>
+template <int QF, int ACT>
 __global__ void __launch_bounds__(256)
 moe_gate_up_few_kernel(const bf16* __restrict__ h, const bf16* __restrict__ W, const int* __restrict__ choice,
                        bf16* __restrict__ y, int D, int F, int top, int n_experts, float limit, float alpha,
@@ -519,7 +580,8 @@ moe_gate_up_few_kernel(const bf16* __restrict__ h, const bf16* __restrict__ W, c
     const uint4* src = reinterpret_cast<const uint4*>(h + (size_t)(pair / top) * D);
     for (int g = threadIdx.x; g < groups; g += 256) row[g] = src[g];
     __syncthreads();
-    const bf16* Wg = W + (size_t)e * 2 * F * D;
+    constexpr bool GATED = ACT == kGatedSwish;
+    const bf16* Wg = W + (size_t)e * (GATED ? 2 : 1) * F * D;
     const int f0 = (blockIdx.x * 8 + warp) * QF;
     if (f0 >= F) return;
     const uint4* g_row[QF];
@@ -528,12 +590,12 @@ moe_gate_up_few_kernel(const bf16* __restrict__ h, const bf16* __restrict__ W, c
     for (int q = 0; q < QF; ++q) {
         const int f = min(f0 + q, F - 1);                       // a feature beyond the last: read the last again, store nothing
         g_row[q] = reinterpret_cast<const uint4*>(Wg + (size_t)f * D);
-        u_row[q] = reinterpret_cast<const uint4*>(Wg + (size_t)(F + f) * D);
+        u_row[q] = GATED ? reinterpret_cast<const uint4*>(Wg + (size_t)(F + f) * D) : nullptr;
     }
     float sg[QF], su[QF];
 #pragma unroll
     for (int q = 0; q < QF; ++q) sg[q] = su[q] = 0.f;
-    constexpr int U = 8 / QF;                                   // steps whose loads are issued together: 16 loads a lane
+    constexpr int U = (GATED ? 8 : 16) / QF;                    // steps whose loads are issued together: 16 loads a lane
     const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
     for (int g0 = lane; g0 < groups; g0 += 32 * U) {
         uint4 wg[U][QF], wu[U][QF];
@@ -543,7 +605,7 @@ moe_gate_up_few_kernel(const bf16* __restrict__ h, const bf16* __restrict__ W, c
 #pragma unroll
             for (int q = 0; q < QF; ++q) {
                 wg[u][q] = g < groups ? __ldg(g_row[q] + g) : zero;
-                wu[u][q] = g < groups ? __ldg(u_row[q] + g) : zero;
+                if constexpr (GATED) wu[u][q] = g < groups ? __ldg(u_row[q] + g) : zero;
             }
         }
 #pragma unroll
@@ -554,21 +616,16 @@ moe_gate_up_few_kernel(const bf16* __restrict__ h, const bf16* __restrict__ W, c
 #pragma unroll
             for (int q = 0; q < QF; ++q) {
                 sg[q] += dot8(x, wg[u][q]);
-                su[q] += dot8(x, wu[u][q]);
+                if constexpr (GATED) su[q] += dot8(x, wu[u][q]);
             }
         }
     }
     const float wt = in_weight ? in_weight[pair] : 1.f;
 #pragma unroll
     for (int q = 0; q < QF; ++q) {
-        float a = warp_sum(sg[q]) * wt, b = warp_sum(su[q]) * wt;
-        if (lane == 0 && f0 + q < F) {
-            if (limit > 0.f) {
-                a = fminf(a, limit);
-                b = fminf(fmaxf(b, -limit), limit);
-            }
-            y[(size_t)pair * F + f0 + q] = from_float<bf16>(a / (1.f + expf(-alpha * a)) * (b + up_shift));
-        }
+        const float a = warp_sum(sg[q]) * wt, b = GATED ? warp_sum(su[q]) * wt : 0.f;
+        if (lane == 0 && f0 + q < F)
+            y[(size_t)pair * F + f0 + q] = from_float<bf16>(expert_act<ACT>(a, b, limit, alpha, up_shift));
     }
 }
 
@@ -679,12 +736,15 @@ extern "C" int hos_moe_tile_rows() { return kTile; }
 
 extern "C" int hos_moe_route(const void* h, int dtype, const float* router, const float* correction,
                              const int* token_seq, int* choice, float* weight, int N, int D, int n_out, int top,
-                             int scoring, float* logits, float renorm, float wscale, cudaStream_t stream) {
+                             int scoring, float* logits, float renorm, float wscale, int groups, int keep,
+                             cudaStream_t stream) {
     if (N <= 0) return 0;
     if (top <= 0 || top > n_out) HOS_REFUSE("moe_route: %d of %d router outputs cannot be chosen", top, n_out);
+    if (groups < 0 || (groups > 0 && (n_out % groups != 0 || keep < 1 || keep > groups)))
+        HOS_REFUSE("moe_route: the best %d of %d groups of %d router outputs", keep, groups, n_out);
     // rows to a block: as many as pay (the router matrix is read once per block) and as shared memory holds
     int rt = N >= 1024 ? 8 : N >= 16 ? 4 : 1;
-    auto smem_of = [&](int r) { return (size_t)(2 + 8) * r * n_out * sizeof(float); };   // scores, flags, a partial sum per warp
+    auto smem_of = [&](int r) { return (size_t)r * ((2 + 8) * n_out + groups) * sizeof(float); };   // scores, flags, a partial sum per warp
     while (rt > 1 && smem_of(rt) > 48 * 1024) rt = rt == 8 ? 4 : 1;
     const size_t smem = smem_of(rt);
     if (smem > 48 * 1024) HOS_REFUSE("moe_route: %d router outputs are more than a block's shared memory holds", n_out);
@@ -694,10 +754,10 @@ extern "C" int hos_moe_route(const void* h, int dtype, const float* router, cons
     // few blocks and more than eight outputs: the outputs' groups of eight go to blocks of their own (grid.y) and a
     // second launch chooses; the caller then gives `logits` [N][n_out]
     if (blocks >= 296u || n_out <= 8) logits = nullptr;
-    const unsigned groups = logits != nullptr ? (unsigned)((n_out + 7) / 8) : 1u;
+    const unsigned eights = logits != nullptr ? (unsigned)((n_out + 7) / 8) : 1u;
 #define HOS_ROUTE(T, RT, VEC)                                                                                        \
-    launch_pdl(moe_route_kernel<T, RT, VEC>, dim3(blocks, groups), dim3(256), smem, stream, (const T*)h, router,     \
-               correction, token_seq, choice, weight, N, D, n_out, top, scoring, logits, renorm, wscale)
+    launch_pdl(moe_route_kernel<T, RT, VEC>, dim3(blocks, eights), dim3(256), smem, stream, (const T*)h, router,     \
+               correction, token_seq, choice, weight, N, D, n_out, top, scoring, logits, renorm, wscale, groups, keep)
 #define HOS_ROUTE_V(T, RT)                                                                                           \
     do {                                                                                                             \
         if (vec) HOS_ROUTE(T, RT, true);                                                                             \
@@ -715,10 +775,10 @@ extern "C" int hos_moe_route(const void* h, int dtype, const float* router, cons
 #undef HOS_ROUTE_V
 #undef HOS_ROUTE
     if (logits != nullptr) {
-        const size_t csmem = (size_t)4 * 2 * n_out * sizeof(float);
+        const size_t csmem = (size_t)4 * (2 * n_out + groups) * sizeof(float);
         if (csmem > 48 * 1024) HOS_REFUSE("moe_route: %d router outputs are more than a block's shared memory holds", n_out);
         launch_pdl(moe_choose_kernel, dim3((N + 3) / 4), dim3(128), csmem, stream, (const float*)logits, correction, token_seq,
-                   choice, weight, N, n_out, top, scoring, renorm, wscale);
+                   choice, weight, N, n_out, top, scoring, renorm, wscale, groups, keep);
     }
     return check_launch("moe_route");
 }
@@ -733,29 +793,44 @@ extern "C" int hos_moe_align(const int* choice, int n_pairs, int n_experts, int*
     return check_launch("moe_align");
 }
 
-extern "C" int hos_moe_gate_up(const void* h, const void* W, int dtype, const int* listed, const int* tile_expert,
-                               void* y, int max_tiles, int D, int F, int top, float limit, float alpha, float up_shift,
-                               const float* in_weight, cudaStream_t stream) {
-    if (max_tiles <= 0) return 0;
+// act: 0 the gated form (W: gate rows, then up rows), 1 relu(u)^2 (W: up rows)
+template <int ACT>
+static int launch_gate_up(const void* h, const void* W, int dtype, const int* listed, const int* tile_expert, void* y,
+                          int max_tiles, int D, int F, int top, float limit, float alpha, float up_shift, const float* in_weight,
+                          cudaStream_t stream) {
     dim3 grid((F + kTile - 1) / kTile, max_tiles);
     if (grid.y > 65535) HOS_REFUSE("moe_gate_up: %d tiles are more than one launch takes", max_tiles);
     if (dtype == kBF16 && D % 8 == 0 && F % 8 == 0 && ((uintptr_t)h | (uintptr_t)W | (uintptr_t)y) % 16 == 0) {
+        constexpr int smem = TcTile<ACT == kGatedSwish ? 2 : 1>::kSmemBytes;
         static bool set = false;
         if (!set) {
-            cudaFuncSetAttribute(moe_gate_up_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, TcTile<2>::kSmemBytes);
+            cudaFuncSetAttribute(moe_gate_up_tc_kernel<ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
             set = true;
         }
-        launch_pdl(moe_gate_up_tc_kernel, grid, dim3(256), (size_t)TcTile<2>::kSmemBytes, stream, (const bf16*)h,
-                   (const bf16*)W, listed, tile_expert, (bf16*)y, D, F, top, limit, alpha, up_shift, in_weight);
+        launch_pdl(moe_gate_up_tc_kernel<ACT>, grid, dim3(256), (size_t)smem, stream, (const bf16*)h, (const bf16*)W, listed,
+                   tile_expert, (bf16*)y, D, F, top, limit, alpha, up_shift, in_weight);
     } else if (dtype == kBF16)
-        launch_pdl(moe_gate_up_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)h, (const bf16*)W, listed, tile_expert,
+        launch_pdl(moe_gate_up_kernel<bf16, ACT>, grid, dim3(256), 0, stream, (const bf16*)h, (const bf16*)W, listed, tile_expert,
                    (bf16*)y, D, F, top, limit, alpha, up_shift, in_weight);
     else if (dtype == kF32)
-        launch_pdl(moe_gate_up_kernel<float>, grid, dim3(256), 0, stream, (const float*)h, (const float*)W, listed,
+        launch_pdl(moe_gate_up_kernel<float, ACT>, grid, dim3(256), 0, stream, (const float*)h, (const float*)W, listed,
                    tile_expert, (float*)y, D, F, top, limit, alpha, up_shift, in_weight);
     else
         HOS_REFUSE("moe_gate_up: unknown dtype %d", dtype);
     return check_launch("moe_gate_up");
+}
+
+extern "C" int hos_moe_gate_up(const void* h, const void* W, int dtype, const int* listed, const int* tile_expert,
+                               void* y, int max_tiles, int D, int F, int top, float limit, float alpha, float up_shift,
+                               const float* in_weight, int act, cudaStream_t stream) {
+    if (max_tiles <= 0) return 0;
+    if (act == kGatedSwish)
+        return launch_gate_up<kGatedSwish>(h, W, dtype, listed, tile_expert, y, max_tiles, D, F, top, limit, alpha, up_shift,
+                                           in_weight, stream);
+    if (act == kReluSquare)
+        return launch_gate_up<kReluSquare>(h, W, dtype, listed, tile_expert, y, max_tiles, D, F, top, limit, alpha, up_shift,
+                                           in_weight, stream);
+    HOS_REFUSE("moe_gate_up: unknown activation %d", act);
 }
 
 extern "C" int hos_moe_down(const void* y, const void* W, int dtype, const int* listed, const int* tile_expert,
@@ -807,22 +882,29 @@ extern "C" int hos_moe_combine(const float* pair_out, const int* choice, const f
 // launches nothing) where the sizes are not the kernels' (K no multiple of 8, rows that do not fit shared memory).
 extern "C" int hos_moe_gate_up_few(const void* h, const void* W, const int* choice, void* y, int n_pairs, int D, int F,
                                    int top, int n_experts, float limit, float alpha, float up_shift, const float* in_weight,
-                                   cudaStream_t stream) {
+                                   int act, cudaStream_t stream) {
     if (n_pairs <= 0) return 0;
     if (D % 8 || F % 8 || D * 2 > 96 * 1024 || ((uintptr_t)h | (uintptr_t)W | (uintptr_t)y) % 16) return 1;
+    if (act != kGatedSwish && act != kReluSquare) HOS_REFUSE("moe_gate_up_few: unknown activation %d", act);
     const long long want = 2LL * sm_count();
     const int qf = (long long)((F + 31) / 32) * n_pairs >= want ? 4 : (long long)((F + 15) / 16) * n_pairs >= want ? 2 : 1;
-#define HOS_GU_FEW(QF)                                                                                               \
+#define HOS_GU_FEW_A(QF, ACT)                                                                                        \
     do {                                                                                                             \
         if (D * 2 > 48 * 1024)                                                                                       \
-            cudaFuncSetAttribute(moe_gate_up_few_kernel<QF>, cudaFuncAttributeMaxDynamicSharedMemorySize, D * 2);    \
-        launch_pdl(moe_gate_up_few_kernel<QF>, dim3((F + 8 * QF - 1) / (8 * QF), n_pairs), dim3(256), (size_t)D * 2, \
+            cudaFuncSetAttribute(moe_gate_up_few_kernel<QF, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, D * 2); \
+        launch_pdl(moe_gate_up_few_kernel<QF, ACT>, dim3((F + 8 * QF - 1) / (8 * QF), n_pairs), dim3(256), (size_t)D * 2, \
                    stream, (const bf16*)h, (const bf16*)W, choice, (bf16*)y, D, F, top, n_experts, limit, alpha,     \
                    up_shift, in_weight);                                                                             \
+    } while (0)
+#define HOS_GU_FEW(QF)                                                                                               \
+    do {                                                                                                             \
+        if (act == kReluSquare) HOS_GU_FEW_A(QF, kReluSquare);                                                       \
+        else HOS_GU_FEW_A(QF, kGatedSwish);                                                                          \
     } while (0)
     if (qf == 4) HOS_GU_FEW(4);
     else if (qf == 2) HOS_GU_FEW(2);
     else HOS_GU_FEW(1);
+#undef HOS_GU_FEW_A
 #undef HOS_GU_FEW
     return check_launch("moe_gate_up_few");
 }

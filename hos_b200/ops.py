@@ -24,7 +24,8 @@ PAGE_TOKENS = 64
 EPI_NONE, EPI_SOFTCAP, EPI_GATED, EPI_BIAS = 0, 1, 2, 3
 ACT_GELU_TANH, ACT_SILU, ACT_CLAMPED_SWISH = 0, 1, 2
 ACTIVATIONS = {"gelu_tanh": ACT_GELU_TANH, "silu": ACT_SILU}
-BIAS_ACTIVATIONS = {"none": 0, "gelu_erf": 1}          # what EPI_BIAS applies after the bias
+BIAS_ACTIVATIONS = {"none": 0, "gelu_erf": 1, "gelu_tanh": 2}      # what EPI_BIAS applies after the bias (or without one)
+EXPERT_ACTIVATIONS = {"gated_swish": 0, "relu_square": 1}          # the routed experts' (csrc/moe.cu)
 # the clamped form as the products' gated epilogues know it: g logistic(SWISH_ALPHA g) (u + SWISH_SHIFT), the limit a parameter
 SWISH_ALPHA, SWISH_SHIFT = 1.702, 1.0
 ROPE_STYLES = {"rotate_half": 0, "interleaved": 1}
@@ -317,7 +318,7 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, add_one: bool, out: to
 def norm_add_norm(y: torch.Tensor, w_post: torch.Tensor, eps_post: float, add_one_post: bool,
                   x: torch.Tensor, w_next: Optional[torch.Tensor] = None, eps_next: float = 0.0,
                   add_one_next: bool = False, h: Optional[torch.Tensor] = None) -> None:
-    """x += RMSNorm(y; w_post); if h is given, h = RMSNorm(x; w_next).  y is [N, D], or
+    """x += RMSNorm(y; w_post); if h is given, h = RMSNorm(x; w_next), or x itself in h's type without w_next.  y is [N, D], or
     [parts, N, D] float32 partial sums (of a matrix product that split K), added here."""
     _check(y, "norm input")
     _check(x, "residual stream", torch.float32, 2)
@@ -328,8 +329,9 @@ def norm_add_norm(y: torch.Tensor, w_post: torch.Tensor, eps_post: float, add_on
         raise KernelError("norm_add_norm: sizes disagree")
     if h is not None:
         _check(h, "next norm output", None, 2)
-        _check(w_next, "next norm weight", torch.float32, 1)
-        if h.shape != x.shape or w_next.shape[0] != d:
+        if w_next is not None:
+            _check(w_next, "next norm weight", torch.float32, 1)
+        if h.shape != x.shape or (w_next is not None and w_next.shape[0] != d):
             raise KernelError("norm_add_norm: sizes of the next norm disagree")
     core().call("hos_norm_add_norm", _ptr(y), dtype_code(y.dtype), n_parts, _ptr(w_post), float(eps_post),
                 int(add_one_post), _ptr(x), _ptr(w_next), float(eps_next), int(add_one_next),
@@ -424,7 +426,8 @@ def gather_rows(x: torch.Tensor, idx: torch.Tensor, out: torch.Tensor) -> None:
 def gemm_plain(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = EPI_NONE,
                cap: float = 0.0, act: int = 0, bias: Optional[torch.Tensor] = None) -> None:
     """out[M, N] = a[M, K] . w[N, K]^T with 32-bit accumulation on the CUDA cores.
-    Gated epilogue: w has 2N rows (gate rows, then up rows), out = act(gate) * up.  Bias epilogue: act(product + bias)."""
+    Gated epilogue: w has 2N rows (gate rows, then up rows), out = act(gate) * up.  Bias epilogue: act(product + bias),
+    or act(product) with no bias."""
     _check(a, "left operand", None, 2)
     _check(w, "weight", None, 2)
     _check(out, "product", None, 2)
@@ -624,31 +627,51 @@ def scaled_add_norms(a: Optional[torch.Tensor], f: Optional[torch.Tensor], mult:
                   dtype_code(h.dtype) if h is not None else 0, n, d, _stream())
 
 
-def latent_prep(proj: torch.Tensor, n_heads: int, dq: int, rank: int, rot: int, w_norm: Optional[torch.Tensor], eps: float,
-                inv_freq: Optional[torch.Tensor], rot_dims: int, step, kc: Optional[torch.Tensor], q_lat: torch.Tensor,
-                cache: Optional[PagedKVArgs]) -> None:
-    """kc None: the rows hold queries only (a call that reads another call's cache): the queries' rotated parts are
-    written and nothing is normed or stored."""
-    _check(proj, "projection rows", None, 2)
-    _check(q_lat, "latent queries", torch.float32, 3)
-    n = proj.shape[0]
-    if kc is None:
-        if proj.shape[1] != n_heads * (dq + rot) or q_lat.shape != (n, n_heads, rank + rot):
+def latent_prep(step, q, n_heads: int, dq: int, rank: int, rot: int, eps: float, inv_freq: Optional[torch.Tensor], rot_dims: int,
+                style: int, q_lat: Optional[torch.Tensor] = None, down=None, w_norm: Optional[torch.Tensor] = None,
+                kc: Optional[torch.Tensor] = None, cache: Optional[PagedKVArgs] = None, cq=None,
+                cq_norm: Optional[torch.Tensor] = None, cq_out: Optional[torch.Tensor] = None) -> None:
+    """Norms, rotations and the cache write between the projections and the latent attention, for the parts that are given.
+    `q`, `down` and `cq` are (rows, first column) or None: the heads' queries [n_heads x (dq + rot)] -> the last `rot` numbers
+    of q_lat's heads; the latent and the shared key part [rank + rot] -> kc and the cache; the queries' own latent ->
+    cq_out, normed with cq_norm.  style: the rotation's pairing (ROPE_STYLES)."""
+    rows = next((p[0] for p in (q, down, cq) if p is not None), None)
+    if rows is None:
+        raise KernelError("latent_prep: no rows")
+    n, dt = rows.shape[0], rows.dtype
+    rq = cq_out.shape[1] if cq_out is not None else 0
+    for part, cols, what in ((q, n_heads * (dq + rot), "query rows"), (down, rank + rot, "latent rows"), (cq, rq, "query latents")):
+        if part is not None:
+            _check(part[0], what, dt, 2)
+            if part[0].shape[0] != n or part[1] + cols > part[0].shape[1]:
+                raise KernelError(f"latent_prep: sizes of the {what} disagree")
+    if q is not None:
+        _check(q_lat, "latent queries", torch.float32, 3)
+        if q_lat.shape != (n, n_heads, rank + rot):
             raise KernelError("latent_prep: sizes disagree")
-        cache = None
+    if down is not None:
+        _check(kc, "latent rows", dt, 2)
+        if kc.shape != (n, rank + rot) or w_norm is None or w_norm.shape[0] != rank:
+            raise KernelError("latent_prep: sizes disagree")
     else:
-        _check(kc, "latent rows", proj.dtype, 2)
-        if proj.shape[1] != n_heads * (dq + rot) + rank + rot or kc.shape != (n, rank + rot) \
-                or q_lat.shape != (n, n_heads, rank + rot) or w_norm is None:
+        cache = None
+    if cq is not None:
+        _check(cq_out, "normed query latents", dt, 2)
+        if cq_out.shape[0] != n or cq_norm is None or cq_norm.shape[0] != rq:
             raise KernelError("latent_prep: sizes disagree")
-    if cache is not None and (cache.k_pages.dtype != proj.dtype or cache.head_dim != rank + rot or cache.n_kv_heads != 1):
+    if cache is not None and (cache.k_pages.dtype != dt or cache.head_dim != rank + rot or cache.n_kv_heads != 1):
         raise KernelError("latent_prep: the cache does not fit the latent rows")
-    blocks().call("hos_latent_prep", _ptr(proj), dtype_code(proj.dtype), proj.shape[1], n_heads, dq, rank, rot,
-                  _ptr(w_norm), float(eps), _ptr(inv_freq), int(rot_dims) if inv_freq is not None else 0,
+
+    def at(part):
+        if part is None:
+            return None, 0
+        return ctypes.c_void_p(part[0].data_ptr() + part[1] * part[0].element_size()), part[0].shape[1]
+    blocks().call("hos_latent_prep", *at(q), *at(down), *at(cq), dtype_code(dt), n_heads, dq, rank, rot, rq, _ptr(w_norm),
+                  _ptr(cq_norm), float(eps), _ptr(inv_freq), int(rot_dims) if inv_freq is not None else 0, int(style),
                   _ptr(step.token_pos), _ptr(step.token_seq), _ptr(step.seq_slot), _ptr(step.seq_len_after),
-                  _ptr(kc), _ptr(q_lat), _ptr(cache.k_pages) if cache else None,
-                  _ptr(cache.page_table) if cache else None, cache.table_stride if cache else 0,
-                  cache.ring_pages if cache else 0, n, _stream())
+                  _ptr(kc) if down is not None else None, _ptr(q_lat), _ptr(cq_out),
+                  _ptr(cache.k_pages) if cache else None, _ptr(cache.page_table) if cache else None,
+                  cache.table_stride if cache else 0, cache.ring_pages if cache else 0, n, _stream())
 
 
 def latent_attn(q_lat: torch.Tensor, kc: Optional[torch.Tensor], cache: Optional[PagedKVArgs], sink: Optional[torch.Tensor],
@@ -737,9 +760,9 @@ MOE_SCORING = {"softmax": 0, "logistic": 1}
 
 
 def moe_route(h, router, correction, token_seq, choice, weight, top: int, scoring: int = 0,
-              renormalise: Optional[float] = None, weight_scale: float = 1.0) -> None:
+              renormalise: Optional[float] = None, weight_scale: float = 1.0, groups: Optional[tuple] = None) -> None:
     """renormalise (a number >= 0): the chosen scores are divided by their sum plus that number; weight_scale: a constant
-    on every weight after that."""
+    on every weight after that.  groups (count, keep): only outputs of the `keep` best of `count` equal groups can be chosen."""
     _check(h, "rows", None, 2)
     _check(router, "router", torch.float32, 2)
     n, d = h.shape
@@ -747,7 +770,7 @@ def moe_route(h, router, correction, token_seq, choice, weight, top: int, scorin
     logits = torch.empty((n, router.shape[0]), dtype=torch.float32, device=h.device) if router.shape[0] > 8 and n < 2048 else None
     experts().call("hos_moe_route", _ptr(h), dtype_code(h.dtype), _ptr(router), _ptr(correction), _ptr(token_seq),
                   _ptr(choice), _ptr(weight), n, d, router.shape[0], int(top), int(scoring), _ptr(logits),
-                  -1.0 if renormalise is None else float(renormalise), float(weight_scale), _stream())
+                  -1.0 if renormalise is None else float(renormalise), float(weight_scale), *(groups or (0, 0)), _stream())
 
 
 def moe_align(choice, n_experts: int, listed, tile_expert) -> None:
@@ -756,12 +779,16 @@ def moe_align(choice, n_experts: int, listed, tile_expert) -> None:
 
 
 def moe_gate_up(h, w, listed, tile_expert, y, top: int, limit: float, alpha: float, up_shift: float = 1.0,
-                in_weight: Optional[torch.Tensor] = None) -> None:
-    """in_weight ([pairs] float32): the pair's weight multiplies the expert's input (then `moe_down` takes none)."""
+                in_weight: Optional[torch.Tensor] = None, act: int = 0) -> None:
+    """w: [experts, 2F, D], gate rows then up rows, or [experts, F, D] for an activation without a gate (act, one of
+    EXPERT_ACTIVATIONS).  in_weight ([pairs] float32): the pair's weight multiplies the expert's input (then `moe_down` takes
+    none)."""
     _check(w, "expert gate/up weights", h.dtype, 3)
+    if w.shape[1] != y.shape[1] * (2 if act == 0 else 1):
+        raise KernelError("moe_gate_up: the experts' weights do not fit the inner rows")
     experts().call("hos_moe_gate_up", _ptr(h), _ptr(w), dtype_code(h.dtype), _ptr(listed), _ptr(tile_expert), _ptr(y),
-                  tile_expert.numel(), h.shape[1], w.shape[1] // 2, int(top), float(limit), float(alpha), float(up_shift),
-                  _ptr(in_weight), _stream())
+                  tile_expert.numel(), h.shape[1], y.shape[1], int(top), float(limit), float(alpha), float(up_shift),
+                  _ptr(in_weight), int(act), _stream())
 
 
 def moe_down(y, w, listed, tile_expert, weight, pair_out) -> None:
@@ -771,7 +798,7 @@ def moe_down(y, w, listed, tile_expert, weight, pair_out) -> None:
 
 
 def moe_few(h, w_gate_up, w_down, choice, weight, y, pair_out, top: int, n_experts: int, limit: float, alpha: float,
-            up_shift: float = 1.0, weight_on_input: bool = False) -> bool:
+            up_shift: float = 1.0, weight_on_input: bool = False, act: int = 0) -> bool:
     """Both expert products for a handful of (row, choice) pairs, without lists or tiles (decoding at small batch):
     y [pairs, F] and pair_out [pairs, D] by pair id.  False: the sizes are not these kernels' and nothing ran."""
     lib = experts()
@@ -790,7 +817,7 @@ def moe_few(h, w_gate_up, w_down, choice, weight, y, pair_out, top: int, n_exper
         return rc
 
     rc = timed("hos_moe_gate_up_few", _ptr(h), _ptr(w_gate_up), _ptr(choice), _ptr(y), pairs, d, f, int(top), int(n_experts),
-               float(limit), float(alpha), float(up_shift), _ptr(weight) if weight_on_input else None, _stream())
+               float(limit), float(alpha), float(up_shift), _ptr(weight) if weight_on_input else None, int(act), _stream())
     if rc == 1:
         return False
     if rc == 0:
@@ -967,14 +994,15 @@ def qk_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional[t
             eps: float, freq: Optional[torch.Tensor], rot_dims: int, magnitude: float, step, q_out: torch.Tensor,
             cache: PagedKVArgs, n_heads: int, n_kv: int, kd: int, vd: int, norm_whole: bool = False,
             v_first: Optional[torch.Tensor] = None, v_first_col: int = 0, v_mix: float = 0.0, q_maps: int = 1,
-            proj_col: int = 0, q_temp=None) -> None:
+            proj_col: int = 0, q_temp=None, style: int = 1, unit_norm: bool = False) -> None:
     """proj: float32 rows whose columns from proj_col on are [q | k | v | ...] (G = n_kv; 0: a call that stores nothing).  Adds the
     biases, norms and rotates the q and k heads, writes q_out float32 [N, H, kd] and stores k, v in the cache.
     norm_whole: one root mean square over all q heads and one over all k heads (weights [H kd], [G kd]).  v_first
     (float32 [N, ld], the values from column v_first_col on): v <- (1 - v_mix) v + v_mix v_first before the store.
     q_maps > 1: a head's kd numbers are q_maps queries, one per attention map over the same key row; q_out is then
     [N, H * q_maps, kd], every query a head of its own that is zero outside its part of the key row.  q_temp = (coef, every): q times
-    1 + coef ln(floor((p + 1) / every) + 1) at position p."""
+    1 + coef ln(floor((p + 1) / every) + 1) at position p.  style: the rotation's pairing (ROPE_STYLES).  unit_norm: every q and
+    k head over its root mean square, without a weight."""
     _check(proj, "projection rows", torch.float32, 2)
     _check(q_out, "queries", torch.float32, 3)
     n = proj.shape[0]
@@ -998,7 +1026,7 @@ def qk_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional[t
                   _ptr(q_out), _ptr(cache.k_pages) if n_kv else None, _ptr(cache.v_pages) if n_kv else None,
                   dtype_code(cache.k_pages.dtype), _ptr(cache.page_table), cache.table_stride, cache.ring_pages, n,
                   int(n_heads), int(n_kv), int(kd), int(vd), 1 if norm_whole else 0, vf_ptr, vf_ld, float(v_mix),
-                  int(q_maps), float(coef), int(every), _stream())
+                  int(q_maps), float(coef), int(every), int(style), 1 if unit_norm else 0, _stream())
 
 
 def qkv_conv_store(proj: torch.Tensor, col: int, bias: Optional[torch.Tensor], conv_w: torch.Tensor, conv_state, step, q_out: torch.Tensor,
@@ -1041,9 +1069,9 @@ def diff_combine(a: torch.Tensor, lam: float, mult: float, eps: float, gate: Opt
 
 def gated_attn(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor],
                gate_col: int, step, out: torch.Tensor, scale: float, chunk: int, window: int, n_splits: int = 1,
-               keep_first: int = 0, out_col: int = 0, out_scale: float = 1.0) -> None:
+               keep_first: int = 0, out_col: int = 0, out_scale: float = 1.0, softcap: float = 0.0) -> None:
     """q: float32 [N, H, kd]; keys and values from the paged cache; out: [N, >= out_col + H * vd], the heads' outputs times
-    out_scale from column out_col on.  gate: float32 rows whose column gate_col + h is head h's gate logit."""
+    out_scale from column out_col on.  softcap (0: none): a score s becomes softcap tanh(s / softcap).  gate: float32 rows whose column gate_col + h is head h's gate logit."""
     _check(q, "queries", torch.float32, 3)
     _check(out, "attention output", None, 2)
     n, heads, kd = q.shape
@@ -1060,12 +1088,12 @@ def gated_attn(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[torch.Tensor]
                   gate.shape[1] if gate is not None else 0, _ptr(step.token_pos), _ptr(step.token_seq), _ptr(step.seq_slot),
                   _at(out, out_col), dtype_code(out.dtype), out.shape[1], float(out_scale), _ptr(part_acc), _ptr(part_ml),
                   int(n_splits), n, heads,
-                  cache.n_kv_heads, kd, vd, float(scale), int(chunk or 0), int(window or 0), int(keep_first or 0), _stream())
+                  cache.n_kv_heads, kd, vd, float(scale), int(chunk or 0), int(window or 0), int(keep_first or 0), float(softcap), _stream())
 
 
 def gated_attn_mma(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor],
                    gate_col: int, step, out: torch.Tensor, scale: float, chunk: int, window: int, n_q_tiles: int,
-                   keep_first: int = 0, out_col: int = 0, out_scale: float = 1.0) -> bool:
+                   keep_first: int = 0, out_col: int = 0, out_scale: float = 1.0, softcap: float = 0.0) -> bool:
     """The same attention on the tensor cores, for bfloat16 caches and rows that come many to a sequence.  False: the
     sizes are not that kernel's and nothing ran."""
     n, heads, kd = q.shape
@@ -1081,13 +1109,15 @@ def gated_attn_mma(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[torch.Ten
                   gate.shape[1] if gate is not None else 0, _ptr(step.cu_seqlens), _ptr(step.token_pos),
                   _ptr(step.token_seq), _ptr(step.seq_slot), _at(out, out_col), 1 if out.dtype == torch.float32 else 0,
                   out.shape[1], float(out_scale), int(step.n_seqs), int(n_q_tiles), heads,
-                  cache.n_kv_heads, kd, vd, float(scale), int(chunk or 0), int(window or 0), int(keep_first or 0), _stream())
+                  cache.n_kv_heads, kd, vd, float(scale), int(chunk or 0), int(window or 0), int(keep_first or 0), float(softcap),
+                  _stream())
     return True
 
 
 def gated_attn_mma_decode(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor],
                           gate_col: int, step, out: torch.Tensor, scale: float, chunk: int, window: int,
-                          n_splits: int = 1, keep_first: int = 0, out_col: int = 0, out_scale: float = 1.0) -> bool:
+                          n_splits: int = 1, keep_first: int = 0, out_col: int = 0, out_scale: float = 1.0,
+                          softcap: float = 0.0) -> bool:
     """Single tokens on the tensor cores: the query heads that share a kv head are the rows of one tile.  False: the
     sizes are not that kernel's and nothing ran."""
     n, heads, kd = q.shape
@@ -1108,7 +1138,7 @@ def gated_attn_mma_decode(q: torch.Tensor, cache: PagedKVArgs, sink: Optional[to
                   _ptr(step.token_seq), _ptr(step.seq_slot), _at(out, out_col), 1 if out.dtype == torch.float32 else 0,
                   out.shape[1], float(out_scale), _ptr(part_acc), _ptr(part_ml), int(n_splits), n,
                   heads, cache.n_kv_heads, kd, vd, float(scale), int(chunk or 0), int(window or 0), int(keep_first or 0),
-                  _stream())
+                  float(softcap), _stream())
     if n_splits > 1:
         gated_attn_lib().call("hos_attn_merge", _ptr(part_acc), _ptr(part_ml), int(n_splits), gate_ptr, gate_ld,
                       _ptr(step.token_seq), _at(out, out_col), dtype_code(out.dtype), out.shape[1], float(out_scale), n, heads,

@@ -15,6 +15,9 @@ sums are 32-bit.
 "postnorm": the norm comes after the sum, and the branches read the residual stream itself,
     x <- post_mixer(alpha * x + mixer(x));  x <- post_ffn(alpha * x + ffn(x))
     (`alpha`: LayerSpec.params["alpha"], default 1; a layer without a feed-forward has the first line only).
+"branch_norm": a norm on each branch's output only, and the branches read the residual stream itself,
+    x += post_mixer(mixer(x));  x += post_ffn(ffn(x))
+    (a layer without a feed-forward has the first line only).
 """
 from __future__ import annotations
 
@@ -215,7 +218,37 @@ class PostNormLayer(Layer):
         return self._sum_norm(f, x, self.norms["post_ffn"], next_norm)
 
 
+class BranchNormLayer(Layer):
+    """x += norm(branch(x)) for the mixer and then for the feed-forward.  The norm, the sum and the copy of the new x that
+    the next branch's products read (or the model's last norm of it) are one kernel where the norm can do that."""
+    norm_roles = ("post_mixer",)
+    chains = True
+
+    def __init__(self, spec: LayerSpec, rt: Runtime):
+        super().__init__(spec, rt)
+        from .feedforward import NoFeedForward
+        from .norm import RowsAsGiven
+        self.has_ffn = not isinstance(self.feed_forward, NoFeedForward)
+        if self.has_ffn and "post_ffn" not in spec.norms:
+            raise SpecError(f"arch spec error: arrangement {spec.arrangement!r} needs norms ['post_ffn']")
+        self._entry = RowsAsGiven(rt)
+
+    def entry_norm(self):
+        return self._entry
+
+    def forward(self, x: torch.Tensor, step: StepInfo, store: CallStore, h_in=None, next_norm=None):
+        n = self.norms
+        h = h_in if h_in is not None else self._entry.forward(x)
+        a = self._branch(self.mixer, getattr(n["post_mixer"], "accepts_partials", False), h, step, store)
+        if not self.has_ffn:
+            return n["post_mixer"].add_to(a, x, then=next_norm)
+        h = n["post_mixer"].add_to(a, x, then=self._entry)
+        f = self._branch(self.feed_forward, getattr(n["post_ffn"], "accepts_partials", False), h, step)
+        return n["post_ffn"].add_to(f, x, then=next_norm)
+
+
 register_part("arrangement", "sandwich", SandwichLayer)
+register_part("arrangement", "branch_norm", BranchNormLayer)
 register_part("arrangement", "postnorm", PostNormLayer)
 register_part("arrangement", "parallel", ParallelLayer)
 register_part("arrangement", "parallel_shared_norm", SharedNormParallelLayer)

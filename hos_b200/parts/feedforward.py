@@ -74,8 +74,8 @@ class GatedMLP(FeedForward):
 
 
 class DenseMLP(FeedForward):
-    """Feed-forward without a gate, with biases: down(act(up(h) + b_up)) + b_down, act "gelu_erf" (0.5 x (1 + erf(x /
-    sqrt 2))) or "none".  The up product's epilogue adds its bias and applies the activation; the output bias is
+    """Feed-forward without a gate: down(act(up(h) + b_up)) + b_down, act "gelu_erf" (0.5 x (1 + erf(x / sqrt 2))),
+    "gelu_tanh" or "none"; `bias` false: without both biases.  The up product's epilogue adds its bias and applies the activation; the output bias is
     `out_bias`, which an arrangement may add itself (`forward_unbiased` leaves it out)."""
     graph_safe = True
 
@@ -86,24 +86,33 @@ class DenseMLP(FeedForward):
         if act not in ops.BIAS_ACTIVATIONS:
             raise SpecError(f"arch spec error: unknown activation {act!r}")
         self.act = ops.BIAS_ACTIVATIONS[act]
-        self.out_bias = None
+        self.has_bias = bool(spec.params.get("bias", True))
+        self.b_up = self.out_bias = None
 
     def weight_specs(self) -> List[WeightSpec]:
         w = self.spec.weights
-        return [WeightSpec(w["up"], (self.inner, self.width), "matrix", 0.02), WeightSpec(w["up_bias"], (self.inner,), "vector", 0.1),
-                WeightSpec(w["down"], (self.width, self.inner), "matrix", 0.02),
-                WeightSpec(w["down_bias"], (self.width,), "vector", 0.1)]
+        out = [WeightSpec(w["up"], (self.inner, self.width), "matrix", 0.02), WeightSpec(w["down"], (self.width, self.inner), "matrix", 0.02)]
+        if self.has_bias:
+            out += [WeightSpec(w["up_bias"], (self.inner,), "vector", 0.1), WeightSpec(w["down_bias"], (self.width,), "vector", 0.1)]
+        return out
 
     def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
         w = self.spec.weights
         self.w_up, self.w_down = self._matrix(tensors[w["up"]]), self._matrix(tensors[w["down"]])
-        self.b_up, self.out_bias = self._vector32(tensors[w["up_bias"]]), self._vector32(tensors[w["down_bias"]])
+        if self.has_bias:
+            self.b_up, self.out_bias = self._vector32(tensors[w["up_bias"]]), self._vector32(tensors[w["down_bias"]])
 
     def _inner(self, h: torch.Tensor) -> torch.Tensor:
         return linear.matmul(h, self.w_up, epilogue=ops.EPI_BIAS, act=self.act, bias=self.b_up)
 
     def forward(self, h: torch.Tensor, step: StepInfo = None) -> torch.Tensor:
+        if not self.has_bias:
+            return linear.matmul(self._inner(h), self.w_down)
         return linear.matmul(self._inner(h), self.w_down, epilogue=ops.EPI_BIAS, bias=self.out_bias)
+
+    def forward_partial(self, h: torch.Tensor, step: StepInfo = None) -> torch.Tensor:
+        """As forward, but without biases the down projection may come back as float32 partial sums."""
+        return self.forward(h, step) if self.has_bias else self.forward_unbiased(h, step)
 
     def forward_unbiased(self, h: torch.Tensor, step: StepInfo = None) -> torch.Tensor:
         """As forward, without `out_bias`, for a consumer that adds it; may hand back 32-bit partial sums."""

@@ -1,8 +1,9 @@
 """Softmax attention with grouped queries whose pieces are all options: keys of `dim` and values of `vdim`
 numbers per head; biases on the q, k, v projections; an RMS norm of every query and key head (`qk_norm` true or
-"head": a weight of `dim` numbers shared by the heads, before the rotation) or one over the whole query
+"head": a weight of `dim` numbers shared by the heads, before the rotation; "unit": no weight, the same before the rotation
+as after it, since a rotation keeps a head's root mean square) or one over the whole query
 projection and one over the whole key projection ("whole": weights of heads x dim numbers); a rotary position
-part on the first numbers of a head; scores (q . k) * scale; a mask of chunks (position i sees j <= i with
+part on the first numbers of a head (either pairing); scores (q . k) * scale, with `softcap` c then c tanh(score / c); a mask of chunks (position i sees j <= i with
 floor(j / C) = floor(i / C), counted from the sequence's position 0) or of a window (the last W keys, and with
 `keep_first` also the sequence's first keep_first keys), or plain causal; a sink (`sink` true: a learned number per
 head whose exponential joins the softmax's denominator, without a key or a value; "zero": the constant 0, which
@@ -61,7 +62,8 @@ class GatedSoftmaxAttention(Mixer):
         self.chunk: Optional[int] = p.get("chunk")
         self.window: Optional[int] = p.get("window")
         self.has_bias, self.qk_norm = bool(p.get("bias", False)), bool(p.get("qk_norm", False))
-        self.norm_whole = p.get("qk_norm") == "whole"
+        self.norm_whole, self.unit_norm = p.get("qk_norm") == "whole", p.get("qk_norm") == "unit"
+        self.softcap = float(p.get("softcap") or 0.0)
         self.has_sink, self.head_gate = bool(p.get("sink", False)), bool(p.get("head_gate", False))
         self.zero_sink = p.get("sink") == "zero"
         self.keep_first = int(p.get("keep_first") or 0)
@@ -88,8 +90,12 @@ class GatedSoftmaxAttention(Mixer):
         for name, v in (("chunk", self.chunk), ("window", self.window)):
             if v is not None and int(v) <= 0:
                 raise SpecError(f"arch spec error: the attention's {name} must be positive")
+        if self.softcap < 0.0:
+            raise SpecError("arch spec error: the attention's soft-cap cannot be negative")
         pos_spec = p.get("position")
         self.position = part_impl("position", pos_spec.kind)(pos_spec, rt) if pos_spec else None
+        if self.unit_norm and getattr(self.position, "magnitude", 1.0) != 1.0:
+            raise SpecError("arch spec error: a norm without a weight goes with a rotation of magnitude 1")
         self.q_cols = self.n_heads * self.dim
         self.kv_cols = 0 if self.shares_kv else self.n_kv_heads * (self.dim + self.vdim)
         self.gate_col = self.q_cols + self.kv_cols
@@ -109,7 +115,7 @@ class GatedSoftmaxAttention(Mixer):
             out += [WeightSpec(w[r + "_conv"], (n, self.taps), "matrix", 0.4) for r, n in roles]
         if self.has_o_bias:
             out.append(WeightSpec(w["o_bias"], (self.width,), "vector", 0.1))
-        if self.qk_norm:
+        if self.qk_norm and not self.unit_norm:
             out += [WeightSpec(w[r + "_norm"], (n if self.norm_whole else self.dim,), "vector", 0.1)
                     for r, n in roles if r != "v"]
         if self.has_sink and not self.zero_sink:
@@ -137,8 +143,9 @@ class GatedSoftmaxAttention(Mixer):
             if self.head_gate:
                 parts.append(torch.zeros(self.n_heads, dtype=torch.float32, device=parts[0].device))
             self.bias = torch.cat(parts).contiguous()
-        self.q_norm = self._vector32(tensors[w["q_norm"]]) if self.qk_norm else None
-        self.k_norm = self._vector32(tensors[w["k_norm"]]) if self.qk_norm and not self.shares_kv else None
+        weighted = self.qk_norm and not self.unit_norm
+        self.q_norm = self._vector32(tensors[w["q_norm"]]) if weighted else None
+        self.k_norm = self._vector32(tensors[w["k_norm"]]) if weighted and not self.shares_kv else None
         self.sink = None
         if self.has_sink:
             self.sink = (torch.zeros(self.n_heads, dtype=torch.float32, device=self.w_in.device) if self.zero_sink
@@ -218,7 +225,7 @@ class GatedSoftmaxAttention(Mixer):
                               "value tensors reads another call's cache, and only such a mixer does)")
         n = proj.shape[0]
         q = torch.empty((n, self.n_heads, self.dim), dtype=torch.float32, device=proj.device)
-        freq, rot_dims, _ = self.position.kernel_args() if self.position else (None, 0, 0)
+        freq, rot_dims, style = self.position.kernel_args() if self.position else (None, 0, 0)
         v_col = col + self.q_cols + self.n_kv_heads * self.dim
         gate_col = col + self.gate_col
         v_first = None
@@ -248,9 +255,9 @@ class GatedSoftmaxAttention(Mixer):
                         getattr(self.position, "magnitude", 1.0), step, q, cache, self.n_heads,
                         0 if self.shares_kv else self.n_kv_heads, self.dim, self.vdim, self.norm_whole,
                         v_first[0] if v_first else None, v_first[1] if v_first else 0, self.v_mix,
-                        proj_col=col if rows is proj else 0, q_temp=self.q_temp)
+                        proj_col=col if rows is proj else 0, q_temp=self.q_temp, style=style, unit_norm=self.unit_norm)
         gate = proj if self.head_gate else None
-        where = dict(keep_first=self.keep_first, out_col=out_col, out_scale=self.out_scale)
+        where = dict(keep_first=self.keep_first, out_col=out_col, out_scale=self.out_scale, softcap=self.softcap)
         if self.use_tensor_cores and att.dtype == torch.bfloat16 and step.max_new > FEW_TOKENS:
             # rows that come many to a sequence: 64 queries to a key tile on the tensor cores
             if step.cu_host:

@@ -13,6 +13,11 @@ numbers) and W_uv is applied to the weighted sum of latents, so the attention ke
 c, angles, scores, softmax, weighted sums) is 32-bit; with bfloat16 rows the two products run on the
 tensor cores with every 32-bit operand as two bfloat16 terms (csrc/latent_attention.cu).
 
+With `q_rank` the queries go through a latent of their own: one product makes [query latent | latent | key part] from
+the layer's input, the query latent is RMS-normed with a weight, and a second product expands it into the heads' queries.
+
+The rotation may pair neighbouring numbers or halves (the position part's style).
+
 Cache: one keys-only group of row size kv_rank + rot_dim, a window ring if `window` is set.
 A sequence that starts at position 0 attends over the step's own rows; one that goes on (by
 one token or many) stores first and attends over the cache.
@@ -24,6 +29,7 @@ rotation are this one's.
 """
 from __future__ import annotations
 
+import functools
 from typing import List, Mapping, Optional
 
 import torch
@@ -55,18 +61,24 @@ class LatentAttention(Mixer):
         self.window: Optional[int] = p.get("window")
         self.has_sink = bool(p.get("sink", False))
         self.shares_kv = bool(p.get("shares_kv", False))
+        self.q_rank = int(p.get("q_rank") or 0)   # 0: queries straight from the layer's input
         if self.shares_kv and self.window:
             raise SpecError("arch spec error: a latent attention that reads another call's cache keeps no window of its own")
         pos_spec = p.get("position")
         self.position = part_impl("position", pos_spec.kind)(pos_spec, rt) if pos_spec else None
-        if min(self.n_heads, self.dim, self.rot_dim, self.vdim, self.rank) <= 0:
+        if min(self.n_heads, self.dim, self.rot_dim, self.vdim, self.rank) <= 0 or self.q_rank < 0:
             raise SpecError("arch spec error: latent attention needs positive sizes")
         self.q_cols = self.n_heads * (self.dim + self.rot_dim)
         self.row = self.rank + self.rot_dim
 
     def weight_specs(self) -> List[WeightSpec]:
         w = self.spec.weights
-        out = [WeightSpec(w["q"], (self.q_cols, self.width), "matrix", 0.02)]
+        if self.q_rank:
+            out = [WeightSpec(w["dq"], (self.q_rank, self.width), "matrix", 0.02),
+                   WeightSpec(w["dq_norm"], (self.q_rank,), "vector", 0.1),
+                   WeightSpec(w["uq"], (self.q_cols, self.q_rank), "matrix", 0.05)]
+        else:
+            out = [WeightSpec(w["q"], (self.q_cols, self.width), "matrix", 0.02)]
         if not self.shares_kv:
             out += [WeightSpec(w["dkv"], (self.row, self.width), "matrix", 0.02),
                     WeightSpec(w["dkv_norm"], (self.rank,), "vector", 0.1)]
@@ -79,15 +91,20 @@ class LatentAttention(Mixer):
 
     def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
         w = self.spec.weights
-        q = self._matrix(tensors[w["q"]])
+        q = self._matrix(tensors[w["dq" if self.q_rank else "q"]])
+        self.q_norm = self._vector32(tensors[w["dq_norm"]]) if self.q_rank else None
+        self.w_uq = linear.pad_rows(self._matrix(tensors[w["uq"]])) if self.q_rank else None
+        self.w_norm = None
         if self.shares_kv:
-            self.w_in, self.w_norm = q, None
+            self.w_in = q
         else:
             dkv = self._matrix(tensors[w["dkv"]])
             if q.dtype != dkv.dtype:
                 q, dkv = q.float(), dkv.float()
             self.w_in = torch.cat([q, dkv], dim=0).contiguous()          # one product for q and the down projection
             self.w_norm = self._vector32(tensors[w["dkv_norm"]])
+        if self.q_rank:
+            self.w_in = linear.pad_rows(self.w_in)
         uk = self._matrix(tensors[w["uk"]]).view(self.n_heads, self.dim, self.rank)
         self.w_uk_t = uk.transpose(1, 2).contiguous()                # [heads, rank, dim]: q'_h = W_uk_h^T q_h
         self.w_uv = self._matrix(tensors[w["uv"]]).view(self.n_heads, self.vdim, self.rank).contiguous()
@@ -111,6 +128,14 @@ class LatentAttention(Mixer):
         return max(1, min(32, (keys + 63) // 64, (2 * sms + blocks - 1) // blocks)), 1
 
     def forward(self, h: torch.Tensor, step: StepInfo, store: CallStore) -> torch.Tensor:
+        return self._run(h, step, store, False)
+
+    def forward_partial(self, h: torch.Tensor, step: StepInfo, store: CallStore) -> torch.Tensor:
+        """As forward, but the output projection may come back as float32 partial sums [parts, N, width] for a consumer
+        that adds them."""
+        return self._run(h, step, store, True)
+
+    def _run(self, h: torch.Tensor, step: StepInfo, store: CallStore, partial_ok: bool) -> torch.Tensor:
         n = h.shape[0]
         cache = store.kv
         if cache is None or store.owns_kv == self.shares_kv:
@@ -121,11 +146,20 @@ class LatentAttention(Mixer):
         kc = None if self.shares_kv else torch.empty((n, D), dtype=h.dtype, device=h.device)
         q_lat = torch.empty((n, H, D), dtype=torch.float32, device=h.device)
         inv_freq, rot_dims, style = self.position.kernel_args() if self.position else (None, 0, 1)
-        if inv_freq is not None and style != ops.ROPE_STYLES["interleaved"]:
-            raise KernelError("latent attention rotates neighbouring pairs only")
-        ops.latent_prep(proj, H, self.dim, R, self.rot_dim, self.w_norm, self.eps, inv_freq, rot_dims, step, kc, q_lat, cache)
+        prep = functools.partial(ops.latent_prep, step, n_heads=H, dq=self.dim, rank=R, rot=self.rot_dim, eps=self.eps,
+                                 inv_freq=inv_freq, rot_dims=rot_dims, style=style)
+        q_first = self.q_rank or self.q_cols                # the column where the down projection's part of `proj` begins
+        keys = {} if self.shares_kv else dict(down=(proj, q_first), w_norm=self.w_norm, kc=kc, cache=cache)
+        if self.q_rank:
+            cq = torch.empty((n, self.q_rank), dtype=h.dtype, device=h.device)
+            prep(q=None, cq=(proj, 0), cq_norm=self.q_norm, cq_out=cq, **keys)
+            q = linear.matmul(cq, self.w_uq)
+            prep(q=(q, 0), q_lat=q_lat)
+        else:
+            q = proj
+            prep(q=(q, 0), q_lat=q_lat, **keys)
         # q'_h = W_uk_h^T q_h into the first `rank` numbers of every head's latent query
-        ops.heads_product(proj, 0, proj.shape[1], self.dim + self.rot_dim, self.w_uk_t, q_lat, 0, H * D, D, n)
+        ops.heads_product(q, 0, q.shape[1], self.dim + self.rot_dim, self.w_uk_t, q_lat, 0, H * D, D, n)
         o_lat = torch.empty((n, H, R), dtype=h.dtype, device=h.device)      # what the value expansion reads
         nf = 0 if self.shares_kv else (n if step.from_zero else step.fresh_tokens)
         if nf > 0:
@@ -146,7 +180,7 @@ class LatentAttention(Mixer):
                             n_splits=shares, rows_per_block=per_block, tensor_cores=self.use_tensor_cores)
         att = torch.empty((n, H * self.vdim), dtype=h.dtype, device=h.device)
         ops.heads_product(o_lat, 0, H * R, R, self.w_uv, att, 0, H * self.vdim, self.vdim, n)
-        return linear.matmul(att, self.w_o)
+        return linear.matmul_or_partials(att, self.w_o) if partial_ok else linear.matmul(att, self.w_o)
 
 
 register_part("mixer", "latent_attention", LatentAttention)

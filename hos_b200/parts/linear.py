@@ -35,7 +35,7 @@ def matmul(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
            epilogue: int = ops.EPI_NONE, cap: float = 0.0, act: int = 0,
            out: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[M, N] = x[M, K] . w[N or 2N, K]^T (2N rows with the gated epilogue; with its clamped activation the limit
-    rides in `cap`; the bias epilogue adds `bias` ([N] float32) and applies `act`, one of ops.BIAS_ACTIVATIONS)."""
+    rides in `cap`; the bias epilogue adds `bias` ([N] float32, or None) and applies `act`, one of ops.BIAS_ACTIVATIONS)."""
     m = x.shape[0]
     n = w.shape[0] // 2 if epilogue == ops.EPI_GATED else w.shape[0]
     if out is None:

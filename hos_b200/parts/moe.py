@@ -7,9 +7,11 @@ expert is weighted by its plain score s, not renormalised: its output is (`weigh
 input, expert(s h) ("input").  With `renormalise` (a number >= 0) the chosen scores are first divided by their sum
 plus that number, and `weight_scale` is a constant on every weight after that.  The last `identity` router outputs are experts without tensors whose
 output is the row itself.
-Expert: g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit), y = g * sigmoid(alpha * g) * (u + up_shift),
+`groups` {"count": g, "keep": k}: the outputs form g equal groups of neighbours, a group's score is the sum of its two
+largest s + correction, and only outputs of the k best groups can be chosen.
+Expert (`activation` "gated_swish"): g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit), y = g * sigmoid(alpha * g) * (u + up_shift),
 output W_down y; no biases (`up_shift` 1 and `alpha` 1.702 by default; 0 and 1 make the plain gated form
-silu(g) * u).  `shared`, the spec of a feed-forward part, is an expert that every row uses; its output is
+silu(g) * u); "relu_square": no gate, W_down relu(W_up h)^2.  `shared`, the spec of a feed-forward part, is an expert that every row uses; its output is
 added.  The step stays on the device: rows are listed expert by expert and the experts' products run as
 tiles of one launch each (csrc/moe.cu); the output is the 32-bit sum.
 """
@@ -48,6 +50,17 @@ class RoutedExperts(FeedForward):
         self.weight_scale = float(p.get("weight_scale", 1.0))
         if self.renormalise is not None and float(self.renormalise) < 0.0:
             raise SpecError("arch spec error: the number added to the chosen scores' sum cannot be negative")
+        act = p.get("activation", "gated_swish")
+        if act not in ops.EXPERT_ACTIVATIONS:
+            raise SpecError(f"arch spec error: unknown expert activation {act!r}")
+        self.act, self.gated = ops.EXPERT_ACTIVATIONS[act], act == "gated_swish"
+        groups = p.get("groups")
+        self.groups = (int(groups["count"]), int(groups["keep"])) if groups else None
+        outputs = self.n_experts + self.n_identity
+        if self.groups:
+            count, keep = self.groups
+            if not 0 < keep <= count or outputs % count != 0 or int(p["top"]) > keep * (outputs // count):
+                raise SpecError(f"arch spec error: {p['top']} of the best {keep} of {count} groups of {outputs} experts")
         shared = p.get("shared")
         self.shared = part_impl("feed_forward", shared.kind)(shared, rt) if shared is not None else None
         if self.n_experts < 0 or self.n_identity < 0 or not 0 < self.top <= self.n_experts + self.n_identity:
@@ -60,8 +73,9 @@ class RoutedExperts(FeedForward):
             out.append(WeightSpec(w["correction"], (self.n_experts + self.n_identity,), "vector", 0.05))
         for e in range(self.n_experts):
             base = w["expert"].format(e)
-            out += [WeightSpec(base + w["gate"], (self.inner, self.width), "matrix", 0.05),
-                    WeightSpec(base + w["up"], (self.inner, self.width), "matrix", 0.05),
+            if self.gated:
+                out.append(WeightSpec(base + w["gate"], (self.inner, self.width), "matrix", 0.05))
+            out += [WeightSpec(base + w["up"], (self.inner, self.width), "matrix", 0.05),
                     WeightSpec(base + w["down"], (self.width, self.inner), "matrix", 0.05)]
         if self.shared is not None:
             out += self.shared.weight_specs()
@@ -75,12 +89,14 @@ class RoutedExperts(FeedForward):
         self.correction = self._vector32(tensors[w["correction"]]) if self.has_correction else None
         dev = self.router.device
         dt = torch.float32 if self.rt.is_fp32 else torch.bfloat16
-        self.w_gate_up = torch.empty((max(1, self.n_experts), 2 * self.inner, self.width), dtype=dt, device=dev)
+        ways = 2 if self.gated else 1                      # gate rows, then up rows; without a gate the up rows alone
+        self.w_gate_up = torch.empty((max(1, self.n_experts), ways * self.inner, self.width), dtype=dt, device=dev)
         self.w_down = torch.empty((max(1, self.n_experts), self.width, self.inner), dtype=dt, device=dev)
         for e in range(self.n_experts):
             base = w["expert"].format(e)
-            self.w_gate_up[e, : self.inner] = tensors[base + w["gate"]]
-            self.w_gate_up[e, self.inner:] = tensors[base + w["up"]]
+            if self.gated:
+                self.w_gate_up[e, : self.inner] = tensors[base + w["gate"]]
+            self.w_gate_up[e, (ways - 1) * self.inner:] = tensors[base + w["up"]]
             self.w_down[e] = tensors[base + w["down"]]
 
     def forward(self, h: torch.Tensor, step: StepInfo = None) -> torch.Tensor:
@@ -90,7 +106,7 @@ class RoutedExperts(FeedForward):
         choice = torch.empty(pairs, dtype=torch.int32, device=dev)
         weight = torch.empty(pairs, dtype=torch.float32, device=dev)
         ops.moe_route(h, self.router, self.correction, step.token_seq, choice, weight, top, self.scoring,
-                      self.renormalise, self.weight_scale)
+                      self.renormalise, self.weight_scale, self.groups)
         out = torch.empty((n, self.width), dtype=torch.float32, device=dev)
         pair_out = None
         if self.n_experts > 0:
@@ -100,7 +116,7 @@ class RoutedExperts(FeedForward):
                 # a handful of pairs: a block per pair and slice of the features, no lists, no tiles
                 y = torch.empty((pairs, self.inner), dtype=h.dtype, device=dev)
                 done = ops.moe_few(h, self.w_gate_up, self.w_down, choice, weight, y, pair_out, top, self.n_experts,
-                                   self.limit, self.alpha, self.up_shift, self.weight_on_input)
+                                   self.limit, self.alpha, self.up_shift, self.weight_on_input, self.act)
             if not done:
                 # every expert's list is padded to whole tiles: at most this many tiles whatever the router chooses
                 max_tiles = min(pairs, self.n_experts) + pairs // tile
@@ -109,7 +125,7 @@ class RoutedExperts(FeedForward):
                 ops.moe_align(choice, self.n_experts, listed, tile_expert)
                 y = torch.empty((max_tiles * tile, self.inner), dtype=h.dtype, device=dev)
                 ops.moe_gate_up(h, self.w_gate_up, listed, tile_expert, y, top, self.limit, self.alpha, self.up_shift,
-                                weight if self.weight_on_input else None)
+                                weight if self.weight_on_input else None, self.act)
                 ops.moe_down(y, self.w_down, listed, tile_expert, None if self.weight_on_input else weight, pair_out)
         extra = self.shared.forward(h, step) if self.shared is not None else None
         ops.moe_combine(pair_out, choice, weight, h, out, top, self.n_experts, extra)

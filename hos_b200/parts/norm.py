@@ -50,7 +50,7 @@ class RMSNorm(Norm):
     accepts_partials = True      # y may be [parts, N, width] float32 partial sums
 
     def add_to(self, y: torch.Tensor, x: torch.Tensor, then: Optional[Norm] = None):
-        """x += self(y); with another RMSNorm as `then`, its output comes from the same kernel."""
+        """x += self(y); with another RMSNorm (or x itself, RowsAsGiven) as `then`, its output comes from the same kernel."""
         if then is None:
             ops.norm_add_norm(y, self.weight, self.eps, self.add_one, x)
             return None
@@ -58,6 +58,10 @@ class RMSNorm(Norm):
             h = torch.empty(x.shape, dtype=self.rt.dtype, device=x.device)
             ops.norm_add_norm(y, self.weight, self.eps, self.add_one, x,
                               then.weight, then.eps, then.add_one, h)
+            return h
+        if isinstance(then, RowsAsGiven) and not self.rt.is_fp32:
+            h = torch.empty(x.shape, dtype=self.rt.dtype, device=x.device)
+            ops.norm_add_norm(y, self.weight, self.eps, self.add_one, x, h=h)
             return h
         ops.norm_add_norm(y, self.weight, self.eps, self.add_one, x)
         return then.forward(x)

@@ -9,7 +9,10 @@ With `scaling` (factor, original, fast, slow: the ramp between scaled and unscal
 extends a trained context) pair i turns at f_i / factor * ramp_i + f_i * (1 - ramp_i), where, with
 turns(t) = rotary_dim * ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(turns(fast)), 0),
 hi = min(ceil(turns(slow)), rotary_dim - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1);
-cosine and sine are then multiplied by `magnitude` = 0.1 ln(factor) + 1.  `table: "float64"` takes the
+cosine and sine are then multiplied by `magnitude` = 0.1 ln(factor) + 1.  With `scaling` of kind "bands" (factor, low, high, original: the rule that Llama 3.1 made common) the frequencies whose
+wavelength 2 pi / f is shorter than original / high stay, those whose wavelength is longer than original / low are divided by
+the factor, and between the two f becomes (1 - s) f / factor + s f with s = (original / wavelength - low) / (high - low);
+cosine and sine are not multiplied.  `table: "float64"` takes the
 frequencies in 64-bit before they are rounded to 32-bit.
 
 A position encoding is used by a mixer: the mixer asks it for `kernel_args()` and
@@ -42,6 +45,25 @@ def _ramped(freqs, dims: int, theta: float, sc) -> list:
     return out
 
 
+def _banded(freqs, sc) -> list:
+    """The frequencies under the rule of bands (see the module's text)."""
+    factor, low, high, original = (float(sc[k]) for k in _SCALINGS["bands"])
+    out = []
+    for f in freqs:
+        turns = original * f / (2.0 * math.pi)         # original / wavelength
+        if turns > high:
+            out.append(f)
+        elif turns < low:
+            out.append(f / factor)
+        else:
+            s = (turns - low) / (high - low) if high > low else 1.0
+            out.append((1.0 - s) * f / factor + s * f)
+    return out
+
+
+_SCALINGS = {"ramp": ("factor", "original", "fast", "slow"), "bands": ("factor", "low", "high", "original")}
+
+
 class Rotary(Part):
     graph_safe = True
 
@@ -58,19 +80,25 @@ class Rotary(Part):
         scaling = spec.params.get("scaling")
         self.magnitude = 1.0            # a factor on cosine and sine (kernels that know no scaling take it as 1)
         if scaling:
-            for k in ("factor", "original", "fast", "slow"):
+            kind = scaling.get("kind", "ramp")
+            if kind not in _SCALINGS:
+                raise SpecError(f"arch spec error: unknown rotary scaling {kind!r}")
+            for k in _SCALINGS[kind]:
                 if k not in scaling:
                     raise SpecError(f"arch spec error: rotary scaling needs {k!r}")
-            self.magnitude = 0.1 * math.log(float(scaling["factor"])) + 1.0
+            if kind == "bands" and float(scaling["high"]) < float(scaling["low"]):
+                raise SpecError("arch spec error: rotary scaling needs high at or above low")
+            if kind == "ramp":
+                self.magnitude = 0.1 * math.log(float(scaling["factor"])) + 1.0
         in64 = bool(scaling) or spec.params.get("table") == "float64"
         key = (str(rt.device), self.theta, self.rotary_dim, in64,
-               tuple(sorted((k, float(v)) for k, v in scaling.items())) if scaling else None)
+               (kind,) + tuple(float(scaling[k]) for k in _SCALINGS[kind]) if scaling else None)
         if key not in _shared:          # layers with the same frequencies share one tensor (and what is derived from it)
             half = self.rotary_dim // 2
             if in64:
                 freqs = [self.theta ** (-2.0 * i / self.rotary_dim) for i in range(half)]
                 if scaling:
-                    freqs = _ramped(freqs, self.rotary_dim, self.theta, scaling)
+                    freqs = (_ramped(freqs, self.rotary_dim, self.theta, scaling) if kind == "ramp" else _banded(freqs, scaling))
                 _shared[key] = torch.tensor(freqs, dtype=torch.float64).to(torch.float32).to(rt.device).contiguous()
             else:
                 i = torch.arange(half, dtype=torch.float32)
