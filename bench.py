@@ -12,7 +12,7 @@ back to the host, where the loop reads them one step late.  `prefill` is one pro
 step must read (every weight once, and the cache of the live sequences) to its time.
 `points` holds decoding at batch 1 and 64.  One JSON line is printed.
 
-`--design satapel` (or `vagonex`, `fobilorn`, `tofodra`, `ravutar`) is another measurement (not the line above): prompt and decode throughput of that design at
+`--design satapel` (or `vagonex`, `fobilorn`, `tofodra`, `ravutar`, `nuvivik`) is another measurement (not the line above): prompt and decode throughput of that design at
 a few sizes beside Gemma-2 at equal size, and each of the design's kernels against its roofline; one JSON line per size.
 With `--profile prefill|decode` it measures nothing and runs two such steps of one block of layers kernel by kernel, for a profiler.
 
@@ -673,6 +673,98 @@ def _vagonex_work_like_ravutar(z, tokens, batch, ctx):
     }
 
 
+# ---- --design nuvivik: the Nuvivik design beside Tofodra at equal size -----------------------------------
+# Layers (latent attention with a dense feed-forward, grouped-query attention with routed experts, latent attention with a
+# dense feed-forward, latent attention with routed experts) x blocks.  The closest existing model is Tofodra (latent
+# attention, attention through the same grouped-query kernels over a window, dense and routed feed-forwards, a norm on each
+# branch's output): "Tofodra at equal size" has the same width, layer count and vocabulary, latent attention of the same
+# heads and latent (its queries straight from the layer's input, every earlier key in sight: the format knows no window
+# there), two-map attention of as many heads over key rows of the same length and the same window where Nuvivik has grouped
+# queries, and gated feed-forwards and experts of as many weights (two thirds as wide).
+NUVIVIK_SIZES = {
+    "s": dict(width=1024, vocab=32000, blocks=2, lat_heads=8, lat_dim=64, lat_rot=32, lat_vdim=64, q_rank=384, rank=256,
+              lat_window=1024, heads=8, kv_heads=2, dim=128, vdim=128, rot=64, window=1024, dense_ff=4096, experts=16, groups=4,
+              keep=2, top=2, ff=1536),
+    "m": dict(width=2048, vocab=32000, blocks=2, lat_heads=16, lat_dim=64, lat_rot=64, lat_vdim=128, q_rank=768, rank=512,
+              lat_window=1024, heads=16, kv_heads=4, dim=128, vdim=128, rot=64, window=1024, dense_ff=8192, experts=16, groups=4,
+              keep=2, top=2, ff=2304),
+    "l": dict(width=4096, vocab=64000, blocks=1, lat_heads=32, lat_dim=64, lat_rot=64, lat_vdim=128, q_rank=1536, rank=512,
+              lat_window=2048, heads=32, kv_heads=8, dim=128, vdim=128, rot=64, window=2048, dense_ff=14400, experts=32, groups=8,
+              keep=4, top=4, ff=1536),
+}
+
+
+def nuvivik_raw(z):
+    dense = {"kind": "dense", "ff": z["dense_ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"]},
+           "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": z["groups"], "keep": z["keep"]}}}
+    lat = {"heads": z["lat_heads"], "dim": z["lat_dim"], "rot_dim": z["lat_rot"], "vdim": z["lat_vdim"], "q_rank": z["q_rank"],
+           "kv_rank": z["rank"], "scale": (z["lat_dim"] + z["lat_rot"]) ** -0.5, "mask": {"size": z["lat_window"]},
+           "rot": {"base": 10000.0, "dims": z["lat_rot"]}}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5,
+           "softcap": 30.0, "mask": {"size": z["window"]},
+           "rot": {"base": 500000.0, "dims": z["rot"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    lat_layer, att_layer = {"type": "latent_attention", "mixer": lat}, {"type": "attention", "mixer": att}
+    layers = [dict(lat_layer, mlp=dense), dict(att_layer, mlp=moe), dict(lat_layer, mlp=dense), dict(lat_layer, mlp=moe)] * z["blocks"]
+    return {"architecture": "Nuvivik", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+            "embedding": {"scale": float(z["width"]) ** 0.5}, "logit_scale": 1.0, "logit_softcap": 30.0, "layers": layers}
+
+
+def _tofodra_sizes_like_nuvivik(z):
+    return dict(z, ret_heads=1, ret_dim=1, ret_vdim=1, dim=z["dim"] // 2, keep=0, dense_ff=z["dense_ff"] * 2 // 3, ff=z["ff"] * 2 // 3)
+
+
+def tofodra_raw_like_nuvivik(z):
+    t = _tofodra_sizes_like_nuvivik(z)
+    raw = tofodra_raw(dict(t, blocks=1, shared=64))
+    for layer in raw["layers"]:
+        if layer["mlp"]["kind"] == "moe":
+            layer["mlp"].pop("shared", None)
+    lat, _, att, _ = raw["layers"]
+    dense, moe = lat["mlp"], raw["layers"][1]["mlp"]
+    return dict(raw, layers=[lat, dict(att, mlp=moe), dict(lat, mlp=dense), dict(lat, mlp=moe)] * z["blocks"])
+
+
+def nuvivik_kernel_work(z, tokens, batch, ctx):
+    """Per launch of each of the design's kernels: (bytes that must move, FLOPs of the mathematics) for a prompt of `tokens`
+    tokens and for a decode step of `batch` sequences at length `ctx` (bfloat16 cache and products, 32-bit rows)."""
+    LH, R, P, rq = z["lat_heads"], z["rank"], z["lat_rot"], z["q_rank"]
+    D, LW = R + P, z["lat_window"]
+    H, G, kd, vd, W = z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["window"]
+    lat_pairs, pairs = (sum(min(p + 1, w) for p in range(tokens)) for w in (LW, W))
+    lat_keys, keys = min(ctx, LW), min(ctx, W)
+    top, ff, width, E = z["top"], z["ff"], z["width"], z["experts"]
+    touched = min(E, batch * top)
+    attn = {"prefill": (tokens * G * (kd + vd) * 2 + tokens * H * (kd * 4 + vd * 2), 2.0 * pairs * H * (kd + vd)),
+            "decode": (batch * keys * G * (kd + vd) * 2, 2.0 * batch * keys * H * (kd + vd))}
+    expert = {"prefill": (E * ff * width * 2, 2.0 * tokens * top * ff * width),
+              "decode": (touched * ff * width * 2, 2.0 * batch * top * ff * width)}
+    few = {"prefill": (0, 0.0), "decode": expert["decode"]}
+    per_head = LH * R * (z["lat_dim"] + z["lat_vdim"])               # both per-head products' weights; a launch is half of it
+    return {
+        "hos_latent_attn": {"prefill": (tokens * D * 2 + tokens * LH * (D * 4 + R * 2), 2.0 * lat_pairs * LH * (D + R)),
+                            "decode": (batch * lat_keys * D * 2, 2.0 * batch * lat_keys * LH * (D + R))},
+        "hos_heads_product": {"prefill": (0, 2.0 * tokens * per_head / 2), "decode": (per_head * 2 / 2, 2.0 * batch * per_head / 2)},
+        # two launches a layer: latents in and out (and to the cache), rotated query parts in and out; the mean of the two
+        "hos_latent_prep": _both(lambda n, q: (n * ((rq + D) * 2 + (rq + 2 * D) * 2 + LH * P * 6) / 2, 0.0), tokens, batch),
+        "hos_gated_attn": attn, "hos_gated_attn_mma": attn, "hos_gated_attn_mma_decode": attn,
+        "hos_qk_prep": _both(lambda n, q: (n * (H * kd * 8 + G * (kd + vd) * 6), 0.0), tokens, batch),
+        # x in and out (32-bit), the branch's output in, the rows in the products' type out
+        "hos_norm_add_norm": _both(lambda n, q: (n * width * 12, 0.0), tokens, batch),
+        "hos_moe_route": _both(lambda n, q: (n * width * 2 + E * width * 4, 0.0), tokens, batch),
+        "hos_moe_gate_up": expert, "hos_moe_down": expert, "hos_moe_gate_up_few": few, "hos_moe_down_few": few,
+        "hos_moe_combine": _both(lambda n, q: (n * width * (4 * top + 4), 0.0), tokens, batch),
+    }
+
+
+def _tofodra_work_like_nuvivik(z, tokens, batch, ctx):
+    t = _tofodra_sizes_like_nuvivik(z)
+    LH, D, P = t["lat_heads"], t["rank"] + t["lat_rot"], t["lat_rot"]
+    return dict(tofodra_kernel_work(t, tokens, batch, ctx),
+                hos_latent_prep=_both(lambda n, q: (n * (D * 2 + 2 * D * 2 + LH * P * 6), 0.0), tokens, batch),
+                hos_moe_route=_both(lambda n, q: (n * z["width"] * 2 + z["experts"] * z["width"] * 4, 0.0), tokens, batch))
+
+
 DESIGNS = {"fobilorn": lambda: (FOBILORN_SIZES, fobilorn_raw, gemma_raw_like_fobilorn, fobilorn_kernel_work,
                                 ("hos_gated_attn",)),
            "satapel": lambda: (SATAPEL_SIZES, satapel_raw, gemma_raw_like, satapel_kernel_work, ("hos_wkv_scan",)),
@@ -682,7 +774,8 @@ DESIGNS = {"fobilorn": lambda: (FOBILORN_SIZES, fobilorn_raw, gemma_raw_like_fob
                                ("hos_state_scan", "hos_gated_attn")),
            "ravutar": lambda: (RAVUTAR_SIZES, ravutar_raw, vagonex_raw_like_ravutar, ravutar_kernel_work,
                                ("hos_state_scan", "hos_state_scan/channel", "hos_state_scan/v_factor", "hos_gated_attn",
-                                "hos_channel_decay"))}
+                                "hos_channel_decay")),
+           "nuvivik": lambda: (NUVIVIK_SIZES, nuvivik_raw, tofodra_raw_like_nuvivik, nuvivik_kernel_work, ("hos_gated_attn",))}
 
 
 def _vagonex_work_like_tofodra(z, tokens, batch, ctx):
@@ -704,8 +797,8 @@ def _vagonex_work_like_tofodra(z, tokens, batch, ctx):
             "hos_scale_add_norm": {"prefill": (tokens * z["width"] * 12, 0.0), "decode": (batch * z["width"] * 12, 0.0)}}
 
 
-OTHER_WORK = {"tofodra": _vagonex_work_like_tofodra, "ravutar": _vagonex_work_like_ravutar}
-OTHER_ARM = {"tofodra": "vagonex_equal_size", "ravutar": "vagonex_equal_size"}      # the closest existing model per design (Gemma-2 where none is named)
+OTHER_WORK = {"tofodra": _vagonex_work_like_tofodra, "ravutar": _vagonex_work_like_ravutar, "nuvivik": _tofodra_work_like_nuvivik}
+OTHER_ARM = {"tofodra": "vagonex_equal_size", "ravutar": "vagonex_equal_size", "nuvivik": "tofodra_equal_size"}      # the closest existing model per design (Gemma-2 where none is named)
 
 
 def run_design_profile_step(args) -> int:

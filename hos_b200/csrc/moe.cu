@@ -50,14 +50,15 @@ __device__ __forceinline__ float expert_act(float g, float u, float limit, float
 }
 
 // One warp: the outputs outside the `keep` best of `groups` equal groups are marked as taken.  gs: [groups] in shared memory;
-// score(e) is what the groups are judged by.  Equal groups: the first wins.
-template <typename Score>
-__device__ __forceinline__ void route_groups(Score score, float* taken, float* gs, int n_out, int groups, int keep, int lane) {
+// value(e) is what the outputs are ordered by, sum(a, b) a group's standing by its two largest values.  Equal groups: the
+// first wins.
+template <typename Value, typename Sum>
+__device__ __forceinline__ void route_groups(Value value, Sum sum, float* taken, float* gs, int n_out, int groups, int keep, int lane) {
     const int size = n_out / groups;
     for (int g = lane; g < groups; g += 32) {
         float a = -INFINITY, b = -INFINITY;
         for (int i = 0; i < size; ++i) {
-            const float c = score(g * size + i);
+            const float c = value(g * size + i);
             if (c > a) {
                 b = a;
                 a = c;
@@ -65,7 +66,7 @@ __device__ __forceinline__ void route_groups(Score score, float* taken, float* g
                 b = c;
             }
         }
-        gs[g] = size > 1 ? a + b : a;
+        gs[g] = sum(a, b);
     }
     for (int e = lane; e < n_out; e += 32) taken[e] = 1.f;
     __syncwarp();
@@ -73,7 +74,7 @@ __device__ __forceinline__ void route_groups(Score score, float* taken, float* g
         float best = -INFINITY;
         int arg = 0x7fffffff;
         for (int g = lane; g < groups; g += 32)
-            if (gs[g] > best || (gs[g] == best && gs[g] != -INFINITY && g < arg)) {
+            if (gs[g] > best || (gs[g] == best && best != -INFINITY && g < arg)) {
                 best = gs[g];
                 arg = g;
             }
@@ -127,8 +128,18 @@ __device__ __forceinline__ void route_choose(float* z, float* taken, const float
     }
     __syncwarp();
     if (groups > 0) {
-        route_groups([&](int e) { return (by_logit ? 1.f / (1.f + expf(-z[e])) : z[e]) + (correction ? correction[e] : 0.f); }, taken,
-                     gs, n_out, groups, keep, lane);
+        // By logits (b is -inf where a group has one output): S = s(a) + s(b) orders the groups; where it is above 1 the
+        // order is told by L = 2 - S = s(-a) + s(-b), which keeps its digits where both scores round to 1.  1 / L
+        // continues S upwards from 1.
+        auto by_logits = [](float a, float b) {
+            if (b == -INFINITY) return a;
+            const float sum = 1.f / (1.f + expf(-a)) + 1.f / (1.f + expf(-b));
+            return sum <= 1.f ? sum : 1.f / (1.f / (1.f + expf(a)) + 1.f / (1.f + expf(b)));
+        };
+        if (by_logit) route_groups([&](int e) { return z[e]; }, by_logits, taken, gs, n_out, groups, keep, lane);
+        else
+            route_groups([&](int e) { return z[e] + (correction ? correction[e] : 0.f); },
+                         [](float a, float b) { return b == -INFINITY ? a : a + b; }, taken, gs, n_out, groups, keep, lane);
         __syncwarp();
     }
     for (int k = 0; k < top; ++k) {
