@@ -711,7 +711,8 @@ def nuvivik_raw(z):
 
 
 def _tofodra_sizes_like_nuvivik(z):
-    return dict(z, ret_heads=1, ret_dim=1, ret_vdim=1, dim=z["dim"] // 2, keep=0, dense_ff=z["dense_ff"] * 2 // 3, ff=z["ff"] * 2 // 3)
+    return dict(z, ret_heads=1, ret_dim=1, ret_vdim=1, dim=z["dim"] // 2, keep=0, dense_ff=z["dense_ff"] * 2 // 3 // 64 * 64,
+                ff=z["ff"] * 2 // 3 // 64 * 64)
 
 
 def tofodra_raw_like_nuvivik(z):
@@ -728,8 +729,8 @@ def tofodra_raw_like_nuvivik(z):
 def nuvivik_kernel_work(z, tokens, batch, ctx):
     """Per launch of each of the design's kernels: (bytes that must move, FLOPs of the mathematics) for a prompt of `tokens`
     tokens and for a decode step of `batch` sequences at length `ctx` (bfloat16 cache and products, 32-bit rows)."""
-    LH, R, P, rq = z["lat_heads"], z["rank"], z["lat_rot"], z["q_rank"]
-    D, LW = R + P, z["lat_window"]
+    LH, R, rq = z["lat_heads"], z["rank"], z["q_rank"]
+    D, LW = R + z["lat_rot"], z["lat_window"]
     H, G, kd, vd, W = z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["window"]
     lat_pairs, pairs = (sum(min(p + 1, w) for p in range(tokens)) for w in (LW, W))
     lat_keys, keys = min(ctx, LW), min(ctx, W)
@@ -745,8 +746,8 @@ def nuvivik_kernel_work(z, tokens, batch, ctx):
         "hos_latent_attn": {"prefill": (tokens * D * 2 + tokens * LH * (D * 4 + R * 2), 2.0 * lat_pairs * LH * (D + R)),
                             "decode": (batch * lat_keys * D * 2, 2.0 * batch * lat_keys * LH * (D + R))},
         "hos_heads_product": {"prefill": (0, 2.0 * tokens * per_head / 2), "decode": (per_head * 2 / 2, 2.0 * batch * per_head / 2)},
-        # two launches a layer: latents in and out (and to the cache), rotated query parts in and out; the mean of the two
-        "hos_latent_prep": _both(lambda n, q: (n * ((rq + D) * 2 + (rq + 2 * D) * 2 + LH * P * 6) / 2, 0.0), tokens, batch),
+        # both latents and the key part in and out, and to the cache
+        "hos_latent_prep": _both(lambda n, q: (n * (2 * rq + 3 * D) * 2, 0.0), tokens, batch),
         "hos_gated_attn": attn, "hos_gated_attn_mma": attn, "hos_gated_attn_mma_decode": attn,
         "hos_qk_prep": _both(lambda n, q: (n * (H * kd * 8 + G * (kd + vd) * 6), 0.0), tokens, batch),
         # x in and out (32-bit), the branch's output in, the rows in the products' type out
@@ -759,9 +760,9 @@ def nuvivik_kernel_work(z, tokens, batch, ctx):
 
 def _tofodra_work_like_nuvivik(z, tokens, batch, ctx):
     t = _tofodra_sizes_like_nuvivik(z)
-    LH, D, P = t["lat_heads"], t["rank"] + t["lat_rot"], t["lat_rot"]
+    D = t["rank"] + t["lat_rot"]
     return dict(tofodra_kernel_work(t, tokens, batch, ctx),
-                hos_latent_prep=_both(lambda n, q: (n * (D * 2 + 2 * D * 2 + LH * P * 6), 0.0), tokens, batch),
+                hos_latent_prep=_both(lambda n, q: (n * 3 * D * 2, 0.0), tokens, batch),
                 hos_moe_route=_both(lambda n, q: (n * z["width"] * 2 + z["experts"] * z["width"] * 4, 0.0), tokens, batch))
 
 

@@ -14,7 +14,7 @@
 // sink: a learned number per head that joins the softmax's denominator as exp(sink), without a key
 // or a value and unscaled.
 //
-// Kernels: latent_prep (norms of c and of the queries' own latent, rotations, cache write), latent_attn and latent_attn_tc (keys from
+// Kernels: latent_prep (norms of c and of the queries' own latent, the key part's rotation, cache write), latent_attn and latent_attn_tc (keys from
 // the step's own rows for sequences that start at position 0, or from the paged cache), latent_merge
 // (the shares of a row's keys put together), heads_product and heads_product_tc (the per-head products
 // W_uk_h^T q_h and W_uv_h o_h as one launch over all heads).
@@ -24,35 +24,56 @@
 
 namespace hos {
 
+// ---- rotary pairs ----------------------------------------------------------------------------
+// The first rot_dims of P numbers are rotated, angle = position * inv_freq[i]; style 0 pairs (i, i + rot_dims / 2), style 1
+// pairs (2i, 2i + 1).
+struct LatentRot {
+    const float* inv_freq;
+    int rot_dims, style;
+};
+
+// number j of the rotated part `src`; tab: (sin, cos) per pair
+template <typename T>
+__device__ __forceinline__ float rotated(const T* __restrict__ src, int j, const float2* tab, const LatentRot& r) {
+    if (j >= r.rot_dims) return to_float(src[j]);
+    const int half = r.rot_dims >> 1;
+    const bool second = r.style == 0 ? j >= half : (j & 1) != 0;
+    const int i = r.style == 0 ? (second ? j - half : j) : j >> 1;
+    const float2 sc = tab[i];
+    const float u = to_float(src[r.style == 0 ? i : 2 * i]), v = to_float(src[r.style == 0 ? i + half : 2 * i + 1]);
+    return second ? v * sc.y + u * sc.x : u * sc.y - v * sc.x;
+}
+
+// The heads' queries as projected: row n, head h at p + n * stride + h * (dq + P), its last P numbers are the rotated part.
+template <typename T>
+struct LatentQuery {
+    const T* p;
+    long long stride;
+    int dq;
+    LatentRot rot;
+};
+
 // ---- latent_prep ---------------------------------------------------------------------------
-// What lies between the projections and the attention, for whichever of the three parts are given:
-//   down[n] = [ c_raw: R | key_rot_raw: P ]      -> kc[n] = [ rms(c_raw) * w_norm | rot(key_rot_raw) ], the row the cache
-//                                                   keeps, also stored at the token's place in the paged cache (rows of
-//                                                   R + P, not permuted)
-//   q[n]    = H heads of [ dq | P ]              -> q_lat[n][h][R : R + P] = rot(q_h[dq : dq + P])          (32-bit)
-//   cq[n]   = the queries' own latent, Rq numbers -> cq_out[n] = rms(cq) * cq_norm, what the queries' up projection reads
-// A call without a part passes null for it (a call that reads another call's cache: no `down`; queries that come straight
-// from the layer's input: no `cq`; queries that are not there yet because they wait for cq_out: no `q`).
-// Rotation: the first rot_dims of the P numbers, angle = position * inv_freq[i]; style 0 pairs (i, i + rot_dims / 2),
-// style 1 pairs (2i, 2i + 1).
+// What lies between the down projections and what reads their latents, for either or both of the two:
+//   down[n] = [ c_raw: R | key_rot_raw: P ]       -> kc[n] = [ rms(c_raw) * w_norm | rot(key_rot_raw) ], the row the cache
+//                                                    keeps, also stored at the token's place in the paged cache (rows of
+//                                                    R + P, not permuted)
+//   cq[n]   = the queries' own latent, Rq numbers  -> cq_out[n] = rms(cq) * cq_norm, what the queries' up projection reads
 template <typename T>
 struct LatentPrep {
-    const T* q;
     const T* down;
     const T* cq;
-    int q_stride, down_stride, cq_stride;
-    int H, dq, R, P, Rq;
+    int down_stride, cq_stride;
+    int R, P, Rq;
     const float* w_norm;
     const float* cq_norm;
     float eps;
-    const float* inv_freq;
-    int rot_dims, style;
+    LatentRot rot;
     const int* token_pos;
     const int* token_seq;
     const int* seq_slot;
     const int* seq_len_after;
     T* kc;
-    float* q_lat;
     T* cq_out;
     T* k_pages;
     const int* page_table;
@@ -67,7 +88,7 @@ __global__ void latent_prep_kernel(LatentPrep<T> a) {
     const int n = blockIdx.x;
     const int seq = a.token_seq[n];
     if (seq < 0) return;
-    const int pos = a.token_pos[n], R = a.R, P = a.P, D = R + P, half = a.rot_dims >> 1;
+    const int pos = a.token_pos[n], R = a.R, P = a.P, D = R + P, half = a.rot.rot_dims >> 1;
     const bool keys = a.down != nullptr;
     int page = -1;
     if (a.k_pages != nullptr && !(a.ring_pages > 0 && pos + a.ring_pages * kPageTokens < a.seq_len_after[seq])) {
@@ -76,69 +97,35 @@ __global__ void latent_prep_kernel(LatentPrep<T> a) {
     }
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float s, c;
-        sincosf((float)pos * a.inv_freq[i], &s, &c);
+        sincosf((float)pos * a.rot.inv_freq[i], &s, &c);
         sincos_tab[i] = make_float2(s, c);
     }
     const T* craw = keys ? a.down + (size_t)n * a.down_stride : nullptr;
-    float ss = 0.f;
+    float ss = 0.f, sq = 0.f;
     if (keys)
         for (int d = threadIdx.x; d < R; d += blockDim.x) {
             const float v = to_float(craw[d]);
             ss = fmaf(v, v, ss);
         }
-    const float rinv = rsqrtf(block_sum(ss, scratch) / (float)R + a.eps);      // (also orders sincos_tab)
-    T* out = keys ? a.kc + (size_t)n * D : nullptr;
-    T* cached = keys && page >= 0 ? a.k_pages + ((size_t)page * kPageTokens + pos % kPageTokens) * D : nullptr;
-    if (keys)
-        for (int d = threadIdx.x; d < R; d += blockDim.x) {
-            const T v = from_float<T>(to_float(craw[d]) * rinv * a.w_norm[d]);
-            out[d] = v;
-            if (cached) cached[d] = v;
-        }
-    if (a.cq != nullptr) {
-        const T* src = a.cq + (size_t)n * a.cq_stride;
-        float sq = 0.f;
+    const T* cq = a.cq != nullptr ? a.cq + (size_t)n * a.cq_stride : nullptr;
+    if (cq)
         for (int d = threadIdx.x; d < a.Rq; d += blockDim.x) {
-            const float v = to_float(src[d]);
+            const float v = to_float(cq[d]);
             sq = fmaf(v, v, sq);
         }
+    if (cq) {
         const float qinv = rsqrtf(block_sum(sq, scratch) / (float)a.Rq + a.eps);
         for (int d = threadIdx.x; d < a.Rq; d += blockDim.x)
-            a.cq_out[(size_t)n * a.Rq + d] = from_float<T>(to_float(src[d]) * qinv * a.cq_norm[d]);
+            a.cq_out[(size_t)n * a.Rq + d] = from_float<T>(to_float(cq[d]) * qinv * a.cq_norm[d]);
     }
-    // the shared rotated key part and every head's rotated query part: items of one pair (or one unrotated number
-    // beyond rot_dims); item group 0 is the key if there is one
-    const int per = half + (P - a.rot_dims), first = keys ? 1 : 0;
-    for (int it = threadIdx.x; it < ((a.q != nullptr ? a.H : 0) + first) * per; it += blockDim.x) {
-        const int who = it / per - first, j = it - (it / per) * per;       // who == -1: the key
-        const T* src = who < 0 ? craw + R : a.q + (size_t)n * a.q_stride + (size_t)who * (a.dq + P) + a.dq;
-        float x, y = 0.f;
-        int d0, d1 = 0;
-        const bool pair = j < half;
-        if (pair) {
-            d0 = a.style == 0 ? j : 2 * j;
-            d1 = a.style == 0 ? j + half : 2 * j + 1;
-            const float2 sc = sincos_tab[j];
-            const float u = to_float(src[d0]), v = to_float(src[d1]);
-            x = u * sc.y - v * sc.x;
-            y = v * sc.y + u * sc.x;
-        } else {
-            d0 = a.rot_dims + (j - half);
-            x = to_float(src[d0]);
-        }
-        if (who < 0) {
-            const T tx = from_float<T>(x), ty = from_float<T>(y);
-            out[R + d0] = tx;
-            if (cached) cached[R + d0] = tx;
-            if (pair) {
-                out[R + d1] = ty;
-                if (cached) cached[R + d1] = ty;
-            }
-        } else {
-            float* q = a.q_lat + ((size_t)n * a.H + who) * D + R;
-            q[d0] = x;
-            if (pair) q[d1] = y;
-        }
+    if (!keys) return;
+    const float rinv = rsqrtf(block_sum(ss, scratch) / (float)R + a.eps);      // (also orders sincos_tab)
+    T* out = a.kc + (size_t)n * D;
+    T* cached = page >= 0 ? a.k_pages + ((size_t)page * kPageTokens + pos % kPageTokens) * D : nullptr;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+        const T v = from_float<T>(d < R ? to_float(craw[d]) * rinv * a.w_norm[d] : rotated(craw + R, d - R, sincos_tab, a.rot));
+        out[d] = v;
+        if (cached) cached[d] = v;
     }
 }
 
@@ -153,7 +140,7 @@ constexpr int kHG = 8, kTK = 32, kAttnThreads = 256;
 
 template <typename T, bool PAGED, int NC, int QT>
 __global__ void __launch_bounds__(kAttnThreads)
-latent_attn_kernel(const float* __restrict__ q_lat, const T* __restrict__ kc, const T* __restrict__ k_pages,
+latent_attn_kernel(const float* __restrict__ q_lat, const LatentQuery<T> q, const T* __restrict__ kc, const T* __restrict__ k_pages,
                    const int* __restrict__ page_table, int table_stride, int ring_pages,
                    const float* __restrict__ sink, T* __restrict__ o_lat, float* __restrict__ part_acc,
                    float* __restrict__ part_ml, const int* __restrict__ token_pos,
@@ -167,6 +154,8 @@ latent_attn_kernel(const float* __restrict__ q_lat, const T* __restrict__ kc, co
     float* ps = ks + kTK * Dk;                 // [QT][kTK][kHG] weights of the tile
     float* alpha = ps + QT * kTK * kHG;        // [QT][kHG] what the running sums are scaled by
     float* denom = alpha + QT * kHG;           // [QT][kHG]
+    const int half = q.rot.rot_dims >> 1;
+    float2* sincos_tab = reinterpret_cast<float2*>(denom + QT * kHG);       // [QT][half]
     __shared__ int key_row[kTK];               // where each key of the tile lies (-1: none)
     __shared__ int row_seq[QT], row_pos[QT];
     const int n0 = row0 + blockIdx.x * QT, h0 = blockIdx.y * kHG;
@@ -178,10 +167,21 @@ latent_attn_kernel(const float* __restrict__ q_lat, const T* __restrict__ kc, co
         row_seq[tid] = n < row_end ? token_seq[n] : -1;
         row_pos[tid] = n < row_end ? token_pos[n] : 0;
     }
+    for (int i = tid; i < QT * half; i += kAttnThreads) {
+        const int t = i / half, n = n0 + t;
+        float sn = 0.f, cs = 1.f;
+        if (n < row_end) sincosf((float)token_pos[n] * q.rot.inv_freq[i - t * half], &sn, &cs);
+        sincos_tab[i] = make_float2(sn, cs);
+    }
+    __syncthreads();
     for (int i = tid; i < QT * kHG * Dq; i += kAttnThreads) {
         const int t = i / (kHG * Dq), rem = i - t * kHG * Dq, h = rem / Dq, d = rem - h * Dq;
         const int n = n0 + t;
-        qs[i] = (n < row_end && h < nh && d < D) ? q_lat[((size_t)n * H + h0 + h) * D + d] : 0.f;
+        float v = 0.f;
+        if (n < row_end && h < nh && d < D)
+            v = d < R ? q_lat[((size_t)n * H + h0 + h) * R + d]
+                      : rotated(q.p + n * q.stride + (size_t)(h0 + h) * (q.dq + D - R) + q.dq, d - R, sincos_tab + t * half, q.rot);
+        qs[i] = v;
     }
     __syncthreads();
     float m_run[QT], l_run[QT];                // of head `warp`, per row (kept by every lane of the warp)
@@ -382,7 +382,7 @@ latent_attn_kernel(const float* __restrict__ q_lat, const T* __restrict__ kc, co
 // 8-wide column tiles of the latent.
 template <bool PAGED, int NT>
 __global__ void __launch_bounds__(kAttnThreads)
-latent_attn_tc_kernel(const float* __restrict__ q_lat, const bf16* __restrict__ kc, const bf16* __restrict__ k_pages,
+latent_attn_tc_kernel(const float* __restrict__ q_lat, const LatentQuery<bf16> q, const bf16* __restrict__ kc, const bf16* __restrict__ k_pages,
                       const int* __restrict__ page_table, int table_stride, int ring_pages,
                       const float* __restrict__ sink, bf16* __restrict__ o_lat, float* __restrict__ part_acc,
                       float* __restrict__ part_ml, const int* __restrict__ token_pos,
@@ -400,6 +400,8 @@ latent_attn_tc_kernel(const float* __restrict__ q_lat, const bf16* __restrict__ 
     float* Sp = reinterpret_cast<float*>(Pl + 16 * kPs);      // [warps][16][kSs] every warp's share of the scores
     float* alpha = Sp + (kAttnThreads / 32) * 16 * kSs;       // [16]
     float* denom = alpha + 16;                  // [16]
+    const int half = q.rot.rot_dims >> 1;
+    float2* sincos_tab = reinterpret_cast<float2*>(denom + 16);             // [2][half]
     __shared__ int row_seq[2], row_pos[2];
     const int n0 = row0 + blockIdx.x * QT, h0 = blockIdx.y * kHG;
     const int split = blockIdx.z, n_splits = gridDim.z;
@@ -411,9 +413,19 @@ latent_attn_tc_kernel(const float* __restrict__ q_lat, const bf16* __restrict__ 
         row_seq[tid] = in ? token_seq[n] : -1;
         row_pos[tid] = in ? token_pos[n] : 0;
     }
+    for (int i = tid; i < QT * half; i += kAttnThreads) {
+        const int t = i / half, n = n0 + t;
+        float sn = 0.f, cs = 1.f;
+        if (n < row_end) sincosf((float)token_pos[n] * q.rot.inv_freq[i - t * half], &sn, &cs);
+        sincos_tab[i] = make_float2(sn, cs);
+    }
+    __syncthreads();
     for (int i = tid; i < 16 * Ds; i += kAttnThreads) {
         const int row = i / Ds, d = i - row * Ds, t = row >> 3, h = row & 7, n = n0 + t;
-        const float v = (t < QT && n < row_end && h < nh && d < D) ? q_lat[((size_t)n * H + h0 + h) * D + d] : 0.f;
+        float v = 0.f;
+        if (t < QT && n < row_end && h < nh && d < D)
+            v = d < R ? q_lat[((size_t)n * H + h0 + h) * R + d]
+                      : rotated(q.p + n * q.stride + (size_t)(h0 + h) * (q.dq + D - R) + q.dq, d - R, sincos_tab + t * half, q.rot);
         const bf16 hi = __float2bfloat16_rn(v);
         Qh[i] = hi;
         Ql[i] = __float2bfloat16_rn(v - __bfloat162float(hi));
@@ -460,19 +472,19 @@ latent_attn_tc_kernel(const float* __restrict__ q_lat, const bf16* __restrict__ 
         auto issue = [&](int tile, int stage) {
             const int p0 = lo + tile * kTK;
             bf16* dst = Kt + stage * kTK * Ds;
-            for (int x = tid; x < kTK * groups; x += kAttnThreads) {
-                const int j = x / groups, gq = x - j * groups, p = p0 + j;
-                const bool ok = p <= pos_last;
-                size_t r = 0;
-                if (ok) {
-                    if (PAGED) {
-                        const int lp = p / kPageTokens;
-                        r = (size_t)table[ring_pages > 0 ? lp % ring_pages : lp] * kPageTokens + p % kPageTokens;
-                    } else {
-                        r = (size_t)(seq_first + p);
-                    }
+            if constexpr (PAGED) {          // a warp to a row: its place in the cache is looked up once
+                for (int j = warp; j < kTK; j += kAttnThreads / 32) {
+                    const int p = p0 + j, lp = p / kPageTokens;
+                    const bool ok = p <= pos_last;
+                    const size_t r = ok ? (size_t)table[ring_pages > 0 ? lp % ring_pages : lp] * kPageTokens + p % kPageTokens : 0;
+                    for (int gq = lane; gq < groups; gq += 32) cp_async16(dst + j * Ds + gq * 8, base + r * D + gq * 8, ok);
                 }
-                cp_async16(dst + j * Ds + gq * 8, base + r * D + gq * 8, ok);
+            } else {
+                for (int x = tid; x < kTK * groups; x += kAttnThreads) {
+                    const int j = x / groups, gq = x - j * groups, p = p0 + j;
+                    const bool ok = p <= pos_last;
+                    cp_async16(dst + j * Ds + gq * 8, base + (ok ? (size_t)(seq_first + p) : 0) * D + gq * 8, ok);
+                }
             }
         };
         if (tile_lo < tile_hi) issue(tile_lo, 0);
@@ -710,17 +722,17 @@ heads_product_tc_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, 
 }
 
 template <typename T, bool PAGED, int NC, int QT>
-static int launch_attn_as(const float* q_lat, const void* kc, const void* k_pages, const int* page_table, int table_stride,
+static int launch_attn_as(const float* q_lat, const LatentQuery<T>& q, const void* kc, const void* k_pages, const int* page_table, int table_stride,
                           int ring_pages, const float* sink, void* o_lat, float* part_acc, float* part_ml, int n_splits,
                           const int* token_pos, const int* token_seq, const int* cu_seqlens, const int* seq_slot, int row0,
                           int rows, int H, int R, int D, float scale, int window, cudaStream_t stream) {
     const int Dq = (D + 3) / 4 * 4;
     const int Dk = 4 * (((D + 3) / 4) | 1);        // rows of 16-byte groups, an odd number of them: no bank conflicts
-    const size_t smem = (size_t)(QT * kHG * Dq + kTK * Dk + QT * kTK * kHG + 2 * QT * kHG) * sizeof(float);
+    const size_t smem = (size_t)(QT * kHG * Dq + kTK * Dk + QT * kTK * kHG + 2 * QT * kHG + QT * q.rot.rot_dims) * sizeof(float);
     if (smem > 200 * 1024) HOS_REFUSE("latent_attn: rows of %d numbers do not fit a block's shared memory", D);
     auto kernel = latent_attn_kernel<T, PAGED, NC, QT>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_pdl(kernel, dim3((rows + QT - 1) / QT, (H + kHG - 1) / kHG, n_splits), dim3(kAttnThreads), smem, stream, q_lat,
+    launch_pdl(kernel, dim3((rows + QT - 1) / QT, (H + kHG - 1) / kHG, n_splits), dim3(kAttnThreads), smem, stream, q_lat, q,
                (const T*)kc, (const T*)k_pages, page_table, table_stride, ring_pages, sink, (T*)o_lat, part_acc, part_ml,
                token_pos, token_seq, cu_seqlens, seq_slot, row0, row0 + rows, H, R, D, Dq, Dk, scale, window);
     int rc = check_launch("latent_attn");
@@ -733,16 +745,16 @@ static int launch_attn_as(const float* q_lat, const void* kc, const void* k_page
 }
 
 template <bool PAGED, int NT>
-static int launch_attn_tc_as(const float* q_lat, const void* kc, const void* k_pages, const int* page_table, int table_stride,
+static int launch_attn_tc_as(const float* q_lat, const LatentQuery<bf16>& q, const void* kc, const void* k_pages, const int* page_table, int table_stride,
                              int ring_pages, const float* sink, void* o_lat, float* part_acc, float* part_ml, int n_splits,
                              int QT, const int* token_pos, const int* token_seq, const int* cu_seqlens, const int* seq_slot,
                              int row0, int rows, int H, int R, int D, float scale, int window, cudaStream_t stream) {
     const int Ds = max((D + 15) / 16 * 16, 64 * NT) + 8;       // rows of 16-byte groups, an odd number of them
-    const size_t smem = (size_t)(2 * 16 * Ds + 2 * kTK * Ds + 2 * 16 * 40) * 2 + (size_t)(8 * 16 * 36 + 32) * 4;
+    const size_t smem = (size_t)(2 * 16 * Ds + 2 * kTK * Ds + 2 * 16 * 40) * 2 + (size_t)(8 * 16 * 36 + 32 + 2 * q.rot.rot_dims) * 4;
     if (smem > 200 * 1024) return 1;                     // does not fit: the caller takes the other kernel
     auto kernel = latent_attn_tc_kernel<PAGED, NT>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_pdl(kernel, dim3((rows + QT - 1) / QT, (H + kHG - 1) / kHG, n_splits), dim3(kAttnThreads), smem, stream, q_lat,
+    launch_pdl(kernel, dim3((rows + QT - 1) / QT, (H + kHG - 1) / kHG, n_splits), dim3(kAttnThreads), smem, stream, q_lat, q,
                (const bf16*)kc, (const bf16*)k_pages, page_table, table_stride, ring_pages, sink, (bf16*)o_lat, part_acc,
                part_ml, token_pos, token_seq, cu_seqlens, seq_slot, row0, row0 + rows, QT, H, R, D, Ds, scale, window);
     int rc = check_launch("latent_attn");
@@ -756,7 +768,7 @@ static int launch_attn_tc_as(const float* q_lat, const void* kc, const void* k_p
 
 // 0: launched; 1: not a case for the tensor-core kernel; negative: an error.
 template <bool PAGED>
-static int launch_attn_tc(const float* q_lat, const void* kc, const void* k_pages, const int* page_table, int table_stride,
+static int launch_attn_tc(const float* q_lat, const LatentQuery<bf16>& q, const void* kc, const void* k_pages, const int* page_table, int table_stride,
                           int ring_pages, const float* sink, void* o_lat, float* part_acc, float* part_ml, int n_splits,
                           int rows_per_block, const int* token_pos, const int* token_seq, const int* cu_seqlens,
                           const int* seq_slot, int row0, int rows, int H, int R, int D, float scale, int window,
@@ -764,7 +776,7 @@ static int launch_attn_tc(const float* q_lat, const void* kc, const void* k_page
     const void* src = PAGED ? k_pages : kc;
     if ((D & 7) != 0 || ((uintptr_t)src & 15) != 0 || R > 1024) return 1;
     const int QT = (rows_per_block > 1 && n_splits == 1) ? 2 : 1;
-#define HOS_TC(NT) return launch_attn_tc_as<PAGED, NT>(q_lat, kc, k_pages, page_table, table_stride, ring_pages, sink, o_lat,   \
+#define HOS_TC(NT) return launch_attn_tc_as<PAGED, NT>(q_lat, q, kc, k_pages, page_table, table_stride, ring_pages, sink, o_lat,   \
                                                        part_acc, part_ml, n_splits, QT, token_pos, token_seq, cu_seqlens,    \
                                                        seq_slot, row0, rows, H, R, D, scale, window, stream)
     if (R <= 128) HOS_TC(2);
@@ -777,13 +789,13 @@ static int launch_attn_tc(const float* q_lat, const void* kc, const void* k_page
 // Rows per block: four where many rows share keys (prompts), fewer where the sums would not fit the registers;
 // one with shares of the keys (decoding).
 template <typename T, bool PAGED>
-static int launch_attn(const float* q_lat, const void* kc, const void* k_pages, const int* page_table, int table_stride,
+static int launch_attn(const float* q_lat, const LatentQuery<T>& q, const void* kc, const void* k_pages, const int* page_table, int table_stride,
                        int ring_pages, const float* sink, void* o_lat, float* part_acc, float* part_ml, int n_splits,
                        int rows_per_block, const int* token_pos, const int* token_seq, const int* cu_seqlens,
                        const int* seq_slot, int row0, int rows, int H, int R, int D, float scale, int window,
                        cudaStream_t stream) {
     const int nc = (R + kAttnThreads - 1) / kAttnThreads;
-#define HOS_AS(NC, QT) return launch_attn_as<T, PAGED, NC, QT>(q_lat, kc, k_pages, page_table, table_stride, ring_pages, sink, \
+#define HOS_AS(NC, QT) return launch_attn_as<T, PAGED, NC, QT>(q_lat, q, kc, k_pages, page_table, table_stride, ring_pages, sink, \
                                                                o_lat, part_acc, part_ml, n_splits, token_pos, token_seq,     \
                                                                cu_seqlens, seq_slot, row0, rows, H, R, D, scale, window, stream)
     if (rows_per_block <= 1 || n_splits > 1) {
@@ -803,24 +815,23 @@ using namespace hos;
 
 extern "C" const char* hos_last_error() { return error_buffer(); }
 
-// q, down, cq: rows q_stride, down_stride, cq_stride elements apart, of one dtype; any of them may be null (see the kernel).
-extern "C" int hos_latent_prep(const void* q, int q_stride, const void* down, int down_stride, const void* cq, int cq_stride,
-                               int dtype, int H, int dq, int R, int P, int Rq, const float* w_norm, const float* cq_norm,
-                               float eps, const float* inv_freq, int rot_dims, int style, const int* token_pos,
-                               const int* token_seq, const int* seq_slot, const int* seq_len_after, void* kc, float* q_lat,
-                               void* cq_out, void* k_pages, const int* page_table, int table_stride, int ring_pages, int N,
-                               cudaStream_t stream) {
+// down, cq: rows down_stride, cq_stride elements apart, of one dtype; either may be null (see the kernel).
+extern "C" int hos_latent_prep(const void* down, int down_stride, const void* cq, int cq_stride, int dtype, int R, int P, int Rq,
+                               const float* w_norm, const float* cq_norm, float eps, const float* inv_freq, int rot_dims,
+                               int style, const int* token_pos, const int* token_seq, const int* seq_slot,
+                               const int* seq_len_after, void* kc, void* cq_out, void* k_pages, const int* page_table,
+                               int table_stride, int ring_pages, int N, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (inv_freq == nullptr) rot_dims = 0;
     if (rot_dims < 0 || rot_dims > P || (rot_dims & 1)) HOS_REFUSE("latent_prep: %d rotated of %d numbers", rot_dims, P);
     if (style != 0 && style != 1) HOS_REFUSE("latent_prep: unknown pairing style %d", style);
-    if ((q && !q_lat) || (down && (!kc || !w_norm)) || (cq && (!cq_out || !cq_norm || Rq <= 0)))
-        HOS_REFUSE("latent_prep: a part comes without its output or its norm's weight");
+    if ((down && (!kc || !w_norm)) || (cq && (!cq_out || !cq_norm || Rq <= 0)))
+        HOS_REFUSE("latent_prep: a latent comes without its output or its norm's weight");
 #define HOS_PREP(T)                                                                                                  \
     do {                                                                                                             \
-        LatentPrep<T> a{(const T*)q, (const T*)down, (const T*)cq, q_stride, down_stride, cq_stride, H, dq, R, P, Rq, w_norm, \
-                        cq_norm, eps, inv_freq, rot_dims, style, token_pos, token_seq, seq_slot, seq_len_after, (T*)kc, \
-                        q_lat, (T*)cq_out, (T*)k_pages, page_table, table_stride, ring_pages};                       \
+        LatentPrep<T> a{(const T*)down, (const T*)cq, down_stride, cq_stride, R, P, Rq, w_norm, cq_norm, eps,        \
+                        LatentRot{inv_freq, rot_dims, style}, token_pos, token_seq, seq_slot, seq_len_after, (T*)kc, \
+                        (T*)cq_out, (T*)k_pages, page_table, table_stride, ring_pages};                              \
         launch_pdl(latent_prep_kernel<T>, dim3(N), dim3(128), (size_t)(rot_dims / 2 + 1) * sizeof(float2), stream, a); \
     } while (0)
     if (dtype == kBF16) HOS_PREP(bf16);
@@ -835,7 +846,10 @@ extern "C" int hos_latent_prep(const void* q, int q_stride, const void* down, in
 // every row are cut into that many shares (part_acc: [rows of the step][H][n_splits][R], part_ml: [..][n_splits][2]).
 // rows_per_block: 1, or more where neighbouring rows share their keys (prompts).  use_tensor_cores: bfloat16 rows
 // whose sizes fit take the MMA kernel (the 32-bit query and weights as two bfloat16 terms each); 0 keeps the FMA kernel.
-extern "C" int hos_latent_attn(int dtype, int paged, const float* q_lat, const void* kc, const void* k_pages,
+// q_lat: [rows of the step][H][R], W_uk_h^T q_h; q: the heads' queries as projected (of `dtype`, rows q_stride apart, heads of dq
+// + D - R numbers whose last D - R are rotated here).
+extern "C" int hos_latent_attn(int dtype, int paged, const float* q_lat, const void* q, long long q_stride, int dq,
+                               const float* inv_freq, int rot_dims, int style, const void* kc, const void* k_pages,
                                const int* page_table, int table_stride, int ring_pages, const float* sink,
                                void* o_lat, float* part_acc, float* part_ml, int n_splits, int rows_per_block,
                                const int* token_pos, const int* token_seq, const int* cu_seqlens,
@@ -844,24 +858,30 @@ extern "C" int hos_latent_attn(int dtype, int paged, const float* q_lat, const v
     if (rows <= 0) return 0;
     if (R > 4 * kAttnThreads) HOS_REFUSE("latent_attn: a latent of %d numbers is more than %d", R, 4 * kAttnThreads);
     if (R > D) HOS_REFUSE("latent_attn: the latent (%d) is longer than the row (%d)", R, D);
+    if (inv_freq == nullptr) rot_dims = 0;
+    if (rot_dims < 0 || rot_dims > D - R || (rot_dims & 1)) HOS_REFUSE("latent_attn: %d rotated of %d numbers", rot_dims, D - R);
+    if (style != 0 && style != 1) HOS_REFUSE("latent_attn: unknown pairing style %d", style);
+    const LatentRot rot{inv_freq, rot_dims, style};
+    const LatentQuery<bf16> q16{(const bf16*)q, q_stride, dq, rot};
+    const LatentQuery<float> q32{(const float*)q, q_stride, dq, rot};
     if (n_splits < 1 || n_splits > 65535 || (n_splits > 1 && (part_acc == nullptr || part_ml == nullptr)))
         HOS_REFUSE("latent_attn: %d shares of the keys need their buffers", n_splits);
-#define HOS_GO(T, PG) return launch_attn<T, PG>(q_lat, kc, k_pages, page_table, table_stride, ring_pages, sink, o_lat, part_acc, \
+#define HOS_GO(T, Q, PG) return launch_attn<T, PG>(q_lat, Q, kc, k_pages, page_table, table_stride, ring_pages, sink, o_lat, part_acc, \
                                                  part_ml, n_splits, rows_per_block, token_pos, token_seq, cu_seqlens, seq_slot,   \
                                                  row0, rows, H, R, D, scale, window, stream)
     if (dtype == kBF16 && use_tensor_cores) {
-        const int rc = paged ? launch_attn_tc<true>(q_lat, kc, k_pages, page_table, table_stride, ring_pages, sink, o_lat, part_acc,
+        const int rc = paged ? launch_attn_tc<true>(q_lat, q16, kc, k_pages, page_table, table_stride, ring_pages, sink, o_lat, part_acc,
                                                     part_ml, n_splits, rows_per_block, token_pos, token_seq, cu_seqlens,
                                                     seq_slot, row0, rows, H, R, D, scale, window, stream)
-                             : launch_attn_tc<false>(q_lat, kc, k_pages, page_table, table_stride, ring_pages, sink, o_lat, part_acc,
+                             : launch_attn_tc<false>(q_lat, q16, kc, k_pages, page_table, table_stride, ring_pages, sink, o_lat, part_acc,
                                                      part_ml, n_splits, rows_per_block, token_pos, token_seq, cu_seqlens,
                                                      seq_slot, row0, rows, H, R, D, scale, window, stream);
         if (rc <= 0) return rc;
     }
-    if (dtype == kBF16 && paged) HOS_GO(bf16, true);
-    if (dtype == kBF16) HOS_GO(bf16, false);
-    if (dtype == kF32 && paged) HOS_GO(float, true);
-    if (dtype == kF32) HOS_GO(float, false);
+    if (dtype == kBF16 && paged) HOS_GO(bf16, q16, true);
+    if (dtype == kBF16) HOS_GO(bf16, q16, false);
+    if (dtype == kF32 && paged) HOS_GO(float, q32, true);
+    if (dtype == kF32) HOS_GO(float, q32, false);
 #undef HOS_GO
     HOS_REFUSE("latent_attn: unknown dtype %d", dtype);
 }

@@ -627,28 +627,22 @@ def scaled_add_norms(a: Optional[torch.Tensor], f: Optional[torch.Tensor], mult:
                   dtype_code(h.dtype) if h is not None else 0, n, d, _stream())
 
 
-def latent_prep(step, q, n_heads: int, dq: int, rank: int, rot: int, eps: float, inv_freq: Optional[torch.Tensor], rot_dims: int,
-                style: int, q_lat: Optional[torch.Tensor] = None, down=None, w_norm: Optional[torch.Tensor] = None,
-                kc: Optional[torch.Tensor] = None, cache: Optional[PagedKVArgs] = None, cq=None,
-                cq_norm: Optional[torch.Tensor] = None, cq_out: Optional[torch.Tensor] = None) -> None:
-    """Norms, rotations and the cache write between the projections and the latent attention, for the parts that are given.
-    `q`, `down` and `cq` are (rows, first column) or None: the heads' queries [n_heads x (dq + rot)] -> the last `rot` numbers
-    of q_lat's heads; the latent and the shared key part [rank + rot] -> kc and the cache; the queries' own latent ->
-    cq_out, normed with cq_norm.  style: the rotation's pairing (ROPE_STYLES)."""
-    rows = next((p[0] for p in (q, down, cq) if p is not None), None)
+def latent_prep(step, rank: int, rot: int, eps: float, inv_freq: Optional[torch.Tensor], rot_dims: int, style: int, down=None,
+                w_norm: Optional[torch.Tensor] = None, kc: Optional[torch.Tensor] = None, cache: Optional[PagedKVArgs] = None,
+                cq=None, cq_norm: Optional[torch.Tensor] = None, cq_out: Optional[torch.Tensor] = None) -> None:
+    """Norms, the key part's rotation and the cache write between the down projections and what reads their latents.  `down`
+    and `cq` are (rows, first column) or None: the latent and the shared key part [rank + rot] -> kc and the cache; the
+    queries' own latent -> cq_out, normed with cq_norm.  style: the rotation's pairing (ROPE_STYLES)."""
+    rows = next((p[0] for p in (down, cq) if p is not None), None)
     if rows is None:
         raise KernelError("latent_prep: no rows")
     n, dt = rows.shape[0], rows.dtype
     rq = cq_out.shape[1] if cq_out is not None else 0
-    for part, cols, what in ((q, n_heads * (dq + rot), "query rows"), (down, rank + rot, "latent rows"), (cq, rq, "query latents")):
+    for part, cols, what in ((down, rank + rot, "latent rows"), (cq, rq, "query latents")):
         if part is not None:
             _check(part[0], what, dt, 2)
             if part[0].shape[0] != n or part[1] + cols > part[0].shape[1]:
                 raise KernelError(f"latent_prep: sizes of the {what} disagree")
-    if q is not None:
-        _check(q_lat, "latent queries", torch.float32, 3)
-        if q_lat.shape != (n, n_heads, rank + rot):
-            raise KernelError("latent_prep: sizes disagree")
     if down is not None:
         _check(kc, "latent rows", dt, 2)
         if kc.shape != (n, rank + rot) or w_norm is None or w_norm.shape[0] != rank:
@@ -666,31 +660,35 @@ def latent_prep(step, q, n_heads: int, dq: int, rank: int, rot: int, eps: float,
         if part is None:
             return None, 0
         return ctypes.c_void_p(part[0].data_ptr() + part[1] * part[0].element_size()), part[0].shape[1]
-    blocks().call("hos_latent_prep", *at(q), *at(down), *at(cq), dtype_code(dt), n_heads, dq, rank, rot, rq, _ptr(w_norm),
-                  _ptr(cq_norm), float(eps), _ptr(inv_freq), int(rot_dims) if inv_freq is not None else 0, int(style),
-                  _ptr(step.token_pos), _ptr(step.token_seq), _ptr(step.seq_slot), _ptr(step.seq_len_after),
-                  _ptr(kc) if down is not None else None, _ptr(q_lat), _ptr(cq_out),
-                  _ptr(cache.k_pages) if cache else None, _ptr(cache.page_table) if cache else None,
+    blocks().call("hos_latent_prep", *at(down), *at(cq), dtype_code(dt), rank, rot, rq, _ptr(w_norm), _ptr(cq_norm), float(eps),
+                  _ptr(inv_freq), int(rot_dims) if inv_freq is not None else 0, int(style), _ptr(step.token_pos),
+                  _ptr(step.token_seq), _ptr(step.seq_slot), _ptr(step.seq_len_after), _ptr(kc) if down is not None else None,
+                  _ptr(cq_out), _ptr(cache.k_pages) if cache else None, _ptr(cache.page_table) if cache else None,
                   cache.table_stride if cache else 0, cache.ring_pages if cache else 0, n, _stream())
 
 
-def latent_attn(q_lat: torch.Tensor, kc: Optional[torch.Tensor], cache: Optional[PagedKVArgs], sink: Optional[torch.Tensor],
+def latent_attn(q_lat: torch.Tensor, q: torch.Tensor, dq: int, inv_freq: Optional[torch.Tensor], rot_dims: int, style: int, kc: Optional[torch.Tensor], cache: Optional[PagedKVArgs], sink: Optional[torch.Tensor],
                 o_lat: torch.Tensor, step, row0: int, rows: int, rank: int, scale: float, window: Optional[int],
                 paged: bool, n_splits: int = 1, rows_per_block: int = 1, tensor_cores: bool = True) -> None:
-    """Rows row0 .. row0+rows-1 of the step: keys from `kc` (the step's own rows; sequences from position 0)
+    """q_lat: float32 [N, heads, rank], the queries' unrotated parts taken to the latent; q: rows whose first columns are the
+    heads' queries as projected, dq unrotated and then the rotated numbers each (rotated here; style: ROPE_STYLES).
+    Rows row0 .. row0+rows-1 of the step: keys from `kc` (the step's own rows; sequences from position 0)
     or from the paged cache.  `n_splits` > 1: every row's keys are cut into that many shares that run side by side
     and are merged (few rows: decoding); `rows_per_block` > 1: neighbouring rows share the keys they read (prompts)."""
     _check(q_lat, "latent queries", torch.float32, 3)
     _check(o_lat, "latent outputs", (cache.k_pages if paged else kc).dtype, 3)
-    n, heads, d = q_lat.shape
-    if o_lat.shape != (n, heads, rank):
-        raise KernelError("latent_attn: sizes disagree")
+    n, heads, r = q_lat.shape
     src = cache.k_pages if paged else kc
+    _check(q, "query rows", src.dtype, 2)
+    d = src.shape[-1]
+    if r != rank or o_lat.shape != (n, heads, rank) or q.shape[0] != n or q.shape[1] < heads * (dq + d - rank):
+        raise KernelError("latent_attn: sizes disagree")
     part_acc = part_ml = None
     if n_splits > 1:
         part_acc = torch.empty((n, heads, n_splits, rank), dtype=torch.float32, device=q_lat.device)
         part_ml = torch.empty((n, heads, n_splits, 2), dtype=torch.float32, device=q_lat.device)
-    blocks().call("hos_latent_attn", dtype_code(src.dtype), int(paged), _ptr(q_lat), _ptr(kc),
+    blocks().call("hos_latent_attn", dtype_code(src.dtype), int(paged), _ptr(q_lat), _ptr(q), q.shape[1], int(dq), _ptr(inv_freq),
+                  int(rot_dims) if inv_freq is not None else 0, int(style), _ptr(kc),
                   _ptr(cache.k_pages) if paged else None, _ptr(cache.page_table) if paged else None,
                   cache.table_stride if paged else 0, cache.ring_pages if paged else 0, _ptr(sink), _ptr(o_lat),
                   _ptr(part_acc), _ptr(part_ml), int(n_splits), int(rows_per_block),

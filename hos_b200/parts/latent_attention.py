@@ -144,28 +144,27 @@ class LatentAttention(Mixer):
         H, R, D = self.n_heads, self.rank, self.row
         proj = linear.matmul(h, self.w_in)
         kc = None if self.shares_kv else torch.empty((n, D), dtype=h.dtype, device=h.device)
-        q_lat = torch.empty((n, H, D), dtype=torch.float32, device=h.device)
+        q_lat = torch.empty((n, H, R), dtype=torch.float32, device=h.device)
         inv_freq, rot_dims, style = self.position.kernel_args() if self.position else (None, 0, 1)
-        prep = functools.partial(ops.latent_prep, step, n_heads=H, dq=self.dim, rank=R, rot=self.rot_dim, eps=self.eps,
-                                 inv_freq=inv_freq, rot_dims=rot_dims, style=style)
         q_first = self.q_rank or self.q_cols                # the column where the down projection's part of `proj` begins
-        keys = {} if self.shares_kv else dict(down=(proj, q_first), w_norm=self.w_norm, kc=kc, cache=cache)
+        parts = {} if self.shares_kv else dict(down=(proj, q_first), w_norm=self.w_norm, kc=kc, cache=cache)
+        q = proj
         if self.q_rank:
             cq = torch.empty((n, self.q_rank), dtype=h.dtype, device=h.device)
-            prep(q=None, cq=(proj, 0), cq_norm=self.q_norm, cq_out=cq, **keys)
+            parts.update(cq=(proj, 0), cq_norm=self.q_norm, cq_out=cq)
+        if parts:
+            ops.latent_prep(step, R, self.rot_dim, self.eps, inv_freq, rot_dims, style, **parts)
+        if self.q_rank:
             q = linear.matmul(cq, self.w_uq)
-            prep(q=(q, 0), q_lat=q_lat)
-        else:
-            q = proj
-            prep(q=(q, 0), q_lat=q_lat, **keys)
-        # q'_h = W_uk_h^T q_h into the first `rank` numbers of every head's latent query
-        ops.heads_product(q, 0, q.shape[1], self.dim + self.rot_dim, self.w_uk_t, q_lat, 0, H * D, D, n)
+        # q'_h = W_uk_h^T q_h
+        ops.heads_product(q, 0, q.shape[1], self.dim + self.rot_dim, self.w_uk_t, q_lat, 0, H * R, R, n)
+        attend = functools.partial(ops.latent_attn, q_lat, q, self.dim, inv_freq, rot_dims, style)
         o_lat = torch.empty((n, H, R), dtype=h.dtype, device=h.device)      # what the value expansion reads
         nf = 0 if self.shares_kv else (n if step.from_zero else step.fresh_tokens)
         if nf > 0:
             shares, per_block = self.plan(nf, step)
-            ops.latent_attn(q_lat, kc, None, self.sink, o_lat, step, 0, nf, R, self.scale, self.window, paged=False,
-                            n_splits=shares, rows_per_block=per_block, tensor_cores=self.use_tensor_cores)
+            attend(kc, None, self.sink, o_lat, step, 0, nf, R, self.scale, self.window, paged=False,
+                   n_splits=shares, rows_per_block=per_block, tensor_cores=self.use_tensor_cores)
         if nf < n:
             if cache.ring_pages > 0 and not step.replayed:
                 room = cache.ring_pages * ops.PAGE_TOKENS - int(self.window) + 1
@@ -176,8 +175,8 @@ class LatentAttention(Mixer):
                                       f"at most {room} fit")
             rows = n - nf
             shares, per_block = self.plan(rows, step)
-            ops.latent_attn(q_lat, None, cache, self.sink, o_lat, step, nf, rows, R, self.scale, self.window, paged=True,
-                            n_splits=shares, rows_per_block=per_block, tensor_cores=self.use_tensor_cores)
+            attend(None, cache, self.sink, o_lat, step, nf, rows, R, self.scale, self.window, paged=True,
+                   n_splits=shares, rows_per_block=per_block, tensor_cores=self.use_tensor_cores)
         att = torch.empty((n, H * self.vdim), dtype=h.dtype, device=h.device)
         ops.heads_product(o_lat, 0, H * R, R, self.w_uv, att, 0, H * self.vdim, self.vdim, n)
         return linear.matmul_or_partials(att, self.w_o) if partial_ok else linear.matmul(att, self.w_o)

@@ -395,19 +395,36 @@ def test_the_two_attention_kernels_agree_in_bfloat16(folders, case):
 def test_the_attention_kernels_alone(heads, rank, rot, n, window, scale):
     """Both kernels (MMA and FMA), one and several rows to a block, on random latent rows against float64: two head
     groups, every count of column tiles, a latent too wide for the MMA kernel's shared memory (it steps aside), a
-    row size that is no multiple of 8.  The output is bfloat16: its rounding is the error."""
+    row size that is no multiple of 8; the queries' rotated parts turned by the kernel in both pairings, all of the
+    part and all but two numbers of it.  The output is bfloat16: its rounding is the error."""
     from hos_b200 import ops
     from hos_b200.parts.base import StepInfo
     torch.manual_seed(heads * 1000 + rank)
     d = rank + rot
-    q = torch.randn(n, heads, d, device="cuda")
+    dq = 6
+    q_lat = torch.randn(n, heads, rank, device="cuda")
+    rows = torch.randn(n, heads * (dq + rot) + 5, device="cuda").to(torch.bfloat16)
     kc = torch.randn(n, d, device="cuda").to(torch.bfloat16)
     sink = torch.randn(heads, device="cuda")
     pos = torch.arange(n, dtype=torch.int32, device="cuda")
     step = StepInfo(n, 1, None, pos, torch.zeros(n, dtype=torch.int32, device="cuda"),
                     torch.tensor([0, n], dtype=torch.int32, device="cuda"), torch.zeros(1, dtype=torch.int32, device="cuda"),
                     None, True, False, n, n)
-    k64, q64 = kc.double().cpu(), q.double().cpu()
+    k64 = kc.double().cpu()
+    for style, dims in (("rotate_half", rot), ("interleaved", rot - 2)):
+        freq = torch.tensor([300.0 ** (-2.0 * e / dims) for e in range(dims // 2)], dtype=torch.float64).float()
+        part = rows.double().cpu()[:, : heads * (dq + rot)].reshape(n, heads, dq + rot)[..., dq:].clone()
+        ang = torch.arange(n).double()[:, None, None] * freq.double()
+        c, sn = torch.cos(ang), torch.sin(ang)
+        a = torch.arange(dims // 2) * (1 if style == "rotate_half" else 2)
+        b = a + (dims // 2 if style == "rotate_half" else 1)
+        u, v = part[..., a].clone(), part[..., b].clone()
+        part[..., a], part[..., b] = u * c - v * sn, v * c + u * sn
+        _check_latent_attn(ops, torch.cat([q_lat.double().cpu(), part], -1), q_lat, rows, dq, freq.cuda(), dims,
+                           ops.ROPE_STYLES[style], kc, k64, sink, step, heads, rank, n, window, scale)
+
+
+def _check_latent_attn(ops, q64, q_lat, rows, dq, freq, dims, style, kc, k64, sink, step, heads, rank, n, window, scale):
     s = torch.einsum("ihd,jd->hij", q64, k64) * scale
     i, j = torch.arange(n)[:, None], torch.arange(n)[None]
     seen = (i >= j) & ((i - j < window) if window else torch.ones(n, n, dtype=torch.bool))
@@ -417,7 +434,7 @@ def test_the_attention_kernels_alone(heads, rank, rot, n, window, scale):
     for tensor_cores in (True, False):
         for per_block in (4, 1):
             out = torch.empty(n, heads, rank, dtype=torch.bfloat16, device="cuda")
-            ops.latent_attn(q, kc, None, sink, out, step, 0, n, rank, scale, window, paged=False, n_splits=1,
+            ops.latent_attn(q_lat, rows, dq, freq, dims, style, kc, None, sink, out, step, 0, n, rank, scale, window, paged=False, n_splits=1,
                             rows_per_block=per_block, tensor_cores=tensor_cores)
             err = float((out.double().cpu() - want).abs().max() / want.abs().max())
             assert err < 4e-3, f"tensor cores {tensor_cores}, {per_block} rows a block: {err:.2e}"
