@@ -8,6 +8,7 @@ checkpoint name.
   frequencies         base^(-2i/dims); with a scaling: unchanged for short wavelengths, divided by the
                       factor for long ones, a straight line between the two in original / wavelength
   rotate_halves       rotary positions on pairs (i, i + dims/2) of the first `dims` numbers
+  capped              c tanh(s / c); no cap: s
   visible             the mask: causal, the last `size` keys
   latent_mixer        queries from a normed latent, keys and values expanded from one normed latent row per
                       position, one rotated key part shared by the heads, one more term in the denominator
@@ -74,6 +75,10 @@ def softmax_with_sink(s, sink=None):
     return e / (e.sum() + (0.0 if sink is None else torch.exp(sink - top)))
 
 
+def capped(s, cap):
+    return cap * torch.tanh(s / cap) if cap else s
+
+
 def latent_mixer(m, eps, w, p, h):
     T, H, d, r, vd, R = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
     cq = rms(h @ w[p + "dq"].T, eps) * w[p + "dq.norm"]
@@ -105,8 +110,7 @@ def attention_mixer(m, eps, w, p, h):
         for hd in range(H):
             g = hd // (H // G)
             s = (k[js, g] @ q[i, hd]) * m["scale"]
-            s = m["softcap"] * torch.tanh(s / m["softcap"])
-            out[i, hd] = softmax_with_sink(s) @ v[js, g]
+            out[i, hd] = softmax_with_sink(capped(s, m.get("softcap"))) @ v[js, g]
     return out.reshape(T, H * vd) @ w[p + "o"].T
 
 
@@ -159,5 +163,4 @@ def forward(cfg, w, tokens: List[int], taps: Optional[list] = None, edit=None):
             x = x + rms(feed_forward(layer["mlp"], w, p + "mlp.", x), eps) * w[p + "norm2"]
         if taps is not None:
             taps.append(x.clone())
-    logits = (rms(x, eps) * w["final.norm"]) @ w["head"].T * cfg["logit_scale"]
-    return cfg["logit_softcap"] * torch.tanh(logits / cfg["logit_softcap"])
+    return capped((rms(x, eps) * w["final.norm"]) @ w["head"].T * cfg["logit_scale"], cfg["logit_softcap"])
