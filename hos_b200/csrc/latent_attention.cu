@@ -174,14 +174,16 @@ latent_attn_kernel(const float* __restrict__ q_lat, const LatentQuery<T> q, cons
         sincos_tab[i] = make_float2(sn, cs);
     }
     __syncthreads();
-    for (int i = tid; i < QT * kHG * Dq; i += kAttnThreads) {
-        const int t = i / (kHG * Dq), rem = i - t * kHG * Dq, h = rem / Dq, d = rem - h * Dq;
+    static_assert(kHG == kAttnThreads / 32, "a warp stages its head's queries");
+    for (int t = 0; t < QT; ++t) {
         const int n = n0 + t;
-        float v = 0.f;
-        if (n < row_end && h < nh && d < D)
-            v = d < R ? q_lat[((size_t)n * H + h0 + h) * R + d]
-                      : rotated(q.p + n * q.stride + (size_t)(h0 + h) * (q.dq + D - R) + q.dq, d - R, sincos_tab + t * half, q.rot);
-        qs[i] = v;
+        const bool in = n < row_end && warp < nh;
+        const float* src = q_lat + ((size_t)n * H + h0 + warp) * R;
+        const T* part = q.p + n * q.stride + (size_t)(h0 + warp) * (q.dq + D - R) + q.dq;
+        float* dst = qs + (t * kHG + warp) * Dq;
+#pragma unroll 4
+        for (int d = lane; d < R; d += 32) dst[d] = in ? src[d] : 0.f;
+        for (int d = R + lane; d < Dq; d += 32) dst[d] = in && d < D ? rotated(part, d - R, sincos_tab + t * half, q.rot) : 0.f;
     }
     __syncthreads();
     float m_run[QT], l_run[QT];                // of head `warp`, per row (kept by every lane of the warp)
@@ -420,15 +422,19 @@ latent_attn_tc_kernel(const float* __restrict__ q_lat, const LatentQuery<bf16> q
         sincos_tab[i] = make_float2(sn, cs);
     }
     __syncthreads();
-    for (int i = tid; i < 16 * Ds; i += kAttnThreads) {
-        const int row = i / Ds, d = i - row * Ds, t = row >> 3, h = row & 7, n = n0 + t;
-        float v = 0.f;
-        if (t < QT && n < row_end && h < nh && d < D)
-            v = d < R ? q_lat[((size_t)n * H + h0 + h) * R + d]
-                      : rotated(q.p + n * q.stride + (size_t)(h0 + h) * (q.dq + D - R) + q.dq, d - R, sincos_tab + t * half, q.rot);
-        const bf16 hi = __float2bfloat16_rn(v);
-        Qh[i] = hi;
-        Ql[i] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    for (int t = 0; t < 2; ++t) {               // MMA row t * 8 + head: a warp stages its head's queries
+        const int n = n0 + t, at = (t * 8 + warp) * Ds;
+        const bool in = t < QT && n < row_end && warp < nh;
+        const float* src = q_lat + ((size_t)n * H + h0 + warp) * R;
+        const bf16* part = q.p + n * q.stride + (size_t)(h0 + warp) * (q.dq + D - R) + q.dq;
+        auto put = [&](int d, float v) {
+            const bf16 hi = __float2bfloat16_rn(v);
+            Qh[at + d] = hi;
+            Ql[at + d] = __float2bfloat16_rn(v - __bfloat162float(hi));
+        };
+#pragma unroll 8
+        for (int d = lane; d < R; d += 32) put(d, in ? src[d] : 0.f);
+        for (int d = R + lane; d < Ds; d += 32) put(d, in && d < D ? rotated(part, d - R, sincos_tab + t * half, q.rot) : 0.f);
     }
     for (int i = tid; i < 2 * kTK * (Ds - D); i += kAttnThreads)       // the padding columns stay zero
         Kt[(i / (Ds - D)) * Ds + D + i % (Ds - D)] = __float2bfloat16_rn(0.f);

@@ -216,7 +216,7 @@ def test_far_keys_and_a_long_decode(tmp_path):
 
 
 @pytest.mark.parametrize("name, layer", [
-    ("latent", latent(2, 24, 4, 8, 16, 16, 1.0, mlp=None)), ("attention", attention(2, 1, 24, 8, 0.8, 4, mlp=None)),
+    ("latent", latent(2, 24, 4, 8, 16, 16, 1.0, mlp=None)), ("attention", attention(2, 1, 48, 8, 0.6, 4, mlp=None)),
     ("latent, window", latent(3, 16, 4, 8, 16, 16, 0.6, window=130, mlp=None)),
     ("attention, window", attention(4, 2, 64, 64, 0.3, 16, softcap=12.0, window=130, mlp=None))])
 def test_one_key_that_stands_out_inside_and_outside_a_window(tmp_path, name, layer):
@@ -384,12 +384,12 @@ def test_the_first_tokens_at_the_tensor_core_kernels_sizes(folders, dtype):
     (c,) = r.admit(1)
     out = r.step([c, b], [seqs[2], seqs[1][11:14]], [list(range(9)), [0, 1, 2]]).cpu()
     got_b.append(out[9:])
-    for g, x in ((torch.cat(got_a), want[0]), (torch.cat(got_b), want[1]), (out[:9], want[2])):
-        if dtype == "float32":
-            e = row_errors(g, x)
-            assert float(e.max()) <= 1e-4, f"worst {float(e.max()):.2e}"
-        else:
-            assert_rows(g, x, dtype, "first tokens")
+    g, x = torch.cat(got_a + got_b + [out[:9]]), torch.cat(want)
+    if dtype == "float32":
+        e = row_errors(g, x)
+        assert float(e.max()) <= 1e-4, f"worst {float(e.max()):.2e}"
+    else:
+        assert_rows(g, x, dtype, "first tokens")
     for s_ in (a, b, c):
         r.release(s_)
     r.cache.check()
@@ -662,16 +662,14 @@ def test_the_router_with_groups_alone_against_float64():
             got, wt = choice.cpu().view(n, top), weight.cpu().view(n, top)
             size, checked = n_out // count, 0
             for r in range(n):
-                # the groups' standing: above 1 by what is missing to 2, which keeps its digits
+                # a group's standing, a number that grows with the sum of its two largest scores and keeps its digits where
+                # the sum is near 2: the sum up to 1, above it one over what is missing to 2 (a group of one: its logit)
                 two = z[r].view(count, size).sort(-1, descending=True).values[:, :2]
-                loss = torch.sigmoid(-two).sum(-1)
-                total = torch.sigmoid(two).sum(-1)
-                order = sorted(range(count), key=lambda g: (float(loss[g]) if total[g] > 1 else 10.0 - float(total[g]), g))
-                last, nxt = order[keep - 1], order[keep] if keep < count else None
-                if nxt is not None:
-                    p, q_ = (loss[last], loss[nxt]) if total[nxt] > 1 else (total[nxt], total[last])
-                    if float((q_ - p) / q_) < 1e-3:
-                        continue                              # a close call in 32-bit too
+                total, missing = torch.sigmoid(two).sum(-1), torch.sigmoid(-two).sum(-1)
+                stand = two[:, 0] if size == 1 else torch.where(total > 1, 1.0 / missing, total)
+                order = sorted(range(count), key=lambda g: (-float(stand[g]), g))
+                if keep < count and float(stand[order[keep - 1]] - stand[order[keep]]) < 1e-3 * abs(float(stand[order[keep]])):
+                    continue                                  # a close call in 32-bit too
                 open_ = [e for e in range(n_out) if e // size in order[:keep]]
                 best = sorted(open_, key=lambda e: (-float(z[r, e]), e))
                 if len(best) > top and float(z[r, best[top - 1]] - z[r, best[top]]) < 1e-3:
