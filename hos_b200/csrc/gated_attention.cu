@@ -85,20 +85,15 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
             inv_all[part] = 1.f / sqrtf(ss / (float)cn + eps);
         }
     }
-    // a lane's numbers of a head are the same columns for every head: their sines and cosines are taken once
+    // the row's sines and cosines, once for all heads
+    __shared__ float2 turn[32 * kPrepPL / 2];
     const int half = rot_dims >> 1;
-    float sn[kPrepPL], cs[kPrepPL];
-#pragma unroll
-    for (int i = 0; i < kPrepPL; ++i) {
-        const int d = lane + 32 * i;
-        sn[i] = 0.f;
-        cs[i] = 1.f;
-        if (d < rot_dims) {
-            sincosf(fpos * freq[style == 0 ? (d < half ? d : d - half) : d >> 1], &sn[i], &cs[i]);
-            sn[i] *= magnitude;
-            cs[i] *= magnitude;
-        }
+    for (int i = threadIdx.x; i < half; i += kThreads) {
+        float sn, cs;
+        sincosf(fpos * freq[i], &sn, &cs);
+        turn[i] = make_float2(sn * magnitude, cs * magnitude);
     }
+    if (rot_dims > 0) __syncthreads();
     // query heads 0..H-1, then key heads H..H+G-1
     for (int item = warp; item < H + G; item += kThreads / 32) {
         const bool is_q = item < H;
@@ -134,7 +129,8 @@ qk_prep_kernel(const float* __restrict__ proj, int ld, const float* __restrict__
                     const int o = upper ? d - half : d + half;
                     other = (row[col0 + o] + (bias ? bias[col0 + o] : 0.f)) * inv * (nw != nullptr ? nw[o] : 1.f);
                 }
-                v[i] = upper ? fmaf(v[i], cs[i], other * sn[i]) : fmaf(v[i], cs[i], -other * sn[i]);
+                const float2 sc = turn[style == 0 ? (upper ? d - half : d) : d >> 1];
+                v[i] = fmaf(v[i], sc.y, upper ? other * sc.x : -other * sc.x);
             }
         }
         if (is_q && q_every > 0)

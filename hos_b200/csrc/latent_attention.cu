@@ -102,19 +102,22 @@ __global__ void latent_prep_kernel(LatentPrep<T> a) {
     }
     const T* craw = keys ? a.down + (size_t)n * a.down_stride : nullptr;
     float ss = 0.f, sq = 0.f;
-    if (keys)
+    if (keys) {
+#pragma unroll 4
         for (int d = threadIdx.x; d < R; d += blockDim.x) {
             const float v = to_float(craw[d]);
             ss = fmaf(v, v, ss);
         }
+    }
     const T* cq = a.cq != nullptr ? a.cq + (size_t)n * a.cq_stride : nullptr;
-    if (cq)
+    if (cq) {
+#pragma unroll 4
         for (int d = threadIdx.x; d < a.Rq; d += blockDim.x) {
             const float v = to_float(cq[d]);
             sq = fmaf(v, v, sq);
         }
-    if (cq) {
         const float qinv = rsqrtf(block_sum(sq, scratch) / (float)a.Rq + a.eps);
+#pragma unroll 4
         for (int d = threadIdx.x; d < a.Rq; d += blockDim.x)
             a.cq_out[(size_t)n * a.Rq + d] = from_float<T>(to_float(cq[d]) * qinv * a.cq_norm[d]);
     }
@@ -835,10 +838,11 @@ extern "C" int hos_latent_prep(const void* down, int down_stride, const void* cq
         HOS_REFUSE("latent_prep: a latent comes without its output or its norm's weight");
 #define HOS_PREP(T)                                                                                                  \
     do {                                                                                                             \
+        const int threads = N <= 592 ? 256 : 128;           /* few rows: a shorter chain of loads to a row */        \
         LatentPrep<T> a{(const T*)down, (const T*)cq, down_stride, cq_stride, R, P, Rq, w_norm, cq_norm, eps,        \
                         LatentRot{inv_freq, rot_dims, style}, token_pos, token_seq, seq_slot, seq_len_after, (T*)kc, \
                         (T*)cq_out, (T*)k_pages, page_table, table_stride, ring_pages};                              \
-        launch_pdl(latent_prep_kernel<T>, dim3(N), dim3(128), (size_t)(rot_dims / 2 + 1) * sizeof(float2), stream, a); \
+        launch_pdl(latent_prep_kernel<T>, dim3(N), dim3(threads), (size_t)(rot_dims / 2 + 1) * sizeof(float2), stream, a); \
     } while (0)
     if (dtype == kBF16) HOS_PREP(bf16);
     else if (dtype == kF32) HOS_PREP(float);
