@@ -622,30 +622,48 @@ latent_attn_tc_kernel(const float* __restrict__ q_lat, const LatentQuery<bf16> q
     }
 }
 
-// o_lat[n][h] = sum_s e^{m_s - M} acc_s / sum_s e^{m_s - M} l_s over the shares s of the keys.
+// o_lat[n][h] = sum_s e^{m_s - M} acc_s / sum_s e^{m_s - M} l_s over the shares s of the keys.  A block takes kMergeCols
+// columns of a (row, head), two to a thread; the shares' weights are formed once, 128 shares at a time, and a column's
+// shares are independent loads.
+constexpr int kMergeCols = 256;
 template <typename T>
-__global__ void latent_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
-                                    T* __restrict__ o_lat, const int* __restrict__ token_seq, int row0, int H, int R,
-                                    int n_splits) {
+__global__ void __launch_bounds__(kMergeCols / 2)
+latent_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, T* __restrict__ o_lat,
+                    const int* __restrict__ token_seq, int row0, int H, int R, int n_splits) {
     pdl_enter();
-    const int n = row0 + blockIdx.x, h = blockIdx.y;
+    __shared__ float weight[kMergeCols / 2];
+    const int n = row0 + blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
+    const int c0 = blockIdx.z * kMergeCols + threadIdx.x, c1 = c0 + kMergeCols / 2;
     T* out = o_lat + ((size_t)n * H + h) * R;
-    if (token_seq[n] < 0) {
-        for (int c = threadIdx.x; c < R; c += blockDim.x) out[c] = from_float<T>(0.f);
-        return;
+    float v0 = 0.f, v1 = 0.f, den = 0.f;
+    if (token_seq[n] >= 0) {
+        const float* ml = part_ml + ((size_t)n * H + h) * n_splits * 2;
+        float M = -INFINITY;
+        for (int s = lane; s < n_splits; s += 32) M = fmaxf(M, ml[2 * s]);
+        M = warp_max(M);
+        for (int s = lane; s < n_splits; s += 32) den += ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - M) * ml[2 * s + 1];
+        den = warp_sum(den);
+        const float* pa = part_acc + ((size_t)n * H + h) * n_splits * R;
+        for (int s0 = 0; s0 < n_splits; s0 += blockDim.x) {
+            const int cnt = min((int)blockDim.x, n_splits - s0);
+            __syncthreads();
+            if ((int)threadIdx.x < cnt) {
+                const float m = ml[2 * (s0 + threadIdx.x)];
+                weight[threadIdx.x] = m == -INFINITY ? 0.f : expf(m - M);
+            }
+            __syncthreads();
+#pragma unroll 8
+            for (int s = 0; s < cnt; ++s) {
+                const float* row = pa + (size_t)(s0 + s) * R;
+                const float x0 = c0 < R ? row[c0] : 0.f, x1 = c1 < R ? row[c1] : 0.f, w = weight[s];
+                v0 = w > 0.f ? fmaf(w, x0, v0) : v0;
+                v1 = w > 0.f ? fmaf(w, x1, v1) : v1;
+            }
+        }
     }
-    const float* ml = part_ml + ((size_t)n * H + h) * n_splits * 2;
-    float M = -INFINITY;
-    for (int s = 0; s < n_splits; ++s) M = fmaxf(M, ml[2 * s]);
-    float den = 0.f;
-    for (int s = 0; s < n_splits; ++s) den += ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - M) * ml[2 * s + 1];
-    const float* pa = part_acc + ((size_t)n * H + h) * n_splits * R;
-    for (int c = threadIdx.x; c < R; c += blockDim.x) {
-        float v = 0.f;
-        for (int s = 0; s < n_splits; ++s)
-            if (ml[2 * s] != -INFINITY) v = fmaf(expf(ml[2 * s] - M), pa[(size_t)s * R + c], v);
-        out[c] = from_float<T>(den > 0.f ? v / den : 0.f);
-    }
+    const float f = den > 0.f ? 1.f / den : 0.f;
+    if (c0 < R) out[c0] = from_float<T>(v0 * f);
+    if (c1 < R) out[c1] = from_float<T>(v1 * f);
 }
 
 // ---- heads_product -------------------------------------------------------------------------
@@ -746,7 +764,7 @@ static int launch_attn_as(const float* q_lat, const LatentQuery<T>& q, const voi
                token_pos, token_seq, cu_seqlens, seq_slot, row0, row0 + rows, H, R, D, Dq, Dk, scale, window);
     int rc = check_launch("latent_attn");
     if (rc == 0 && n_splits > 1) {
-        launch_pdl(latent_merge_kernel<T>, dim3(rows, H), dim3(128), 0, stream, (const float*)part_acc, (const float*)part_ml,
+        launch_pdl(latent_merge_kernel<T>, dim3(rows, H, (R + kMergeCols - 1) / kMergeCols), dim3(kMergeCols / 2), 0, stream, (const float*)part_acc, (const float*)part_ml,
                    (T*)o_lat, token_seq, row0, H, R, n_splits);
         rc = check_launch("latent_merge");
     }
@@ -768,7 +786,7 @@ static int launch_attn_tc_as(const float* q_lat, const LatentQuery<bf16>& q, con
                part_ml, token_pos, token_seq, cu_seqlens, seq_slot, row0, row0 + rows, QT, H, R, D, Ds, scale, window);
     int rc = check_launch("latent_attn");
     if (rc == 0 && n_splits > 1) {
-        launch_pdl(latent_merge_kernel<bf16>, dim3(rows, H), dim3(128), 0, stream, (const float*)part_acc,
+        launch_pdl(latent_merge_kernel<bf16>, dim3(rows, H, (R + kMergeCols - 1) / kMergeCols), dim3(kMergeCols / 2), 0, stream, (const float*)part_acc,
                    (const float*)part_ml, (bf16*)o_lat, token_seq, row0, H, R, n_splits);
         rc = check_launch("latent_merge");
     }
