@@ -126,11 +126,13 @@ scale_add_norm_vec_kernel(const TY* __restrict__ y, int n_parts, long long part_
     }
 }
 
-template <typename TH>
+template <typename TH, int VEC>
 __global__ void cast_rows_kernel(const float* __restrict__ x, TH* __restrict__ h, long long n) {
     pdl_enter();
-    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) h[i] = from_float<TH>(x[i]);
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (i >= n) return;
+    if constexpr (VEC == 4) store4(h + i, load4(x + i));
+    else h[i] = from_float<TH>(x[i]);
 }
 
 template <typename TH>
@@ -311,9 +313,14 @@ extern "C" int hos_scale_add_norm(const void* y, int y_dtype, int n_parts, float
 
 extern "C" int hos_cast_rows(const float* x, void* h, int h_dtype, long long n, cudaStream_t stream) {
     if (n <= 0) return 0;
-    const unsigned blocks = (unsigned)((n + 255) / 256);
-    if (h_dtype == kBF16) launch_pdl(cast_rows_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, x, (bf16*)h, n);
-    else launch_pdl(cast_rows_kernel<float>, dim3(blocks), dim3(256), 0, stream, x, (float*)h, n);
+    const bool vec = n % 4 == 0 && ((uintptr_t)x | (uintptr_t)h) % 16 == 0;
+    const unsigned blocks = (unsigned)((n / (vec ? 4 : 1) + 255) / 256);
+#define HOS_CAST(TH, VEC) launch_pdl(cast_rows_kernel<TH, VEC>, dim3(blocks), dim3(256), 0, stream, x, (TH*)h, n)
+    if (h_dtype == kBF16 && vec) HOS_CAST(bf16, 4);
+    else if (h_dtype == kBF16) HOS_CAST(bf16, 1);
+    else if (vec) HOS_CAST(float, 4);
+    else HOS_CAST(float, 1);
+#undef HOS_CAST
     return check_launch("cast_rows");
 }
 
